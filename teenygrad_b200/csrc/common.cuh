@@ -464,6 +464,21 @@ __device__ __forceinline__ uint4 head_norm_rope(const uint4 raw, const uint4 wra
   return make_uint4(out[0], out[1], out[2], out[3]);
 }
 
+// Gated linear units on two projections of the same channel.
+//   kGluSilu  SwiGLU with the rounding points of the unfused bf16 graph: both projections are bf16 tensors, silu is
+//             evaluated in f32 and rounded to bf16, the product is rounded by the caller.
+//   kGluGelu  0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * up in f32, one rounding by the caller; the bracket is
+//             twice a sigmoid: (1 + tanh(t)) / 2 = 1 / (1 + exp(-2 t)).
+constexpr int kGluSilu = 1, kGluGelu = 2;
+__device__ __forceinline__ float gelu_tanh_f(float g) {
+  return g / (1.0f + expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g)));
+}
+__device__ __forceinline__ float glu_f(int kind, float gate_acc, float up_acc) {
+  if (kind == kGluGelu) return gelu_tanh_f(gate_acc) * up_acc;
+  const float g = bf16_round(gate_acc), u = bf16_round(up_acc);
+  return bf16_round(g * (1.0f / (1.0f + expf(-g)))) * u;
+}
+
 // A {32-bit payload, 32-bit stamp} pair as ONE 64-bit word in (possibly another GPU's) global memory: a 64-bit scalar
 // access is single-copy atomic, so a reader that sees the stamp sees the payload written with it.  (A 16-byte vector
 // store of two pairs carries no such guarantee between its halves, let alone inside one.)  Layout = uint2{payload, stamp}.

@@ -51,7 +51,7 @@ struct GemmArgs {
   int group;              // persistent kernel: P-tiles per raster group
   int kb_per_split;       // skinny kernel: k-blocks per cluster rank
   int l2_ahead;           // skinny kernel: weight k-blocks asked into L2 beyond the shared-memory ring at start
-  int swiglu;             // W rows interleave 64 gate / 64 up channels; Y[M, N/2] = silu(gate) * up
+  int swiglu;             // GLU kind (glu_f): W rows interleave 64 gate / 64 up channels; Y[M, N/2] = act(gate) * up
   // Tensor-parallel push (skinny kernel only): instead of Y, the f32 row sums go to slot `rank` of every rank's
   // receive buffer (peer-mapped memory, [M][N] f32 each) and each CTA then bumps every rank's arrival counter.
   uint2* const* push_recv;    // device array [push_world]: where this rank writes inside rank p's buffer (or null)
@@ -91,13 +91,6 @@ __device__ __forceinline__ void tile_coords(int tile, int tiles_p, int tiles_q, 
   const int r = tile - g * per_group;
   tp = first_p + r % size_p;
   tq = r / size_p;
-}
-
-// SwiGLU on two projections of the same channel, with the rounding points of the unfused graph: both projections
-// are bf16 tensors, silu is evaluated in f32 and rounded to bf16, the product is rounded to bf16 by the caller.
-__device__ __forceinline__ float swiglu_f(float gate_acc, float up_acc) {
-  const float g = bf16_round(gate_acc), u = bf16_round(up_acc);
-  return bf16_round(g * (1.0f / (1.0f + expf(-g)))) * u;
 }
 
 // The four K=16 steps of a 64-deep product as one block of straight-line code, D[tmem] (+)= A * B with B in shared
@@ -292,7 +285,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_consta
                   float f[8];
 #pragma unroll
                   for (int e = 0; e < 8; ++e)
-                    f[e] = swiglu_f(__uint_as_float(gr[v * 8 + e]), __uint_as_float(ur[v * 8 + e]));
+                    f[e] = glu_f(args.swiglu, __uint_as_float(gr[v * 8 + e]), __uint_as_float(ur[v * 8 + e]));
                   if (vec_ok) {
                     uint4 o;
                     o.x = pack_bf16x2(f[0], f[1]); o.y = pack_bf16x2(f[2], f[3]);
@@ -812,7 +805,8 @@ gemm_bf16_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid
           us.x *= row_scale(wr + 64); us.y *= row_scale(wr + 65); us.z *= row_scale(wr + 66); us.w *= row_scale(wr + 67);
         }
         if (c < args.M) {
-          const float o[4] = {swiglu_f(gs.x, us.x), swiglu_f(gs.y, us.y), swiglu_f(gs.z, us.z), swiglu_f(gs.w, us.w)};
+          const float o[4] = {glu_f(args.swiglu, gs.x, us.x), glu_f(args.swiglu, gs.y, us.y), glu_f(args.swiglu, gs.z, us.z),
+                              glu_f(args.swiglu, gs.w, us.w)};
           bf16* dst = args.y + static_cast<size_t>(c) * args.ldy + n_out;
           if (vec_ok && n_out + 3 < args.N / 2) {
             *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]));
@@ -992,10 +986,11 @@ size_t gemm_bf16_scratch_bytes(int, int, int) { return 0; }
 
 // Y[M,N] = X[M,K] W^T (+bias).  w_is_kn: W given as [K, N] row-major (matmul_forward's B) instead of [N, K].
 int gemm_bf16(const bf16* x, int ldx, const bf16* w, int ldw, bool w_is_kn, const bf16* bias, bf16* y, int ldy,
-              int M, int N, int K, void*, size_t, cudaStream_t stream, bool swiglu, const GemmPush* push, float* y32,
+              int M, int N, int K, void*, size_t, cudaStream_t stream, int swiglu, const GemmPush* push, float* y32,
               int l2_ahead) {
   if (!x || !w || (!y && !y32) || M <= 0 || N <= 0 || K <= 0) return TEENY_ERR_BAD_ARG;
   if (y32 && (!w_is_kn || swiglu || push || bias)) return TEENY_ERR_BAD_ARG;  // f32 output: the [K, N] form only
+  if (swiglu < 0 || swiglu > kGluGelu) return TEENY_ERR_BAD_ARG;
   if (swiglu && (w_is_kn || bias || N % 128 != 0)) return TEENY_ERR_BAD_ARG;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) || (ldx & 7) || (ldw & 7))
     return TEENY_ERR_ALIGNMENT;
@@ -1005,7 +1000,7 @@ int gemm_bf16(const bf16* x, int ldx, const bf16* w, int ldw, bool w_is_kn, cons
   a.k_blocks = ceil_div(K, kBK);
   a.kb_per_split = a.k_blocks;
   a.group = 8;
-  a.swiglu = swiglu ? 1 : 0;
+  a.swiglu = swiglu;
   {
     static const int ahead = [] { const char* e = getenv("TEENY_L2_AHEAD"); return e ? atoi(e) : kL2Ahead; }();
     a.l2_ahead = l2_ahead >= 0 ? l2_ahead : (ahead < 0 ? 0 : ahead);

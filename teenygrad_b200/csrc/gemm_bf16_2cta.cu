@@ -43,7 +43,7 @@ struct Args2 {
   int tiles_m, tiles_n;   // 256 x 256 tiles
   int k_blocks;
   int group;
-  int swiglu;             // W rows interleave 64 gate / 64 up channels; Y[M, N/2] = silu(gate) * up
+  int swiglu;             // GLU kind (glu_f): W rows interleave 64 gate / 64 up channels; Y[M, N/2] = act(gate) * up
   int qkv;                // the fused QKV projection with head norms, rotary embedding and cache fill in the epilogue
   QkvEpilogue f;
   int* err;
@@ -86,12 +86,6 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
       "tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;"
       ::"r"(bar), "h"(static_cast<uint16_t>(3))
       : "memory");
-}
-
-// SwiGLU with the rounding points of the unfused bf16 graph (both projections, silu, product).
-__device__ __forceinline__ float swiglu2_f(float gate_acc, float up_acc) {
-  const float g = bf16_round(gate_acc), u = bf16_round(up_acc);
-  return bf16_round(g * (1.0f / (1.0f + expf(-g)))) * u;
 }
 
 __device__ __forceinline__ void tile_coords2(int tile, int tiles_m, int tiles_n, int group, int& tm, int& tn) {
@@ -322,7 +316,7 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
                 float f[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e)
-                  f[e] = swiglu2_f(__uint_as_float(gr[v * 8 + e]), __uint_as_float(ur[v * 8 + e]));
+                  f[e] = glu_f(args.swiglu, __uint_as_float(gr[v * 8 + e]), __uint_as_float(ur[v * 8 + e]));
                 if (vec_ok) {
                   uint4 o;
                   o.x = pack_bf16x2(f[0], f[1]); o.y = pack_bf16x2(f[2], f[3]);
@@ -410,7 +404,7 @@ int gemm_bf16_2cta_prepare() {
 
 // Y[M, N] = X[M, K] W[N, K]^T (+ bias) for large M and N; caller has checked pointers / alignment.
 int gemm_bf16_2cta(const bf16* x, int ldx, const bf16* w, int ldw, const bf16* bias, bf16* y, int ldy, int M, int N,
-                   int K, cudaStream_t stream, bool swiglu, const QkvEpilogue* qkv) {
+                   int K, cudaStream_t stream, int swiglu, const QkvEpilogue* qkv) {
   int rc = gemm_bf16_2cta_prepare();
   if (rc) return rc;
   if (qkv) {
@@ -443,7 +437,7 @@ int gemm_bf16_2cta(const bf16* x, int ldx, const bf16* w, int ldw, const bf16* b
   a.tiles_n = (N + 255) / 256;
   a.k_blocks = (K + kBK - 1) / kBK;
   a.group = 16;  // 16 x 256 rows of X share each 256-row block of W before moving on (best of 4/8/16/32 measured)
-  a.swiglu = swiglu ? 1 : 0;
+  a.swiglu = swiglu;
   if (qkv) {
     a.qkv = 1;
     a.f = *qkv;

@@ -23,7 +23,8 @@ int gemm_bf16_prepare();
 int attention_prefill_prepare();
 int attention_decode_prepare();
 // swiglu: W is [N, K] with rows interleaved in blocks of 64 gate channels / 64 up channels (N = 2 * channels) and
-// Y is [M, N / 2] = silu(gate) * up, rounded as the unfused bf16 graph rounds (both projections, silu, product).
+// Y is [M, N / 2] = act(gate) * up.  1 = silu, rounded as the unfused bf16 graph rounds (both projections, silu,
+// product); 2 = gelu in its tanh form, f32 up to one rounding (glu_f, common.cuh).
 // Tensor-parallel push mode of the decode GEMM (M <= 128): y is not written; every rank receives this rank's f32
 // result in its receive buffer as {value, stamp} pairs (8 bytes per element, element (row, col) at row * N + col),
 // stamp = *epoch * 1024 + round + 1.  The receiver recognises arrived data by the stamp, so the sender needs no
@@ -36,7 +37,7 @@ struct GemmPush {
   int owner_rows;         // 0: every rank receives every row; > 0: row r goes only to rank r / owner_rows, which sums it
 };
 int gemm_bf16(const bf16* x, int ldx, const bf16* w, int ldw, bool w_is_kn, const bf16* bias, bf16* y, int ldy,
-              int M, int N, int K, void* scratch, size_t scratch_bytes, cudaStream_t stream, bool swiglu = false,
+              int M, int N, int K, void* scratch, size_t scratch_bytes, cudaStream_t stream, int swiglu = 0,
               const GemmPush* push = nullptr, float* y32 = nullptr, int l2_ahead = -1);
 // y32 (w_is_kn only): store the f32 accumulators to y32[M, ldy] instead of rounding them to bf16 into y.
 // l2_ahead (decode-shaped GEMMs, M <= 128): how many of its 16 KB weight tiles beyond the shared-memory ring each CTA
@@ -102,7 +103,7 @@ struct QkvEpilogue {
 };
 int gemm_bf16_2cta_prepare();
 int gemm_bf16_2cta(const bf16* x, int ldx, const bf16* w, int ldw, const bf16* bias, bf16* y, int ldy, int M, int N,
-                   int K, cudaStream_t stream, bool swiglu = false, const QkvEpilogue* qkv = nullptr);
+                   int K, cudaStream_t stream, int swiglu = 0, const QkvEpilogue* qkv = nullptr);
 // Whether gemm_bf16 hands an [M, N] problem to the CTA-pair kernel (enough 256 x 256 tiles for every SM pair).
 bool gemm_bf16_uses_2cta(int M, int N);
 // C[M, N] = A[M, K] B[K, N], all f32 row-major and contiguous, on the tensor cores at f32 accuracy: each operand is
@@ -218,5 +219,105 @@ int sample_merge(const unsigned long long* lists, int parts, size_t list_stride,
                  float top_p, const float* u, int* out_idx, float* out_prob, cudaStream_t st);
 // u[row] = uniform in [0, 1) from (seed, step, row) by a stateless hash; step from *step_dev when given.
 int sampling_uniform(unsigned long long seed, int step, const int* step_dev, float* u, int rows, cudaStream_t st);
+
+// ---- layers of the hybrid decoders (recurrent mixers, windowed attention) ------------------------
+// One entry of a step: `len` tokens of the sequence in state slot `slot`, the first at position `pos`, in rows row0 ..
+// row0 + len - 1 of the step's activations.  pos == 0 starts the sequence: the slot's old contents are not read.
+struct SeqDesc { int slot, pos, row0, len; };
+
+// Element type of activations: bf16, or f32 where `f32` is set; then pointers to void hold floats.
+// Per-head matrix state S [DK, DV] (f32), one step per token, o = S^T q:
+//   kScanDelta  S <- diag(w) S - (a u)(u^T S) + k v^T, both terms on the old S, u = k / sqrt(sum k^2 + unit_eps),
+//               w = exp(-decay_coef * sigmoid(wz + w_bias)), a = sigmoid(a_raw + a_bias), q = the raw projection
+//   kScanDecay  S <- decay[head] S + k v^T, with silu on q, k and v
+constexpr int kScanDelta = 0, kScanDecay = 1;
+struct StateScan {
+  int mode, f32;
+  const void* proj;          // [T, ld]: the fused input projection; off_* = column of head 0 of each part
+  long long ld;
+  int off_q, off_k, off_v, off_a;
+  const void* wz;            // kScanDelta: [T, ld_wz], the decay's low-rank product
+  long long ld_wz;
+  const float *w_bias, *a_bias;  // [H * DK]
+  const float* decay;            // kScanDecay: [H]
+  float decay_coef, unit_eps;
+  float* state;              // [slots, H, DK, DV]
+  float* o;                  // [T, ldo], head h at column h * DV
+  long long ldo;
+  int H, DK, DV;
+};
+int state_scan_prepare();
+int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+bool state_scan_supports(int dk, int dv);
+// out[t, c] = o[t, c] / rms(group of c) * w[c] * sigmoid(gate[t, c]) * scale; groups of group_size consecutive columns
+int gated_rms_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, void* out, long long ldout,
+                   int T, int cols, int group_size, float eps, float scale, bool f32, cudaStream_t st);
+// Element-wise gated recurrence S <- (1 - z) S + z g(u), z = sigmoid(proj[off_z] + z_bias), u = proj[off_x] + x_bias, g(u) =
+// u + 1/2 for u >= 0, sigmoid(u) below; out = S * silu(proj[off_g]) * scale.  state [slots, W].
+struct MinGru {
+  int f32;
+  const void* proj;
+  long long ld;
+  int off_z, off_x, off_g;
+  const float *z_bias, *x_bias;
+  float* state;
+  void* out;
+  long long ldout;
+  int W;
+  float scale;
+};
+int min_gru(const MinGru& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+
+// Sliding-window grouped-query attention over a ring cache.  Query i sees keys i - window + 1 .. i.  Keys of positions
+// below the entry's `pos` come from the ring (row position % ring of [slots, Hkv, ring, D]); those of the entry itself
+// from k_new / v_new (row of the token, head at column head * D).
+struct WindowAttn {
+  int f32;
+  const void* q;             // [T, ldq], normed and rotated
+  long long ldq;
+  const void* k_new;         // [T, ldk]
+  long long ldk;
+  const void* v_new;         // [T, ldv]
+  long long ldv;
+  void* k_ring;
+  void* v_ring;
+  int ring, window;
+  void* out;                 // [T, ldo]
+  long long ldo;
+  int Hq, Hkv, D, DV;
+  float scale, out_scale;
+};
+// Per-head RMSNorm of q (in place) and k (k_raw -> k_out), then rotary positions on the first rot_dims dimensions
+// (i with i + rot_dims / 2), angles position * inv_freq[i] in f32.  q_w / k_w null: no norm.
+struct HeadNormRope {
+  int f32;
+  void* q;
+  long long ldq;
+  const void* k_raw;
+  long long ldkr;
+  void* k_out;
+  long long ldk;
+  const float *q_w, *k_w, *inv_freq;
+  int Hq, Hkv, D, rot_dims;
+  float eps;
+};
+int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+int window_attention_prepare();
+int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+// The last min(len, ring) tokens of every entry into the ring.
+int ring_append(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+
+// f32 residual stream: x = embed[id] * scale; x += delta, y = rms_norm(x) * w (y in the activation type).
+int embedding_scaled(const int* ids, const void* table, float* x, int T, int width, int vocab, float scale, bool f32,
+                     cudaStream_t st);
+// delta null: nothing is added.  rows null: row i -> y row i, and x is updated; else y row i comes from x row rows[i] (plus
+// its delta) and x stays as it is.
+int residual_rms_norm(float* x, const void* delta, long long ldd, void* y, long long ldy, const float* w, int M, int N, float eps,
+                      const int* rows, bool f32, cudaStream_t st);
+int tanh_rows(const void* x, long long ldx, void* y, long long ldy, int M, int N, bool f32, cudaStream_t st);
+// act(gate) * up from rows interleaved in blocks of 64 (kGlu* of common.cuh), f32
+int glu_interleaved_f32(const float* gu, long long ld, float* out, long long ldo, int T, int inter, int kind, cudaStream_t st);
+int argmax_f32(const float* logits, long long ld, float* best_val, int* best_idx, int rows, int cols, cudaStream_t st);
+int f32_to_bf16(const float* x, bf16* y, long long n, cudaStream_t st);
 
 }  // namespace teeny

@@ -31,8 +31,7 @@
 
 #include "../../include/teeny_b200.h"
 #include "../../include/teeny_qwen3.h"
-#include "common.cuh"
-#include "kernels.h"
+#include "decoder_base.h"
 #include <cstdio>
 
 namespace teeny {
@@ -266,37 +265,6 @@ int tp_enable_peer(TpContext* c, size_t rows, size_t cols, cudaStream_t st) {
   return 0;
 }
 
-__global__ void finish_step_kernel(const int* __restrict__ next_ids, int* __restrict__ cur_ids,
-                                   int* __restrict__ history, int* __restrict__ state, int B, int max_steps,
-                                   unsigned* __restrict__ tp_epoch) {
-  pdl_wait();
-  // state[0] = position of the next token to append, state[1] = live KV length during the step (= state[0] + 1),
-  // state[2] = number of generated tokens so far
-  const int b = blockIdx.x * blockDim.x + threadIdx.x;
-  const int step = state[2];
-  if (b < B) {
-    const int id = next_ids[b];
-    cur_ids[b] = id;
-    if (step < max_steps) history[static_cast<size_t>(step) * B + b] = id;
-  }
-  __syncthreads();  // single block: every thread has read `step`
-  if (b == 0) {
-    state[0] += 1;
-    state[1] += 1;
-    state[2] = step + 1;
-    if (tp_epoch) *tp_epoch += 1u;  // the pushes of the next step carry new stamps
-  }
-}
-
-__global__ void set_state_kernel(int* state, int pos, int len, int steps) {
-  pdl_wait();
-  state[0] = pos;
-  state[1] = len;
-  state[2] = steps;
-}
-
-size_t align_up(size_t v, size_t a = 256) { return (v + a - 1) / a * a; }
-
 }  // namespace
 
 // A projection weight in the form it was given: bf16 [N, K], or FP8 (E4M3) bytes [N, K] with f32 scales
@@ -329,7 +297,7 @@ struct Workspace {
 
 using namespace teeny;
 
-struct teeny_qwen3 {
+struct teeny_qwen3 : DecoderBase {
   teeny_qwen3_config cfg;
   int Hq, Hkv, I, Vl;  // local (per-rank) q heads, kv heads, intermediate, vocab rows
   std::vector<LayerWeights> layers;
@@ -338,7 +306,6 @@ struct teeny_qwen3 {
   void* fp8_scratch = nullptr;  // where a large prefill converts one FP8 projection at a time to bf16
   size_t fp8_scratch_bytes = 0;
   const float* inv_freq = nullptr;
-  uint8_t* ws = nullptr;
   Workspace off;
   ncclComm_t comm = nullptr;
   TpContext* tp = nullptr;
@@ -346,24 +313,12 @@ struct teeny_qwen3 {
   bool pending_gather = false;  // a pushed projection waits to be summed by the next norm
   int pending_parity = 0;
   unsigned pending_round = 0;
-  cudaGraphExec_t graph_exec = nullptr;
-  cudaStream_t capture_stream = nullptr;
   // tensor-parallel prefill in two half-batches: the all-reduce of one half runs on comm_stream while the other
   // half computes (ev_ready: projection written; ev_done[half]: its all-reduce finished)
   cudaStream_t comm_stream = nullptr;
   cudaEvent_t ev_ready = nullptr, ev_done[2] = {nullptr, nullptr};
   bool overlap_prefill = false;
-  // token selection: greedy unless a temperature > 0 was set
-  float sample_temperature = 0.0f, sample_top_p = 1.0f;
-  int sample_top_k = 1;
-  unsigned long long sample_seed = 0;
-  int graph_batch = 0;
-  unsigned long long graph_kernels = 0;  // kernels recorded in graph_exec (launch accounting)
-  int batch = 0;  // batch of the running generation (set by prefill)
-  int next_pos = 0;  // host mirror of state[0]: cache position the next decode step appends at (prefill sets it to S)
   bool tables_ready = false;
-
-  template <typename T> T* at(size_t o) const { return reinterpret_cast<T*>(ws + o); }
 };
 
 namespace {
@@ -439,12 +394,6 @@ Workspace plan(const teeny_qwen3_config& c) {
   w.total = o;
   return w;
 }
-
-#define TEENY_TRY(expr)                  \
-  do {                                   \
-    const int rc_ = (expr);              \
-    if (rc_ != 0) return rc_;            \
-  } while (0)
 
 int all_reduce(teeny_qwen3* m, bf16* buf, size_t count, cudaStream_t st) {
   if (m->cfg.tp_size == 1) return 0;
@@ -721,16 +670,7 @@ int run_head(teeny_qwen3* m, int B, int S, cudaStream_t st, const int* step_dev 
   int* ci = m->at<int>(m->off.cand_idx);
   int* next = m->at<int>(m->off.next_ids);
   if (c.tp_size == 1) {
-    if (m->sample_temperature > 0.0f) {
-      // token t of a generation draws u from (seed, t, row): t = 0 at prefill, the running count in decode
-      float* u = m->at<float>(m->off.sample_u);
-      TEENY_TRY(sampling_uniform(m->sample_seed, 0, S > 1 || !step_dev ? nullptr : step_dev, u, B, st));
-      TEENY_TRY(sample_top_k_top_p_bf16(logits, Vl, B, Vl, m->sample_temperature, m->sample_top_k, m->sample_top_p, u, next,
-                                        nullptr, st));
-      return 0;
-    }
-    TEENY_TRY(argmax_bf16(logits, Vl, cv, next, B, Vl, 0, st));
-    return 0;
+    return select_tokens(m, logits, Vl, B, Vl, S > 1 ? nullptr : step_dev, m->at<float>(m->off.sample_u), cv, next, st);
   }
   if (!m->comm) return TEENY_ERR_NCCL;
   if (m->sample_temperature > 0.0f) {
@@ -761,13 +701,6 @@ int run_head(teeny_qwen3* m, int B, int S, cudaStream_t st, const int* step_dev 
   return 0;
 }
 
-// While alive, this thread's launches carry the programmatic-dependent-launch attribute, so each kernel's set-up
-// (and the decode GEMMs' first weight tiles) overlaps the tail of the kernel before it.
-struct PdlScope {
-  PdlScope() { pdl_set_enabled(true); }
-  ~PdlScope() { pdl_set_enabled(false); }
-};
-
 int decode_body(teeny_qwen3* m, int B, cudaStream_t st) {
   PdlScope pdl;
   m->push_round = 0;  // every step issues an even number of pushes, so the parity sequence repeats
@@ -778,9 +711,8 @@ int decode_body(teeny_qwen3* m, int B, cudaStream_t st) {
   TEENY_TRY(run_layers(m, B, 1, 0, state + 0, state + 1, true, st));
   TEENY_TRY(run_head(m, B, 1, st, state + 2));
   unsigned* tp_epoch = (m->tp && m->tp->peer_ok) ? m->tp->epoch() : nullptr;
-  launch_kernel(finish_step_kernel, dim3(1), dim3(1024), 0, st, 1, m->at<int>(m->off.next_ids), m->at<int>(m->off.cur_ids),
-                                         m->at<int>(m->off.history), state, B, c.max_new_tokens, tp_epoch);
-  return static_cast<int>(cudaGetLastError());
+  return finish_step(m->at<int>(m->off.next_ids), m->at<int>(m->off.cur_ids), m->at<int>(m->off.history), state, B,
+                     c.max_new_tokens, tp_epoch, nullptr, st);
 }
 
 }  // namespace
@@ -865,8 +797,7 @@ int teeny_qwen3_create(const teeny_qwen3_config* cfg, void* workspace, size_t wo
 
 void teeny_qwen3_destroy(teeny_qwen3* m) {
   if (!m) return;
-  if (m->graph_exec) cudaGraphExecDestroy(m->graph_exec);
-  if (m->capture_stream) cudaStreamDestroy(m->capture_stream);
+  destroy_base(m);
   if (m->comm_stream) cudaStreamDestroy(m->comm_stream);
   if (m->ev_ready) cudaEventDestroy(m->ev_ready);
   for (cudaEvent_t ev : m->ev_done)
@@ -976,11 +907,9 @@ int teeny_qwen3_prefill(teeny_qwen3* m, const int* ids, int B, int S, teeny_stre
     TEENY_TRY(run_layers(m, B, S, 0, nullptr, nullptr, false, st));
   TEENY_TRY(run_head(m, B, S, st));
   // generation state: next position S, live length during the next step S + 1, no tokens recorded yet
-  launch_kernel(set_state_kernel, dim3(1), dim3(1), 0, st, 1, state, S - 1, S, 0);
-  launch_kernel(finish_step_kernel, dim3(1), dim3(1024), 0, st, 1, m->at<int>(m->off.next_ids), m->at<int>(m->off.cur_ids),
-                                         m->at<int>(m->off.history), state, B, c.max_new_tokens,
-                                         static_cast<unsigned*>(nullptr));
-  return static_cast<int>(cudaGetLastError());
+  TEENY_TRY(set_generation_state(state, S - 1, S, 0, st));
+  return finish_step(m->at<int>(m->off.next_ids), m->at<int>(m->off.cur_ids), m->at<int>(m->off.history), state, B,
+                     c.max_new_tokens, nullptr, nullptr, st);
 }
 
 int teeny_qwen3_decode(teeny_qwen3* m, teeny_stream_t stream) {
@@ -994,59 +923,18 @@ int teeny_qwen3_decode(teeny_qwen3* m, teeny_stream_t stream) {
 }
 
 int teeny_qwen3_set_sampling(teeny_qwen3* m, float temperature, int top_k, float top_p, unsigned long long seed) {
-  if (!m) return TEENY_ERR_BAD_ARG;
-  if (temperature > 0.0f) {
-    if (top_k < 1 || top_k > 1024 || !(top_p > 0.0f) || top_p > 1.0f) return TEENY_ERR_BAD_ARG;
-    m->sample_temperature = temperature; m->sample_top_k = top_k; m->sample_top_p = top_p; m->sample_seed = seed;
-  } else {
-    m->sample_temperature = 0.0f;
-  }
-  if (m->graph_exec) {  // the captured step has the old selection baked in
-    cudaGraphExecDestroy(m->graph_exec);
-    m->graph_exec = nullptr;
-  }
-  return TEENY_OK;
+  return m ? set_sampling(m, temperature, top_k, top_p, seed) : static_cast<int>(TEENY_ERR_BAD_ARG);
 }
 
 int teeny_qwen3_capture_decode(teeny_qwen3* m, teeny_stream_t stream) {
-  if (!m || m->batch <= 0) return TEENY_ERR_BAD_ARG;
-  (void)stream;  // recording needs a non-default stream of its own; the graph is replayed on the caller's stream
-  if (m->graph_exec) {
-    cudaGraphExecDestroy(m->graph_exec);
-    m->graph_exec = nullptr;
-  }
-  cudaError_t e = cudaSuccess;
-  if (!m->capture_stream) e = cudaStreamCreateWithFlags(&m->capture_stream, cudaStreamNonBlocking);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  cudaStream_t st = m->capture_stream;
-  e = cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  const unsigned long long launches_before = launches_so_far();
-  const int rc = decode_body(m, m->batch, st);
-  m->graph_kernels = launches_so_far() - launches_before;
-  cudaGraph_t graph = nullptr;
-  e = cudaStreamEndCapture(st, &graph);
-  if (rc != 0) {
-    if (graph) cudaGraphDestroy(graph);
-    return rc;
-  }
-  if (e != cudaSuccess) return static_cast<int>(e);
-  e = cudaGraphInstantiate(&m->graph_exec, graph, 0);
-  cudaGraphDestroy(graph);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  m->graph_batch = m->batch;
-  return 0;
+  (void)stream;
+  if (!m) return TEENY_ERR_BAD_ARG;
+  return capture_step(m, [m](cudaStream_t st) { return decode_body(m, m->batch, st); });
 }
 
 int teeny_qwen3_decode_replay(teeny_qwen3* m, teeny_stream_t stream) {
-  if (!m || !m->graph_exec || m->graph_batch != m->batch) return TEENY_ERR_BAD_ARG;
-  if (m->next_pos >= m->cfg.max_len) return TEENY_ERR_BAD_ARG;  // cache full (see teeny_qwen3_decode)
-  const int rc = static_cast<int>(cudaGraphLaunch(m->graph_exec, reinterpret_cast<cudaStream_t>(stream)));
-  if (rc == 0) {
-    ++m->next_pos;
-    count_launches(m->graph_kernels);
-  }
-  return rc;
+  if (!m) return TEENY_ERR_BAD_ARG;
+  return replay_step(m, m->cfg.max_len, reinterpret_cast<cudaStream_t>(stream));
 }
 
 void* teeny_qwen3_buffer(teeny_qwen3* m, int which) {

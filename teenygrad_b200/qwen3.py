@@ -12,6 +12,7 @@ import torch
 
 from . import _lib, tp as tpmod
 from ._lib import lib, check, vp, i32, f32, sz
+from .runner import BUF_HISTORY, BUF_LOGITS, BUF_NEXT_IDS, BUF_STATE, DecoderRunner, stream as _stream  # noqa: F401
 
 _BF16 = torch.bfloat16
 
@@ -48,7 +49,7 @@ _lib.bind(SIGNATURES)
 
 W_QKV, W_O, W_GATE_UP, W_DOWN, W_INPUT_LN, W_POST_LN, W_Q_NORM, W_K_NORM = range(8)
 W_EMBED, W_FINAL_NORM, W_LM_HEAD, W_INV_FREQ = 100, 101, 102, 103
-BUF_LOGITS, BUF_NEXT_IDS, BUF_HISTORY, BUF_STATE, BUF_HIDDEN, BUF_K_CACHE, BUF_V_CACHE, BUF_RESIDUAL, BUF_LAST_DELTA = range(9)
+BUF_HIDDEN, BUF_K_CACHE, BUF_V_CACHE, BUF_RESIDUAL, BUF_LAST_DELTA = range(4, 9)
 _LAYER_SLOTS = {"qkv": W_QKV, "o": W_O, "gate_up": W_GATE_UP, "down": W_DOWN, "input_ln": W_INPUT_LN,
                 "post_ln": W_POST_LN, "q_norm": W_Q_NORM, "k_norm": W_K_NORM}
 
@@ -76,10 +77,6 @@ def default_inv_freq(cfg):
     return 1.0 / (cfg.rope_theta ** (torch.arange(0, cfg.head_dim, 2, dtype=torch.int64).float() / cfg.head_dim))
 
 
-def _stream():
-    return C.c_void_p(torch.cuda.current_stream().cuda_stream)
-
-
 def check_generation_fits(prompt_len, max_new_tokens, max_len, history_capacity):
     """Raises unless a generation of ``max_new_tokens`` after a prompt of ``prompt_len`` fits the runner: the first
     token comes out of the prefill, each later one appends one cache row, so rows 0 .. prompt_len + max_new_tokens - 2
@@ -91,13 +88,14 @@ def check_generation_fits(prompt_len, max_new_tokens, max_len, history_capacity)
                          f"cache rows; the runner was created with max_len={max_len}")
 
 
-class Qwen3Runner:
-    """Greedy Qwen3 decoding on one GPU (or one tensor-parallel rank)."""
+class Qwen3Runner(DecoderRunner):
+    """Qwen3 decoding on one GPU (or one tensor-parallel rank)."""
+
+    PREFIX = "teeny_qwen3"
 
     def __init__(self, cfg, max_batch, max_len, max_tokens=None, max_new_tokens=256, tp_rank=0, tp_size=1,
                  comm=None, device=None):
         self.cfg = cfg
-        self.device = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
         tpmod.check_divisible(cfg, tp_size)
         c = _Cfg()
         c.num_layers, c.hidden, c.num_q_heads, c.num_kv_heads = cfg.num_layers, cfg.hidden, cfg.num_q_heads, cfg.num_kv_heads
@@ -106,31 +104,19 @@ class Qwen3Runner:
         c.max_tokens = max_tokens if max_tokens is not None else max_batch * max_len
         c.max_new_tokens, c.tp_rank, c.tp_size = max_new_tokens, tp_rank, tp_size
         self._c = c
-        self.tp_rank, self.tp_size, self.max_batch, self.max_new_tokens = tp_rank, tp_size, max_batch, max_new_tokens
-        self.max_len = max_len
+        self.tp_rank, self.tp_size, self.max_batch = tp_rank, tp_size, max_batch
         nbytes = lib.teeny_qwen3_workspace_bytes(C.byref(c))
         if nbytes == 0:
             raise ValueError("unsupported Qwen3 configuration for this backend")
-        self.workspace = torch.empty(nbytes, dtype=torch.uint8, device=self.device)
+        self._init_runner(nbytes, max_len, max_new_tokens, device)
         self._h = vp()
         self._comm = comm
         check(lib.teeny_qwen3_create(C.byref(c), C.c_void_p(self.workspace.data_ptr()), nbytes, comm, _stream(),
                                      C.byref(self._h)), "teeny_qwen3_create")
-        self._weights = []  # keeps device tensors alive
-        self._captured = False
-        self.batch = 0
-
-    def __del__(self):
-        h = getattr(self, "_h", None)
-        if h and lib is not None:  # at interpreter shutdown the module globals may already be gone
-            lib.teeny_qwen3_destroy(h)
-            self._h = None
 
     # ---- weights ----
     def _set(self, layer, which, t):
-        t = t.to(self.device).contiguous()
-        self._weights.append(t)
-        check(lib.teeny_qwen3_set_weight(self._h, layer, which, C.c_void_p(t.data_ptr())), "teeny_qwen3_set_weight")
+        self._call("set_weight", self._h, layer, which, self._upload(t))
 
     def load_layer_shards(self, layer, shards):
         for name, slot in _LAYER_SLOTS.items():
@@ -219,24 +205,9 @@ class Qwen3Runner:
         self.load_head_shards(tpmod.shard_head(sd, self.cfg, self.tp_rank, self.tp_size), inv_freq)
 
     # ---- buffers ----
-    def _view(self, which, shape, dtype):
-        ptr = lib.teeny_qwen3_buffer(self._h, which)
-        off = ptr - self.workspace.data_ptr()
-        n = int(torch.tensor(shape).prod()) * torch.empty(0, dtype=dtype).element_size()
-        return self.workspace[off:off + n].view(dtype).view(*shape)
-
     def logits(self):
         """bf16 [batch, vocab/tp]: this rank's slice of the last step's LM-head output."""
         return self._view(BUF_LOGITS, (self.batch, self.cfg.vocab // self.tp_size), _BF16)
-
-    def next_ids(self):
-        return self._view(BUF_NEXT_IDS, (self.batch,), torch.int32)
-
-    def history(self):
-        return self._view(BUF_HISTORY, (self.max_new_tokens, self.batch), torch.int32)
-
-    def state(self):
-        return self._view(BUF_STATE, (3,), torch.int32)
 
     def residual_stream(self, tokens):
         """(residual, last_delta), bf16 [tokens, hidden] each: their sum is the hidden state after the last layer
@@ -249,34 +220,14 @@ class Qwen3Runner:
         """ids: int [B, S] (any device).  Runs the prompt, records the first generated token."""
         ids = ids.to(self.device, dtype=torch.int32).contiguous()
         B, S = ids.shape
-        if B != self.batch:
-            self._captured = False  # the recorded decode step has the batch baked in; everything else is a fixed address
-        self.batch = B
+        self._set_batch(B)
         check(lib.teeny_qwen3_prefill(self._h, C.c_void_p(ids.data_ptr()), B, S, _stream()), "teeny_qwen3_prefill")
 
-    def set_sampling(self, temperature, top_k=50, top_p=1.0, seed=0):
-        """Token selection for the following generations: ``temperature <= 0`` is greedy; otherwise temperature /
-        top-k / top-p sampling with u for token t and row r a stateless hash of (seed, t, r) (single GPU only)."""
-        check(lib.teeny_qwen3_set_sampling(self._h, float(temperature), int(top_k), float(top_p), int(seed)),
-              "teeny_qwen3_set_sampling")
-        self._captured = False
-
-    def decode_step(self, graph=False):
-        if graph:
-            if not self._captured:
-                check(lib.teeny_qwen3_capture_decode(self._h, _stream()), "teeny_qwen3_capture_decode")
-                self._captured = True
-            check(lib.teeny_qwen3_decode_replay(self._h, _stream()), "teeny_qwen3_decode_replay")
-        else:
-            check(lib.teeny_qwen3_decode(self._h, _stream()), "teeny_qwen3_decode")
-
     def generate(self, prompt_ids, max_new_tokens, use_graph=True):
-        """Greedy decode; returns int32 [B, max_new_tokens] on the device (no host sync inside)."""
+        """Returns int32 [B, max_new_tokens] on the device (no host sync inside)."""
         check_generation_fits(prompt_ids.shape[1], max_new_tokens, self.max_len, self.max_new_tokens)
         self.prefill(prompt_ids)
-        for _ in range(max_new_tokens - 1):
-            self.decode_step(graph=use_graph)
-        return self.history()[:max_new_tokens].t()
+        return self._decode_loop(max_new_tokens, use_graph)
 
 
 def random_weights_device(cfg, seed, device, std=0.02):
