@@ -1,0 +1,120 @@
+/*
+ * teeny_hybrid -- C ABI of the hybrid decoder runner (libteeny_b200.so): decoders whose layers mix recurrent token
+ * mixers and sliding-window attention, in any order, over an f32 residual stream.
+ *
+ * A layer is   x <- x + sum of branches(norm1(x))   and, when it has a feed-forward,   x <- x + ff(norm2(x)).
+ * All branches of a layer read one fused input projection W_in norm1(x) and write one row that the fused output
+ * projection W_out takes back to the width, so parallel branches cost no extra matrix products.
+ *
+ * A sequence's state has a constant size (per branch: a ring of keys and values, a matrix state per head, or a vector
+ * state) and lives in a slot; a step runs any number of entries, each the next tokens of one slot.
+ *
+ * The reference has no such models; execution follows the same scheme as its model executor and as teeny_qwen3.h.
+ * All pointers are device pointers owned by the caller unless stated; nothing here allocates device memory.
+ * Status codes are those of teeny_b200.h.
+ */
+#ifndef TEENY_HYBRID_H_
+#define TEENY_HYBRID_H_
+
+#include "teeny_b200.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* Branch kinds.  pad8(n) = n rounded up to a multiple of 8; h = norm1(x).
+ *   ATTENTION  grouped-query attention over the last `window` tokens.  Input rows: q [heads * dim], k [kv_heads * dim] and,
+ *              unless KEYS_ARE_VALUES, v [kv_heads * vdim].  QK_NORM: per-head RMS norms of q and k before the rotation.
+ *              Rotate-half positions on the first rot_dims dimensions, score = (q . k) * score_scale.
+ *   DELTA      generalized delta rule, S <- diag(w) S - (a u)(u^T S) + k v^T, o = S^T r, w = exp(-decay_coef *
+ *              sigmoid(W_low tanh(W_1 h) + DECAY_BIAS)), a = sigmoid(A h + RATE_BIAS), u = k / sqrt(sum k^2 + unit_eps); each
+ *              head's o is RMS-normed, times O_NORM, times sigmoid(G h).
+ *              Input rows: r, k, v, a, g [heads * dim each], W_1 [rank].
+ *   DECAY      S <- decay_head S + k v^T, o = S^T q with silu on q, k, v; o is RMS-normed over all heads together, times
+ *              O_NORM, times sigmoid(G h).  Input rows: q, k [heads * dim], v, g [heads * vdim].
+ *   MIN_GRU    S <- (1 - z) S + z g(u), z = sigmoid(Z h + Z_BIAS), u = X h + X_BIAS, output S * silu(G h).
+ *              Input rows: z, x, g [dim each].
+ * Every part of the input rows starts at a multiple of 8 (zero rows in between), in the order given; branches follow one
+ * another.  A branch's output (heads * vdim, or dim for MIN_GRU; attention with KEYS_ARE_VALUES: heads * dim) is
+ * multiplied by out_scale and also starts at a multiple of 8. */
+enum { TEENY_HYBRID_ATTENTION = 0, TEENY_HYBRID_DELTA, TEENY_HYBRID_DECAY, TEENY_HYBRID_MIN_GRU };
+enum { TEENY_HYBRID_QK_NORM = 1, TEENY_HYBRID_KEYS_ARE_VALUES = 2 };
+/* Feed-forward activations of the gated dense kind: act(gate) * up. */
+enum { TEENY_HYBRID_ACT_SILU = 1, TEENY_HYBRID_ACT_GELU_TANH = 2 };
+
+typedef struct {
+  int num_layers, num_branches, width, vocab;
+  float eps;          /* of every norm of the model */
+  float embed_scale;
+  int f32;            /* 0: weights, activations and caches bf16; 1: everything f32 (true f32 products) */
+  int max_batch;      /* state slots, and most entries of a step */
+  int max_len;        /* most positions of a sequence */
+  int max_tokens;     /* most tokens of a step */
+  int max_rows;       /* most rows of logits of a step */
+  int max_new_tokens; /* capacity of the generated-token history */
+} teeny_hybrid_config;
+
+typedef struct {
+  int first_branch, num_branches;
+  int ff, act;        /* ff = 0: no feed-forward */
+} teeny_hybrid_layer;
+
+typedef struct {
+  int kind, heads, kv_heads, dim, vdim, rank, window, rot_dims, flags;
+  float score_scale, out_scale, decay_coef, unit_eps;
+} teeny_hybrid_branch;
+
+typedef struct teeny_hybrid teeny_hybrid;
+
+/* Weights.  Matrices are row-major in the model's element type with rows pad8(columns) elements apart; vectors are f32.
+ * Per layer (branch ignored): NORM1, NORM2 [width]; IN [input rows, width]; OUT [width, output columns]; GATE_UP [2 * pad64(ff),
+ * width], gate and up rows interleaved in blocks of 64 (zero rows beyond ff); DOWN [width, pad64(ff)].
+ * Per branch of the layer: Q_NORM, K_NORM [dim]; O_NORM; LOW [heads * dim, rank] (a matrix); DECAY_BIAS, RATE_BIAS [heads *
+ * dim]; Z_BIAS, X_BIAS [dim]; DECAY [heads]; INV_FREQ [rot_dims / 2].
+ * Model: EMBED [vocab, width] (rows width apart), FINAL_NORM, LM_HEAD [vocab, width]. */
+enum {
+  TEENY_HYBRID_W_NORM1 = 0, TEENY_HYBRID_W_NORM2, TEENY_HYBRID_W_IN, TEENY_HYBRID_W_OUT, TEENY_HYBRID_W_GATE_UP,
+  TEENY_HYBRID_W_DOWN,
+  TEENY_HYBRID_W_Q_NORM = 50, TEENY_HYBRID_W_K_NORM, TEENY_HYBRID_W_O_NORM, TEENY_HYBRID_W_LOW, TEENY_HYBRID_W_DECAY_BIAS,
+  TEENY_HYBRID_W_RATE_BIAS, TEENY_HYBRID_W_Z_BIAS, TEENY_HYBRID_W_X_BIAS, TEENY_HYBRID_W_DECAY, TEENY_HYBRID_W_INV_FREQ,
+  TEENY_HYBRID_W_EMBED = 100, TEENY_HYBRID_W_FINAL_NORM, TEENY_HYBRID_W_LM_HEAD
+};
+enum {
+  TEENY_HYBRID_BUF_LOGITS = 0, /* element type [rows, pad8(vocab)]: logits of the last step's rows */
+  TEENY_HYBRID_BUF_NEXT_IDS,   /* int32 [batch]: token chosen by the last step (input of the next) */
+  TEENY_HYBRID_BUF_HISTORY,    /* int32 [max_new_tokens, batch] */
+  TEENY_HYBRID_BUF_STATE,      /* int32 [3]: position, live length, tokens generated (of the first sequence) */
+  TEENY_HYBRID_BUF_RESIDUAL,   /* f32 [tokens, width]: the residual stream before the last sublayer's output was added ... */
+  TEENY_HYBRID_BUF_LAST_DELTA  /* ... and that output, element type [tokens, pad8(width)] */
+};
+
+/* Bytes of workspace (activations, states, caches, generation state); 0 if the configuration is not supported.  The
+ * arrays are host memory: num_layers layers, num_branches branches. */
+size_t teeny_hybrid_workspace_bytes(const teeny_hybrid_config* cfg, const teeny_hybrid_layer* layers, const teeny_hybrid_branch* branches);
+/* Bytes of state one slot holds over all branches (the part of the workspace that grows with max_batch alone). */
+size_t teeny_hybrid_slot_bytes(const teeny_hybrid_config* cfg, const teeny_hybrid_layer* layers, const teeny_hybrid_branch* branches);
+int teeny_hybrid_create(const teeny_hybrid_config* cfg, const teeny_hybrid_layer* layers, const teeny_hybrid_branch* branches,
+                        void* workspace, size_t workspace_bytes, teeny_stream_t stream, teeny_hybrid** out);
+void teeny_hybrid_destroy(teeny_hybrid* model);
+int teeny_hybrid_set_weight(teeny_hybrid* model, int layer, int branch, int which, const void* device_ptr);
+/* One step: entry e brings the next lens[e] tokens of slot slots[e], the first at position positions[e]; position 0 starts a
+ * new sequence in the slot.  slots, positions, lens (n entries each) and rows (n_rows) are host arrays; ids: device
+ * int32, the entries' tokens one after the other.  rows: which of the step's tokens get logits (row numbers in ids).  A
+ * slot must not appear twice in a step. */
+int teeny_hybrid_step(teeny_hybrid* model, const int* ids, const int* slots, const int* positions, const int* lens, int n,
+                      const int* rows, int n_rows, teeny_stream_t stream);
+/* Generation over the sequences of the last step: begin picks every entry's first token from the logits of its last
+ * token (the step must have asked for exactly one row per entry, in order) and records it; each decode then appends one
+ * token per sequence.  decode launches the kernels; capture_decode records one step as a CUDA graph, decode_replay
+ * launches it. */
+int teeny_hybrid_begin(teeny_hybrid* model, teeny_stream_t stream);
+int teeny_hybrid_decode(teeny_hybrid* model, teeny_stream_t stream);
+int teeny_hybrid_set_sampling(teeny_hybrid* model, float temperature, int top_k, float top_p, unsigned long long seed);
+int teeny_hybrid_capture_decode(teeny_hybrid* model, teeny_stream_t stream);
+int teeny_hybrid_decode_replay(teeny_hybrid* model, teeny_stream_t stream);
+void* teeny_hybrid_buffer(teeny_hybrid* model, int which);
+
+#ifdef __cplusplus
+}
+#endif
+#endif /* TEENY_HYBRID_H_ */

@@ -10,7 +10,7 @@ import os
 import re
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-HEADERS = ("teeny_b200.h", "teeny_qwen3.h")
+HEADERS = ("teeny_b200.h", "teeny_qwen3.h", "teeny_hybrid.h")
 RUST_FILE = os.path.join(ROOT, "integration", "teeny-cuda", "src", "b200.rs")
 BEGIN, END = "// ---- generated from include/*.h: begin ----", "// ---- generated from include/*.h: end ----"
 
@@ -24,8 +24,14 @@ TYPES = {
     "void**": "*mut *mut c_void", "const char*": "*const c_char",
     "const teeny_attn_shape*": "*const TeenyAttnShape", "const teeny_qwen3_config*": "*const TeenyQwen3Config",
     "teeny_qwen3*": "*mut TeenyQwen3", "teeny_qwen3**": "*mut *mut TeenyQwen3",
+    "const teeny_hybrid_config*": "*const TeenyHybridConfig", "const teeny_hybrid_layer*": "*const TeenyHybridLayer",
+    "const teeny_hybrid_branch*": "*const TeenyHybridBranch", "teeny_hybrid*": "*mut TeenyHybrid",
+    "teeny_hybrid**": "*mut *mut TeenyHybrid",
 }
-STRUCT_NAMES = {"teeny_attn_shape": "TeenyAttnShape", "teeny_qwen3_config": "TeenyQwen3Config"}
+STRUCT_NAMES = {"teeny_attn_shape": "TeenyAttnShape", "teeny_qwen3_config": "TeenyQwen3Config",
+                "teeny_hybrid_config": "TeenyHybridConfig", "teeny_hybrid_layer": "TeenyHybridLayer",
+                "teeny_hybrid_branch": "TeenyHybridBranch"}
+OPAQUE = {"teeny_qwen3": "TeenyQwen3", "teeny_hybrid": "TeenyHybrid"}
 
 
 def _strip_comments(text):
@@ -96,7 +102,8 @@ def render_rust(functions, structs, enums):
         for ctype, f in fields:
             out.append(f"    pub {rust_arg_name(f)}: {TYPES[ctype]},")
         out.append("}")
-    out.append("/// Opaque runner handle (`teeny_qwen3`).\n#[repr(C)]\npub struct TeenyQwen3 {\n    _private: [u8; 0],\n}")
+    for cname, rname in OPAQUE.items():
+        out.append(f"/// Opaque runner handle (`{cname}`).\n#[repr(C)]\npub struct {rname} {{\n    _private: [u8; 0],\n}}")
     for name, value in enums.items():
         out.append(f"pub const {name}: c_int = {value};")
     out.append('#[link(name = "teeny_b200")]\nextern "C" {')

@@ -67,9 +67,55 @@ pub struct TeenyQwen3Config {
     pub tp_rank: c_int,
     pub tp_size: c_int,
 }
+#[repr(C)]
+#[derive(Clone, Copy, Debug, Default)]
+pub struct TeenyHybridConfig {
+    pub num_layers: c_int,
+    pub num_branches: c_int,
+    pub width: c_int,
+    pub vocab: c_int,
+    pub eps: f32,
+    pub embed_scale: f32,
+    pub f32: c_int,
+    pub max_batch: c_int,
+    pub max_len: c_int,
+    pub max_tokens: c_int,
+    pub max_rows: c_int,
+    pub max_new_tokens: c_int,
+}
+#[repr(C)]
+#[derive(Clone, Copy, Debug, Default)]
+pub struct TeenyHybridLayer {
+    pub first_branch: c_int,
+    pub num_branches: c_int,
+    pub ff: c_int,
+    pub act: c_int,
+}
+#[repr(C)]
+#[derive(Clone, Copy, Debug, Default)]
+pub struct TeenyHybridBranch {
+    pub kind: c_int,
+    pub heads: c_int,
+    pub kv_heads: c_int,
+    pub dim: c_int,
+    pub vdim: c_int,
+    pub rank: c_int,
+    pub window: c_int,
+    pub rot_dims: c_int,
+    pub flags: c_int,
+    pub score_scale: f32,
+    pub out_scale: f32,
+    pub decay_coef: f32,
+    pub unit_eps: f32,
+}
 /// Opaque runner handle (`teeny_qwen3`).
 #[repr(C)]
 pub struct TeenyQwen3 {
+    _private: [u8; 0],
+}
+/// Opaque runner handle (`teeny_hybrid`).
+#[repr(C)]
+pub struct TeenyHybrid {
     _private: [u8; 0],
 }
 pub const TEENY_OK: c_int = 0;
@@ -101,6 +147,39 @@ pub const TEENY_QWEN3_BUF_K_CACHE: c_int = 5;
 pub const TEENY_QWEN3_BUF_V_CACHE: c_int = 6;
 pub const TEENY_QWEN3_BUF_RESIDUAL: c_int = 7;
 pub const TEENY_QWEN3_BUF_LAST_DELTA: c_int = 8;
+pub const TEENY_HYBRID_ATTENTION: c_int = 0;
+pub const TEENY_HYBRID_DELTA: c_int = 1;
+pub const TEENY_HYBRID_DECAY: c_int = 2;
+pub const TEENY_HYBRID_MIN_GRU: c_int = 3;
+pub const TEENY_HYBRID_QK_NORM: c_int = 1;
+pub const TEENY_HYBRID_KEYS_ARE_VALUES: c_int = 2;
+pub const TEENY_HYBRID_ACT_SILU: c_int = 1;
+pub const TEENY_HYBRID_ACT_GELU_TANH: c_int = 2;
+pub const TEENY_HYBRID_W_NORM1: c_int = 0;
+pub const TEENY_HYBRID_W_NORM2: c_int = 1;
+pub const TEENY_HYBRID_W_IN: c_int = 2;
+pub const TEENY_HYBRID_W_OUT: c_int = 3;
+pub const TEENY_HYBRID_W_GATE_UP: c_int = 4;
+pub const TEENY_HYBRID_W_DOWN: c_int = 5;
+pub const TEENY_HYBRID_W_Q_NORM: c_int = 50;
+pub const TEENY_HYBRID_W_K_NORM: c_int = 51;
+pub const TEENY_HYBRID_W_O_NORM: c_int = 52;
+pub const TEENY_HYBRID_W_LOW: c_int = 53;
+pub const TEENY_HYBRID_W_DECAY_BIAS: c_int = 54;
+pub const TEENY_HYBRID_W_RATE_BIAS: c_int = 55;
+pub const TEENY_HYBRID_W_Z_BIAS: c_int = 56;
+pub const TEENY_HYBRID_W_X_BIAS: c_int = 57;
+pub const TEENY_HYBRID_W_DECAY: c_int = 58;
+pub const TEENY_HYBRID_W_INV_FREQ: c_int = 59;
+pub const TEENY_HYBRID_W_EMBED: c_int = 100;
+pub const TEENY_HYBRID_W_FINAL_NORM: c_int = 101;
+pub const TEENY_HYBRID_W_LM_HEAD: c_int = 102;
+pub const TEENY_HYBRID_BUF_LOGITS: c_int = 0;
+pub const TEENY_HYBRID_BUF_NEXT_IDS: c_int = 1;
+pub const TEENY_HYBRID_BUF_HISTORY: c_int = 2;
+pub const TEENY_HYBRID_BUF_STATE: c_int = 3;
+pub const TEENY_HYBRID_BUF_RESIDUAL: c_int = 4;
+pub const TEENY_HYBRID_BUF_LAST_DELTA: c_int = 5;
 #[link(name = "teeny_b200")]
 extern "C" {
     pub fn teeny_version() -> c_int;
@@ -167,6 +246,18 @@ extern "C" {
     pub fn teeny_tp_all_reduce_bf16(comm: *mut c_void, buf: *mut u16, count: usize, stream: CUstream) -> c_int;
     pub fn teeny_tp_peer_enabled(comm: *mut c_void) -> c_int;
     pub fn teeny_tp_gather_add_rms_norm_bf16(recv: *const c_void, slot_elems: usize, world: c_int, epoch: *const u32, round: u32, residual: *mut u16, y: *mut u16, weight: *const u16, m: c_int, n: c_int, eps: f32, wait_limit_ns: c_ulonglong, stream: CUstream) -> c_int;
+    pub fn teeny_hybrid_workspace_bytes(cfg: *const TeenyHybridConfig, layers: *const TeenyHybridLayer, branches: *const TeenyHybridBranch) -> usize;
+    pub fn teeny_hybrid_slot_bytes(cfg: *const TeenyHybridConfig, layers: *const TeenyHybridLayer, branches: *const TeenyHybridBranch) -> usize;
+    pub fn teeny_hybrid_create(cfg: *const TeenyHybridConfig, layers: *const TeenyHybridLayer, branches: *const TeenyHybridBranch, workspace: *mut c_void, workspace_bytes: usize, stream: CUstream, out: *mut *mut TeenyHybrid) -> c_int;
+    pub fn teeny_hybrid_destroy(model: *mut TeenyHybrid);
+    pub fn teeny_hybrid_set_weight(model: *mut TeenyHybrid, layer: c_int, branch: c_int, which: c_int, device_ptr: *const c_void) -> c_int;
+    pub fn teeny_hybrid_step(model: *mut TeenyHybrid, ids: *const c_int, slots: *const c_int, positions: *const c_int, lens: *const c_int, n: c_int, rows: *const c_int, n_rows: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_hybrid_begin(model: *mut TeenyHybrid, stream: CUstream) -> c_int;
+    pub fn teeny_hybrid_decode(model: *mut TeenyHybrid, stream: CUstream) -> c_int;
+    pub fn teeny_hybrid_set_sampling(model: *mut TeenyHybrid, temperature: f32, top_k: c_int, top_p: f32, seed: c_ulonglong) -> c_int;
+    pub fn teeny_hybrid_capture_decode(model: *mut TeenyHybrid, stream: CUstream) -> c_int;
+    pub fn teeny_hybrid_decode_replay(model: *mut TeenyHybrid, stream: CUstream) -> c_int;
+    pub fn teeny_hybrid_buffer(model: *mut TeenyHybrid, which: c_int) -> *mut c_void;
 }
 // ---- generated from include/*.h: end ----
 

@@ -808,6 +808,171 @@ __global__ void argmax_combine_kernel(const float* __restrict__ vals, const int*
   out_idx[r] = i;
 }
 
+
+// ---- f32 residual stream (decoders whose residual sum is kept in 32 bits) ----
+__device__ __forceinline__ void st_as(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st_as(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+// four consecutive elements
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld4(const bf16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(bf16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+template <typename T>
+__global__ void embedding_scaled_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x, int width,
+                                        int vocab, float scale) {
+  pdl_wait();
+  pdl_trigger();
+  int id = ids[blockIdx.x];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // ids are validated on the host; clamp keeps loads in range
+  const T* src = table + static_cast<size_t>(id) * width;
+  float* dst = x + static_cast<size_t>(blockIdx.x) * width;
+  if ((width & 3) == 0) {
+    for (int c = threadIdx.x; c < (width >> 2); c += blockDim.x) {
+      const float4 v = ld4(src + 4 * c);
+      st4(dst + 4 * c, make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale));
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = ldf<T>(src + c) * scale;
+  }
+}
+
+// One CTA per row, the row held in registers (VPT vectors of four per thread) between the statistics and the scaling.
+template <typename T, int VPT>
+__global__ void residual_rms_norm_kernel(float* __restrict__ x, const T* __restrict__ delta, long long ldd, T* __restrict__ y,
+                                         long long ldy, const float* __restrict__ w, int N, float eps, const int* __restrict__ rows) {
+  const int nv = N >> 2;
+  float4 g[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    g[i] = idx < nv ? __ldg(reinterpret_cast<const float4*>(w) + idx) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const size_t row = rows ? rows[blockIdx.x] : blockIdx.x;
+  float* xr = x + row * N;
+  float4 v[VPT], d[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    v[i] = d[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (idx < nv) {
+      v[i] = ld4(xr + 4 * idx);
+      if (delta) d[i] = ld4(delta + row * ldd + 4 * idx);
+    }
+  }
+  float sq = 0.0f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    v[i] = make_float4(v[i].x + d[i].x, v[i].y + d[i].y, v[i].z + d[i].z, v[i].w + d[i].w);
+    if (delta && !rows && idx < nv) st4(xr + 4 * idx, v[i]);
+    sq = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, sq))));
+  }
+  sq = block_sum(sq, red);
+  const float rr = 1.0f / sqrtf(sq / static_cast<float>(N) + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx < nv)
+      st4(y + static_cast<size_t>(blockIdx.x) * ldy + 4 * idx,
+          make_float4(v[i].x * rr * g[i].x, v[i].y * rr * g[i].y, v[i].z * rr * g[i].z, v[i].w * rr * g[i].w));
+  }
+}
+// any N: scalar accesses
+template <typename T>
+__global__ void residual_rms_norm_scalar_kernel(float* __restrict__ x, const T* __restrict__ delta, long long ldd, T* __restrict__ y,
+                                                long long ldy, const float* __restrict__ w, int N, float eps,
+                                                const int* __restrict__ rows) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const size_t row = rows ? rows[blockIdx.x] : blockIdx.x;
+  float* xr = x + row * N;
+  float sq = 0.0f;
+  for (int c = threadIdx.x; c < N; c += blockDim.x) {
+    const float v = xr[c] + (delta ? ldf<T>(delta + row * ldd + c) : 0.0f);
+    sq = fmaf(v, v, sq);
+  }
+  sq = block_sum(sq, red);
+  const float rr = 1.0f / sqrtf(sq / static_cast<float>(N) + eps);
+  for (int c = threadIdx.x; c < N; c += blockDim.x) {
+    const float v = xr[c] + (delta ? ldf<T>(delta + row * ldd + c) : 0.0f);
+    if (delta && !rows) xr[c] = v;
+    st_as(y + static_cast<size_t>(blockIdx.x) * ldy + c, v * rr * w[c]);
+  }
+}
+
+template <typename T>
+__global__ void tanh_rows_kernel(const T* __restrict__ x, long long ldx, T* __restrict__ y, long long ldy, int M, int N) {
+  pdl_wait();
+  pdl_trigger();
+  const long long total = static_cast<long long>(M) * N;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / N;
+    const int c = static_cast<int>(i - r * N);
+    st_as(y + r * ldy + c, tanhf(ldf<T>(x + r * ldx + c)));
+  }
+}
+
+__global__ void glu_interleaved_f32_kernel(const float* __restrict__ gu, long long ld, float* __restrict__ out, long long ldo, int T,
+                                           int inter, int kind) {
+  pdl_wait();
+  pdl_trigger();
+  const long long total = static_cast<long long>(T) * inter;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / inter;
+    const int c = static_cast<int>(i - r * inter);
+    const float* p = gu + r * ld + (c >> 6) * 128 + (c & 63);
+    out[r * ldo + c] = (kind == kGluGelu ? gelu_tanh_f(p[0]) : silu_f(p[0])) * p[64];
+  }
+}
+
+__global__ void argmax_f32_kernel(const float* __restrict__ logits, long long ld, float* __restrict__ best_val,
+                                  int* __restrict__ best_idx, int cols) {
+  pdl_wait();
+  __shared__ float sv[32];
+  __shared__ int si[32];
+  const float* row = logits + static_cast<size_t>(blockIdx.x) * ld;
+  float v = -INFINITY;
+  int idx = 0x7fffffff;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) argmax_merge(v, idx, row[c], c);
+  for (int pass = 0; pass < 2; ++pass) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
+      argmax_merge(v, idx, ov, oi);
+    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (pass == 0) {
+      if (lane == 0) { sv[warp] = v; si[warp] = idx; }
+      __syncthreads();
+      v = lane < (blockDim.x >> 5) ? sv[lane] : -INFINITY;
+      idx = lane < (blockDim.x >> 5) ? si[lane] : 0x7fffffff;
+    } else if (threadIdx.x == 0) {
+      best_val[blockIdx.x] = v;
+      best_idx[blockIdx.x] = idx;
+    }
+  }
+}
+
+__global__ void f32_to_bf16_kernel(const float* __restrict__ x, bf16* __restrict__ y, long long n) {
+  pdl_wait();
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x)
+    y[i] = __float2bfloat16_rn(x[i]);
+}
+
 }  // namespace
 
 int rms_norm_f32(const float* x, float* y, const float* w, float* rrms, int M, int N, float eps, cudaStream_t st) {
@@ -944,6 +1109,79 @@ int argmax_combine(const float* vals, const int* idx, int* out_idx, int parts, i
   if (!vals || !idx || !out_idx || parts <= 0 || rows < 0) return TEENY_ERR_BAD_ARG;
   if (rows == 0) return TEENY_OK;
   launch_kernel(argmax_combine_kernel, dim3((rows + 127) / 128), dim3(128), 0, st, 1, vals, idx, out_idx, parts, rows);
+  return static_cast<int>(cudaGetLastError());
+}
+
+
+int embedding_scaled(const int* ids, const void* table, float* x, int T, int width, int vocab, float scale, bool f32,
+                     cudaStream_t st) {
+  if (!ids || !table || !x || T <= 0 || width <= 0 || vocab <= 0) return TEENY_ERR_BAD_ARG;
+  const int threads = width >= 1024 ? 256 : 64;
+  if (f32) launch_kernel(embedding_scaled_kernel<float>, dim3(T), dim3(threads), 0, st, 1, ids, static_cast<const float*>(table), x, width, vocab, scale);
+  else launch_kernel(embedding_scaled_kernel<bf16>, dim3(T), dim3(threads), 0, st, 1, ids, static_cast<const bf16*>(table), x, width, vocab, scale);
+  return static_cast<int>(cudaGetLastError());
+}
+
+namespace {
+template <typename T>
+int launch_residual_norm(float* x, const void* delta, long long ldd, void* y, long long ldy, const float* w, int M, int N, float eps,
+                         const int* rows, cudaStream_t st) {
+  const T* d = static_cast<const T*>(delta);
+  T* yo = static_cast<T*>(y);
+  const int nv = N / 4;
+  const bool vec = N % 4 == 0 && ldy % 4 == 0 && (!delta || ldd % 4 == 0) && aligned16(x) && aligned16(y) && aligned16(w) &&
+                   (!delta || aligned16(delta)) && nv <= 8 * 512;
+  if (!vec) {
+    launch_kernel(residual_rms_norm_scalar_kernel<T>, dim3(M), dim3(256), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps, rows);
+    return static_cast<int>(cudaGetLastError());
+  }
+  // a few rows (decode) are one chain of latencies: one vector per thread
+  int threads = (nv + 31) / 32 * 32;
+  const int most = M <= 512 ? 1024 : 256;
+  if (threads > most) threads = most;
+  if (nv > 8 * threads) threads = 512;
+  const int vpt = (nv + threads - 1) / threads;
+#define TEENY_RRN(V) launch_kernel(residual_rms_norm_kernel<T, V>, dim3(M), dim3(threads), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps, rows)
+  if (vpt <= 1) TEENY_RRN(1);
+  else if (vpt <= 2) TEENY_RRN(2);
+  else if (vpt <= 4) TEENY_RRN(4);
+  else TEENY_RRN(8);
+#undef TEENY_RRN
+  return static_cast<int>(cudaGetLastError());
+}
+}  // namespace
+
+int residual_rms_norm(float* x, const void* delta, long long ldd, void* y, long long ldy, const float* w, int M, int N, float eps,
+                      const int* rows, bool f32, cudaStream_t st) {
+  if (!x || !y || !w || M <= 0 || N <= 0) return TEENY_ERR_BAD_ARG;
+  return f32 ? launch_residual_norm<float>(x, delta, ldd, y, ldy, w, M, N, eps, rows, st)
+             : launch_residual_norm<bf16>(x, delta, ldd, y, ldy, w, M, N, eps, rows, st);
+}
+
+int tanh_rows(const void* x, long long ldx, void* y, long long ldy, int M, int N, bool f32, cudaStream_t st) {
+  if (!x || !y || M <= 0 || N <= 0) return TEENY_ERR_BAD_ARG;
+  const dim3 grid(ew_grid(static_cast<long long>(M) * N, kEwThreads));
+  if (f32) launch_kernel(tanh_rows_kernel<float>, grid, dim3(kEwThreads), 0, st, 1, static_cast<const float*>(x), ldx, static_cast<float*>(y), ldy, M, N);
+  else launch_kernel(tanh_rows_kernel<bf16>, grid, dim3(kEwThreads), 0, st, 1, static_cast<const bf16*>(x), ldx, static_cast<bf16*>(y), ldy, M, N);
+  return static_cast<int>(cudaGetLastError());
+}
+
+int glu_interleaved_f32(const float* gu, long long ld, float* out, long long ldo, int T, int inter, int kind, cudaStream_t st) {
+  if (!gu || !out || T <= 0 || inter <= 0 || inter % 64 || (kind != kGluSilu && kind != kGluGelu)) return TEENY_ERR_BAD_ARG;
+  launch_kernel(glu_interleaved_f32_kernel, dim3(ew_grid(static_cast<long long>(T) * inter, kEwThreads)), dim3(kEwThreads), 0, st, 1, gu, ld,
+                out, ldo, T, inter, kind);
+  return static_cast<int>(cudaGetLastError());
+}
+
+int argmax_f32(const float* logits, long long ld, float* best_val, int* best_idx, int rows, int cols, cudaStream_t st) {
+  if (!logits || !best_val || !best_idx || rows <= 0 || cols <= 0) return TEENY_ERR_BAD_ARG;
+  launch_kernel(argmax_f32_kernel, dim3(rows), dim3(256), 0, st, 1, logits, ld, best_val, best_idx, cols);
+  return static_cast<int>(cudaGetLastError());
+}
+
+int f32_to_bf16(const float* x, bf16* y, long long n, cudaStream_t st) {
+  if (!x || !y || n <= 0) return TEENY_ERR_BAD_ARG;
+  launch_kernel(f32_to_bf16_kernel, dim3(ew_grid(n, kEwThreads)), dim3(kEwThreads), 0, st, 1, x, y, n);
   return static_cast<int>(cudaGetLastError());
 }
 

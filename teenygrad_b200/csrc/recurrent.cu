@@ -1,0 +1,477 @@
+// Recurrent token mixers: per-head matrix states (generalized delta rule, scalar-decay linear attention) and the
+// element-wise minimal GRU, plus the gated group norm behind the matrix states.  Everything that enters a recurrence
+// and the states themselves are f32.
+//
+// state_scan_kernel.  The columns of a head's state are independent of one another given the head's key-side vectors:
+// S[:, j] <- w o S[:, j] - (a o u)(u . S[:, j]) + k v_j, o_j = q . S[:, j].  So a CTA owns a block of columns of one
+// (sequence, head), KS neighbouring lanes share a column pair and hold kRows key channels of it each in registers, and
+// the tokens go by one after the other: exact f32 arithmetic, and the result does not depend on how a prompt was cut.
+//   warps 0 .. n-1    consumers: per token 5 (delta) or 3 (decay) packed f32x2 operations per channel pair and column,
+//                     key-side vectors by 16-byte broadcast loads from shared memory, one butterfly over the KS lanes
+//                     for u . S and one for the output.
+//   last four warps   producers: read the raw projections of the next kChunk tokens, evaluate unit norms, decays,
+//                     rates and activations once per (token, channel) and leave them in the other shared-memory buffer.
+// The buffers change hands through named barriers (bar.sync / bar.arrive).
+#include <atomic>
+
+#include "common.cuh"
+#include "kernels.h"
+
+namespace teeny {
+
+namespace {
+
+constexpr int kRows = 16;        // key channels per consumer lane
+constexpr int kChunk = 16;       // tokens per shared-memory buffer
+constexpr int kProducers = 128;  // threads
+constexpr int kMaxConsumers = 512;
+
+template <typename T> __device__ __forceinline__ float ldf(const T* p);
+template <> __device__ __forceinline__ float ldf<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float ldf<bf16>(const bf16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void stf(float* p, float v) { *p = v; }
+__device__ __forceinline__ void stf(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+
+// Barrier FIRST + buf (buf 0 or 1); the numbers are immediates so that the kernel claims no more barriers than it uses.
+template <int FIRST>
+__device__ __forceinline__ void buffer_sync(int buf, int nthreads) {
+  if (buf == 0) asm volatile("bar.sync %0, %1;" ::"n"(FIRST), "r"(nthreads) : "memory");
+  else asm volatile("bar.sync %0, %1;" ::"n"(FIRST + 1), "r"(nthreads) : "memory");
+}
+template <int FIRST>
+__device__ __forceinline__ void buffer_arrive(int buf, int nthreads) {
+  if (buf == 0) asm volatile("bar.arrive %0, %1;" ::"n"(FIRST), "r"(nthreads) : "memory");
+  else asm volatile("bar.arrive %0, %1;" ::"n"(FIRST + 1), "r"(nthreads) : "memory");
+}
+constexpr int kBarFull = 1, kBarEmpty = 3;
+
+typedef unsigned long long f32x2;  // two packed f32
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+template <int KS>
+__device__ __forceinline__ float lane_group_sum(float v) {
+#pragma unroll
+  for (int o = KS / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
+constexpr int scan_vectors(int mode) { return mode == kScanDelta ? 5 : 2; }  // key-side vectors per token
+
+template <typename T, int MODE, int KS>
+__global__ void __launch_bounds__(kMaxConsumers + kProducers)
+state_scan_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int col_groups) {
+  constexpr int DKP = KS * kRows, NV = scan_vectors(MODE), NCH = (DKP + 31) / 32;
+  extern __shared__ __align__(16) float scan_smem[];
+  const int cols = 2 * col_groups;
+  float* vec = scan_smem;                              // [2][kChunk][NV][DKP]
+  float* val = scan_smem + 2 * kChunk * NV * DKP;      // [2][kChunk][cols]
+  const int n_cons = blockDim.x - kProducers, all = blockDim.x;
+  pdl_wait();
+  const SeqDesc seq = seqs[blockIdx.z];
+  const int h = blockIdx.y, col0 = blockIdx.x * cols;
+  const int n_chunks = (seq.len + kChunk - 1) / kChunk;
+
+  if (static_cast<int>(threadIdx.x) >= n_cons) {
+    // ---------------- producers ----------------
+    const int pw = (threadIdx.x - n_cons) >> 5, lane = threadIdx.x & 31;
+    float wb[NCH], ab[NCH];
+    if (MODE == kScanDelta) {
+#pragma unroll
+      for (int i = 0; i < NCH; ++i) {
+        const int ch = lane + 32 * i;
+        wb[i] = ch < a.DK ? a.w_bias[h * a.DK + ch] : 0.0f;
+        ab[i] = ch < a.DK ? a.a_bias[h * a.DK + ch] : 0.0f;
+      }
+    }
+    const T* proj = static_cast<const T*>(a.proj);
+    for (int c = 0; c < n_chunks; ++c) {
+      const int buf = c & 1;
+      if (c >= 2) buffer_sync<kBarEmpty>(buf, all);
+      const int n = min(kChunk, seq.len - c * kChunk);
+#pragma unroll 2
+      for (int t = pw; t < n; t += kProducers / 32) {
+        const size_t row = static_cast<size_t>(seq.row0) + c * kChunk + t;
+        const T* pr = proj + row * a.ld;
+        float* dst = vec + (buf * kChunk + t) * NV * DKP;
+        float kk[NCH], rr[NCH];
+#pragma unroll
+        for (int i = 0; i < NCH; ++i) {
+          const int ch = lane + 32 * i;
+          const bool in = ch < a.DK;
+          kk[i] = in ? ldf(pr + a.off_k + h * a.DK + ch) : 0.0f;
+          rr[i] = in ? ldf(pr + a.off_q + h * a.DK + ch) : 0.0f;
+        }
+        if (MODE == kScanDelta) {
+          float wz[NCH], az[NCH], ss = 0.0f;
+          const T* wr = static_cast<const T*>(a.wz) + row * a.ld_wz;
+#pragma unroll
+          for (int i = 0; i < NCH; ++i) {
+            const int ch = lane + 32 * i;
+            const bool in = ch < a.DK;
+            wz[i] = in ? ldf(wr + h * a.DK + ch) : 0.0f;
+            az[i] = in ? ldf(pr + a.off_a + h * a.DK + ch) : 0.0f;
+            ss = fmaf(kk[i], kk[i], ss);
+          }
+          const float inv = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
+#pragma unroll
+          for (int i = 0; i < NCH; ++i) {
+            const int ch = lane + 32 * i;
+            if (ch < DKP) {
+              const float u = kk[i] * inv;
+              dst[ch] = u;
+              dst[DKP + ch] = expf(-a.decay_coef * sigmoid_f(wz[i] + wb[i]));
+              dst[2 * DKP + ch] = -sigmoid_f(az[i] + ab[i]) * u;
+              dst[3 * DKP + ch] = kk[i];
+              dst[4 * DKP + ch] = rr[i];
+            }
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < NCH; ++i) {
+            const int ch = lane + 32 * i;
+            if (ch < DKP) {
+              dst[ch] = silu_f(kk[i]);
+              dst[DKP + ch] = silu_f(rr[i]);
+            }
+          }
+        }
+        for (int cc = lane; cc < cols; cc += 32) {
+          float v = col0 + cc < a.DV ? ldf(pr + a.off_v + h * a.DV + col0 + cc) : 0.0f;
+          if (MODE == kScanDecay) v = silu_f(v);
+          val[(buf * kChunk + t) * cols + cc] = v;
+        }
+      }
+      buffer_arrive<kBarFull>(buf, all);
+    }
+    return;
+  }
+
+  // ---------------- consumers ----------------
+  const int ks = threadIdx.x % KS, cg = threadIdx.x / KS;
+  const bool live = cg < col_groups;
+  const int col = col0 + 2 * cg;
+  const bool in0 = live && col < a.DV, in1 = live && col + 1 < a.DV;
+  const bool pair = in1 && (a.DV & 1) == 0;  // the two columns as one 8-byte access
+  float* state = a.state + (static_cast<size_t>(seq.slot) * a.H + h) * a.DK * a.DV;
+  f32x2 S0[kRows / 2], S1[kRows / 2];  // columns col, col + 1; channels 4 (m KS + ks) + {0, 1}, {2, 3}
+#pragma unroll
+  for (int m = 0; m < kRows / 4; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float s[2][2];
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        const int ch = 4 * (m * KS + ks) + 2 * e + f;
+        const bool in = seq.pos > 0 && ch < a.DK;
+        if (pair) {
+          const float2 p = in ? *reinterpret_cast<const float2*>(state + static_cast<size_t>(ch) * a.DV + col) : make_float2(0.0f, 0.0f);
+          s[f][0] = p.x; s[f][1] = p.y;
+        } else {
+          s[f][0] = in && in0 ? state[static_cast<size_t>(ch) * a.DV + col] : 0.0f;
+          s[f][1] = in && in1 ? state[static_cast<size_t>(ch) * a.DV + col + 1] : 0.0f;
+        }
+      }
+      S0[2 * m + e] = pack2(s[0][0], s[1][0]);
+      S1[2 * m + e] = pack2(s[0][1], s[1][1]);
+    }
+  const f32x2 dec2 = MODE == kScanDecay ? pack2(a.decay[h], a.decay[h]) : 0ull;
+  const int vcol = live ? 2 * cg : 0;
+  float* orow = a.o + static_cast<size_t>(seq.row0) * a.ldo + h * a.DV + col;
+  const bool opair = pair && (a.ldo & 1) == 0;
+
+  for (int c = 0; c < n_chunks; ++c) {
+    const int buf = c & 1;
+    buffer_sync<kBarFull>(buf, all);
+    const int n = min(kChunk, seq.len - c * kChunk);
+    const ulonglong2* vp = reinterpret_cast<const ulonglong2*>(vec + buf * kChunk * NV * DKP) + ks;
+    const float* vv = val + buf * kChunk * cols + vcol;
+#pragma unroll 2
+    for (int t = 0; t < n; ++t, vp += NV * DKP / 4, vv += cols) {
+      const float2 v = *reinterpret_cast<const float2*>(vv);
+      const f32x2 v0 = pack2(v.x, v.x), v1 = pack2(v.y, v.y);
+      f32x2 o0 = 0ull, o1 = 0ull;
+      if (MODE == kScanDelta) {
+        f32x2 p0 = 0ull, p1 = 0ull, q0 = 0ull, q1 = 0ull;
+#pragma unroll
+        for (int m = 0; m < kRows / 4; ++m) {
+          const ulonglong2 u = vp[m * KS];
+          p0 = fma2(u.x, S0[2 * m], p0);
+          p1 = fma2(u.x, S1[2 * m], p1);
+          q0 = fma2(u.y, S0[2 * m + 1], q0);
+          q1 = fma2(u.y, S1[2 * m + 1], q1);
+        }
+        const float2 a0 = unpack2(p0), b0 = unpack2(q0), a1 = unpack2(p1), b1 = unpack2(q1);
+        const float s0 = lane_group_sum<KS>((a0.x + a0.y) + (b0.x + b0.y));
+        const float s1 = lane_group_sum<KS>((a1.x + a1.y) + (b1.x + b1.y));
+        const f32x2 x0 = pack2(s0, s0), x1 = pack2(s1, s1);
+#pragma unroll
+        for (int m = 0; m < kRows / 4; ++m) {
+          const ulonglong2 w = vp[DKP / 4 + m * KS], na = vp[2 * DKP / 4 + m * KS], k = vp[3 * DKP / 4 + m * KS],
+                           r = vp[4 * DKP / 4 + m * KS];
+          S0[2 * m] = fma2(w.x, S0[2 * m], fma2(na.x, x0, mul2(k.x, v0)));
+          S1[2 * m] = fma2(w.x, S1[2 * m], fma2(na.x, x1, mul2(k.x, v1)));
+          S0[2 * m + 1] = fma2(w.y, S0[2 * m + 1], fma2(na.y, x0, mul2(k.y, v0)));
+          S1[2 * m + 1] = fma2(w.y, S1[2 * m + 1], fma2(na.y, x1, mul2(k.y, v1)));
+          o0 = fma2(r.y, S0[2 * m + 1], fma2(r.x, S0[2 * m], o0));
+          o1 = fma2(r.y, S1[2 * m + 1], fma2(r.x, S1[2 * m], o1));
+        }
+      } else {
+#pragma unroll
+        for (int m = 0; m < kRows / 4; ++m) {
+          const ulonglong2 k = vp[m * KS], r = vp[DKP / 4 + m * KS];
+          S0[2 * m] = fma2(dec2, S0[2 * m], mul2(k.x, v0));
+          S1[2 * m] = fma2(dec2, S1[2 * m], mul2(k.x, v1));
+          S0[2 * m + 1] = fma2(dec2, S0[2 * m + 1], mul2(k.y, v0));
+          S1[2 * m + 1] = fma2(dec2, S1[2 * m + 1], mul2(k.y, v1));
+          o0 = fma2(r.y, S0[2 * m + 1], fma2(r.x, S0[2 * m], o0));
+          o1 = fma2(r.y, S1[2 * m + 1], fma2(r.x, S1[2 * m], o1));
+        }
+      }
+      const float2 e0 = unpack2(o0), e1 = unpack2(o1);
+      const float y0 = lane_group_sum<KS>(e0.x + e0.y), y1 = lane_group_sum<KS>(e1.x + e1.y);
+      if (ks == 0) {
+        if (opair) {
+          *reinterpret_cast<float2*>(orow) = make_float2(y0, y1);
+        } else {
+          if (in0) orow[0] = y0;
+          if (in1) orow[1] = y1;
+        }
+      }
+      orow += a.ldo;
+    }
+    if (c + 2 < n_chunks) buffer_arrive<kBarEmpty>(buf, all);
+  }
+  pdl_trigger();
+#pragma unroll
+  for (int m = 0; m < kRows / 4; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const float2 s0 = unpack2(S0[2 * m + e]), s1 = unpack2(S1[2 * m + e]);
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        const int ch = 4 * (m * KS + ks) + 2 * e + f;
+        if (ch >= a.DK) continue;
+        float* p = state + static_cast<size_t>(ch) * a.DV + col;
+        const float c0 = f ? s0.y : s0.x, c1 = f ? s1.y : s1.x;
+        if (pair) {
+          *reinterpret_cast<float2*>(p) = make_float2(c0, c1);
+        } else {
+          if (in0) p[0] = c0;
+          if (in1) p[1] = c1;
+        }
+      }
+    }
+}
+
+// ---- group norm with a sigmoid gate behind a matrix-state mixer: one warp or one CTA per (token, group) ----
+template <typename T, bool CTA>
+__global__ void gated_rms_norm_kernel(const float* __restrict__ o, long long ldo, const T* __restrict__ gate, long long ldg,
+                                      const float* __restrict__ w, T* __restrict__ out, long long ldout, int T_rows, int groups,
+                                      int group_size, float eps, float scale) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const int per = CTA ? 1 : blockDim.x >> 5, lanes = CTA ? blockDim.x : 32;
+  const int me = CTA ? threadIdx.x : threadIdx.x & 31;
+  const long long unit = static_cast<long long>(blockIdx.x) * per + (CTA ? 0 : threadIdx.x >> 5);
+  if (unit >= static_cast<long long>(T_rows) * groups) return;
+  const long long row = unit / groups;
+  const int c0 = static_cast<int>(unit % groups) * group_size;
+  const float* src = o + row * ldo + c0;
+  float sq = 0.0f;
+  for (int c = me; c < group_size; c += lanes) sq = fmaf(src[c], src[c], sq);
+  sq = warp_sum(sq);
+  if (CTA) {
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+    __syncthreads();
+    sq = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.0f);
+  }
+  const float rr = scale / sqrtf(sq / static_cast<float>(group_size) + eps);
+  const T* g = gate + row * ldg + c0;
+  T* dst = out + row * ldout + c0;
+  for (int c = me; c < group_size; c += lanes) stf(dst + c, src[c] * rr * w[c0 + c] * sigmoid_f(ldf(g + c)));
+}
+
+// ---- minimal GRU.  The gates read only the current token, so S_t = A_t S_{t-1} + B_t is a scan of affine maps: warp w of
+// a CTA takes TS consecutive tokens of 32 channels, composes their maps, the compositions meet in shared memory, and every
+// warp finishes its own tokens from the state that enters them. ----
+template <typename T, int TS>
+__global__ void min_gru_kernel(const MinGru a, const SeqDesc* __restrict__ seqs) {
+  __shared__ float sA[2][8][32], sB[2][8][32];
+  pdl_wait();
+  pdl_trigger();
+  const SeqDesc seq = seqs[blockIdx.y];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int ch = blockIdx.x * 32 + lane;
+  const bool in = ch < a.W;
+  const float zb = in ? a.z_bias[ch] : 0.0f, xb = in ? a.x_bias[ch] : 0.0f;
+  float* st = a.state + static_cast<size_t>(seq.slot) * a.W + ch;
+  float S = (in && seq.pos > 0) ? *st : 0.0f;
+  const int tile = warps * TS;
+  int par = 0;
+  for (int t0 = 0; t0 < seq.len; t0 += tile, par ^= 1) {
+    const int first = t0 + warp * TS;
+    float A[TS], B[TS];
+    float pa = 1.0f, pb = 0.0f;
+#pragma unroll
+    for (int i = 0; i < TS; ++i) {
+      A[i] = 1.0f;
+      B[i] = 0.0f;
+      if (in && first + i < seq.len) {
+        const T* p = static_cast<const T*>(a.proj) + (static_cast<size_t>(seq.row0) + first + i) * a.ld + ch;
+        const float z = sigmoid_f(ldf(p + a.off_z) + zb), u = ldf(p + a.off_x) + xb;
+        A[i] = 1.0f - z;
+        B[i] = z * (u >= 0.0f ? u + 0.5f : sigmoid_f(u));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TS; ++i) {
+      pa *= A[i];
+      pb = fmaf(A[i], pb, B[i]);
+    }
+    float mine = S;
+    if (warps > 1) {
+      sA[par][warp][lane] = pa;
+      sB[par][warp][lane] = pb;
+      __syncthreads();  // the other parity's buffer is rewritten only behind the next tile's barrier
+      for (int w = 0; w < warps; ++w) {
+        if (w == warp) mine = S;
+        S = fmaf(sA[par][w][lane], S, sB[par][w][lane]);
+      }
+    } else {
+      S = fmaf(pa, S, pb);
+    }
+#pragma unroll
+    for (int i = 0; i < TS; ++i) {
+      if (in && first + i < seq.len) {
+        mine = fmaf(A[i], mine, B[i]);
+        const size_t row = static_cast<size_t>(seq.row0) + first + i;
+        const float g = ldf(static_cast<const T*>(a.proj) + row * a.ld + a.off_g + ch);
+        stf(static_cast<T*>(a.out) + row * a.ldout + ch, mine * silu_f(g) * a.scale);
+      }
+    }
+  }
+  if (in && warp == 0) *st = S;
+}
+
+template <typename T, int MODE, int KS>
+int launch_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool prepare_only, cudaStream_t st) {
+  constexpr int NV = scan_vectors(MODE), DKP = KS * kRows;
+  constexpr int max_groups = kMaxConsumers / KS;
+  static std::atomic<unsigned long long> done{0};  // one bit per device; threads may race to set it
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!(dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull)) {
+    const int most = 2 * kChunk * (NV * DKP + 2 * max_groups) * static_cast<int>(sizeof(float));
+    const cudaError_t e = cudaFuncSetAttribute(state_scan_kernel<T, MODE, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
+  }
+  if (prepare_only) return 0;
+  int groups = (a.DV + 1) / 2;
+  if (groups > max_groups) groups = max_groups;
+  const int threads = (groups * KS + 31) / 32 * 32 + kProducers;
+  const int smem = 2 * kChunk * (NV * DKP + 2 * groups) * static_cast<int>(sizeof(float));
+  const dim3 grid((a.DV + 2 * groups - 1) / (2 * groups), a.H, n_seqs);
+  launch_kernel(state_scan_kernel<T, MODE, KS>, grid, dim3(threads), smem, st, 1, a, seqs, groups);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int MODE>
+int dispatch_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool prep, cudaStream_t st) {
+  if (a.DK <= 16) return launch_scan<T, MODE, 1>(a, seqs, n_seqs, prep, st);
+  if (a.DK <= 32) return launch_scan<T, MODE, 2>(a, seqs, n_seqs, prep, st);
+  if (a.DK <= 64) return launch_scan<T, MODE, 4>(a, seqs, n_seqs, prep, st);
+  if (a.DK <= 128) return launch_scan<T, MODE, 8>(a, seqs, n_seqs, prep, st);
+  return launch_scan<T, MODE, 16>(a, seqs, n_seqs, prep, st);
+}
+
+int scan_any(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool prep, cudaStream_t st) {
+  if (a.mode == kScanDelta)
+    return a.f32 ? dispatch_scan<float, kScanDelta>(a, seqs, n_seqs, prep, st) : dispatch_scan<bf16, kScanDelta>(a, seqs, n_seqs, prep, st);
+  return a.f32 ? dispatch_scan<float, kScanDecay>(a, seqs, n_seqs, prep, st) : dispatch_scan<bf16, kScanDecay>(a, seqs, n_seqs, prep, st);
+}
+
+}  // namespace
+
+bool state_scan_supports(int dk, int dv) { return dk >= 1 && dk <= 256 && dv >= 1; }
+
+// Function attributes of every variant, outside any stream capture.
+int state_scan_prepare() {
+  for (int mode = 0; mode < 2; ++mode)
+    for (int f32 = 0; f32 < 2; ++f32)
+      for (int dk : {16, 32, 64, 128, 256}) {
+        StateScan a{};
+        a.mode = mode; a.f32 = f32; a.DK = dk;
+        const int rc = scan_any(a, nullptr, 0, true, nullptr);
+        if (rc) return rc;
+      }
+  return 0;
+}
+
+int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
+  if (!a.proj || !a.state || !a.o || !seqs || n_seqs <= 0 || n_seqs > 65535 || max_len <= 0 || a.H <= 0 || a.H > 65535 ||
+      !state_scan_supports(a.DK, a.DV))
+    return TEENY_ERR_BAD_ARG;
+  if (a.mode == kScanDelta ? (!a.wz || !a.w_bias || !a.a_bias) : (a.mode != kScanDecay || !a.decay)) return TEENY_ERR_BAD_ARG;
+  return scan_any(a, seqs, n_seqs, false, st);
+}
+
+int gated_rms_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, void* out, long long ldout,
+                   int T, int cols, int group_size, float eps, float scale, bool f32, cudaStream_t st) {
+  if (!o || !gate || !w || !out || T <= 0 || cols <= 0 || group_size <= 0 || cols % group_size) return TEENY_ERR_BAD_ARG;
+  const int groups = cols / group_size;
+  const bool cta = group_size > 512;
+  const long long units = static_cast<long long>(T) * groups;
+  const long long blocks = cta ? units : (units + 7) / 8;
+  if (blocks > 0x7fffffffLL) return TEENY_ERR_BAD_ARG;
+  const dim3 grid(static_cast<unsigned>(blocks)), block(256);
+#define TEENY_GRN(TT, C)                                                                                                     \
+  launch_kernel(gated_rms_norm_kernel<TT, C>, grid, block, 0, st, 1, o, ldo, static_cast<const TT*>(gate), ldg, w,           \
+                static_cast<TT*>(out), ldout, T, groups, group_size, eps, scale)
+  if (f32) { if (cta) TEENY_GRN(float, true); else TEENY_GRN(float, false); }
+  else { if (cta) TEENY_GRN(bf16, true); else TEENY_GRN(bf16, false); }
+#undef TEENY_GRN
+  return static_cast<int>(cudaGetLastError());
+}
+
+int min_gru(const MinGru& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
+  if (!a.proj || !a.z_bias || !a.x_bias || !a.state || !a.out || !seqs || n_seqs <= 0 || n_seqs > 65535 || max_len <= 0 || a.W <= 0)
+    return TEENY_ERR_BAD_ARG;
+  const dim3 grid((a.W + 31) / 32, n_seqs);
+  constexpr int TS = 16;
+  if (max_len == 1) {
+    if (a.f32) launch_kernel(min_gru_kernel<float, 1>, grid, dim3(32), 0, st, 1, a, seqs);
+    else launch_kernel(min_gru_kernel<bf16, 1>, grid, dim3(32), 0, st, 1, a, seqs);
+  } else {
+    int warps = (max_len + TS - 1) / TS;
+    if (warps > 8) warps = 8;
+    if (a.f32) launch_kernel(min_gru_kernel<float, TS>, grid, dim3(32 * warps), 0, st, 1, a, seqs);
+    else launch_kernel(min_gru_kernel<bf16, TS>, grid, dim3(32 * warps), 0, st, 1, a, seqs);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace teeny

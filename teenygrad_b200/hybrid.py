@@ -1,0 +1,376 @@
+"""Hybrid decoder runner: host wrapper over the C++ executor of include/teeny_hybrid.h.
+
+``HybridConfig`` describes a decoder as layers of parallel branches (windowed attention, delta rule, scalar-decay
+state, minimal GRU) and an optional gated feed-forward; a design's own module turns its config.json into one and hands
+the weights over layer by layer (``HybridRunner.load_layer``).  Sequences live in state slots: ``open`` / ``step`` /
+``close`` feed any tokens of any sequences, ``generate`` runs whole prompts and decodes with CUDA-graph replay.
+"""
+import ctypes as C
+from dataclasses import dataclass, field
+
+import torch
+
+from . import _lib
+from ._lib import lib, check, vp, i32, f32, sz
+from .runner import BUF_LOGITS, DecoderRunner, stream
+
+ATTENTION, DELTA, DECAY, MIN_GRU = range(4)
+QK_NORM, KEYS_ARE_VALUES = 1, 2
+ACT_SILU, ACT_GELU_TANH = 1, 2
+
+W_NORM1, W_NORM2, W_IN, W_OUT, W_GATE_UP, W_DOWN = range(6)
+BRANCH_VECTORS = {"q_norm": 50, "k_norm": 51, "o_norm": 52, "decay_bias": 54, "rate_bias": 55, "z_bias": 56, "x_bias": 57,
+                  "decay": 58, "inv_freq": 59}
+W_LOW = 53
+W_EMBED, W_FINAL_NORM, W_LM_HEAD = 100, 101, 102
+BUF_RESIDUAL, BUF_LAST_DELTA = 4, 5
+
+
+class _Cfg(C.Structure):
+    """teeny_hybrid_config"""
+    _fields_ = [(n, i32) for n in ("num_layers", "num_branches", "width", "vocab")] + [("eps", f32), ("embed_scale", f32)] + \
+               [(n, i32) for n in ("f32", "max_batch", "max_len", "max_tokens", "max_rows", "max_new_tokens")]
+
+
+class _Layer(C.Structure):
+    """teeny_hybrid_layer"""
+    _fields_ = [(n, i32) for n in ("first_branch", "num_branches", "ff", "act")]
+
+
+class _Branch(C.Structure):
+    """teeny_hybrid_branch"""
+    _fields_ = [(n, i32) for n in ("kind", "heads", "kv_heads", "dim", "vdim", "rank", "window", "rot_dims", "flags")] + \
+               [(n, f32) for n in ("score_scale", "out_scale", "decay_coef", "unit_eps")]
+
+
+_P = C.POINTER
+_DESC = [_P(_Cfg), _P(_Layer), _P(_Branch)]
+SIGNATURES = {
+    "teeny_hybrid_workspace_bytes": (sz, _DESC),
+    "teeny_hybrid_slot_bytes": (sz, _DESC),
+    "teeny_hybrid_create": (i32, _DESC + [vp, sz, vp, _P(vp)]),
+    "teeny_hybrid_destroy": (None, [vp]),
+    "teeny_hybrid_set_weight": (i32, [vp, i32, i32, i32, vp]),
+    "teeny_hybrid_step": (i32, [vp, vp, _P(i32), _P(i32), _P(i32), i32, _P(i32), i32, vp]),
+    "teeny_hybrid_begin": (i32, [vp, vp]),
+    "teeny_hybrid_decode": (i32, [vp, vp]),
+    "teeny_hybrid_set_sampling": (i32, [vp, f32, i32, f32, C.c_ulonglong]),
+    "teeny_hybrid_capture_decode": (i32, [vp, vp]),
+    "teeny_hybrid_decode_replay": (i32, [vp, vp]),
+    "teeny_hybrid_buffer": (vp, [vp, i32]),
+}
+_lib.bind(SIGNATURES)
+
+
+@dataclass
+class Branch:
+    kind: int
+    dim: int
+    heads: int = 1
+    kv_heads: int = 0
+    vdim: int = 0
+    rank: int = 0
+    window: int = 0
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    flags: int = 0
+    score_scale: float = 1.0
+    out_scale: float = 1.0
+    decay_coef: float = 0.0
+    unit_eps: float = 0.0
+    decay: tuple = ()  # per head, for DECAY
+
+    def input_sizes(self):
+        """Rows of the parts of the fused input projection, in order (include/teeny_hybrid.h)."""
+        n, nv = self.heads * self.dim, self.heads * self.vdim
+        if self.kind == ATTENTION:
+            k = self.kv_heads * self.dim
+            return [n, k] if self.flags & KEYS_ARE_VALUES else [n, k, self.kv_heads * self.vdim]
+        if self.kind == DELTA:
+            return [n] * 5 + [self.rank]
+        if self.kind == DECAY:
+            return [n, n, nv, nv]
+        return [self.dim] * 3
+
+    def output_size(self):
+        return self.dim if self.kind == MIN_GRU else self.heads * self.vdim
+
+
+@dataclass
+class Layer:
+    branches: list
+    ff: int = 0
+    act: int = 0
+
+
+@dataclass
+class HybridConfig:
+    width: int
+    vocab: int
+    eps: float
+    embed_scale: float
+    layers: list = field(default_factory=list)
+
+
+@dataclass
+class Sequence:
+    """A live request: its state slot and how many of its tokens have been run."""
+    slot: int
+    pos: int = 0
+
+
+def pad_to(n, m):
+    return (n + m - 1) // m * m
+
+
+def fuse_rows(parts, dtype):
+    """Matrices stacked with every part starting at a multiple of 8 rows, rows padded to a multiple of 8 columns."""
+    k = parts[0].shape[1]
+    out = torch.zeros(sum(pad_to(p.shape[0], 8) for p in parts), pad_to(k, 8), dtype=dtype)
+    r = 0
+    for p in parts:
+        out[r:r + p.shape[0], :k] = p
+        r += pad_to(p.shape[0], 8)
+    return out
+
+
+def fuse_columns(parts, dtype):
+    """Matrices side by side with every part starting at a multiple of 8 columns."""
+    out = torch.zeros(parts[0].shape[0], sum(pad_to(p.shape[1], 8) for p in parts), dtype=dtype)
+    c = 0
+    for p in parts:
+        out[:, c:c + p.shape[1]] = p
+        c += pad_to(p.shape[1], 8)
+    return out
+
+
+def interleave_glu(gate, up, dtype):
+    """Gate and up rows in alternating blocks of 64, zero rows beyond the feed-forward size; columns padded to 8."""
+    ff, k = gate.shape
+    f = pad_to(ff, 64)
+    both = torch.zeros(2, f, pad_to(k, 8), dtype=dtype)
+    both[0, :ff, :k], both[1, :ff, :k] = gate, up
+    return both.view(2, f // 64, 64, -1).transpose(0, 1).reshape(2 * f, -1).contiguous()
+
+
+def pad_columns(w, multiple, dtype):
+    out = torch.zeros(w.shape[0], pad_to(w.shape[1], multiple), dtype=dtype)
+    out[:, :w.shape[1]] = w
+    return out
+
+
+def plan_steps(entries, max_tokens, max_rows):
+    """Cuts entries (length, wanted places in ascending order) into steps of at most ``max_tokens`` tokens and
+    ``max_rows`` wanted rows: yields lists of (entry, first, count, wanted places in [first, first + count)).  An entry's
+    portions come in order, one per step."""
+    step, tokens, rows = [], 0, 0
+    for e, (n, want) in enumerate(entries):
+        at, w = 0, 0
+        while at < n:
+            if tokens == max_tokens or rows == max_rows or (step and step[-1][0] == e):
+                yield step
+                step, tokens, rows = [], 0, 0
+            count = min(n - at, max_tokens - tokens)
+            here = [p for p in want[w:] if p < at + count]
+            if rows + len(here) > max_rows:  # stop in front of the first place that has no row left
+                here = here[:max_rows - rows]
+                count = want[w + len(here)] - at
+                if count == 0:
+                    yield step
+                    step, tokens, rows = [], 0, 0
+                    continue
+            step.append((e, at, count, here))
+            at, w, tokens, rows = at + count, w + len(here), tokens + count, rows + len(here)
+    if step:
+        yield step
+
+
+class HybridRunner(DecoderRunner):
+    """A hybrid decoder on one GPU; ``dtype`` torch.bfloat16, or torch.float32 for true 32-bit throughout."""
+
+    PREFIX = "teeny_hybrid"
+
+    def __init__(self, cfg, max_batch, max_len, max_tokens=None, max_rows=None, max_new_tokens=256, dtype=torch.bfloat16,
+                 device=None):
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"hybrid decoders run in bfloat16 or float32, not {dtype}")
+        self.cfg, self.dtype, self.max_batch = cfg, dtype, max_batch
+        self.max_tokens = max(max_batch, max_tokens if max_tokens is not None else min(max_batch * max_len, 65536))
+        self.max_rows = max(max_batch, max_rows or 0)
+        branches = [b for layer in cfg.layers for b in layer.branches]
+        c = _Cfg(len(cfg.layers), len(branches), cfg.width, cfg.vocab, cfg.eps, cfg.embed_scale, int(dtype == torch.float32),
+                 max_batch, max_len, self.max_tokens, self.max_rows, max_new_tokens)
+        ls, bs, at = (_Layer * len(cfg.layers))(), (_Branch * len(branches))(), 0
+        for i, layer in enumerate(cfg.layers):
+            ls[i] = _Layer(at, len(layer.branches), layer.ff, layer.act)
+            at += len(layer.branches)
+        for i, b in enumerate(branches):
+            bs[i] = _Branch(b.kind, b.heads, b.kv_heads, b.dim, b.vdim, b.rank, b.window, b.rot_dims, b.flags, b.score_scale,
+                            b.out_scale, b.decay_coef, b.unit_eps)
+        nbytes = lib.teeny_hybrid_workspace_bytes(C.byref(c), ls, bs)
+        if nbytes == 0:
+            raise ValueError("unsupported hybrid decoder configuration for this backend")
+        self.slot_bytes = lib.teeny_hybrid_slot_bytes(C.byref(c), ls, bs)
+        self._init_runner(nbytes, max_len, max_new_tokens, device)
+        self._h = vp()
+        check(lib.teeny_hybrid_create(C.byref(c), ls, bs, C.c_void_p(self.workspace.data_ptr()), nbytes, stream(),
+                                      C.byref(self._h)), "teeny_hybrid_create")
+        self._free = list(range(max_batch))[::-1]
+        self._rows = self._tokens = 0
+
+    # ---- weights ----
+    def _set(self, layer, branch, which, t):
+        self._call("set_weight", self._h, layer, branch, which, self._upload(t))
+
+    def load_layer(self, i, norm1, branches, norm2=None, gate=None, up=None, down=None):
+        """``branches``: per branch a dict with ``inputs`` (matrices in the order of ``Branch.input_sizes``), ``out`` [width,
+        output size], and the vectors (and ``low``) its kind has."""
+        layer = self.cfg.layers[i]
+        if len(branches) != len(layer.branches):
+            raise ValueError(f"layer {i} has {len(layer.branches)} branches, got {len(branches)}")
+        for b, w in zip(layer.branches, branches):
+            got = [tuple(p.shape) for p in w["inputs"]]
+            want = [(n, self.cfg.width) for n in b.input_sizes()]
+            if got != want or tuple(w["out"].shape) != (self.cfg.width, b.output_size()):
+                raise ValueError(f"layer {i}: weight shapes {got}, {tuple(w['out'].shape)}; the configuration says {want}, "
+                                 f"{(self.cfg.width, b.output_size())}")
+        self._set(i, 0, W_NORM1, norm1.float())
+        self._set(i, 0, W_IN, fuse_rows([p for w in branches for p in w["inputs"]], self.dtype))
+        self._set(i, 0, W_OUT, fuse_columns([w["out"] for w in branches], self.dtype))
+        for j, (b, w) in enumerate(zip(layer.branches, branches)):
+            for name, which in BRANCH_VECTORS.items():
+                if name in w:
+                    self._set(i, j, which, w[name].float())
+            if "low" in w:
+                self._set(i, j, W_LOW, pad_columns(w["low"], 8, self.dtype))
+            if b.kind == DECAY:
+                self._set(i, j, BRANCH_VECTORS["decay"], torch.tensor(b.decay, dtype=torch.float64).float())
+            if b.kind == ATTENTION and b.rot_dims:
+                e = torch.arange(b.rot_dims // 2, dtype=torch.float64) * (-2.0 / b.rot_dims)
+                self._set(i, j, BRANCH_VECTORS["inv_freq"], (float(b.rot_base) ** e).float())
+        if layer.ff:
+            self._set(i, 0, W_NORM2, norm2.float())
+            self._set(i, 0, W_GATE_UP, interleave_glu(gate, up, self.dtype))
+            self._set(i, 0, W_DOWN, pad_columns(down, 64, self.dtype))
+
+    def load_head(self, embed, final_norm, lm_head):
+        self._set(0, 0, W_EMBED, embed.to(self.dtype))
+        self._set(0, 0, W_FINAL_NORM, final_norm.float())
+        self._set(0, 0, W_LM_HEAD, pad_columns(lm_head, 8, self.dtype))
+
+    # ---- sequences ----
+    def open(self):
+        if not self._free:
+            raise RuntimeError(f"all {self.max_batch} state slots are in use")
+        return Sequence(self._free.pop())
+
+    def close(self, seq):
+        """Gives the slot back; its next sequence starts at position 0, which ignores what the slot holds."""
+        if seq.slot in self._free:
+            raise ValueError("the sequence is closed already")
+        self._free.append(seq.slot)
+
+    def _run(self, ids, seqs, lens, rows):
+        """One step of the C runner: ``ids`` device int32, entry i = the next lens[i] tokens of seqs[i]."""
+        n = len(seqs)
+        arr = lambda v: (i32 * max(len(v), 1))(*v)  # noqa: E731
+        self._call("step", self._h, C.c_void_p(ids.data_ptr()), arr([s.slot for s in seqs]), arr([s.pos for s in seqs]), arr(lens),
+                   n, arr(rows), len(rows), stream())
+        self.batch = 0
+        self._rows, self._tokens = len(rows), int(sum(lens))
+        for s, c in zip(seqs, lens):
+            s.pos += c
+
+    def _check_ids(self, ids):
+        if ids.numel() and (int(ids.min()) < 0 or int(ids.max()) >= self.cfg.vocab):
+            raise ValueError("token id outside the vocabulary")
+        return ids
+
+    def step(self, entries):
+        """``entries``: (sequence, token ids, wanted places among them in ascending order).  Runs the tokens from the state
+        earlier steps left; returns the wanted places' logits, float32 [wanted, vocab] per entry, on the device."""
+        toks = [self._check_ids(torch.as_tensor(t, dtype=torch.int32).reshape(-1)) for _, t, _ in entries]
+        for s, t in zip((e[0] for e in entries), toks):
+            if t.numel() == 0 or s.pos + t.numel() > self.max_len:
+                raise ValueError(f"{t.numel()} tokens at position {s.pos}: the runner was created with max_len={self.max_len}")
+        out = [[] for _ in entries]
+        for portion in plan_steps([(t.numel(), list(w)) for t, (_, _, w) in zip(toks, entries)], self.max_tokens, self.max_rows):
+            ids = torch.cat([toks[e][at:at + c] for e, at, c, _ in portion]).to(self.device)
+            rows, row0 = [], 0
+            for e, at, c, want in portion:
+                rows += [row0 + p - at for p in want]
+                row0 += c
+            self._run(ids, [entries[e][0] for e, _, _, _ in portion], [c for _, _, c, _ in portion], rows)
+            if rows:
+                got, r = self.logits().float(), 0
+                for e, _, _, want in portion:
+                    out[e].append(got[r:r + len(want)])
+                    r += len(want)
+        empty = torch.empty(0, self.cfg.vocab, device=self.device)
+        return [torch.cat(o) if o else empty for o in out]
+
+    # ---- buffers ----
+    def logits(self):
+        """Element type [rows, vocab]: logits of the last step's wanted rows (of every sequence after a decode step)."""
+        ld = pad_to(self.cfg.vocab, 8)
+        return self._view(BUF_LOGITS, (self.batch or self._rows, ld), self.dtype)[:, :self.cfg.vocab]
+
+    def residual_stream(self):
+        """float32 [tokens, width]: the residual stream after the last layer of the last step."""
+        n, ld = self.batch or self._tokens, pad_to(self.cfg.width, 8)
+        return self._view(BUF_RESIDUAL, (n, self.cfg.width), torch.float32) + \
+            self._view(BUF_LAST_DELTA, (n, ld), self.dtype)[:, :self.cfg.width].float()
+
+    # ---- generation ----
+    def prefill(self, prompts, seqs):
+        """Runs the prompts (int [B, S] or a list of unequal ones) into ``seqs`` and picks every first token."""
+        B = len(seqs)
+        if isinstance(prompts, torch.Tensor):
+            rows = prompts.to(torch.int32)
+            lens = [rows.shape[1]] * B
+        else:
+            rows = [torch.as_tensor(p, dtype=torch.int32).reshape(-1) for p in prompts]
+            lens = [int(r.numel()) for r in rows]
+        # the last step holds an equal share of every prompt's end, so that all first tokens are picked together
+        tail = [min(n, self.max_tokens // B) for n in lens]
+        head = [n - t for n, t in zip(lens, tail)]
+        if any(head):
+            self.step([(s, r[:h], []) for s, r, h in zip(seqs, rows, head) if h])
+        if isinstance(rows, torch.Tensor):
+            ids = rows[:, head[0]:].to(self.device, non_blocking=True).contiguous().view(-1)
+        else:
+            ids = torch.cat([r[h:] for r, h in zip(rows, head)]).to(self.device)
+        ends = torch.tensor(tail).cumsum(0) - 1
+        before = self.batch
+        self._run(ids, seqs, tail, ends.tolist())
+        self._call("begin", self._h, stream())
+        self.batch = before
+        self._set_batch(B)
+
+    def _generate_group(self, prompts, max_new_tokens, use_graph):
+        seqs = [self.open() for _ in range(len(prompts))]
+        try:
+            self.prefill(prompts, seqs)
+            return self._decode_loop(max_new_tokens, use_graph)
+        finally:
+            for s in seqs[::-1]:
+                self.close(s)
+
+    def generate(self, prompts, max_new_tokens, use_graph=True):
+        """``prompts``: int [B, S], or a list of prompts of any lengths.  Returns int32 [B, max_new_tokens] on the device.
+        More prompts than state slots run in groups."""
+        lens = [prompts.shape[1]] * len(prompts) if isinstance(prompts, torch.Tensor) else [len(p) for p in prompts]
+        if max_new_tokens > self.max_new_tokens:
+            raise ValueError("max_new_tokens exceeds the runner's history capacity")
+        if not lens or min(lens) == 0 or max(lens) + max_new_tokens - 1 > self.max_len:
+            raise ValueError(f"prompts of {lens} tokens + {max_new_tokens} new ones; the runner was created with max_len={self.max_len}")
+        if not (isinstance(prompts, torch.Tensor) and prompts.is_cuda):  # device-resident ids are clamped by the kernel
+            for p in prompts:
+                self._check_ids(torch.as_tensor(p))
+        room = len(self._free)
+        if not room:
+            raise RuntimeError(f"all {self.max_batch} state slots are in use")
+        groups = [prompts[i:i + room] for i in range(0, len(lens), room)]
+        if len(groups) == 1:
+            return self._generate_group(prompts, max_new_tokens, use_graph)
+        return torch.cat([self._generate_group(g, max_new_tokens, use_graph).clone() for g in groups])

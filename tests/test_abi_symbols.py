@@ -32,11 +32,8 @@ def test_every_declared_symbol_is_exported_and_bound(lib):
     for name in declared:
         assert hasattr(lib.lib, name), f"{name} declared in include/ but not exported"
     bound = set(lib.SIGNATURES)
-    try:
-        from teenygrad_b200 import qwen3
-        bound |= set(getattr(qwen3, "SIGNATURES", {}))
-    except ImportError:
-        pass
+    from teenygrad_b200 import hybrid, qwen3
+    bound |= set(qwen3.SIGNATURES) | set(hybrid.SIGNATURES)
     assert set(declared) <= bound, sorted(set(declared) - bound)
 
 
