@@ -14,6 +14,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "mma.cuh"
 
 namespace teeny {
 
@@ -21,19 +22,6 @@ namespace {
 
 constexpr int kDecChunk = 512;
 constexpr int kHD = 128;
-
-__device__ __forceinline__ void mma_bf16_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
-                                               uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 
 // ---- decode kernel: TMA-fed shared-memory ring + mma.sync ----
 // CTA = one (batch, kv head, share of the live keys).  Warp 4 is the producer: for every 64-key tile it requests the
@@ -74,15 +62,6 @@ constexpr int kDecBox = kDecTile * 64 * 2;       // 8 KB: [64 keys][64 d]
 constexpr int kDecStageBytes = 4 * kDecBox;      // K (2 boxes) + V (2 boxes) = 32 KB
 constexpr int dec_smem_bytes(int stages) { return stages * kDecStageBytes + 1024 + 128; }
 constexpr int kDecThreads = 160;                 // 4 consumer warps + 1 producer warp
-
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
 
 template <int G>
 __global__ void __launch_bounds__(kDecThreads, 2)

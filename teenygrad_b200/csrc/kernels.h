@@ -249,6 +249,10 @@ struct StateScan {
 int state_scan_prepare();
 int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
 bool state_scan_supports(int dk, int dv);
+// The same over prompts on the tensor cores (state_scan chooses it).
+bool chunk_scan_supports(const StateScan& a, int max_len);
+int chunk_scan_prepare();
+int chunk_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, cudaStream_t st);
 // out[t, c] = o[t, c] / rms(group of c) * w[c] * sigmoid(gate[t, c]) * scale; groups of group_size consecutive columns
 int gated_rms_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, void* out, long long ldout,
                    int T, int cols, int group_size, float eps, float scale, bool f32, cudaStream_t st);

@@ -428,7 +428,7 @@ int state_scan_prepare() {
         const int rc = scan_any(a, nullptr, 0, true, nullptr);
         if (rc) return rc;
       }
-  return 0;
+  return chunk_scan_prepare();
 }
 
 int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
@@ -436,6 +436,8 @@ int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len,
       !state_scan_supports(a.DK, a.DV))
     return TEENY_ERR_BAD_ARG;
   if (a.mode == kScanDelta ? (!a.wz || !a.w_bias || !a.a_bias) : (a.mode != kScanDecay || !a.decay)) return TEENY_ERR_BAD_ARG;
+  // prompts in bf16: 16 tokens at a time on the tensor cores; single tokens and f32: token by token
+  if (chunk_scan_supports(a, max_len)) return chunk_scan(a, seqs, n_seqs, st);
   return scan_any(a, seqs, n_seqs, false, st);
 }
 

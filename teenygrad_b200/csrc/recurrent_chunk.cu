@@ -1,0 +1,481 @@
+// Matrix-state recurrences over a prompt, 16 tokens at a time on the tensor cores (bf16 activations).
+//
+// Delta rule.  With L_t the running sum of log w over a chunk and W_t = exp(L_t) (per key channel), S_t = diag(W_t) X_t
+// turns the recurrence into rank-one updates without a decay:
+//   p_t = u_t^T S_{t-1} = U_t X_0 + sum_{s<t} (U_t . Ka_s) p_s + (U_t . Kk_s) v_s      U_t = W_{t-1} o u_t
+//   o_t = r_t^T S_t     = R_t X_0 + sum_{s<=t} (R_t . Ka_s) p_s + (R_t . Kk_s) v_s     R_t = W_t o r_t
+//   S_16 = diag(W_16) (X_0 + sum_s Ka_s p_s + Kk_s v_s)                                Ka_s = -a_s u_s / W_s, Kk_s = k_s / W_s
+// so a chunk is four 16 x 16 matrices, one triangular inverse T = (1 - U Ka^T)^{-1} and products with the state.
+// Scalar decay.  o_t = d^{t+1} q_t^T S_0 + sum_{s<=t} d^{t-s} (q_t . k_s) v_s, S_n = d^n S_0 + sum_s d^{n-1-s} k_s v_s; no
+// division by a power of d, however small d is.
+//
+// 32-bit accuracy from bf16 tensor cores: every f32 operand goes in as hi + lo (2^-17), a product as hi hi + hi lo +
+// lo hi with f32 accumulation; the carried state itself is never rounded (f32 accumulators from chunk to chunk).
+//
+// One CTA per (head, sequence).  Warps 0 .. n-1, the consumers, own 16 value columns each and keep S^T [16, DK] as C
+// fragments: those are, packed, the A operand of S^T U^T and S^T R^T, whose results (P^T, O^T) are in turn the A operand
+// and the layout of the update, so the chain never leaves the registers.  The last four warps, the producers, build the
+// B operands of the next chunk in the other shared-memory buffer.  Buffers change hands through named barriers.
+#include <atomic>
+
+#include "common.cuh"
+#include "kernels.h"
+#include "mma.cuh"
+
+namespace teeny {
+
+namespace {
+
+constexpr int kC = 16;          // tokens per chunk
+constexpr int kProducers = 128;
+constexpr int kMatLd = 24;      // row stride of the 16 x 16 matrices (48 bytes: conflict-free ldmatrix)
+constexpr int kMaxDV = 192;     // 12 consumer warps
+constexpr int kBarFull = 1, kBarEmpty = 3, kBarProducers = 5;
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+
+template <int FIRST>
+__device__ __forceinline__ void buffer_sync(int buf, int nthreads) {
+  if (buf == 0) asm volatile("bar.sync %0, %1;" ::"n"(FIRST), "r"(nthreads) : "memory");
+  else asm volatile("bar.sync %0, %1;" ::"n"(FIRST + 1), "r"(nthreads) : "memory");
+}
+template <int FIRST>
+__device__ __forceinline__ void buffer_arrive(int buf, int nthreads) {
+  if (buf == 0) asm volatile("bar.arrive %0, %1;" ::"n"(FIRST), "r"(nthreads) : "memory");
+  else asm volatile("bar.arrive %0, %1;" ::"n"(FIRST + 1), "r"(nthreads) : "memory");
+}
+__device__ __forceinline__ void producers_sync() {
+  asm volatile("bar.sync %0, %1;" ::"n"(kBarProducers), "n"(kProducers) : "memory");
+}
+
+// Shared memory of one buffer, byte offsets.  Delta: rows are U, R, Ka, Kk; decay: q, R, k, Kk (q and k without powers of d
+// are the producers' own).  Each as hi then lo, [16][DKP + 8] bf16.
+template <int DKP>
+struct Lay {
+  static constexpr int kLd = DKP + 8;
+  static constexpr int kTile = kC * kLd * 2;
+  static constexpr int tile(int which, int lo) { return (2 * which + lo) * kTile; }
+  static constexpr int kMats = 8 * kTile;                      // T, A2, B1, B2: hi, lo [16][24] bf16 each
+  static constexpr int mat(int which, int lo) { return kMats + (2 * which + lo) * kC * kMatLd * 2; }
+  static constexpr int kScale = kMats + 8 * kC * kMatLd * 2;   // f32 [DKP]: decay of the chunk per key channel
+  static constexpr int kV = kScale + DKP * 4;                  // V hi, then lo: [16][DVP + 8] bf16
+  static __host__ __device__ constexpr int bytes(int dvp) { return kV + 2 * kC * (dvp + 8) * 2; }
+};
+constexpr int kU = 0, kR = 1, kKa = 2, kKk = 3;
+constexpr int kT = 0, kA2 = 1, kB1 = 2, kB2 = 3;
+
+// two neighbouring elements of a bf16 row; vec: the pair is 4-byte aligned
+__device__ __forceinline__ float2 ld_pair(const bf16* p, int i, int n, bool vec) {
+  if (vec) {
+    if (i >= n) return make_float2(0.0f, 0.0f);
+    const uint32_t v = *reinterpret_cast<const uint32_t*>(p + i);
+    return make_float2(bf16_lo(v), bf16_hi(v));
+  }
+  return make_float2(i < n ? __bfloat162float(p[i]) : 0.0f, i + 1 < n ? __bfloat162float(p[i + 1]) : 0.0f);
+}
+
+__device__ __forceinline__ void st_split(uint8_t* tile_hi, uint8_t* tile_lo, int byte_off, float x, float y) {
+  uint32_t hi, lo;
+  split_bf16x2(x, y, hi, lo);
+  *reinterpret_cast<uint32_t*>(tile_hi + byte_off) = hi;
+  *reinterpret_cast<uint32_t*>(tile_lo + byte_off) = lo;
+}
+
+// acc[2][4] (16 rows x 16 columns) += A B^T for row tiles A, B [16][LD] given as hi / lo, over NK 16-deep steps.
+template <int NK, int LD>
+__device__ __forceinline__ void rows_product(float (&acc)[2][4], uint32_t a_hi, uint32_t a_lo, uint32_t b_hi, uint32_t b_lo, int lane) {
+  const uint32_t ao = static_cast<uint32_t>(((lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8) * 2;
+  const uint32_t bo = static_cast<uint32_t>(((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+  for (int k = 0; k < NK; ++k) {
+    uint32_t ah[4], al[4], bh[4], bl[4];
+    ldsm_x4(ah, a_hi + ao + k * 32);
+    ldsm_x4(al, a_lo + ao + k * 32);
+    ldsm_x4(bh, b_hi + bo + k * 32);
+    ldsm_x4(bl, b_lo + bo + k * 32);
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      mma_bf16_16816(acc[n], ah[0], ah[1], ah[2], ah[3], bh[2 * n], bh[2 * n + 1]);
+      mma_bf16_16816(acc[n], ah[0], ah[1], ah[2], ah[3], bl[2 * n], bl[2 * n + 1]);
+      mma_bf16_16816(acc[n], al[0], al[1], al[2], al[3], bh[2 * n], bh[2 * n + 1]);
+    }
+  }
+}
+
+// acc += A B for an A fragment given as hi / lo and a 16 x 16 matrix stored [n][k] as hi / lo.
+__device__ __forceinline__ void frag_mat(float (&acc)[2][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], bool has_lo,
+                                         uint32_t m_hi, uint32_t m_lo, uint32_t bo) {
+  uint32_t bh[4], bl[4];
+  ldsm_x4(bh, m_hi + bo);
+  ldsm_x4(bl, m_lo + bo);
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    mma_bf16_16816(acc[n], ah[0], ah[1], ah[2], ah[3], bh[2 * n], bh[2 * n + 1]);
+    mma_bf16_16816(acc[n], ah[0], ah[1], ah[2], ah[3], bl[2 * n], bl[2 * n + 1]);
+    if (has_lo) mma_bf16_16816(acc[n], al[0], al[1], al[2], al[3], bh[2 * n], bh[2 * n + 1]);
+  }
+}
+
+__device__ __forceinline__ void split_frag(const float (&x)[4], const float (&y)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+  split_bf16x2(x[0], x[1], hi[0], lo[0]);
+  split_bf16x2(x[2], x[3], hi[1], lo[1]);
+  split_bf16x2(y[0], y[1], hi[2], lo[2]);
+  split_bf16x2(y[2], y[3], hi[3], lo[3]);
+}
+
+template <int MODE, int NK>
+__global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int dvp) {
+  constexpr int DKP = 16 * NK, NP = DKP / 64, LD = DKP + 8;
+  constexpr bool DELTA = MODE == kScanDelta;
+  using L = Lay<DKP>;
+  extern __shared__ __align__(128) uint8_t chunk_smem[];
+  __shared__ float sh_tot[4][DKP];        // producers: log-decay sums of each warp's four tokens
+  __shared__ float sh_a1[kC][kC + 1];     // producers: U Ka^T, strictly lower
+  __shared__ float sh_pow[kC + 1];
+  const int buf_bytes = L::bytes(dvp), ldv = dvp + 8;
+  const int n_cons = blockDim.x - kProducers, all = blockDim.x;
+  const int lane = threadIdx.x & 31;
+  pdl_wait();
+  const SeqDesc seq = seqs[blockIdx.y];
+  const int h = blockIdx.x;
+  const int n_chunks = (seq.len + kC - 1) / kC;
+  if (!DELTA) {  // powers of the head's decay
+    if (threadIdx.x <= kC) sh_pow[threadIdx.x] = powf(a.decay[h], static_cast<float>(threadIdx.x));
+    __syncthreads();
+  }
+
+  if (static_cast<int>(threadIdx.x) >= n_cons) {
+    // ---------------- producers: warp pw takes tokens 4 pw .. 4 pw + 3 of a chunk, a lane NP channel pairs ----------------
+    const int pw = (threadIdx.x - n_cons) >> 5;
+    const bf16* proj = static_cast<const bf16*>(a.proj);
+    const bf16* wzp = static_cast<const bf16*>(a.wz);
+    const int hk = h * a.DK, hv = h * a.DV;
+    const bool vec = ((a.DK | a.off_q | a.off_k | a.off_a) & 1) == 0 && (a.ld & 1) == 0 && (!DELTA || (a.ld_wz & 1) == 0);
+    const bool vecv = ((a.DV | a.off_v) & 1) == 0 && (a.ld & 1) == 0;
+    float2 wb[NP], ab[NP];
+    if (DELTA) {
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int c = 2 * lane + 64 * i;
+        wb[i] = make_float2(c < a.DK ? a.w_bias[hk + c] : 0.0f, c + 1 < a.DK ? a.w_bias[hk + c + 1] : 0.0f);
+        ab[i] = make_float2(c < a.DK ? a.a_bias[hk + c] : 0.0f, c + 1 < a.DK ? a.a_bias[hk + c + 1] : 0.0f);
+      }
+    }
+    float2 kk[4][NP], rr[4][NP], wz[4][NP], az[4][NP];
+    auto fetch = [&](int c) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int t = c * kC + 4 * pw + j;
+        const bool in = t < seq.len;
+        const size_t row = static_cast<size_t>(seq.row0) + (in ? t : 0);
+        const bf16* pr = proj + row * a.ld;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int ch = 2 * lane + 64 * i, n = in ? a.DK : 0;
+          kk[j][i] = ld_pair(pr + a.off_k + hk, ch, n, vec);
+          rr[j][i] = ld_pair(pr + a.off_q + hk, ch, n, vec);
+          if (DELTA) {
+            wz[j][i] = ld_pair(wzp + row * a.ld_wz + hk, ch, n, vec);
+            az[j][i] = ld_pair(pr + a.off_a + hk, ch, n, vec);
+          }
+        }
+      }
+    };
+    if (n_chunks > 0) fetch(0);
+    for (int c = 0; c < n_chunks; ++c) {
+      const int buf = c & 1, n = min(kC, seq.len - c * kC);
+      uint8_t* sb = chunk_smem + buf * buf_bytes;
+      const uint32_t sa = smem_u32(sb);
+      if (c >= 2) buffer_sync<kBarEmpty>(buf, all);
+      // V: copied (delta) or silu, split (decay)
+      for (int j = 0; j < 4; ++j) {
+        const int t = 4 * pw + j;
+        const bool in = t < n;
+        const bf16* pr = proj + (static_cast<size_t>(seq.row0) + c * kC + (in ? t : 0)) * a.ld + a.off_v + hv;
+        uint8_t* v_hi = sb + L::kV + t * ldv * 2;
+        for (int x = 2 * lane; x < dvp; x += 64) {
+          const float2 v = ld_pair(pr, x, in ? a.DV : 0, vecv);
+          if (DELTA) *reinterpret_cast<uint32_t*>(v_hi + 2 * x) = pack_bf16x2(v.x, v.y);
+          else st_split(v_hi, v_hi + kC * ldv * 2, 2 * x, silu_f(v.x), silu_f(v.y));
+        }
+      }
+      if (DELTA) {
+        float2 lw[4][NP];
+        float inv[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const bool in = 4 * pw + j < n;
+          float ss = 0.0f;
+#pragma unroll
+          for (int i = 0; i < NP; ++i) {
+            ss = fmaf(kk[j][i].x, kk[j][i].x, fmaf(kk[j][i].y, kk[j][i].y, ss));
+            lw[j][i] = in ? make_float2(-a.decay_coef * sigmoid_f(wz[j][i].x + wb[i].x), -a.decay_coef * sigmoid_f(wz[j][i].y + wb[i].y))
+                          : make_float2(0.0f, 0.0f);
+            if (j > 0) { lw[j][i].x += lw[j - 1][i].x; lw[j][i].y += lw[j - 1][i].y; }
+            az[j][i] = make_float2(sigmoid_f(az[j][i].x + ab[i].x), sigmoid_f(az[j][i].y + ab[i].y));
+          }
+          inv[j] = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
+        }
+#pragma unroll
+        for (int i = 0; i < NP; ++i) *reinterpret_cast<float2*>(&sh_tot[pw][2 * lane + 64 * i]) = lw[3][i];
+        producers_sync();
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int ch = 2 * lane + 64 * i;
+          float2 base = make_float2(0.0f, 0.0f);
+#pragma unroll
+          for (int q = 0; q < 3; ++q)
+            if (q < pw) { base.x += sh_tot[q][ch]; base.y += sh_tot[q][ch + 1]; }
+          float2 prev = make_float2(expf(base.x), expf(base.y));  // W_{t-1}
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float2 l = make_float2(base.x + lw[j][i].x, base.y + lw[j][i].y);
+            const float2 W = make_float2(expf(l.x), expf(l.y)), iW = make_float2(expf(-l.x), expf(-l.y));
+            const float2 k = kk[j][i], r = rr[j][i], al = az[j][i];
+            const float2 u = make_float2(k.x * inv[j], k.y * inv[j]);
+            const int off = ((4 * pw + j) * LD + ch) * 2;
+            st_split(sb + L::tile(kU, 0), sb + L::tile(kU, 1), off, prev.x * u.x, prev.y * u.y);
+            st_split(sb + L::tile(kR, 0), sb + L::tile(kR, 1), off, W.x * r.x, W.y * r.y);
+            st_split(sb + L::tile(kKa, 0), sb + L::tile(kKa, 1), off, -al.x * u.x * iW.x, -al.y * u.y * iW.y);
+            st_split(sb + L::tile(kKk, 0), sb + L::tile(kKk, 1), off, k.x * iW.x, k.y * iW.y);
+            prev = W;
+          }
+          if (pw == 3) *reinterpret_cast<float2*>(sb + L::kScale + ch * 4) = prev;
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int t = 4 * pw + j;
+          const float dr = sh_pow[t + 1], dk = t < n ? sh_pow[n - 1 - t] : 0.0f;
+#pragma unroll
+          for (int i = 0; i < NP; ++i) {
+            const float2 q = make_float2(silu_f(rr[j][i].x), silu_f(rr[j][i].y)), k = make_float2(silu_f(kk[j][i].x), silu_f(kk[j][i].y));
+            const int off = (t * LD + 2 * lane + 64 * i) * 2;
+            st_split(sb + L::tile(kU, 0), sb + L::tile(kU, 1), off, q.x, q.y);
+            st_split(sb + L::tile(kR, 0), sb + L::tile(kR, 1), off, q.x * dr, q.y * dr);
+            st_split(sb + L::tile(kKa, 0), sb + L::tile(kKa, 1), off, k.x, k.y);
+            st_split(sb + L::tile(kKk, 0), sb + L::tile(kKk, 1), off, k.x * dk, k.y * dk);
+          }
+        }
+      }
+      if (c + 1 < n_chunks) fetch(c + 1);  // in flight while the matrices are built
+      producers_sync();
+      // the 16 x 16 matrices: warp 0 U Ka^T (and its inverse), 1 U Kk^T, 2 R Ka^T, 3 R Kk^T; decay: warp 3 q k^T alone
+      const int g = lane >> 2, cc = lane & 3;
+      if (DELTA || pw == 3) {
+        float acc[2][4] = {};
+        const int ta = DELTA ? (pw < 2 ? kU : kR) : kU, tb = DELTA ? ((pw & 1) ? kKk : kKa) : kKa;
+        rows_product<NK, LD>(acc, sa + L::tile(ta, 0), sa + L::tile(ta, 1), sa + L::tile(tb, 0), sa + L::tile(tb, 1), lane);
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int t = g + 8 * half, s = 8 * nb + 2 * cc;
+            float x = acc[nb][2 * half], y = acc[nb][2 * half + 1];
+            const int reach = DELTA && pw < 2 ? t - 1 : t;  // largest s that contributes
+            if (!DELTA) {
+              x *= sh_pow[s <= t ? t - s : 0];
+              y *= sh_pow[s + 1 <= t ? t - s - 1 : 0];
+            }
+            x = s <= reach ? x : 0.0f;
+            y = s + 1 <= reach ? y : 0.0f;
+            if (DELTA && pw == 0) {
+              sh_a1[t][s] = x;
+              sh_a1[t][s + 1] = y;
+            } else {
+              const int m = DELTA ? (pw == 1 ? kA2 : (pw == 2 ? kB1 : kB2)) : kB2;
+              st_split(sb + L::mat(m, 0), sb + L::mat(m, 1), (t * kMatLd + s) * 2, x, y);
+            }
+          }
+        if (DELTA && pw == 0) {
+          __syncwarp();
+          // column (lane % 16) of the inverse of a unit lower triangular matrix, row by row
+          const int col = lane & 15;
+          float T[kC];
+#pragma unroll
+          for (int t = 0; t < kC; ++t) {
+            float v = t == col ? 1.0f : 0.0f, v2 = 0.0f;
+#pragma unroll
+            for (int s = 0; s < t; ++s) {
+              if (s & 1) v2 = fmaf(sh_a1[t][s], T[s], v2);
+              else v = fmaf(sh_a1[t][s], T[s], v);
+            }
+            T[t] = v + v2;
+          }
+#pragma unroll
+          for (int t = 0; t < kC; ++t) {
+            const bf16 hi = __float2bfloat16_rn(T[t]);
+            bf16* dst = reinterpret_cast<bf16*>(sb + L::mat(kT, lane < 16 ? 0 : 1)) + t * kMatLd + col;
+            *dst = lane < 16 ? hi : __float2bfloat16_rn(T[t] - __bfloat162float(hi));
+          }
+        }
+      }
+      buffer_arrive<kBarFull>(buf, all);
+    }
+    return;
+  }
+
+  // ---------------- consumers ----------------
+  const int g = lane >> 2, cc = lane & 3;
+  const int v0 = (threadIdx.x >> 5) * 16;
+  float S[2 * NK][4];  // S^T: value columns v0 + g, v0 + g + 8; key channels 8 j + 2 cc, + 1
+  float* state = a.state + (static_cast<size_t>(seq.slot) * a.H + h) * a.DK * a.DV;
+#pragma unroll
+  for (int j = 0; j < 2 * NK; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int ch = 8 * j + 2 * cc + (e & 1), v = v0 + g + 8 * (e >> 1);
+      S[j][e] = seq.pos > 0 && ch < a.DK && v < a.DV ? state[static_cast<size_t>(ch) * a.DV + v] : 0.0f;
+    }
+  const uint32_t row_b = static_cast<uint32_t>((lane & 7) + (lane >> 4) * 8), col_b = static_cast<uint32_t>((lane >> 3) & 1) * 8;
+  const uint32_t bo = (row_b * LD + col_b) * 2, mo = (row_b * kMatLd + col_b) * 2;
+  const uint32_t row_t = static_cast<uint32_t>((lane & 7) + ((lane >> 3) & 1) * 8);
+  const uint32_t to = (row_t * LD + static_cast<uint32_t>(lane >> 4) * 8) * 2;
+  const uint32_t vo = (row_b * static_cast<uint32_t>(ldv) + v0 + col_b) * 2;
+
+  for (int c = 0; c < n_chunks; ++c) {
+    const int buf = c & 1, n = min(kC, seq.len - c * kC);
+    const uint32_t sa = smem_u32(chunk_smem) + buf * buf_bytes;
+    const float* scale = reinterpret_cast<const float*>(chunk_smem + buf * buf_bytes + L::kScale);
+    buffer_sync<kBarFull>(buf, all);
+    float O[2][4] = {}, P[2][4] = {}, O2[2][4] = {}, P2[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < NK; ++k) {
+      uint32_t sh[4], sl[4], bh[4], bl[4];
+      split_frag(S[2 * k], S[2 * k + 1], sh, sl);
+      if (DELTA) {
+        ldsm_x4(bh, sa + L::tile(kU, 0) + bo + k * 32);
+        ldsm_x4(bl, sa + L::tile(kU, 1) + bo + k * 32);
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb) {
+          mma_bf16_16816(P[nb], sh[0], sh[1], sh[2], sh[3], bh[2 * nb], bh[2 * nb + 1]);
+          mma_bf16_16816(P2[nb], sh[0], sh[1], sh[2], sh[3], bl[2 * nb], bl[2 * nb + 1]);
+          mma_bf16_16816(P2[nb], sl[0], sl[1], sl[2], sl[3], bh[2 * nb], bh[2 * nb + 1]);
+        }
+      }
+      ldsm_x4(bh, sa + L::tile(kR, 0) + bo + k * 32);
+      ldsm_x4(bl, sa + L::tile(kR, 1) + bo + k * 32);
+#pragma unroll
+      for (int nb = 0; nb < 2; ++nb) {
+        mma_bf16_16816(O[nb], sh[0], sh[1], sh[2], sh[3], bh[2 * nb], bh[2 * nb + 1]);
+        mma_bf16_16816(O2[nb], sh[0], sh[1], sh[2], sh[3], bl[2 * nb], bl[2 * nb + 1]);
+        mma_bf16_16816(O2[nb], sl[0], sl[1], sl[2], sl[3], bh[2 * nb], bh[2 * nb + 1]);
+      }
+    }
+    uint32_t vh[4], vl[4] = {};
+    ldsm_x4_trans(vh, sa + L::kV + vo);
+    uint32_t ph[4], pl[4];
+    if (DELTA) {
+      frag_mat(P, vh, vl, false, sa + L::mat(kA2, 0), sa + L::mat(kA2, 1), mo);
+#pragma unroll
+      for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) P[nb][e] += P2[nb][e];
+      split_frag(P[0], P[1], ph, pl);
+      float Q[2][4] = {};
+      frag_mat(Q, ph, pl, true, sa + L::mat(kT, 0), sa + L::mat(kT, 1), mo);
+      split_frag(Q[0], Q[1], ph, pl);
+      frag_mat(O, ph, pl, true, sa + L::mat(kB1, 0), sa + L::mat(kB1, 1), mo);
+    } else {
+      ldsm_x4_trans(vl, sa + L::kV + kC * ldv * 2 + vo);
+    }
+    frag_mat(O2, vh, vl, !DELTA, sa + L::mat(kB2, 0), sa + L::mat(kB2, 1), mo);
+    // ---- output: token 8 nb + 2 cc + (e & 1), value column v0 + g + 8 (e >> 1) ----
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = 8 * nb + 2 * cc + (e & 1), v = v0 + g + 8 * (e >> 1);
+        if (t < n && v < a.DV)
+          a.o[(static_cast<size_t>(seq.row0) + c * kC + t) * a.ldo + h * a.DV + v] = O[nb][e] + O2[nb][e];
+      }
+    // ---- state ----
+    const float dn = DELTA ? 1.0f : sh_pow[n];
+#pragma unroll
+    for (int j = 0; j < 2 * NK; j += 2) {
+      uint32_t kh[4], kl[4];
+      if (DELTA) {
+        ldsm_x4_trans(kh, sa + L::tile(kKa, 0) + to + j * 16);
+        ldsm_x4_trans(kl, sa + L::tile(kKa, 1) + to + j * 16);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          mma_bf16_16816(S[j + e], ph[0], ph[1], ph[2], ph[3], kh[2 * e], kh[2 * e + 1]);
+          mma_bf16_16816(S[j + e], ph[0], ph[1], ph[2], ph[3], kl[2 * e], kl[2 * e + 1]);
+          mma_bf16_16816(S[j + e], pl[0], pl[1], pl[2], pl[3], kh[2 * e], kh[2 * e + 1]);
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int f = 0; f < 4; ++f) S[j + e][f] *= dn;
+      }
+      ldsm_x4_trans(kh, sa + L::tile(kKk, 0) + to + j * 16);
+      ldsm_x4_trans(kl, sa + L::tile(kKk, 1) + to + j * 16);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        mma_bf16_16816(S[j + e], vh[0], vh[1], vh[2], vh[3], kh[2 * e], kh[2 * e + 1]);
+        mma_bf16_16816(S[j + e], vh[0], vh[1], vh[2], vh[3], kl[2 * e], kl[2 * e + 1]);
+        if (!DELTA) mma_bf16_16816(S[j + e], vl[0], vl[1], vl[2], vl[3], kh[2 * e], kh[2 * e + 1]);
+      }
+      if (DELTA) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float2 w = *reinterpret_cast<const float2*>(scale + 8 * (j + e) + 2 * cc);
+          S[j + e][0] *= w.x; S[j + e][1] *= w.y; S[j + e][2] *= w.x; S[j + e][3] *= w.y;
+        }
+      }
+    }
+    if (c + 2 < n_chunks) buffer_arrive<kBarEmpty>(buf, all);
+  }
+  pdl_trigger();
+#pragma unroll
+  for (int j = 0; j < 2 * NK; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int ch = 8 * j + 2 * cc + (e & 1), v = v0 + g + 8 * (e >> 1);
+      if (ch < a.DK && v < a.DV) state[static_cast<size_t>(ch) * a.DV + v] = S[j][e];
+    }
+}
+
+template <int MODE, int NK>
+int launch_chunk(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool prepare_only, cudaStream_t st) {
+  static std::atomic<unsigned long long> done{0};  // one bit per device; threads may race to set it
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!(dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull)) {
+    const cudaError_t e = cudaFuncSetAttribute(chunk_scan_kernel<MODE, NK>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               2 * Lay<16 * NK>::bytes(kMaxDV));
+    if (e != cudaSuccess) return static_cast<int>(e);
+    if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
+  }
+  if (prepare_only) return 0;
+  const int dvp = (a.DV + 15) / 16 * 16;
+  launch_kernel(chunk_scan_kernel<MODE, NK>, dim3(a.H, n_seqs), dim3(dvp * 2 + kProducers), 2 * Lay<16 * NK>::bytes(dvp), st, 1, a, seqs,
+                dvp);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace
+
+bool chunk_scan_supports(const StateScan& a, int max_len) {
+  // 1 / W_t must stay far from overflow within a chunk
+  return !a.f32 && max_len >= kC && a.DK <= 128 && a.DV <= kMaxDV && (a.mode != kScanDelta || a.decay_coef * kC <= 40.0f);
+}
+
+int chunk_scan_prepare() {
+  StateScan a{};
+  int rc = launch_chunk<kScanDelta, 4>(a, nullptr, 0, true, nullptr);
+  if (!rc) rc = launch_chunk<kScanDelta, 8>(a, nullptr, 0, true, nullptr);
+  if (!rc) rc = launch_chunk<kScanDecay, 4>(a, nullptr, 0, true, nullptr);
+  if (!rc) rc = launch_chunk<kScanDecay, 8>(a, nullptr, 0, true, nullptr);
+  return rc;
+}
+
+int chunk_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, cudaStream_t st) {
+  if (a.mode == kScanDelta)
+    return a.DK <= 64 ? launch_chunk<kScanDelta, 4>(a, seqs, n_seqs, false, st) : launch_chunk<kScanDelta, 8>(a, seqs, n_seqs, false, st);
+  return a.DK <= 64 ? launch_chunk<kScanDecay, 4>(a, seqs, n_seqs, false, st) : launch_chunk<kScanDecay, 8>(a, seqs, n_seqs, false, st);
+}
+
+}  // namespace teeny
