@@ -21,7 +21,7 @@ namespace teeny {
 namespace {
 
 constexpr int kDecChunk = 512;
-constexpr int kHD = 128;
+constexpr int kHD = 128;  // head size of the combine kernel and of the fused front end
 
 // ---- decode kernel: TMA-fed shared-memory ring + mma.sync ----
 // CTA = one (batch, kv head, share of the live keys).  Warp 4 is the producer: for every 64-key tile it requests the
@@ -51,6 +51,9 @@ struct DecodeArgs {
   unsigned* counters;  // [B * Hkv] arrival counters (zero between calls) for the in-kernel merge, or null
   float scale_log2;
   int* err;
+  const SeqDesc* seqs;  // ring caches: per-sequence slot and position (kv_len / kv_len_dev unused), ring rows
+  int ring;
+  float out_scale;
   DecodeRope rope;  // rope.k_new == nullptr: q is final and the caches already hold the new rows
   long long kc_sb, kc_sh, kc_ss, vc_sb, vc_sh, vc_ss;  // cache strides for the append
 };
@@ -59,18 +62,19 @@ constexpr int kDecTile = 64;                     // keys per ring stage
 constexpr int kDecStagesShared = 3;  // ring depth when two CTAs share an SM
 constexpr int kDecStagesAlone = 6;   // ring depth when the grid has at most one CTA per SM
 constexpr int kDecBox = kDecTile * 64 * 2;       // 8 KB: [64 keys][64 d]
-constexpr int kDecStageBytes = 4 * kDecBox;      // K (2 boxes) + V (2 boxes) = 32 KB
-constexpr int dec_smem_bytes(int stages) { return stages * kDecStageBytes + 1024 + 128; }
+constexpr int dec_stage_bytes(int hd) { return 2 * (hd / 64) * kDecBox; }  // K and V boxes: 32 KB for head size 128
+constexpr int dec_smem_bytes(int stages, int hd) { return stages * dec_stage_bytes(hd) + 1024 + 128; }
 constexpr int kDecThreads = 160;                 // 4 consumer warps + 1 producer warp
 
-template <int G>
+template <int G, int HD>
 __global__ void __launch_bounds__(kDecThreads, 2)
 attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                         const DecodeArgs a) {
   extern __shared__ uint8_t dec_smem_raw[];
   __shared__ float sm_ml[4][8][2];
-  __shared__ float sm_o[4][G][kHD];
-  __shared__ __align__(16) bf16 sm_q[4][G][kHD];  // normed, rotated q heads, one copy per consumer warp (fused front end)
+  constexpr int kDecStageBytes = dec_stage_bytes(HD), kVTile = (HD / 64) * kDecBox;
+  __shared__ float sm_o[4][G][HD];
+  __shared__ __align__(16) bf16 sm_q[4][G][HD];  // normed, rotated q heads, one copy per consumer warp (fused front end)
   const uint32_t base = (smem_u32(dec_smem_raw) + 1023u) & ~1023u;
   uint8_t* gen = dec_smem_raw + (base - smem_u32(dec_smem_raw));
   const int n_stages = a.stages;
@@ -91,8 +95,17 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
   __syncthreads();
   // the live keys are divided evenly (in whole 64-key tiles) over the gridDim.x CTAs of this (batch, kv head)
   int L = 0, span = 0, key_begin = 0, key_end = 0, n_tiles = 0;
+  int cb = b, newest = 0;  // row of the cache tensors; cache row of the newest key
   auto plan = [&]() {
-    L = a.kv_len_dev ? *a.kv_len_dev : a.kv_len;
+    if (a.seqs) {
+      const SeqDesc sq = a.seqs[b];
+      cb = sq.slot;
+      L = min(sq.pos + 1, a.ring);
+      newest = sq.pos % a.ring;
+    } else {
+      L = a.kv_len_dev ? *a.kv_len_dev : a.kv_len;
+      newest = L - 1;
+    }
     span = ((L + static_cast<int>(gridDim.x) - 1) / static_cast<int>(gridDim.x) + kDecTile - 1) / kDecTile * kDecTile;
     key_begin = chunk * span;
     key_end = min(L, key_begin + span);
@@ -102,10 +115,11 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     const uint32_t dst = base + st * kDecStageBytes;
     const int key0 = key_begin + t * kDecTile;
     mbar_expect_tx(full_bar(st), kDecStageBytes);
-    tma_load_4d(dst, &tmap_k, full_bar(st), 0, key0, hk, b);
-    tma_load_4d(dst + kDecBox, &tmap_k, full_bar(st), 64, key0, hk, b);
-    tma_load_4d(dst + 2 * kDecBox, &tmap_v, full_bar(st), 0, key0, hk, b);
-    tma_load_4d(dst + 3 * kDecBox, &tmap_v, full_bar(st), 64, key0, hk, b);
+#pragma unroll
+    for (int x = 0; x < HD / 64; ++x) {
+      tma_load_4d(dst + x * kDecBox, &tmap_k, full_bar(st), 64 * x, key0, hk, cb);
+      tma_load_4d(dst + kVTile + x * kDecBox, &tmap_v, full_bar(st), 64 * x, key0, hk, cb);
+    }
   };
   int pre = 0;  // tiles requested ahead of the wait (producer thread only)
   int rope_pos = 0;
@@ -114,7 +128,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     if (a.rope.k_new) rope_pos = a.rope.pos_dev ? *a.rope.pos_dev : a.rope.pos;
     if (threadIdx.x == 128) {
       // first ring of tiles that hold none of the rows the previous kernel is still writing
-      while (pre < n_tiles && pre < n_stages && key_begin + (pre + 1) * kDecTile <= L - a.fresh_rows) {
+      // (the fresh rows end at the newest key; in a ring older rows may follow it)
+      while (pre < n_tiles && pre < n_stages &&
+             (key_begin + (pre + 1) * kDecTile <= newest + 1 - a.fresh_rows || key_begin + pre * kDecTile > newest)) {
         load_tile(pre, pre);
         ++pre;
       }
@@ -126,14 +142,14 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     if (a.rope.k_new) rope_pos = a.rope.pos_dev ? *a.rope.pos_dev : a.rope.pos;
   }
   const int g = lane >> 2, c = lane & 3;
-  float acc[16][4];
+  float acc[HD / 8][4];
   float m = -INFINITY, l = 0.0f;
   if (n_tiles == 0) return;  // chunk lies beyond the live length (uniform for the CTA)
 
   // Fused front end (per-head RMSNorm + RoPE + cache append), one 128-wide head per half-warp.  No CTA-wide barrier:
   // the producer warp norms / rotates the new key, appends it and the new value to the caches and goes on streaming;
   // every consumer warp prepares its own copy of the G query heads.
-  const bool fused = a.rope.k_new != nullptr;
+  const bool fused = HD == kHD && a.rope.k_new != nullptr;
   const int sub = lane & 15, hw = lane >> 4;
   auto rope_head = [&](const bf16* src, const bf16* w, uint4& raw) {
     raw = *reinterpret_cast<const uint4*>(src + sub * 8);
@@ -173,9 +189,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
   } else {
     // ---------------- consumers: warp w owns keys [16 w, 16 w + 16) of every tile ----------------
 #pragma unroll
-    for (int i = 0; i < 16; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    for (int i = 0; i < HD / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
     // Q fragments: head hk * G + g; a0 = d 16 ks + 2c.., a2 = d 16 ks + 8 + 2c..; rows >= G are zero
-    uint32_t qa[8][2];
+    uint32_t qa[HD / 16][2];
     {
       if (fused) {
 #pragma unroll
@@ -189,7 +205,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       }
       const bf16* qp = fused ? &sm_q[warp][g < G ? g : 0][0] : a.q + b * a.q_sb + (hk * G + (g < G ? g : 0)) * a.q_sh;
 #pragma unroll
-      for (int ks = 0; ks < 8; ++ks) {
+      for (int ks = 0; ks < HD / 16; ++ks) {
         const uint32_t lo = *reinterpret_cast<const uint32_t*>(qp + 16 * ks + 2 * c);
         const uint32_t hi = *reinterpret_cast<const uint32_t*>(qp + 16 * ks + 8 + 2 * c);
         qa[ks][0] = g < G ? lo : 0u;
@@ -203,15 +219,15 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     uint32_t ph = 0;
     for (int t = 0; t < n_tiles; ++t, st = (st + 1 == n_stages ? 0 : st + 1), ph ^= (st == 0 ? 1u : 0u)) {
       if (!mbar_wait(full_bar(st), ph, a.err, DEVERR_ATTN_SOFTMAX)) { ok = false; break; }
-      const uint32_t kt = base + st * kDecStageBytes, vt = kt + 2 * kDecBox;
+      const uint32_t kt = base + st * kDecStageBytes, vt = kt + kVTile;
       const int kb = key_begin + t * kDecTile + 16 * warp;  // first key of this warp's slice
       if (kb < key_end) {
         if (kb + 16 > key_end) {
           // rows past the live length hold whatever the cache had (possibly NaN patterns): their probabilities are
           // zero, but 0 * NaN is NaN inside the MMA, so clear those V rows first
-          uint8_t* vrow = gen + st * kDecStageBytes + 2 * kDecBox;
-          for (int i = lane; i < 256; i += 32) {
-            const int r = i >> 4, ch = i & 15;
+          uint8_t* vrow = gen + st * kDecStageBytes + kVTile;
+          for (int i = lane; i < 2 * HD; i += 32) {
+            const int r = i / (HD / 8), ch = i % (HD / 8);
             if (kb + r >= key_end)
               *reinterpret_cast<uint4*>(vrow + (ch >> 3) * kDecBox + (16 * warp + r) * 128 + (ch & 7) * 16) =
                   make_uint4(0, 0, 0, 0);
@@ -225,7 +241,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
           s[nb][0] = s[nb][1] = s[nb][2] = s[nb][3] = 0.0f;
           const int row = row_k + 8 * nb;
 #pragma unroll
-          for (int p = 0; p < 4; ++p) {  // 32 d per ldmatrix.x4: matrices = four 8-d chunks
+          for (int p = 0; p < HD / 32; ++p) {  // 32 d per ldmatrix.x4: matrices = four 8-d chunks
             uint32_t kf[4];
             ldsm_x4(kf, kt + (p >> 1) * kDecBox + row * 128 + ((((p & 1) * 4 + mat) ^ (row & 7)) << 4));
             mma_bf16_16816(s[nb], qa[2 * p][0], 0u, qa[2 * p][1], 0u, kf[0], kf[1]);
@@ -259,7 +275,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
         psum += __shfl_xor_sync(0xffffffffu, psum, 2);
         l = l * alpha + psum;
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
+        for (int i = 0; i < HD / 8; ++i) {
           acc[i][0] *= alpha;
           acc[i][1] *= alpha;
         }
@@ -268,7 +284,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
         // ---- O += P V: ldmatrix.trans yields (key pair, d) fragments; one x4 covers two 8-wide d blocks ----
         const int row_v = 16 * warp + (mat & 1) * 8 + (lane & 7);
 #pragma unroll
-        for (int nbp = 0; nbp < 8; ++nbp) {
+        for (int nbp = 0; nbp < HD / 16; ++nbp) {
           const int chunk16 = 2 * nbp + (mat >> 1);  // 8-d chunk index 0..15
           uint32_t vf[4];
           ldsm_x4_trans(vf, vt + (chunk16 >> 3) * kDecBox + row_v * 128 + (((chunk16 & 7) ^ (row_v & 7)) << 4));
@@ -291,7 +307,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     }
     if (g < G) {
 #pragma unroll
-      for (int nb = 0; nb < 16; ++nb) {
+      for (int nb = 0; nb < HD / 8; ++nb) {
         sm_o[warp][g][8 * nb + 2 * c] = acc[nb][0];
         sm_o[warp][g][8 * nb + 2 * c + 1] = acc[nb][1];
       }
@@ -299,8 +315,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
   }
   __syncthreads();
   const size_t slot = (static_cast<size_t>(b) * a.Hkv + hk) * a.max_chunks + chunk;
-  for (int idx = threadIdx.x; idx < G * kHD; idx += kDecThreads) {
-    const int gg = idx / kHD, d = idx - gg * kHD;
+  for (int idx = threadIdx.x; idx < G * HD; idx += kDecThreads) {
+    const int gg = idx / HD, d = idx - gg * HD;
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sm_ml[w][gg][0]);  // warps without keys hold -inf
@@ -313,10 +329,10 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       oo += sm_o[w][gg][d] * sc;
     }
     if (gridDim.x == 1) {  // whole sequence in this CTA: finish here, no partials
-      a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo / ll);
+      a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo / ll * a.out_scale);
       continue;
     }
-    a.part_o[(slot * G + gg) * kHD + d] = oo;
+    a.part_o[(slot * G + gg) * HD + d] = oo;
     if (d == 0) {
       a.part_ml[(slot * G + gg) * 2 + 0] = mm;
       a.part_ml[(slot * G + gg) * 2 + 1] = ll;
@@ -338,8 +354,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     if (sm_last) {
       __threadfence();
       const size_t slot0 = (static_cast<size_t>(b) * a.Hkv + hk) * a.max_chunks;
-      for (int idx = threadIdx.x; idx < G * kHD; idx += kDecThreads) {
-        const int gg = idx / kHD, d = idx - gg * kHD;
+      for (int idx = threadIdx.x; idx < G * HD; idx += kDecThreads) {
+        const int gg = idx / HD, d = idx - gg * HD;
         float mm = -INFINITY;
         for (int ch = 0; ch < chunks; ++ch) mm = fmaxf(mm, __ldcg(a.part_ml + ((slot0 + ch) * G + gg) * 2));
         float ll = 0.0f, oo = 0.0f;
@@ -347,9 +363,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
           const size_t sl = (slot0 + ch) * G + gg;
           const float sc = ex2(__ldcg(a.part_ml + sl * 2) - mm);
           ll += __ldcg(a.part_ml + sl * 2 + 1) * sc;
-          oo += __ldcg(a.part_o + sl * kHD + d) * sc;
+          oo += __ldcg(a.part_o + sl * HD + d) * sc;
         }
-        a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo / ll);
+        a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo / ll * a.out_scale);
       }
     }
   }
@@ -450,10 +466,15 @@ int attention_decode_prepare() {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull) return 0;
-  cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, dec_smem_bytes(kDecStagesAlone));
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_decode_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, dec_smem_bytes(kDecStagesAlone));
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_decode_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, dec_smem_bytes(kDecStagesAlone));
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_decode_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, dec_smem_bytes(kDecStagesAlone));
+  cudaError_t e = cudaSuccess;
+  auto raise = [&](auto kernel, int hd) {
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, dec_smem_bytes(kDecStagesAlone, hd));
+  };
+  raise(attention_decode_kernel<1, 128>, 128); raise(attention_decode_kernel<2, 128>, 128);
+  raise(attention_decode_kernel<4, 128>, 128); raise(attention_decode_kernel<8, 128>, 128);
+  raise(attention_decode_kernel<1, 64>, 64); raise(attention_decode_kernel<2, 64>, 64);
+  raise(attention_decode_kernel<4, 64>, 64); raise(attention_decode_kernel<8, 64>, 64);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
   return 0;
@@ -467,10 +488,11 @@ size_t attention_decode_scratch_bytes(int B, int Hq, int D, int max_kv) {
 
 int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, const AttnShape& s, int kv_len,
                           const int* kv_len_dev, void* scratch, size_t scratch_bytes, cudaStream_t stream,
-                          int fresh_rows, const DecodeRope* rope, unsigned* counters) {
+                          int fresh_rows, const DecodeRope* rope, unsigned* counters, const DecodeRing* ring) {
   if (!q || !k || !v || !o || !scratch || s.B <= 0 || s.Hq <= 0 || s.Hkv <= 0 || s.Skv <= 0) return TEENY_ERR_BAD_ARG;
-  if (s.D != kHD || s.Hq % s.Hkv != 0 || s.Sq != 1) return TEENY_ERR_BAD_ARG;
-  if (!kv_len_dev && (kv_len <= 0 || kv_len > s.Skv)) return TEENY_ERR_BAD_ARG;
+  if ((s.D != kHD && !(s.D == 64 && ring)) || s.Hq % s.Hkv != 0 || s.Sq != 1) return TEENY_ERR_BAD_ARG;
+  if (ring && (!ring->seqs || ring->slots <= 0 || rope || !counters)) return TEENY_ERR_BAD_ARG;
+  if (!ring && !kv_len_dev && (kv_len <= 0 || kv_len > s.Skv)) return TEENY_ERR_BAD_ARG;
   const int G = s.Hq / s.Hkv;
   if (G != 1 && G != 2 && G != 4 && G != 8) return TEENY_ERR_BAD_ARG;
   const long long strides[] = {s.q_sb, s.q_sh, s.k_sb, s.k_sh, s.k_ss, s.v_sb, s.v_sh, s.v_ss};
@@ -486,7 +508,8 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
   // K and V caches as 4-D tensors (d, key, kv head, batch); a tile is two [64 keys][64 d] boxes
   CUtensorMap mk, mv;
   {
-    const uint64_t dims[4] = {kHD, static_cast<uint64_t>(s.Skv), static_cast<uint64_t>(s.Hkv), static_cast<uint64_t>(s.B)};
+    const uint64_t dims[4] = {static_cast<uint64_t>(s.D), static_cast<uint64_t>(s.Skv), static_cast<uint64_t>(s.Hkv),
+                              static_cast<uint64_t>(ring ? ring->slots : s.B)};
     const uint32_t box[4] = {64, kDecTile, 1, 1};
     auto nz = [](long long st, long long fb) { return static_cast<uint64_t>(st > 0 ? st : fb) * 2; };
     const uint64_t ks[3] = {static_cast<uint64_t>(s.k_ss) * 2, nz(s.k_sh, s.k_ss), nz(s.k_sb, s.k_ss)};
@@ -503,12 +526,15 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
   DecodeArgs a{};
   a.q = q;
   a.part_o = static_cast<float*>(scratch);
-  a.part_ml = a.part_o + static_cast<size_t>(s.B) * s.Hq * max_chunks * kHD;
+  a.part_ml = a.part_o + static_cast<size_t>(s.B) * s.Hq * max_chunks * s.D;
   a.q_sb = s.q_sb; a.q_sh = s.q_sh;
   a.o = o; a.o_sb = s.o_sb; a.o_sh = s.o_sh;
   a.Hkv = s.Hkv; a.G = G; a.max_chunks = max_chunks;
   a.kv_len = kv_len; a.kv_len_dev = kv_len_dev;
   a.fresh_rows = fresh_rows;
+  a.seqs = ring ? ring->seqs : nullptr;
+  a.ring = s.Skv;
+  a.out_scale = s.out_scale;
   if (rope) {
     if (!rope->k_new || !rope->v_new || !rope->k_cache || !rope->v_cache || !rope->q_w || !rope->k_w || !rope->cos_t ||
         !rope->sin_t || rope->max_len <= 0)
@@ -539,14 +565,18 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
     if (n_split < 1) n_split = 1;
   }
   a.counters = n_split > 1 ? counters : nullptr;
-  const int smem = dec_smem_bytes(a.stages);
+  const int smem = dec_smem_bytes(a.stages, s.D);
   dim3 grid(n_split, s.Hkv, s.B);
+#define TEENY_DEC(GG)                                                                                                     \
+  if (s.D == 64) launch_kernel(attention_decode_kernel<GG, 64>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a);      \
+  else launch_kernel(attention_decode_kernel<GG, 128>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a)
   switch (G) {
-    case 1: launch_kernel(attention_decode_kernel<1>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a); break;
-    case 2: launch_kernel(attention_decode_kernel<2>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a); break;
-    case 4: launch_kernel(attention_decode_kernel<4>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a); break;
-    default: launch_kernel(attention_decode_kernel<8>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a); break;
+    case 1: TEENY_DEC(1); break;
+    case 2: TEENY_DEC(2); break;
+    case 4: TEENY_DEC(4); break;
+    default: TEENY_DEC(8); break;
   }
+#undef TEENY_DEC
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
   if (n_split == 1 || a.counters) return 0;

@@ -77,6 +77,8 @@ struct PrefillArgs {  // (Q, K, V and O travel as tensor maps)
   int B, Hq, Hkv, Sq, Skv;
   float scale_log2;
   int causal;
+  int window;        // > 0: query i sees only the last `window` keys up to its own (causal only)
+  float out_scale;
   int n_pair_tiles;  // 256-row query tiles per (batch, head)
   int n_items;       // n_pair_tiles * Hq * B work items; CTA pair p takes items p, p + pairs, ...
   int* err;
@@ -196,7 +198,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
   const int pair_id = static_cast<int>(blockIdx.x >> 1), n_pairs = static_cast<int>(gridDim.x >> 1);
   const int off = args.Skv - args.Sq;                           // causal: query i sees keys <= i + off
   const int heads_x_batch = args.Hq * args.B;
-  struct Item { int pt, h, b, hk, n_tiles; };
+  struct Item { int pt, h, b, hk, t0, n_tiles; };  // t0: first key tile
   auto item_at = [&](int item) {
     Item it;
     it.pt = args.n_pair_tiles - 1 - item / heads_x_batch;
@@ -206,7 +208,9 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
     it.hk = it.h / (args.Hq / args.Hkv);
     int kv_end = args.Skv;
     if (args.causal) kv_end = min(args.Skv, it.pt * 2 * kQT + 2 * kQT + off);   // of the pair's last row
-    it.n_tiles = (kv_end + kKT - 1) / kKT;  // >= 1 (host guarantees Skv >= Sq >= 1 when causal)
+    // the window of the pair's first row begins here; tiles before it are no row's
+    it.t0 = args.window > 0 ? max(0, it.pt * 2 * kQT + off - args.window + 1) / kKT : 0;
+    it.n_tiles = (kv_end + kKT - 1) / kKT - it.t0;  // >= 1 (host guarantees Skv >= Sq >= 1 when causal)
     return it;
   };
 
@@ -252,7 +256,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
           if (!mbar_wait(bar(K_EMPTY + st), ph ^ 1, err, DEVERR_ATTN_PRODUCER)) { ok = false; break; }
           if (leader) mbar_expect_tx(bar(K_FULL + st), 2 * kHalfBytes);  // both CTAs' halves
           const uint32_t dst = base + kSmemK + st * kHalfBytes;
-          const int key0 = j * kKT + static_cast<int>(rank) * 64;
+          const int key0 = (it.t0 + j) * kKT + static_cast<int>(rank) * 64;
           tma_load_4d_pair(dst, &tmap_k, bar(K_FULL + st), 0, key0, it.hk, it.b);
           tma_load_4d_pair(dst + kKBoxBytes, &tmap_k, bar(K_FULL + st), 64, key0, it.hk, it.b);
         }
@@ -268,7 +272,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
           const uint32_t ph = (g / kKV) & 1;
           if (!mbar_wait(bar(V_EMPTY + st), ph ^ 1, err, DEVERR_ATTN_PRODUCER)) { ok = false; break; }
           if (leader) mbar_expect_tx(bar(V_FULL + st), 2 * kHalfBytes);
-          tma_load_4d_pair(base + kSmemV + st * kHalfBytes, &tmap_v, bar(V_FULL + st), static_cast<int>(rank) * 64, j * kKT,
+          tma_load_4d_pair(base + kSmemV + st * kHalfBytes, &tmap_v, bar(V_FULL + st), static_cast<int>(rank) * 64, (it.t0 + j) * kKT,
                            it.hk, it.b);
         }
       }
@@ -455,13 +459,15 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         }
         tc_fence_before();
         mbar_arrive_cluster(s_empty_leader);  // the buffer can take QK^T of tile g + 2 (once the peer's group is here too)
-        const int k0 = j * kKT;
-        const bool need_mask = (k0 + kKT > args.Skv) || (args.causal && (k0 + kKT - 1 > q0 + off));
+        const int k0 = (it.t0 + j) * kKT;
+        const int first = args.window > 0 ? qi + off - args.window + 1 : 0;  // first visible key
+        const bool need_mask = (k0 + kKT > args.Skv) || (args.causal && (k0 + kKT - 1 > q0 + off)) ||
+                               (args.window > 0 && k0 < q0 + kQT + off - args.window);
         if (need_mask) {
           const int limit = args.causal ? min(args.Skv - 1, qi + off) : args.Skv - 1;  // last visible key
 #pragma unroll
           for (int e = 0; e < 128; ++e)
-            if (k0 + e > limit) s[e] = -INFINITY;
+            if (k0 + e > limit || k0 + e < first) s[e] = -INFINITY;
         }
         // row maximum: four independent chains of three-input maxima
         float tm[4] = {s[0], s[1], s[2], s[3]};
@@ -480,7 +486,9 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         // ---- the running maximum: tile j's decision follows tile j-1's (made by the other group) ----
         float m;
         if (j == 0) {
-          m = tmax;  // key 0 is visible to every row, so m is finite from here on
+          // finite from here on: without a window key 0 is visible to every row; with one a row may see nothing of the
+          // first tiles, and its (zero) sums are then scaled away with the first key it sees
+          m = fmaxf(tmax, -1e30f);
         } else {
           if (!mbar_wait(bar(m_ready + (wg ^ 1)), (m_seen + ((j - 1 - j_other) >> 1)) & 1, err, DEVERR_ATTN_SOFTMAX)) { ok = false; break; }
           m = m_sh[r];
@@ -575,6 +583,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
           tc_fence_after();
           float inv;
           asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(inv) : "f"(l));  // l >= 1 (the row's maximum contributes 2^0); 1 ulp
+          inv *= args.out_scale;
           const float2 inv2 = {inv, inv};
           const bool valid = qi < args.Sq;
           uint32_t t[4][32];  // the whole row in flight, so that the accumulator is free for the next item at once
@@ -675,6 +684,7 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   if (!q || !k || !v || !o || s.B <= 0 || s.Hq <= 0 || s.Hkv <= 0 || s.Sq <= 0 || s.Skv <= 0) return TEENY_ERR_BAD_ARG;
   if (s.D != kHD || s.Hq % s.Hkv != 0) return TEENY_ERR_BAD_ARG;
   if (s.causal && s.Skv < s.Sq) return TEENY_ERR_BAD_ARG;
+  if (s.window < 0 || (s.window > 0 && !s.causal)) return TEENY_ERR_BAD_ARG;
   const long long strides[] = {s.q_sb, s.q_sh, s.q_ss, s.k_sb, s.k_sh, s.k_ss, s.v_sb, s.v_sh, s.v_ss, s.o_ss, s.o_sh, s.o_sb};
   for (long long st : strides)
     if (st % 8 != 0) return TEENY_ERR_ALIGNMENT;
@@ -695,6 +705,8 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   a.lse = lse; a.B = s.B; a.Hq = s.Hq; a.Hkv = s.Hkv; a.Sq = s.Sq; a.Skv = s.Skv;
   a.scale_log2 = s.scale * 1.4426950408889634f;
   a.causal = s.causal;
+  a.window = s.window;
+  a.out_scale = s.out_scale;
   a.err = device_error_word();
   if (!a.err) return TEENY_ERR_DRIVER;  // kernels report expired waits through this word: no launch without it
 

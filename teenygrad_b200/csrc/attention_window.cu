@@ -4,12 +4,17 @@
 // ring and its own tokens' keys from the step's activations, and leaves its last `ring` keys in the ring afterwards,
 // so portions may be cut anywhere and a long prompt never overwrites a key that one of its own queries still needs.
 //
-// window_attention_rows_kernel<T>: one warp per (token, query head), any head size up to 256, f32 or bf16 storage, f32
-// arithmetic.
+// window_attention chooses among
+//   attention_prefill_bf16   whole prompts of one length, head size 128 (tcgen05 on CTA pairs, attention_prefill.cu)
+//   attention_decode_bf16    single tokens, head size 64 or 128 (TMA-streamed ring, attention_decode.cu)
+//   window_attention_mma_kernel   any other bf16 step, head sizes up to 256 in multiples of 8 (mma.sync tiles, cp.async rows
+//                            from ring and step): portions, unequal prompts, other head sizes
+//   window_attention_rows_kernel<T>   anything, f32 included: one or eight warps per (token, query head)
 #include <atomic>
 
 #include "common.cuh"
 #include "kernels.h"
+#include "mma.cuh"
 
 namespace teeny {
 
@@ -44,11 +49,16 @@ __global__ void head_norm_rope_rows_kernel(const HeadNormRope a, const SeqDesc* 
     const int hd = is_q ? u : u - a.Hq;
     const T* src = is_q ? static_cast<const T*>(a.q) + row * a.ldq + hd * a.D : static_cast<const T*>(a.k_raw) + row * a.ldkr + hd * a.D;
     T* dst = is_q ? static_cast<T*>(a.q) + row * a.ldq + hd * a.D : static_cast<T*>(a.k_out) + row * a.ldk + hd * a.D;
+    // single tokens: the rotated key (and, where the values are the raw keys, the value) straight into the ring as well
+    const size_t rr0 = ((static_cast<size_t>(seq.slot) * a.Hkv + hd) * a.ring + (a.ring ? seq.pos % a.ring : 0)) * a.D;
+    T* kring = !is_q && a.ring ? static_cast<T*>(a.k_ring) + rr0 : nullptr;
+    T* vring = !is_q && a.ring && a.v_ring ? static_cast<T*>(a.v_ring) + rr0 : nullptr;
     const float* w = is_q ? a.q_w : a.k_w;
     float* buf = rowbuf[warp];
     float sq = 0.0f;
     for (int d = lane; d < a.D; d += 32) {
       const float v = ldf(src + d);
+      if (vring) stf(vring + d, v);
       buf[d] = v;
       sq = fmaf(v, v, sq);
     }
@@ -63,6 +73,7 @@ __global__ void head_norm_rope_rows_kernel(const HeadNormRope a, const SeqDesc* 
       if (d < half) v = v * cs[d] - buf[d + half] * sn[d];
       else if (d < 2 * half) v = v * cs[d - half] + buf[d - half] * sn[d - half];
       stf(dst + d, v);
+      if (kring) stf(kring + d, v);
     }
     __syncwarp();
   }
@@ -83,12 +94,16 @@ __global__ void ring_append_kernel(const WindowAttn a, const SeqDesc* __restrict
     static_cast<T*>(a.v_ring)[((dst + c / a.DV) * a.ring + r) * a.DV + c % a.DV] = static_cast<const T*>(a.v_new)[row * a.ldv + c];
 }
 
-template <typename T>
-__global__ void window_attention_rows_kernel(const WindowAttn a, const SeqDesc* __restrict__ seqs) {
+// WPU warps share a (token, query head): each takes every WPU-th key with an online softmax, merged through shared memory.
+template <typename T, int WPU>
+__global__ void __launch_bounds__(WPU > 1 ? 32 * WPU : 128) window_attention_rows_kernel(const WindowAttn a, const SeqDesc* __restrict__ seqs) {
+  __shared__ float sm_ml[WPU][2];
+  __shared__ float sm_o[WPU > 1 ? WPU : 1][kMaxHead];
   pdl_wait();
   pdl_trigger();
   const SeqDesc seq = seqs[blockIdx.y];
-  const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int unit = WPU > 1 ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + warp;
   const int i = unit / a.Hq, h = unit % a.Hq;
   if (i >= seq.len) return;
   const int hk = h / (a.Hq / a.Hkv), pos = seq.pos + i;
@@ -106,7 +121,7 @@ __global__ void window_attention_rows_kernel(const WindowAttn a, const SeqDesc* 
     acc[e] = 0.0f;
   }
   float m = -INFINITY, l = 0.0f;
-  for (int j = max(0, pos - a.window + 1); j <= pos; ++j) {
+  for (int j = max(0, pos - a.window + 1) + (WPU > 1 ? warp : 0); j <= pos; j += WPU) {
     const bool fresh = j >= seq.pos;
     const T* kp = fresh ? kn + static_cast<size_t>(j - seq.pos) * a.ldk : kr + static_cast<size_t>(j % a.ring) * a.D;
     const T* vp = fresh ? vn + static_cast<size_t>(j - seq.pos) * a.ldv : vr + static_cast<size_t>(j % a.ring) * a.DV;
@@ -128,11 +143,207 @@ __global__ void window_attention_rows_kernel(const WindowAttn a, const SeqDesc* 
     m = m_new;
   }
   T* orow = static_cast<T*>(a.out) + row * a.ldo + h * a.DV;
-  const float inv = a.out_scale / l;
+  if (WPU == 1) {
+    const float inv = a.out_scale / l;
 #pragma unroll
-  for (int e = 0; e < kMaxHead / 32; ++e) {
-    const int d = lane + 32 * e;
-    if (d < a.DV) stf(orow + d, acc[e] * inv);
+    for (int e = 0; e < kMaxHead / 32; ++e) {
+      const int d = lane + 32 * e;
+      if (d < a.DV) stf(orow + d, acc[e] * inv);
+    }
+    return;
+  }
+  if (lane == 0) {
+    sm_ml[warp][0] = m;
+    sm_ml[warp][1] = l;
+  }
+#pragma unroll
+  for (int e = 0; e < kMaxHead / 32; ++e) sm_o[WPU > 1 ? warp : 0][lane + 32 * e] = acc[e];
+  __syncthreads();
+  float mm = -INFINITY, ll = 0.0f;
+#pragma unroll
+  for (int w = 0; w < WPU; ++w) mm = fmaxf(mm, sm_ml[w][0]);
+  for (int d = threadIdx.x; d < a.DV; d += blockDim.x) {
+    float o = 0.0f;
+    ll = 0.0f;
+#pragma unroll
+    for (int w = 0; w < WPU; ++w) {  // warps without keys hold -inf: factor 0
+      const float sc = expf(sm_ml[w][0] - mm);
+      ll = fmaf(sm_ml[w][1], sc, ll);
+      o = fmaf(sm_o[WPU > 1 ? w : 0][d], sc, o);
+    }
+    stf(orow + d, o / ll * a.out_scale);
+  }
+}
+
+// ---- tensor-core tiles for bf16 steps of any shape ----
+// CTA = 64 queries of one head of one entry, four warps of 16 rows; keys in tiles of 64 through a two-stage cp.async ring.
+// Rows come by address (ring or step), so tiles start anywhere; columns beyond the head size and rows beyond the last key
+// are zero.  S = Q K^T, online softmax in the fragments (log2 domain), O += P V with P packed straight from the S fragments.
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+constexpr int kQRows = 64, kKeys = 64;
+constexpr int mma_smem_bytes(int nd) { return (kQRows + 4 * kKeys) * (16 * nd + 8) * 2; }
+
+template <int ND>  // padded head size / 16
+__global__ void __launch_bounds__(128) window_attention_mma_kernel(const WindowAttn a, const SeqDesc* __restrict__ seqs) {
+  constexpr int DP = 16 * ND, LD = DP + 8, CH = DP / 8;
+  constexpr bool kHoldQ = ND <= 8;
+  extern __shared__ __align__(16) bf16 wa_smem[];
+  pdl_wait();
+  const SeqDesc seq = seqs[blockIdx.z];
+  const int i0 = blockIdx.x * kQRows;
+  if (i0 >= seq.len) return;
+  const int h = blockIdx.y, hk = h / (a.Hq / a.Hkv);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  bf16* sq = wa_smem;
+  const uint32_t sq_a = smem_u32(sq);
+  auto tile_addr = [&](int stage, int v) { return sq_a + (kQRows + (2 * stage + v) * kKeys) * LD * 2; };
+
+  const bf16* kn = static_cast<const bf16*>(a.k_new) + static_cast<size_t>(seq.row0) * a.ldk + hk * a.D;
+  const bf16* vn = static_cast<const bf16*>(a.v_new) + static_cast<size_t>(seq.row0) * a.ldv + hk * a.DV;
+  const bf16* kr = static_cast<const bf16*>(a.k_ring) + (static_cast<size_t>(seq.slot) * a.Hkv + hk) * a.ring * a.D;
+  const bf16* vr = static_cast<const bf16*>(a.v_ring) + (static_cast<size_t>(seq.slot) * a.Hkv + hk) * a.ring * a.DV;
+  const bf16* qb = static_cast<const bf16*>(a.q) + static_cast<size_t>(seq.row0) * a.ldq + h * a.D;
+  const int last_i = min(i0 + kQRows, seq.len) - 1;
+  const int key_lo = max(0, seq.pos + i0 - a.window + 1), key_hi = seq.pos + last_i;  // keys any row of the tile sees
+  const int n_tiles = (key_hi - key_lo) / kKeys + 1;
+
+  auto zero16 = [&](uint32_t dst) { asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(dst), "r"(0u) : "memory"); };
+  auto load_tile = [&](int t) {
+    const uint32_t kt = tile_addr(t & 1, 0), vt = tile_addr(t & 1, 1);
+    for (int idx = threadIdx.x; idx < kKeys * CH; idx += 128) {
+      const int r = idx / CH, ch = idx % CH, j = key_lo + t * kKeys + r;
+      const uint32_t off = static_cast<uint32_t>(r * LD + ch * 8) * 2;
+      const bool in = j <= key_hi, fresh = j >= seq.pos;
+      if (in && ch * 8 < a.D)
+        cp_async16(kt + off, (fresh ? kn + static_cast<size_t>(j - seq.pos) * a.ldk : kr + static_cast<size_t>(j % a.ring) * a.D) + ch * 8);
+      else zero16(kt + off);
+      if (in && ch * 8 < a.DV)
+        cp_async16(vt + off, (fresh ? vn + static_cast<size_t>(j - seq.pos) * a.ldv : vr + static_cast<size_t>(j % a.ring) * a.DV) + ch * 8);
+      else zero16(vt + off);
+    }
+    cp_async_commit();
+  };
+  for (int idx = threadIdx.x; idx < kQRows * CH; idx += 128) {
+    const int r = idx / CH, ch = idx % CH;
+    const uint32_t dst = sq_a + static_cast<uint32_t>(r * LD + ch * 8) * 2;
+    if (i0 + r <= last_i && ch * 8 < a.D) cp_async16(dst, qb + static_cast<size_t>(i0 + r) * a.ldq + ch * 8);
+    else zero16(dst);
+  }
+  load_tile(0);
+
+  const uint32_t qa_addr = sq_a + static_cast<uint32_t>((warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8) * 2;
+  const uint32_t ko = static_cast<uint32_t>(((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t vo = static_cast<uint32_t>(((lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8) * 2;
+  uint32_t qf[kHoldQ ? ND : 1][4];
+  float O[2 * ND][4];
+#pragma unroll
+  for (int n = 0; n < 2 * ND; ++n) O[n][0] = O[n][1] = O[n][2] = O[n][3] = 0.0f;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+  const float sc = a.scale * 1.4426950408889634f;
+  const int p_lo = seq.pos + i0 + warp * 16;  // position of the warp's first row; rows g and g + 8
+  for (int t = 0; t < n_tiles; ++t) {
+    if (t + 1 < n_tiles) {
+      load_tile(t + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    if (kHoldQ && t == 0) {
+#pragma unroll
+      for (int k = 0; k < ND; ++k) ldsm_x4(qf[kHoldQ ? k : 0], qa_addr + k * 32);
+    }
+    const int j0 = key_lo + t * kKeys;
+    if (j0 <= p_lo + 15 && j0 + kKeys > p_lo - a.window + 1) {  // some row of the warp sees some key of the tile
+      const uint32_t kt = tile_addr(t & 1, 0), vt = tile_addr(t & 1, 1);
+      float s[kKeys / 8][4];
+#pragma unroll
+      for (int n = 0; n < kKeys / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.0f;
+#pragma unroll
+      for (int k = 0; k < ND; ++k) {
+        uint32_t q[4];
+        if (kHoldQ) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) q[e] = qf[kHoldQ ? k : 0][e];
+        } else {
+          ldsm_x4(q, qa_addr + k * 32);
+        }
+#pragma unroll
+        for (int n = 0; n < kKeys / 8; n += 2) {
+          uint32_t b[4];
+          ldsm_x4(b, kt + ko + static_cast<uint32_t>(n * 8 * LD) * 2 + k * 32);
+          mma_bf16_16816(s[n], q[0], q[1], q[2], q[3], b[0], b[1]);
+          mma_bf16_16816(s[n + 1], q[0], q[1], q[2], q[3], b[2], b[3]);
+        }
+      }
+      const bool mask = j0 + kKeys - 1 > p_lo || j0 < p_lo + 16 - a.window;
+      float mx[2] = {m[0], m[1]};
+#pragma unroll
+      for (int n = 0; n < kKeys / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int p = p_lo + g + 8 * (e >> 1), j = j0 + 8 * n + 2 * c + (e & 1);
+          s[n][e] = mask && (j > p || j <= p - a.window) ? -INFINITY : s[n][e] * sc;
+          mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
+        }
+      float alpha[2], base[2];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+        base[r] = mx[r] == -INFINITY ? 0.0f : mx[r];  // a row that has seen no key yet
+        alpha[r] = ex2(m[r] - base[r]);
+        m[r] = mx[r];
+        l[r] *= alpha[r];
+      }
+#pragma unroll
+      for (int n = 0; n < 2 * ND; ++n) {
+        O[n][0] *= alpha[0]; O[n][1] *= alpha[0]; O[n][2] *= alpha[1]; O[n][3] *= alpha[1];
+      }
+#pragma unroll
+      for (int k = 0; k < kKeys / 16; ++k) {
+        uint32_t pf[4];
+#pragma unroll
+        for (int f = 0; f < 2; ++f) {
+          float* x = s[2 * k + f];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[e] = ex2(x[e] - base[e >> 1]);
+          l[0] += x[0] + x[1];
+          l[1] += x[2] + x[3];
+          pf[2 * f] = pack_bf16x2(x[0], x[1]);
+          pf[2 * f + 1] = pack_bf16x2(x[2], x[3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2 * ND; n += 2) {
+          uint32_t b[4];
+          ldsm_x4_trans(b, vt + vo + static_cast<uint32_t>(k * 16 * LD + n * 8) * 2);
+          mma_bf16_16816(O[n], pf[0], pf[1], pf[2], pf[3], b[0], b[1]);
+          mma_bf16_16816(O[n + 1], pf[0], pf[1], pf[2], pf[3], b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();  // the stage is free for the tile after the next
+  }
+  pdl_trigger();
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    const int i = i0 + warp * 16 + g + 8 * r;
+    if (i > last_i) continue;
+    const float inv = a.out_scale / l[r];
+    bf16* orow = static_cast<bf16*>(a.out) + (static_cast<size_t>(seq.row0) + i) * a.ldo + h * a.DV;
+#pragma unroll
+    for (int n = 0; n < 2 * ND; ++n) {
+      const int d = 8 * n + 2 * c;
+      if (d < a.DV) *reinterpret_cast<uint32_t*>(orow + d) = pack_bf16x2(O[n][2 * r] * inv, O[n][2 * r + 1] * inv);
+    }
   }
 }
 
@@ -153,14 +364,75 @@ int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, 
   return static_cast<int>(cudaGetLastError());
 }
 
-int window_attention_prepare() { return 0; }
+int window_attention_prepare() {
+  static std::atomic<unsigned long long> done{0};  // one bit per device; threads may race to set it
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull) return 0;
+  cudaError_t e = cudaFuncSetAttribute(window_attention_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, mma_smem_bytes(4));
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(window_attention_mma_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, mma_smem_bytes(8));
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(window_attention_mma_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, mma_smem_bytes(16));
+  if (e != cudaSuccess) return static_cast<int>(e);
+  int rc = attention_prefill_prepare();
+  if (rc == 0) rc = attention_decode_prepare();
+  if (rc == 0 && dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
+  return rc;
+}
 
 int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
   if (!valid(a, seqs, n_seqs, max_len) || !a.q || !a.out) return TEENY_ERR_BAD_ARG;
+  {
+    const int rc = window_attention_prepare();
+    if (rc) return rc;
+  }
+  const int G = a.Hq / a.Hkv;
+  // 16-byte rows everywhere
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k_new) | reinterpret_cast<uintptr_t>(a.v_new) |
+                          reinterpret_cast<uintptr_t>(a.k_ring) | reinterpret_cast<uintptr_t>(a.v_ring) | reinterpret_cast<uintptr_t>(a.out);
+  const bool rows16 = !a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && ((a.ldq | a.ldk | a.ldv | a.ldo) & 7) == 0 && (bases & 15) == 0;
+  AttnShape s{};
+  s.Hq = a.Hq; s.Hkv = a.Hkv; s.D = a.D; s.scale = a.scale; s.out_scale = a.out_scale;
+  if (rows16 && max_len == 1 && a.in_ring && a.D == a.DV && (a.D == 64 || a.D == 128) && (G == 1 || G == 2 || G == 4 || G == 8) && a.scratch &&
+      a.scratch_bytes >= attention_decode_scratch_bytes(n_seqs, a.Hq, a.D, a.ring)) {
+    s.B = n_seqs; s.Sq = 1; s.Skv = a.ring;
+    s.q_sb = a.ldq; s.q_sh = a.D; s.q_ss = a.ldq;
+    s.k_ss = s.v_ss = a.D;
+    s.k_sh = s.v_sh = static_cast<long long>(a.ring) * a.D;
+    s.k_sb = s.v_sb = s.k_sh * a.Hkv;
+    s.o_sb = a.ldo; s.o_sh = a.D; s.o_ss = a.ldo;
+    const DecodeRing ring{seqs, a.slots};
+    // (the kernel before this one, head_norm_rope_rows, wrote q and each sequence's newest ring row)
+    return attention_decode_bf16(static_cast<const bf16*>(a.q), static_cast<const bf16*>(a.k_ring), static_cast<const bf16*>(a.v_ring),
+                                 static_cast<bf16*>(a.out), s, 0, nullptr, a.scratch, a.scratch_bytes, st, 1, nullptr, a.counters, &ring);
+  }
+  if (rows16 && a.uniform_fresh && a.D == 128 && a.DV == 128 && max_len >= 128 && a.scale > 0.0f) {
+    s.B = n_seqs; s.Sq = s.Skv = max_len; s.causal = 1;
+    s.window = a.window < max_len ? a.window : 0;
+    s.q_sb = max_len * a.ldq; s.q_sh = a.D; s.q_ss = a.ldq;
+    s.k_sb = max_len * a.ldk; s.k_sh = a.D; s.k_ss = a.ldk;
+    s.v_sb = max_len * a.ldv; s.v_sh = a.D; s.v_ss = a.ldv;
+    s.o_sb = max_len * a.ldo; s.o_sh = a.D; s.o_ss = a.ldo;
+    return attention_prefill_bf16(static_cast<const bf16*>(a.q), static_cast<const bf16*>(a.k_new), static_cast<const bf16*>(a.v_new),
+                                  static_cast<bf16*>(a.out), nullptr, s, st);
+  }
+  if (rows16 && max_len >= 8) {
+    const dim3 grid((max_len + kQRows - 1) / kQRows, a.Hq, n_seqs), block(128);
+    const int d = a.D > a.DV ? a.D : a.DV;
+    if (d <= 64) launch_kernel(window_attention_mma_kernel<4>, grid, block, mma_smem_bytes(4), st, 1, a, seqs);
+    else if (d <= 128) launch_kernel(window_attention_mma_kernel<8>, grid, block, mma_smem_bytes(8), st, 1, a, seqs);
+    else launch_kernel(window_attention_mma_kernel<16>, grid, block, mma_smem_bytes(16), st, 1, a, seqs);
+    return static_cast<int>(cudaGetLastError());
+  }
   const long long units = static_cast<long long>(max_len) * a.Hq;
-  const dim3 grid(static_cast<unsigned>((units + 3) / 4), n_seqs), block(128);
-  if (a.f32) launch_kernel(window_attention_rows_kernel<float>, grid, block, 0, st, 1, a, seqs);
-  else launch_kernel(window_attention_rows_kernel<bf16>, grid, block, 0, st, 1, a, seqs);
+  if (max_len <= 16 && a.window > 32) {  // few rows: eight warps each
+    const dim3 grid(static_cast<unsigned>(units), n_seqs), block(256);
+    if (a.f32) launch_kernel(window_attention_rows_kernel<float, 8>, grid, block, 0, st, 1, a, seqs);
+    else launch_kernel(window_attention_rows_kernel<bf16, 8>, grid, block, 0, st, 1, a, seqs);
+  } else {
+    const dim3 grid(static_cast<unsigned>((units + 3) / 4), n_seqs), block(128);
+    if (a.f32) launch_kernel(window_attention_rows_kernel<float, 1>, grid, block, 0, st, 1, a, seqs);
+    else launch_kernel(window_attention_rows_kernel<bf16, 1>, grid, block, 0, st, 1, a, seqs);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -52,6 +52,7 @@ struct Layer {
 struct Plan {
   std::vector<Layer> layers;
   size_t x, y, proj, mix, delta, act, gu, o32, low, wz, kbuf, yrows, logits, logits16;
+  size_t attn_scratch, attn_counters, attn_scratch_bytes;
   size_t seqs, rows, sample_u, best_val, next_ids, cur_ids, history, state, total;
   size_t slot_bytes;
   int proj_ld, mix_ld, act_ld, o_ld, low_ld, wz_ld, k_ld, vocab_ld, width_ld;
@@ -81,6 +82,8 @@ bool make_plan(const teeny_hybrid_config& c, const teeny_hybrid_layer* layers, c
   p.layers.assign(c.num_layers, Layer());
   p.proj_ld = p.mix_ld = p.o_ld = p.low_ld = p.wz_ld = p.k_ld = 8;
   p.act_ld = 64;
+  p.attn_scratch_bytes = 0;
+  int kv_heads = 1;
   const size_t es = c.f32 ? 4 : 2;
   const size_t T = c.max_tokens, Bm = c.max_batch;
   size_t o = 0;
@@ -111,6 +114,11 @@ bool make_plan(const teeny_hybrid_config& c, const teeny_hybrid_layer* layers, c
           b.v_ring = take(Bm * b.c.kv_heads * static_cast<size_t>(b.ring) * V * es);
           p.slot_bytes += b.c.kv_heads * static_cast<size_t>(b.ring) * (D + V) * es;
           up(p.k_ld, pad8(b.c.kv_heads * D));
+          up(kv_heads, b.c.kv_heads);
+          if (!c.f32) {
+            const size_t need = attention_decode_scratch_bytes(c.max_batch, H, D, b.ring);
+            if (need > p.attn_scratch_bytes) p.attn_scratch_bytes = need;
+          }
           break;
         case TEENY_HYBRID_DELTA:
           for (; n < 5; ++n) sizes[n] = H * D;
@@ -163,6 +171,8 @@ bool make_plan(const teeny_hybrid_config& c, const teeny_hybrid_layer* layers, c
   p.yrows = take(static_cast<size_t>(c.max_rows) * p.width_ld * es);
   p.logits = take(static_cast<size_t>(c.max_rows) * p.vocab_ld * es);
   p.logits16 = take(c.f32 ? Bm * p.vocab_ld * 2 : 0);
+  p.attn_scratch = take(p.attn_scratch_bytes);
+  p.attn_counters = take(Bm * kv_heads * 4);
   p.seqs = take(Bm * sizeof(SeqDesc));
   p.rows = take(static_cast<size_t>(c.max_rows) * 4);
   p.sample_u = take(Bm * 4);
@@ -211,6 +221,7 @@ int linear(teeny_hybrid* m, const void* x, int ldx, const void* w, int ldw, void
 
 struct StepShape {
   int T, n, max_len;  // tokens, entries, longest entry
+  bool uniform_fresh; // whole prompts of one length from position 0
 };
 
 // Address of column `col` of row 0 of an activation buffer in the model's element type.
@@ -232,6 +243,12 @@ int run_attention(teeny_hybrid* m, const Layer& L, const Branch& b, const StepSh
   r.q_w = b.q_norm; r.k_w = b.k_norm; r.inv_freq = b.inv_freq;
   r.Hq = c.heads; r.Hkv = c.kv_heads; r.D = c.dim; r.rot_dims = c.rot_dims;
   r.eps = m->cfg.eps;
+  const bool single = s.max_len == 1 && b.keys_are_values();  // decode: the new key goes into the ring on the way
+  if (single) {
+    r.k_ring = m->at<void>(b.state);
+    r.v_ring = m->at<void>(b.v_ring);
+    r.ring = b.ring;
+  }
   TEENY_TRY(head_norm_rope_rows(r, m->seqs(), s.n, s.max_len, st));
   WindowAttn a{};
   a.f32 = m->cfg.f32;
@@ -246,8 +263,14 @@ int run_attention(teeny_hybrid* m, const Layer& L, const Branch& b, const StepSh
   a.ldo = L.n_out;
   a.Hq = c.heads; a.Hkv = c.kv_heads; a.D = c.dim; a.DV = c.vdim;
   a.scale = c.score_scale; a.out_scale = c.out_scale;
+  a.slots = m->cfg.max_batch;
+  a.uniform_fresh = s.uniform_fresh;
+  a.in_ring = single;
+  a.scratch = m->at<void>(p.attn_scratch);
+  a.scratch_bytes = p.attn_scratch_bytes;
+  a.counters = m->at<unsigned>(p.attn_counters);
   TEENY_TRY(window_attention(a, m->seqs(), s.n, s.max_len, st));
-  return ring_append(a, m->seqs(), s.n, s.max_len, st);
+  return single ? 0 : ring_append(a, m->seqs(), s.n, s.max_len, st);
 }
 
 int run_matrix_state(teeny_hybrid* m, const Layer& L, const Branch& b, const StepShape& s, cudaStream_t st) {
@@ -359,7 +382,7 @@ int record(teeny_hybrid* m, int n, cudaStream_t st) {
 
 int decode_body(teeny_hybrid* m, int n, cudaStream_t st) {
   PdlScope pdl;
-  TEENY_TRY(run_layers(m, m->at<int>(m->p.cur_ids), StepShape{n, n, 1}, st));
+  TEENY_TRY(run_layers(m, m->at<int>(m->p.cur_ids), StepShape{n, n, 1, false}, st));
   TEENY_TRY(run_head(m, nullptr, n, st));
   TEENY_TRY(pick(m, n, m->at<int>(m->p.state) + 2, st));
   return record(m, n, st);
@@ -416,8 +439,8 @@ int teeny_hybrid_create(const teeny_hybrid_config* cfg, const teeny_hybrid_layer
   if (rc == 0) rc = window_attention_prepare();
   m->cfg = *cfg;
   m->ws = static_cast<uint8_t*>(workspace);
-  // Everything starts finite: padding columns are multiplied by zero weights, and rings and states of fresh slots are never
-  // read, so nothing below depends on the zeros themselves.
+  // Arrival counters start at zero, and everything starts finite: padding columns are multiplied by zero weights.  (Rings and
+  // states of fresh slots are never read.)
   if (rc == 0) rc = static_cast<int>(cudaMemsetAsync(workspace, 0, m->p.total, reinterpret_cast<cudaStream_t>(stream)));
   if (rc != 0) {
     delete m;
@@ -480,7 +503,7 @@ int teeny_hybrid_step(teeny_hybrid* m, const int* ids, const int* slots, const i
   TEENY_TRY(check_ready(m));
   std::vector<SeqDesc> seqs(n);
   std::vector<char> used(m->cfg.max_batch, 0);
-  StepShape s{0, n, 0};
+  StepShape s{0, n, 0, true};
   for (int e = 0; e < n; ++e) {
     if (slots[e] < 0 || slots[e] >= m->cfg.max_batch || used[slots[e]] || positions[e] < 0 || lens[e] <= 0 ||
         positions[e] > m->cfg.max_len - lens[e] || lens[e] > m->cfg.max_tokens - s.T)
@@ -489,6 +512,7 @@ int teeny_hybrid_step(teeny_hybrid* m, const int* ids, const int* slots, const i
     seqs[e] = SeqDesc{slots[e], positions[e], s.T, lens[e]};
     s.T += lens[e];
     if (lens[e] > s.max_len) s.max_len = lens[e];
+    s.uniform_fresh = s.uniform_fresh && positions[e] == 0 && lens[e] == lens[0];
   }
   for (int r = 0; r < n_rows; ++r)
     if (rows[r] < 0 || rows[r] >= s.T) return TEENY_ERR_BAD_ARG;

@@ -121,6 +121,10 @@ int gemm_bf16_generic(const bf16* a, long long sam, long long sak, const bf16* b
                       const bf16* bias, bf16* c, long long scm, long long scn, int M, int N, int K,
                       cudaStream_t stream);
 
+// One entry of a step: `len` tokens of the sequence in state slot `slot`, the first at position `pos`, in rows row0 ..
+// row0 + len - 1 of the step's activations.  pos == 0 starts the sequence: the slot's old contents are not read.
+struct SeqDesc { int slot, pos, row0, len; };
+
 // ---- attention ---------------------------------------------------------------------------------
 struct AttnShape {
   int B, Hq, Hkv, Sq, Skv, D;
@@ -130,6 +134,8 @@ struct AttnShape {
   long long o_sb, o_sh, o_ss;
   float scale;
   int causal;
+  int window = 0;           // attention_prefill_bf16, causal: query i sees only its last `window` keys (0 = all)
+  float out_scale = 1.0f;   // factor of the output (attention_prefill_bf16, attention_decode_bf16)
 };
 int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, float* lse, const AttnShape& s,
                            cudaStream_t stream);
@@ -152,6 +158,13 @@ struct DecodeRope {
   int max_len;
   float eps;
 };
+// Decode over ring caches with per-sequence positions: sequence b's cache is row seqs[b].slot of the cache tensors (`slots`
+// of them, s.Skv = ring rows), its new key is already in row pos % ring, and it attends over min(pos + 1, ring) rows.
+// Head size 64 or 128.
+struct DecodeRing {
+  const SeqDesc* seqs;
+  int slots;
+};
 // One query token per sequence against the first *kv_len_dev (or kv_len if the pointer is null) cache entries.
 // fresh_rows >= 0 is a promise that matters only under programmatic dependent launch: the kernel launched just before
 // this one writes nothing this call reads except q (and rope->k_new / v_new) and the last fresh_rows live cache rows,
@@ -160,7 +173,8 @@ struct DecodeRope {
 // by the last CTA to finish instead of by a second kernel (calls sharing the counters must not overlap).
 int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, const AttnShape& s, int kv_len,
                           const int* kv_len_dev, void* scratch, size_t scratch_bytes, cudaStream_t stream,
-                          int fresh_rows = -1, const DecodeRope* rope = nullptr, unsigned* counters = nullptr);
+                          int fresh_rows = -1, const DecodeRope* rope = nullptr, unsigned* counters = nullptr,
+                          const DecodeRing* ring = nullptr);
 // Same as attention_decode_bf16 with the partials in a fixed-size array inside the library image (no caller scratch).
 size_t attention_decode_static_scratch_limit();
 int attention_decode_bf16_static(const bf16* q, const bf16* k, const bf16* v, bf16* o, const AttnShape& s, int kv_len,
@@ -221,9 +235,6 @@ int sample_merge(const unsigned long long* lists, int parts, size_t list_stride,
 int sampling_uniform(unsigned long long seed, int step, const int* step_dev, float* u, int rows, cudaStream_t st);
 
 // ---- layers of the hybrid decoders (recurrent mixers, windowed attention) ------------------------
-// One entry of a step: `len` tokens of the sequence in state slot `slot`, the first at position `pos`, in rows row0 ..
-// row0 + len - 1 of the step's activations.  pos == 0 starts the sequence: the slot's old contents are not read.
-struct SeqDesc { int slot, pos, row0, len; };
 
 // Element type of activations: bf16, or f32 where `f32` is set; then pointers to void hold floats.
 // Per-head matrix state S [DK, DV] (f32), one step per token, o = S^T q:
@@ -290,6 +301,12 @@ struct WindowAttn {
   long long ldo;
   int Hq, Hkv, D, DV;
   float scale, out_scale;
+  int slots;                 // state slots: rows of the ring tensors
+  int uniform_fresh;         // every entry starts at position 0 and has the step's longest length, rows in order
+  int in_ring;               // single tokens: k_new / v_new are in the ring already (head_norm_rope_rows)
+  void* scratch;             // attention_decode_scratch_bytes(entries, Hq, D, ring), or null
+  size_t scratch_bytes;
+  unsigned* counters;        // entries * Hkv words, zero between calls
 };
 // Per-head RMSNorm of q (in place) and k (k_raw -> k_out), then rotary positions on the first rot_dims dimensions
 // (i with i + rot_dims / 2), angles position * inv_freq[i] in f32.  q_w / k_w null: no norm.
@@ -304,6 +321,10 @@ struct HeadNormRope {
   const float *q_w, *k_w, *inv_freq;
   int Hq, Hkv, D, rot_dims;
   float eps;
+  // ring > 0 (single tokens): the rotated key also goes to its row of the ring, and with v_ring the raw key to the value ring
+  void* k_ring;
+  void* v_ring;
+  int ring;
 };
 int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
 int window_attention_prepare();
