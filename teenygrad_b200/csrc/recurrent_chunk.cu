@@ -14,8 +14,11 @@
 //
 // One CTA per (head, sequence).  Warps 0 .. n-1, the consumers, own 16 value columns each and keep S^T [16, DK] as C
 // fragments: those are, packed, the A operand of S^T U^T and S^T R^T, whose results (P^T, O^T) are in turn the A operand
-// and the layout of the update, so the chain never leaves the registers.  The last four warps, the producers, build the
-// B operands of the next chunk in the other shared-memory buffer.  Buffers change hands through named barriers.
+// and the layout of the update, so the chain never leaves the registers.  The last eight warps, the producers, build the
+// B operands: nothing in them depends on the state, so two groups of four warps take alternate chunks, each in its own
+// shared-memory buffer.  Buffers change hands through named barriers.  A group requests the raw projections of its
+// next chunk before it turns to the matrices of the current one, in one batch of unconditional loads (branches around
+// the loads made every one of them wait for its predecessor: 13 000 cycles per chunk instead of a few hundred).
 #include <atomic>
 
 #include "common.cuh"
@@ -27,13 +30,14 @@ namespace teeny {
 namespace {
 
 constexpr int kC = 16;          // tokens per chunk
-constexpr int kProducers = 128;
+constexpr int kGroup = 128;     // threads of a producer group
+constexpr int kProducers = 2 * kGroup;
 constexpr int kMatLd = 24;      // row stride of the 16 x 16 matrices (48 bytes: conflict-free ldmatrix)
 constexpr int kMaxDV = 192;     // 12 consumer warps
 constexpr int kBarFull = 1, kBarEmpty = 3, kBarProducers = 5;
 
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
 template <int FIRST>
 __device__ __forceinline__ void buffer_sync(int buf, int nthreads) {
@@ -45,9 +49,7 @@ __device__ __forceinline__ void buffer_arrive(int buf, int nthreads) {
   if (buf == 0) asm volatile("bar.arrive %0, %1;" ::"n"(FIRST), "r"(nthreads) : "memory");
   else asm volatile("bar.arrive %0, %1;" ::"n"(FIRST + 1), "r"(nthreads) : "memory");
 }
-__device__ __forceinline__ void producers_sync() {
-  asm volatile("bar.sync %0, %1;" ::"n"(kBarProducers), "n"(kProducers) : "memory");
-}
+__device__ __forceinline__ void group_sync(int group) { buffer_sync<kBarProducers>(group, kGroup); }
 
 // Shared memory of one buffer, byte offsets.  Delta: rows are U, R, Ka, Kk; decay: q, R, k, Kk (q and k without powers of d
 // are the producers' own).  Each as hi then lo, [16][DKP + 8] bf16.
@@ -65,15 +67,19 @@ struct Lay {
 constexpr int kU = 0, kR = 1, kKa = 2, kKk = 3;
 constexpr int kT = 0, kA2 = 1, kB1 = 2, kB2 = 3;
 
-// two neighbouring elements of a bf16 row; vec: the pair is 4-byte aligned
-__device__ __forceinline__ float2 ld_pair(const bf16* p, int i, int n, bool vec) {
-  if (vec) {
-    if (i >= n) return make_float2(0.0f, 0.0f);
-    const uint32_t v = *reinterpret_cast<const uint32_t*>(p + i);
-    return make_float2(bf16_lo(v), bf16_hi(v));
+// Two neighbouring elements of a bf16 row as loaded; zero beyond n.  VEC: the pair is 4-byte aligned and n even; the load is
+// unconditional (element 0 where i is beyond).
+template <bool VEC>
+__device__ __forceinline__ uint32_t ld_pair(const bf16* p, int i, int n) {
+  if (VEC) {
+    const uint32_t v = *reinterpret_cast<const uint32_t*>(p + (i < n ? i : 0));
+    return i < n ? v : 0u;
   }
-  return make_float2(i < n ? __bfloat162float(p[i]) : 0.0f, i + 1 < n ? __bfloat162float(p[i + 1]) : 0.0f);
+  const uint16_t* q = reinterpret_cast<const uint16_t*>(p);
+  const uint32_t lo = q[i < n ? i : 0], hi = q[i + 1 < n ? i + 1 : 0];
+  return (i < n ? lo : 0u) | (i + 1 < n ? hi << 16 : 0u);
 }
+__device__ __forceinline__ float2 f2(uint32_t v) { return make_float2(bf16_lo(v), bf16_hi(v)); }
 
 __device__ __forceinline__ void st_split(uint8_t* tile_hi, uint8_t* tile_lo, int byte_off, float x, float y) {
   uint32_t hi, lo;
@@ -124,17 +130,17 @@ __device__ __forceinline__ void split_frag(const float (&x)[4], const float (&y)
   split_bf16x2(y[2], y[3], hi[3], lo[3]);
 }
 
-template <int MODE, int NK>
-__global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int dvp) {
+template <int MODE, int NK, bool VEC, int THREADS, int BLOCKS>
+__global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int dvp) {
   constexpr int DKP = 16 * NK, NP = DKP / 64, LD = DKP + 8;
   constexpr bool DELTA = MODE == kScanDelta;
   using L = Lay<DKP>;
   extern __shared__ __align__(128) uint8_t chunk_smem[];
-  __shared__ float sh_tot[4][DKP];        // producers: log-decay sums of each warp's four tokens
-  __shared__ float sh_a1[kC][kC + 1];     // producers: U Ka^T, strictly lower
+  __shared__ float sh_tot[2][4][DELTA ? DKP : 1];   // producer groups: log-decay sums of each warp's four tokens
+  __shared__ float sh_a1[2][kC][kC + 1];  // producer groups: U Ka^T, strictly lower
   __shared__ float sh_pow[kC + 1];
   const int buf_bytes = L::bytes(dvp), ldv = dvp + 8;
-  const int n_cons = blockDim.x - kProducers, all = blockDim.x;
+  const int n_cons = blockDim.x - kProducers;
   const int lane = threadIdx.x & 31;
   pdl_wait();
   const SeqDesc seq = seqs[blockIdx.y];
@@ -146,13 +152,12 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
   }
 
   if (static_cast<int>(threadIdx.x) >= n_cons) {
-    // ---------------- producers: warp pw takes tokens 4 pw .. 4 pw + 3 of a chunk, a lane NP channel pairs ----------------
-    const int pw = (threadIdx.x - n_cons) >> 5;
+    // ---------------- producers: warp pw of a group takes tokens 4 pw .. 4 pw + 3 of a chunk, a lane NP channel pairs ----
+    const int grp = (threadIdx.x - n_cons) / kGroup, pw = ((threadIdx.x - n_cons) >> 5) & 3;
     const bf16* proj = static_cast<const bf16*>(a.proj);
     const bf16* wzp = static_cast<const bf16*>(a.wz);
     const int hk = h * a.DK, hv = h * a.DV;
-    const bool vec = ((a.DK | a.off_q | a.off_k | a.off_a) & 1) == 0 && (a.ld & 1) == 0 && (!DELTA || (a.ld_wz & 1) == 0);
-    const bool vecv = ((a.DV | a.off_v) & 1) == 0 && (a.ld & 1) == 0;
+    constexpr int NV = kMaxDV / 64;  // value pairs per lane and token
     float2 wb[NP], ab[NP];
     if (DELTA) {
 #pragma unroll
@@ -162,77 +167,87 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
         ab[i] = make_float2(c < a.DK ? a.a_bias[hk + c] : 0.0f, c + 1 < a.DK ? a.a_bias[hk + c + 1] : 0.0f);
       }
     }
-    float2 kk[4][NP], rr[4][NP], wz[4][NP], az[4][NP];
+    uint32_t rk[4][NP], rq[4][NP], rw[4][NP], ra[4][NP];  // raw projections of the chunk, bf16 pairs; zero for absent tokens
     auto fetch = [&](int c) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int t = c * kC + 4 * pw + j;
         const bool in = t < seq.len;
         const size_t row = static_cast<size_t>(seq.row0) + (in ? t : 0);
-        const bf16* pr = proj + row * a.ld;
+        const bf16* pr = proj + row * a.ld + hk;
+        const int n = in ? a.DK : 0;
 #pragma unroll
         for (int i = 0; i < NP; ++i) {
-          const int ch = 2 * lane + 64 * i, n = in ? a.DK : 0;
-          kk[j][i] = ld_pair(pr + a.off_k + hk, ch, n, vec);
-          rr[j][i] = ld_pair(pr + a.off_q + hk, ch, n, vec);
+          const int ch = 2 * lane + 64 * i;
+          rk[j][i] = ld_pair<VEC>(pr + a.off_k, ch, n);
+          rq[j][i] = ld_pair<VEC>(pr + a.off_q, ch, n);
           if (DELTA) {
-            wz[j][i] = ld_pair(wzp + row * a.ld_wz + hk, ch, n, vec);
-            az[j][i] = ld_pair(pr + a.off_a + hk, ch, n, vec);
+            rw[j][i] = ld_pair<VEC>(wzp + row * a.ld_wz + hk, ch, n);
+            ra[j][i] = ld_pair<VEC>(pr + a.off_a, ch, n);
           }
         }
       }
     };
-    if (n_chunks > 0) fetch(0);
-    for (int c = 0; c < n_chunks; ++c) {
-      const int buf = c & 1, n = min(kC, seq.len - c * kC);
-      uint8_t* sb = chunk_smem + buf * buf_bytes;
+    if (grp < n_chunks) fetch(grp);
+    for (int c = grp; c < n_chunks; c += 2) {
+      const int n = min(kC, seq.len - c * kC);
+      uint8_t* sb = chunk_smem + grp * buf_bytes;
       const uint32_t sa = smem_u32(sb);
-      if (c >= 2) buffer_sync<kBarEmpty>(buf, all);
-      // V: copied (delta) or silu, split (decay)
+      uint32_t rv[4][NV];
+#pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int t = 4 * pw + j;
-        const bool in = t < n;
-        const bf16* pr = proj + (static_cast<size_t>(seq.row0) + c * kC + (in ? t : 0)) * a.ld + a.off_v + hv;
-        uint8_t* v_hi = sb + L::kV + t * ldv * 2;
-        for (int x = 2 * lane; x < dvp; x += 64) {
-          const float2 v = ld_pair(pr, x, in ? a.DV : 0, vecv);
-          if (DELTA) *reinterpret_cast<uint32_t*>(v_hi + 2 * x) = pack_bf16x2(v.x, v.y);
-          else st_split(v_hi, v_hi + kC * ldv * 2, 2 * x, silu_f(v.x), silu_f(v.y));
-        }
+        const bf16* pr = proj + (static_cast<size_t>(seq.row0) + c * kC + (t < n ? t : 0)) * a.ld + a.off_v + hv;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (64 * i < dvp) rv[j][i] = ld_pair<VEC>(pr, 2 * lane + 64 * i, t < n ? a.DV : 0);
       }
+      float2 lw[4][NP];  // delta: running log decay over the warp's four tokens
+      float inv[4];
       if (DELTA) {
-        float2 lw[4][NP];
-        float inv[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const bool in = 4 * pw + j < n;
           float ss = 0.0f;
 #pragma unroll
           for (int i = 0; i < NP; ++i) {
-            ss = fmaf(kk[j][i].x, kk[j][i].x, fmaf(kk[j][i].y, kk[j][i].y, ss));
-            lw[j][i] = in ? make_float2(-a.decay_coef * sigmoid_f(wz[j][i].x + wb[i].x), -a.decay_coef * sigmoid_f(wz[j][i].y + wb[i].y))
+            const float2 k = f2(rk[j][i]), wz = f2(rw[j][i]);
+            ss = fmaf(k.x, k.x, fmaf(k.y, k.y, ss));
+            lw[j][i] = in ? make_float2(-a.decay_coef * sigmoid_f(wz.x + wb[i].x), -a.decay_coef * sigmoid_f(wz.y + wb[i].y))
                           : make_float2(0.0f, 0.0f);
             if (j > 0) { lw[j][i].x += lw[j - 1][i].x; lw[j][i].y += lw[j - 1][i].y; }
-            az[j][i] = make_float2(sigmoid_f(az[j][i].x + ab[i].x), sigmoid_f(az[j][i].y + ab[i].y));
           }
-          inv[j] = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
+          inv[j] = ss;
         }
 #pragma unroll
-        for (int i = 0; i < NP; ++i) *reinterpret_cast<float2*>(&sh_tot[pw][2 * lane + 64 * i]) = lw[3][i];
-        producers_sync();
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) inv[j] += __shfl_xor_sync(0xffffffffu, inv[j], o);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) inv[j] = 1.0f / sqrtf(inv[j] + a.unit_eps);
+#pragma unroll
+        for (int i = 0; i < NP; ++i) *reinterpret_cast<float2*>(&sh_tot[grp][pw][DELTA ? 2 * lane + 64 * i : 0]) = lw[3][i];
+      }
+      if (c >= 2) buffer_sync<kBarEmpty>(grp, n_cons + kGroup);
+      if (DELTA) {
+        group_sync(grp);
 #pragma unroll
         for (int i = 0; i < NP; ++i) {
           const int ch = 2 * lane + 64 * i;
           float2 base = make_float2(0.0f, 0.0f);
 #pragma unroll
           for (int q = 0; q < 3; ++q)
-            if (q < pw) { base.x += sh_tot[q][ch]; base.y += sh_tot[q][ch + 1]; }
-          float2 prev = make_float2(expf(base.x), expf(base.y));  // W_{t-1}
+            if (q < pw) {
+              const float2 o = *reinterpret_cast<const float2*>(&sh_tot[grp][q][DELTA ? ch : 0]);
+              base.x += o.x; base.y += o.y;
+            }
+          float2 prev = make_float2(__expf(base.x), __expf(base.y));  // W_{t-1}
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
-            const float2 l = make_float2(base.x + lw[j][i].x, base.y + lw[j][i].y);
-            const float2 W = make_float2(expf(l.x), expf(l.y)), iW = make_float2(expf(-l.x), expf(-l.y));
-            const float2 k = kk[j][i], r = rr[j][i], al = az[j][i];
+            const float2 W = make_float2(__expf(base.x + lw[j][i].x), __expf(base.y + lw[j][i].y));
+            const float2 iW = make_float2(__fdividef(1.0f, W.x), __fdividef(1.0f, W.y));
+            const float2 k = f2(rk[j][i]), r = f2(rq[j][i]), az = f2(ra[j][i]);
+            const float2 al = make_float2(sigmoid_f(az.x + ab[i].x), sigmoid_f(az.y + ab[i].y));
             const float2 u = make_float2(k.x * inv[j], k.y * inv[j]);
             const int off = ((4 * pw + j) * LD + ch) * 2;
             st_split(sb + L::tile(kU, 0), sb + L::tile(kU, 1), off, prev.x * u.x, prev.y * u.y);
@@ -250,7 +265,8 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
           const float dr = sh_pow[t + 1], dk = t < n ? sh_pow[n - 1 - t] : 0.0f;
 #pragma unroll
           for (int i = 0; i < NP; ++i) {
-            const float2 q = make_float2(silu_f(rr[j][i].x), silu_f(rr[j][i].y)), k = make_float2(silu_f(kk[j][i].x), silu_f(kk[j][i].y));
+            const float2 qr = f2(rq[j][i]), kr = f2(rk[j][i]);
+            const float2 q = make_float2(silu_f(qr.x), silu_f(qr.y)), k = make_float2(silu_f(kr.x), silu_f(kr.y));
             const int off = (t * LD + 2 * lane + 64 * i) * 2;
             st_split(sb + L::tile(kU, 0), sb + L::tile(kU, 1), off, q.x, q.y);
             st_split(sb + L::tile(kR, 0), sb + L::tile(kR, 1), off, q.x * dr, q.y * dr);
@@ -259,8 +275,24 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
           }
         }
       }
-      if (c + 1 < n_chunks) fetch(c + 1);  // in flight while the matrices are built
-      producers_sync();
+      // V: copied (delta) or silu, split (decay)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        uint8_t* v_hi = sb + L::kV + (4 * pw + j) * ldv * 2;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int x = 2 * lane + 64 * i;
+          if (x >= dvp) continue;
+          if (DELTA) {
+            *reinterpret_cast<uint32_t*>(v_hi + 2 * x) = rv[j][i];
+          } else {
+            const float2 v = f2(rv[j][i]);
+            st_split(v_hi, v_hi + kC * ldv * 2, 2 * x, silu_f(v.x), silu_f(v.y));
+          }
+        }
+      }
+      if (c + 2 < n_chunks) fetch(c + 2);  // in flight while the matrices are built
+      group_sync(grp);
       // the 16 x 16 matrices: warp 0 U Ka^T (and its inverse), 1 U Kk^T, 2 R Ka^T, 3 R Kk^T; decay: warp 3 q k^T alone
       const int g = lane >> 2, cc = lane & 3;
       if (DELTA || pw == 3) {
@@ -281,8 +313,8 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
             x = s <= reach ? x : 0.0f;
             y = s + 1 <= reach ? y : 0.0f;
             if (DELTA && pw == 0) {
-              sh_a1[t][s] = x;
-              sh_a1[t][s + 1] = y;
+              sh_a1[grp][t][s] = x;
+              sh_a1[grp][t][s + 1] = y;
             } else {
               const int m = DELTA ? (pw == 1 ? kA2 : (pw == 2 ? kB1 : kB2)) : kB2;
               st_split(sb + L::mat(m, 0), sb + L::mat(m, 1), (t * kMatLd + s) * 2, x, y);
@@ -298,8 +330,8 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
             float v = t == col ? 1.0f : 0.0f, v2 = 0.0f;
 #pragma unroll
             for (int s = 0; s < t; ++s) {
-              if (s & 1) v2 = fmaf(sh_a1[t][s], T[s], v2);
-              else v = fmaf(sh_a1[t][s], T[s], v);
+              if (s & 1) v2 = fmaf(sh_a1[grp][t][s], T[s], v2);
+              else v = fmaf(sh_a1[grp][t][s], T[s], v);
             }
             T[t] = v + v2;
           }
@@ -311,7 +343,7 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
           }
         }
       }
-      buffer_arrive<kBarFull>(buf, all);
+      buffer_arrive<kBarFull>(grp, n_cons + kGroup);
     }
     return;
   }
@@ -338,7 +370,7 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
     const int buf = c & 1, n = min(kC, seq.len - c * kC);
     const uint32_t sa = smem_u32(chunk_smem) + buf * buf_bytes;
     const float* scale = reinterpret_cast<const float*>(chunk_smem + buf * buf_bytes + L::kScale);
-    buffer_sync<kBarFull>(buf, all);
+    buffer_sync<kBarFull>(buf, n_cons + kGroup);
     float O[2][4] = {}, P[2][4] = {}, O2[2][4] = {}, P2[2][4] = {};
 #pragma unroll
     for (int k = 0; k < NK; ++k) {
@@ -426,7 +458,7 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
         }
       }
     }
-    if (c + 2 < n_chunks) buffer_arrive<kBarEmpty>(buf, all);
+    if (c + 2 < n_chunks) buffer_arrive<kBarEmpty>(buf, n_cons + kGroup);
   }
   pdl_trigger();
 #pragma unroll
@@ -438,22 +470,38 @@ __global__ void __launch_bounds__(512, 1) chunk_scan_kernel(const StateScan a, c
     }
 }
 
-template <int MODE, int NK>
-int launch_chunk(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool prepare_only, cudaStream_t st) {
+template <int MODE, int NK, bool VEC, int THREADS, int BLOCKS>
+int launch_chunk(const StateScan& a, const SeqDesc* seqs, int n_seqs, int dvp, bool prepare_only, cudaStream_t st) {
   static std::atomic<unsigned long long> done{0};  // one bit per device; threads may race to set it
   int dev = 0;
   cudaGetDevice(&dev);
+  const auto kernel = chunk_scan_kernel<MODE, NK, VEC, THREADS, BLOCKS>;
   if (!(dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull)) {
-    const cudaError_t e = cudaFuncSetAttribute(chunk_scan_kernel<MODE, NK>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               2 * Lay<16 * NK>::bytes(kMaxDV));
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * Lay<16 * NK>::bytes(kMaxDV));
     if (e != cudaSuccess) return static_cast<int>(e);
     if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
   }
   if (prepare_only) return 0;
-  const int dvp = (a.DV + 15) / 16 * 16;
-  launch_kernel(chunk_scan_kernel<MODE, NK>, dim3(a.H, n_seqs), dim3(dvp * 2 + kProducers), 2 * Lay<16 * NK>::bytes(dvp), st, 1, a, seqs,
-                dvp);
+  launch_kernel(kernel, dim3(a.H, n_seqs), dim3(dvp * 2 + kProducers), 2 * Lay<16 * NK>::bytes(dvp), st, 1, a, seqs, dvp);
   return static_cast<int>(cudaGetLastError());
+}
+
+// Registers: a thread of the 64-channel kernel gets 80 with up to 64 value columns (two CTAs per SM), 96 above; of the
+// 128-channel kernel 128 with up to 128 value columns, 96 above.
+template <int MODE>
+int dispatch_chunk(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool prep, cudaStream_t st) {
+  const bool vec = ((a.DK | a.DV | a.off_q | a.off_k | a.off_v) & 1) == 0 && (a.ld & 1) == 0 &&
+                   (a.mode != kScanDelta || ((a.off_a & 1) == 0 && (a.ld_wz & 1) == 0));
+  const int dvp = (a.DV + 15) / 16 * 16;
+#define TEENY_CHUNK(NK, T, B) \
+  return vec ? launch_chunk<MODE, NK, true, T, B>(a, seqs, n_seqs, dvp, prep, st) : launch_chunk<MODE, NK, false, T, B>(a, seqs, n_seqs, dvp, prep, st)
+  if (a.DK <= 64) {
+    if (dvp <= 64) TEENY_CHUNK(4, 384, 2);
+    TEENY_CHUNK(4, 640, 1);
+  }
+  if (dvp <= 128) TEENY_CHUNK(8, 512, 1);
+  TEENY_CHUNK(8, 640, 1);
+#undef TEENY_CHUNK
 }
 
 }  // namespace
@@ -464,18 +512,20 @@ bool chunk_scan_supports(const StateScan& a, int max_len) {
 }
 
 int chunk_scan_prepare() {
-  StateScan a{};
-  int rc = launch_chunk<kScanDelta, 4>(a, nullptr, 0, true, nullptr);
-  if (!rc) rc = launch_chunk<kScanDelta, 8>(a, nullptr, 0, true, nullptr);
-  if (!rc) rc = launch_chunk<kScanDecay, 4>(a, nullptr, 0, true, nullptr);
-  if (!rc) rc = launch_chunk<kScanDecay, 8>(a, nullptr, 0, true, nullptr);
-  return rc;
+  for (int odd = 0; odd < 2; ++odd)
+    for (int dk : {64, 128})
+      for (int dv : {64, 128, 192}) {
+        StateScan a{};
+        a.DK = dk; a.DV = dv; a.off_k = odd;
+        int rc = dispatch_chunk<kScanDelta>(a, nullptr, 0, true, nullptr);
+        if (!rc) rc = dispatch_chunk<kScanDecay>(a, nullptr, 0, true, nullptr);
+        if (rc) return rc;
+      }
+  return 0;
 }
 
 int chunk_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, cudaStream_t st) {
-  if (a.mode == kScanDelta)
-    return a.DK <= 64 ? launch_chunk<kScanDelta, 4>(a, seqs, n_seqs, false, st) : launch_chunk<kScanDelta, 8>(a, seqs, n_seqs, false, st);
-  return a.DK <= 64 ? launch_chunk<kScanDecay, 4>(a, seqs, n_seqs, false, st) : launch_chunk<kScanDecay, 8>(a, seqs, n_seqs, false, st);
+  return a.mode == kScanDelta ? dispatch_chunk<kScanDelta>(a, seqs, n_seqs, false, st) : dispatch_chunk<kScanDecay>(a, seqs, n_seqs, false, st);
 }
 
 }  // namespace teeny
