@@ -79,6 +79,82 @@ __global__ void head_norm_rope_rows_kernel(const HeadNormRope a, const SeqDesc* 
   }
 }
 
+// The same for bf16 heads of whole 16-byte vectors: `lph` (a power of two) lanes hold a head, eight elements each; the
+// rotation partner of a lane is rot_dims / 16 lanes away.
+constexpr int kRopeTasks = 4;  // (head, lane) tasks per thread whose loads are in flight together
+__global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormRope a, const SeqDesc* __restrict__ seqs, int lph) {
+  __shared__ __align__(16) float cs[kMaxHead / 2], sn[kMaxHead / 2];
+  const SeqDesc seq = seqs[blockIdx.y];  // written well before the kernel in front of this one
+  const int i = blockIdx.x;
+  const int half = a.rot_dims >> 1;
+  if (i < seq.len)
+    for (int d = threadIdx.x; d < half; d += blockDim.x)
+      sincosf(static_cast<float>(seq.pos + i) * a.inv_freq[d], &sn[d], &cs[d]);
+  pdl_wait();
+  pdl_trigger();
+  if (i >= seq.len) return;
+  const size_t row = static_cast<size_t>(seq.row0) + i;
+  const bf16* qr = static_cast<const bf16*>(a.q) + row * a.ldq;
+  const bf16* kr = static_cast<const bf16*>(a.k_raw) + row * a.ldkr;
+  const int lane = threadIdx.x & 31, sub = lane & (lph - 1), d0 = sub * 8;
+  const int per = 256 / lph, heads = a.Hq + a.Hkv, h0 = threadIdx.x / lph;
+  const int step = half >> 3;
+  const int partner = (lane - sub) + (sub < step ? sub + step : (sub < 2 * step ? sub - step : sub));
+  const bool in_head = d0 < a.D;
+  for (int base = 0; base < heads; base += per * kRopeTasks) {
+    uint4 raw[kRopeTasks];
+#pragma unroll
+    for (int t = 0; t < kRopeTasks; ++t) {
+      const int u = base + t * per + h0;
+      raw[t] = make_uint4(0u, 0u, 0u, 0u);
+      if (u < heads && in_head) raw[t] = *reinterpret_cast<const uint4*>((u < a.Hq ? qr + u * a.D : kr + (u - a.Hq) * a.D) + d0);
+    }
+    if (base == 0) __syncthreads();  // the angles
+#pragma unroll
+    for (int t = 0; t < kRopeTasks; ++t) {
+      const int u = base + t * per + h0;
+      if (base + t * per >= heads) break;  // uniform over the CTA
+      const bool is_q = u < a.Hq;
+      const uint32_t rw[4] = {raw[t].x, raw[t].y, raw[t].z, raw[t].w};
+      float x[8], sq = 0.0f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        x[2 * e] = bf16_lo(rw[e]);
+        x[2 * e + 1] = bf16_hi(rw[e]);
+        sq = fmaf(x[2 * e], x[2 * e], fmaf(x[2 * e + 1], x[2 * e + 1], sq));
+      }
+      for (int o = lph >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      const float* w = is_q ? a.q_w : a.k_w;
+      if (w && in_head) {
+        const float rr = 1.0f / sqrtf(sq / static_cast<float>(a.D) + a.eps);
+        const float4 w0 = __ldg(reinterpret_cast<const float4*>(w + d0)), w1 = __ldg(reinterpret_cast<const float4*>(w + d0 + 4));
+        x[0] *= rr * w0.x; x[1] *= rr * w0.y; x[2] *= rr * w0.z; x[3] *= rr * w0.w;
+        x[4] *= rr * w1.x; x[5] *= rr * w1.y; x[6] *= rr * w1.z; x[7] *= rr * w1.w;
+      }
+      const int ca = (sub < step ? sub : sub - step) * 8;
+      const float sign = sub < step ? -1.0f : 1.0f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float y = __shfl_sync(0xffffffffu, x[e], partner);
+        if (sub < 2 * step) x[e] = x[e] * cs[ca + e] + sign * y * sn[ca + e];
+      }
+      if (u >= heads || !in_head) continue;
+      const uint4 out = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+      if (is_q) {
+        *reinterpret_cast<uint4*>(static_cast<bf16*>(a.q) + row * a.ldq + u * a.D + d0) = out;
+      } else {
+        const int hk = u - a.Hq;
+        *reinterpret_cast<uint4*>(static_cast<bf16*>(a.k_out) + row * a.ldk + hk * a.D + d0) = out;
+        if (a.ring) {
+          const size_t r = ((static_cast<size_t>(seq.slot) * a.Hkv + hk) * a.ring + seq.pos % a.ring) * a.D + d0;
+          *reinterpret_cast<uint4*>(static_cast<bf16*>(a.k_ring) + r) = out;
+          if (a.v_ring) *reinterpret_cast<uint4*>(static_cast<bf16*>(a.v_ring) + r) = raw[t];
+        }
+      }
+    }
+  }
+}
+
 template <typename T>
 __global__ void ring_append_kernel(const WindowAttn a, const SeqDesc* __restrict__ seqs) {
   pdl_wait();
@@ -359,6 +435,15 @@ int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, 
       a.rot_dims < 0 || a.rot_dims > a.D || (a.rot_dims & 1) || (a.rot_dims && !a.inv_freq))
     return TEENY_ERR_BAD_ARG;
   const dim3 grid(max_len, n_seqs), block(256);
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k_raw) | reinterpret_cast<uintptr_t>(a.k_out) |
+                          reinterpret_cast<uintptr_t>(a.k_ring) | reinterpret_cast<uintptr_t>(a.v_ring) | reinterpret_cast<uintptr_t>(a.q_w) |
+                          reinterpret_cast<uintptr_t>(a.k_w);
+  if (!a.f32 && a.D % 8 == 0 && a.rot_dims % 16 == 0 && ((a.ldq | a.ldkr | a.ldk) & 7) == 0 && (bases & 15) == 0) {
+    int lph = 1;
+    while (lph * 8 < a.D) lph *= 2;
+    launch_kernel(head_norm_rope_vec_kernel, grid, block, 0, st, 1, a, seqs, lph);
+    return static_cast<int>(cudaGetLastError());
+  }
   if (a.f32) launch_kernel(head_norm_rope_rows_kernel<float>, grid, block, 0, st, 1, a, seqs);
   else launch_kernel(head_norm_rope_rows_kernel<bf16>, grid, block, 0, st, 1, a, seqs);
   return static_cast<int>(cudaGetLastError());

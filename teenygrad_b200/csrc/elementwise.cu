@@ -914,13 +914,9 @@ template <typename T>
 __global__ void tanh_rows_kernel(const T* __restrict__ x, long long ldx, T* __restrict__ y, long long ldy, int M, int N) {
   pdl_wait();
   pdl_trigger();
-  const long long total = static_cast<long long>(M) * N;
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
-       i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / N;
-    const int c = static_cast<int>(i - r * N);
-    st_as(y + r * ldy + c, tanhf(ldf<T>(x + r * ldx + c)));
-  }
+  // a thread per element of a few rows at a time: blockDim = (columns in flight, rows)
+  for (int r = blockIdx.x * blockDim.y + threadIdx.y; r < M; r += gridDim.x * blockDim.y)
+    for (int c = threadIdx.x; c < N; c += blockDim.x) st_as(y + r * ldy + c, tanhf(ldf<T>(x + r * ldx + c)));
 }
 
 __global__ void glu_interleaved_f32_kernel(const float* __restrict__ gu, long long ld, float* __restrict__ out, long long ldo, int T,
@@ -1160,9 +1156,10 @@ int residual_rms_norm(float* x, const void* delta, long long ldd, void* y, long 
 
 int tanh_rows(const void* x, long long ldx, void* y, long long ldy, int M, int N, bool f32, cudaStream_t st) {
   if (!x || !y || M <= 0 || N <= 0) return TEENY_ERR_BAD_ARG;
-  const dim3 grid(ew_grid(static_cast<long long>(M) * N, kEwThreads));
-  if (f32) launch_kernel(tanh_rows_kernel<float>, grid, dim3(kEwThreads), 0, st, 1, static_cast<const float*>(x), ldx, static_cast<float*>(y), ldy, M, N);
-  else launch_kernel(tanh_rows_kernel<bf16>, grid, dim3(kEwThreads), 0, st, 1, static_cast<const bf16*>(x), ldx, static_cast<bf16*>(y), ldy, M, N);
+  const dim3 block(N <= 32 ? 32 : (N <= 64 ? 64 : 128), N <= 32 ? 8 : (N <= 64 ? 4 : 2));
+  const dim3 grid(ew_grid(M, block.y));
+  if (f32) launch_kernel(tanh_rows_kernel<float>, grid, block, 0, st, 1, static_cast<const float*>(x), ldx, static_cast<float*>(y), ldy, M, N);
+  else launch_kernel(tanh_rows_kernel<bf16>, grid, block, 0, st, 1, static_cast<const bf16*>(x), ldx, static_cast<bf16*>(y), ldy, M, N);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -296,10 +296,18 @@ int run_matrix_state(teeny_hybrid* m, const Layer& L, const Branch& b, const Ste
     a.ld_wz = p.wz_ld;
     a.w_bias = b.decay_bias; a.a_bias = b.rate_bias;
     a.decay_coef = c.decay_coef; a.unit_eps = c.unit_eps;
+    a.norm_w = b.o_norm;
+    a.off_g = b.in[4];
+    a.out = column(m, p.mix, b.out_col);
+    a.ldout = L.n_out;
+    a.norm_eps = m->cfg.eps;
+    a.out_scale = c.out_scale;
   } else {
     a.decay = b.decay;
   }
-  TEENY_TRY(state_scan(a, m->seqs(), s.n, s.max_len, st));
+  bool normed = false;
+  TEENY_TRY(state_scan(a, m->seqs(), s.n, s.max_len, st, &normed));
+  if (normed) return 0;
   return gated_rms_norm(a.o, a.ldo, column(m, p.proj, b.in[delta ? 4 : 3]), L.n_in, b.o_norm, column(m, p.mix, b.out_col), L.n_out,
                         s.T, b.n_out, delta ? c.vdim : b.n_out, m->cfg.eps, c.out_scale, m->cfg.f32 != 0, st);
 }

@@ -256,9 +256,17 @@ struct StateScan {
   float* o;                  // [T, ldo], head h at column h * DV
   long long ldo;
   int H, DK, DV;
+  // Per-head group norm and gate behind the state, for the kernels that can apply them on the way out (see state_scan):
+  // out[t, h DV + c] = o / rms(o of the head) * norm_w * sigmoid(proj[off_g]) * out_scale
+  const float* norm_w;       // [H * DV], or null
+  int off_g;
+  void* out;
+  long long ldout;
+  float norm_eps, out_scale;
 };
 int state_scan_prepare();
-int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+// *normed (when given) <- whether the norm fields were applied and `o` not written; otherwise gated_rms_norm follows.
+int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st, bool* normed = nullptr);
 bool state_scan_supports(int dk, int dv);
 // The same over prompts on the tensor cores (state_scan chooses it).
 bool chunk_scan_supports(const StateScan& a, int max_len);

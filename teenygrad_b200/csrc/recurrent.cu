@@ -285,95 +285,309 @@ state_scan_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int col_g
     }
 }
 
-// ---- group norm with a sigmoid gate behind a matrix-state mixer: one warp or one CTA per (token, group) ----
-template <typename T, bool CTA>
+// four consecutive elements
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld4(const bf16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(bf16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// ---- group norm with a sigmoid gate behind a matrix-state mixer ----
+// Vector form: LPG lanes hold a whole group of 4 * LPG elements; LPG = 0: the CTA holds the whole row, which is one group
+// (VPT vectors per thread).
+template <typename T, int LPG, int VPT>
+__global__ void __launch_bounds__(256) gated_rms_norm_vec_kernel(const float* __restrict__ o, long long ldo, const T* __restrict__ gate,
+                                                                 long long ldg, const float* __restrict__ w, T* __restrict__ out,
+                                                                 long long ldout, int T_rows, int cols, float eps, float scale) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const int nv = cols >> 2;
+  float4 v[VPT], g[VPT];
+  long long row[VPT];
+  int c[VPT];
+  bool in[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    if (LPG) {
+      const unsigned idx = (blockIdx.x * VPT + i) * 256u + threadIdx.x;  // vectors of all rows in order
+      in[i] = idx < static_cast<unsigned>(T_rows) * static_cast<unsigned>(nv);
+      row[i] = in[i] ? idx / static_cast<unsigned>(nv) : 0;
+      c[i] = in[i] ? static_cast<int>(idx % static_cast<unsigned>(nv)) * 4 : 0;
+    } else {
+      row[i] = blockIdx.x;
+      in[i] = static_cast<int>(threadIdx.x) + i * 256 < nv;
+      c[i] = in[i] ? (threadIdx.x + i * 256) * 4 : 0;
+    }
+    v[i] = ld4(o + row[i] * ldo + c[i]);
+    g[i] = ld4(gate + row[i] * ldg + c[i]);
+  }
+  float total = 0.0f, sq[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    sq[i] = in[i] ? fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, v[i].w * v[i].w))) : 0.0f;
+    if (LPG) {
+#pragma unroll
+      for (int d = LPG / 2; d > 0; d >>= 1) sq[i] += __shfl_xor_sync(0xffffffffu, sq[i], d);
+    }
+    total += sq[i];
+  }
+  if (!LPG) {
+    total = warp_sum(total);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = total;
+    __syncthreads();
+    total = warp_sum((threadIdx.x & 31) < 8 ? red[threadIdx.x & 31] : 0.0f);
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    if (!in[i]) continue;
+    const float rr = scale / sqrtf(LPG ? sq[i] / (4.0f * LPG) + eps : total / static_cast<float>(cols) + eps);
+    const float4 wv = __ldg(reinterpret_cast<const float4*>(w + c[i]));
+    st4(out + row[i] * ldout + c[i],
+        make_float4(v[i].x * rr * wv.x * sigmoid_f(g[i].x), v[i].y * rr * wv.y * sigmoid_f(g[i].y),
+                    v[i].z * rr * wv.z * sigmoid_f(g[i].z), v[i].w * rr * wv.w * sigmoid_f(g[i].w)));
+  }
+}
+
+// Any group size and alignment: a warp per (token, group), scalar accesses.
+template <typename T>
 __global__ void gated_rms_norm_kernel(const float* __restrict__ o, long long ldo, const T* __restrict__ gate, long long ldg,
                                       const float* __restrict__ w, T* __restrict__ out, long long ldout, int T_rows, int groups,
                                       int group_size, float eps, float scale) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[32];
-  const int per = CTA ? 1 : blockDim.x >> 5, lanes = CTA ? blockDim.x : 32;
-  const int me = CTA ? threadIdx.x : threadIdx.x & 31;
-  const long long unit = static_cast<long long>(blockIdx.x) * per + (CTA ? 0 : threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  const long long unit = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (unit >= static_cast<long long>(T_rows) * groups) return;
   const long long row = unit / groups;
   const int c0 = static_cast<int>(unit % groups) * group_size;
   const float* src = o + row * ldo + c0;
   float sq = 0.0f;
-  for (int c = me; c < group_size; c += lanes) sq = fmaf(src[c], src[c], sq);
-  sq = warp_sum(sq);
-  if (CTA) {
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
-    __syncthreads();
-    sq = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.0f);
-  }
-  const float rr = scale / sqrtf(sq / static_cast<float>(group_size) + eps);
+  for (int c = lane; c < group_size; c += 32) sq = fmaf(src[c], src[c], sq);
+  const float rr = scale / sqrtf(warp_sum(sq) / static_cast<float>(group_size) + eps);
   const T* g = gate + row * ldg + c0;
   T* dst = out + row * ldout + c0;
-  for (int c = me; c < group_size; c += lanes) stf(dst + c, src[c] * rr * w[c0 + c] * sigmoid_f(ldf(g + c)));
+  for (int c = lane; c < group_size; c += 32) stf(dst + c, src[c] * rr * w[c0 + c] * sigmoid_f(ldf(g + c)));
 }
 
 // ---- minimal GRU.  The gates read only the current token, so S_t = A_t S_{t-1} + B_t is a scan of affine maps: warp w of
-// a CTA takes TS consecutive tokens of 32 channels, composes their maps, the compositions meet in shared memory, and every
-// warp finishes its own tokens from the state that enters them. ----
-template <typename T, int TS>
-__global__ void min_gru_kernel(const MinGru a, const SeqDesc* __restrict__ seqs) {
-  __shared__ float sA[2][8][32], sB[2][8][32];
+// a CTA takes TS consecutive tokens of 64 channels (a pair per lane), composes their maps, the compositions meet in shared
+// memory, and every warp finishes its own tokens from the state that enters them.  The raw projections of the next tile are
+// requested before the exchange. ----
+template <bool VEC>
+__device__ __forceinline__ float2 ld_two(const float* p, bool second) {
+  if (VEC) return *reinterpret_cast<const float2*>(p);
+  return make_float2(p[0], second ? p[1] : 0.0f);
+}
+template <bool VEC>
+__device__ __forceinline__ float2 ld_two(const bf16* p, bool second) {
+  if (VEC) {
+    const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
+    return make_float2(bf16_lo(v), bf16_hi(v));
+  }
+  return make_float2(__bfloat162float(p[0]), second ? __bfloat162float(p[1]) : 0.0f);
+}
+template <bool VEC>
+__device__ __forceinline__ void st_two(float* p, float2 v, bool second) {
+  if (VEC) { *reinterpret_cast<float2*>(p) = v; return; }
+  p[0] = v.x;
+  if (second) p[1] = v.y;
+}
+template <bool VEC>
+__device__ __forceinline__ void st_two(bf16* p, float2 v, bool second) {
+  if (VEC) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); return; }
+  p[0] = __float2bfloat16_rn(v.x);
+  if (second) p[1] = __float2bfloat16_rn(v.y);
+}
+
+__device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_f(u); }
+
+template <typename T, int TS, bool VEC>
+__global__ void __launch_bounds__(256) min_gru_kernel(const MinGru a, const SeqDesc* __restrict__ seqs) {
+  __shared__ float2 sA[2][8][32], sB[2][8][32];
+  const SeqDesc seq = seqs[blockIdx.y];  // written well before the kernel in front of this one
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int ch = blockIdx.x * 64 + 2 * lane;
+  const bool in = ch < a.W, second = ch + 1 < a.W;
+  const int cl = in ? ch : 0;
+  const float2 zb = in ? make_float2(a.z_bias[ch], second ? a.z_bias[ch + 1] : 0.0f) : make_float2(0.0f, 0.0f);
+  const float2 xb = in ? make_float2(a.x_bias[ch], second ? a.x_bias[ch + 1] : 0.0f) : make_float2(0.0f, 0.0f);
   pdl_wait();
   pdl_trigger();
-  const SeqDesc seq = seqs[blockIdx.y];
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-  const int ch = blockIdx.x * 32 + lane;
-  const bool in = ch < a.W;
-  const float zb = in ? a.z_bias[ch] : 0.0f, xb = in ? a.x_bias[ch] : 0.0f;
-  float* st = a.state + static_cast<size_t>(seq.slot) * a.W + ch;
-  float S = (in && seq.pos > 0) ? *st : 0.0f;
+  float* st = a.state + static_cast<size_t>(seq.slot) * a.W + cl;
+  float2 S = make_float2(0.0f, 0.0f);
+  if (seq.pos > 0) S = make_float2(st[0], second ? st[1] : 0.0f);
   const int tile = warps * TS;
+  float2 z[TS], u[TS], g[TS];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < TS; ++i) {
+      const int t = t0 + warp * TS + i;
+      const T* p = static_cast<const T*>(a.proj) + (static_cast<size_t>(seq.row0) + (t < seq.len ? t : 0)) * a.ld + cl;
+      z[i] = ld_two<VEC>(p + a.off_z, second);
+      u[i] = ld_two<VEC>(p + a.off_x, second);
+      g[i] = ld_two<VEC>(p + a.off_g, second);
+    }
+  };
+  fetch(0);
   int par = 0;
   for (int t0 = 0; t0 < seq.len; t0 += tile, par ^= 1) {
     const int first = t0 + warp * TS;
-    float A[TS], B[TS];
-    float pa = 1.0f, pb = 0.0f;
+    float2 A[TS], B[TS], G[TS], pa = make_float2(1.0f, 1.0f), pb = make_float2(0.0f, 0.0f);
 #pragma unroll
     for (int i = 0; i < TS; ++i) {
-      A[i] = 1.0f;
-      B[i] = 0.0f;
-      if (in && first + i < seq.len) {
-        const T* p = static_cast<const T*>(a.proj) + (static_cast<size_t>(seq.row0) + first + i) * a.ld + ch;
-        const float z = sigmoid_f(ldf(p + a.off_z) + zb), u = ldf(p + a.off_x) + xb;
-        A[i] = 1.0f - z;
-        B[i] = z * (u >= 0.0f ? u + 0.5f : sigmoid_f(u));
-      }
+      const float2 zz = make_float2(sigmoid_f(z[i].x + zb.x), sigmoid_f(z[i].y + zb.y));
+      const bool on = first + i < seq.len;
+      A[i] = on ? make_float2(1.0f - zz.x, 1.0f - zz.y) : make_float2(1.0f, 1.0f);
+      B[i] = on ? make_float2(zz.x * gru_candidate(u[i].x + xb.x), zz.y * gru_candidate(u[i].y + xb.y)) : make_float2(0.0f, 0.0f);
+      G[i] = make_float2(silu_f(g[i].x) * a.scale, silu_f(g[i].y) * a.scale);
+      pa = make_float2(pa.x * A[i].x, pa.y * A[i].y);
+      pb = make_float2(fmaf(A[i].x, pb.x, B[i].x), fmaf(A[i].y, pb.y, B[i].y));
     }
-#pragma unroll
-    for (int i = 0; i < TS; ++i) {
-      pa *= A[i];
-      pb = fmaf(A[i], pb, B[i]);
-    }
-    float mine = S;
+    if (t0 + tile < seq.len) fetch(t0 + tile);
+    float2 mine = S;
     if (warps > 1) {
       sA[par][warp][lane] = pa;
       sB[par][warp][lane] = pb;
       __syncthreads();  // the other parity's buffer is rewritten only behind the next tile's barrier
       for (int w = 0; w < warps; ++w) {
         if (w == warp) mine = S;
-        S = fmaf(sA[par][w][lane], S, sB[par][w][lane]);
+        const float2 wa = sA[par][w][lane], wb = sB[par][w][lane];
+        S = make_float2(fmaf(wa.x, S.x, wb.x), fmaf(wa.y, S.y, wb.y));
       }
     } else {
-      S = fmaf(pa, S, pb);
+      S = make_float2(fmaf(pa.x, S.x, pb.x), fmaf(pa.y, S.y, pb.y));
     }
 #pragma unroll
     for (int i = 0; i < TS; ++i) {
       if (in && first + i < seq.len) {
-        mine = fmaf(A[i], mine, B[i]);
-        const size_t row = static_cast<size_t>(seq.row0) + first + i;
-        const float g = ldf(static_cast<const T*>(a.proj) + row * a.ld + a.off_g + ch);
-        stf(static_cast<T*>(a.out) + row * a.ldout + ch, mine * silu_f(g) * a.scale);
+        mine = make_float2(fmaf(A[i].x, mine.x, B[i].x), fmaf(A[i].y, mine.y, B[i].y));
+        st_two<VEC>(static_cast<T*>(a.out) + (static_cast<size_t>(seq.row0) + first + i) * a.ldout + ch,
+                    make_float2(mine.x * G[i].x, mine.y * G[i].y), second);
       }
     }
   }
-  if (in && warp == 0) *st = S;
+  if (in && warp == 0) {
+    st[0] = S.x;
+    if (second) st[1] = S.y;
+  }
+}
+
+// ---- one token per sequence (decode): the state streams through once ----
+// CTA = one (sequence, head): a thread holds RPT rows x 4 columns of the state, requested before the dependency wait (the
+// state was written a whole step ago), so the whole state of the head is in flight while the projections are finished
+// and the key-side vectors are built in shared memory.  Row groups meet in shared memory for u^T S and for the output.
+// With a.norm_w (delta) the head's group norm and gate are applied on the way out.
+template <typename T, int MODE, int RPT>
+__global__ void __launch_bounds__(512) state_step_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int groups) {
+  constexpr bool DELTA = MODE == kScanDelta;
+  extern __shared__ __align__(16) float step_sh[];
+  const int dkp = (a.DK + 3) & ~3;
+  float* vec = step_sh;                          // [5][dkp], rows 1 .. 4: w, -a, k, q
+  float* val = vec + 5 * dkp;                    // [DV]
+  float* red = val + a.DV;                       // [groups][DV]
+  const SeqDesc seq = seqs[blockIdx.y];
+  const int h = blockIdx.x, c4 = (threadIdx.x % (a.DV >> 2)) * 4, rg = threadIdx.x / (a.DV >> 2);
+  const bool live = rg < groups;
+  float* state = a.state + (static_cast<size_t>(seq.slot) * a.H + h) * a.DK * a.DV + c4;
+  float4 S[RPT];
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+    const int ch = rg * RPT + r;
+    S[r] = live && seq.pos > 0 && ch < a.DK ? ld4(state + static_cast<size_t>(ch) * a.DV) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  pdl_wait();
+  pdl_trigger();
+  const size_t row = seq.row0;
+  const T* pr = static_cast<const T*>(a.proj) + row * a.ld;
+  const int hk = h * a.DK, hv = h * a.DV;
+  for (int c = threadIdx.x; c < a.DK; c += blockDim.x) {
+    const float k = ldf(pr + a.off_k + hk + c), q = ldf(pr + a.off_q + hk + c);
+    if (DELTA) {
+      vec[dkp + c] = expf(-a.decay_coef * sigmoid_f(ldf(static_cast<const T*>(a.wz) + row * a.ld_wz + hk + c) + a.w_bias[hk + c]));
+      vec[2 * dkp + c] = -sigmoid_f(ldf(pr + a.off_a + hk + c) + a.a_bias[hk + c]);
+    }
+    vec[3 * dkp + c] = DELTA ? k : silu_f(k);
+    vec[4 * dkp + c] = DELTA ? q : silu_f(q);
+  }
+  for (int c = threadIdx.x; c < a.DV; c += blockDim.x) {
+    const float v = ldf(pr + a.off_v + hv + c);
+    val[c] = DELTA ? v : silu_f(v);
+  }
+  __syncthreads();
+  const float4 v = live ? *reinterpret_cast<const float4*>(val + c4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  float4 p = make_float4(0.0f, 0.0f, 0.0f, 0.0f), o = p;
+  float inv = 1.0f;
+  if (DELTA) {
+    float ss = 0.0f;
+    for (int c = threadIdx.x & 31; c < a.DK; c += 32) ss = fmaf(vec[3 * dkp + c], vec[3 * dkp + c], ss);
+    inv = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);  // u = k * inv, the same in every warp
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) {
+      const int ch = rg * RPT + r;
+      const float k = live && ch < a.DK ? vec[3 * dkp + ch] * inv : 0.0f;
+      p = make_float4(fmaf(k, S[r].x, p.x), fmaf(k, S[r].y, p.y), fmaf(k, S[r].z, p.z), fmaf(k, S[r].w, p.w));
+    }
+    if (live) *reinterpret_cast<float4*>(red + rg * a.DV + c4) = p;
+    __syncthreads();
+    p = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (live)
+      for (int g = 0; g < groups; ++g) {
+        const float4 x = *reinterpret_cast<const float4*>(red + g * a.DV + c4);
+        p = make_float4(p.x + x.x, p.y + x.y, p.z + x.z, p.w + x.w);
+      }
+    __syncthreads();
+  }
+  const float dec = DELTA ? 0.0f : a.decay[h];
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+    const int ch = rg * RPT + r;
+    if (!live || ch >= a.DK) continue;
+    const float w = DELTA ? vec[dkp + ch] : dec, k = vec[3 * dkp + ch], q = vec[4 * dkp + ch];
+    const float au = DELTA ? vec[2 * dkp + ch] * k * inv : 0.0f;
+    S[r] = make_float4(fmaf(w, S[r].x, fmaf(au, p.x, k * v.x)), fmaf(w, S[r].y, fmaf(au, p.y, k * v.y)),
+                       fmaf(w, S[r].z, fmaf(au, p.z, k * v.z)), fmaf(w, S[r].w, fmaf(au, p.w, k * v.w)));
+    o = make_float4(fmaf(q, S[r].x, o.x), fmaf(q, S[r].y, o.y), fmaf(q, S[r].z, o.z), fmaf(q, S[r].w, o.w));
+    st4(state + static_cast<size_t>(ch) * a.DV, S[r]);
+  }
+  if (live) *reinterpret_cast<float4*>(red + rg * a.DV + c4) = o;
+  __syncthreads();
+  float sq = 0.0f;
+  for (int c = threadIdx.x; c < a.DV; c += blockDim.x) {
+    float y = 0.0f;
+    for (int g = 0; g < groups; ++g) y += red[g * a.DV + c];
+    if (a.norm_w) val[c] = y;  // (v has been read)
+    else a.o[row * a.ldo + hv + c] = y;
+    sq = fmaf(y, y, sq);
+  }
+  if (!a.norm_w) return;
+  __syncthreads();
+  sq = 0.0f;
+  for (int c = threadIdx.x & 31; c < a.DV; c += 32) sq = fmaf(val[c], val[c], sq);
+  const float rr = a.out_scale / sqrtf(warp_sum(sq) / static_cast<float>(a.DV) + a.norm_eps);
+  for (int c = threadIdx.x; c < a.DV; c += blockDim.x)
+    stf(static_cast<T*>(a.out) + row * a.ldout + hv + c, val[c] * rr * a.norm_w[hv + c] * sigmoid_f(ldf(pr + a.off_g + hv + c)));
+}
+
+// Rows per thread and row groups of the one-token kernel; false if the head does not fit it.
+bool step_shape(const StateScan& a, int& rpt, int& groups) {
+  if (a.DV & 3) return false;
+  rpt = (a.DV / 4) * ((a.DK + 7) / 8) <= 512 ? 8 : 16;
+  groups = (a.DK + rpt - 1) / rpt;
+  return (a.DV / 4) * groups <= 512;
+}
+int step_smem(const StateScan& a, int groups) { return (5 * ((a.DK + 3) & ~3) + a.DV + groups * a.DV) * static_cast<int>(sizeof(float)); }
+
+template <typename T, int MODE>
+int launch_step(const StateScan& a, const SeqDesc* seqs, int n_seqs, int rpt, int groups, cudaStream_t st) {
+  const int threads = ((a.DV / 4) * groups + 31) / 32 * 32, smem = step_smem(a, groups);
+  if (rpt == 8) launch_kernel(state_step_kernel<T, MODE, 8>, dim3(a.H, n_seqs), dim3(threads), smem, st, 1, a, seqs, groups);
+  else launch_kernel(state_step_kernel<T, MODE, 16>, dim3(a.H, n_seqs), dim3(threads), smem, st, 1, a, seqs, groups);
+  return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T, int MODE, int KS>
@@ -431,49 +645,89 @@ int state_scan_prepare() {
   return chunk_scan_prepare();
 }
 
-int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
+int state_scan(const StateScan& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st, bool* normed) {
   if (!a.proj || !a.state || !a.o || !seqs || n_seqs <= 0 || n_seqs > 65535 || max_len <= 0 || a.H <= 0 || a.H > 65535 ||
       !state_scan_supports(a.DK, a.DV))
     return TEENY_ERR_BAD_ARG;
   if (a.mode == kScanDelta ? (!a.wz || !a.w_bias || !a.a_bias) : (a.mode != kScanDecay || !a.decay)) return TEENY_ERR_BAD_ARG;
-  // prompts in bf16: 16 tokens at a time on the tensor cores; single tokens and f32: token by token
+  if (normed) *normed = false;
+  // prompts in bf16: 16 tokens at a time on the tensor cores; single tokens: one pass over the state; else token by token
   if (chunk_scan_supports(a, max_len)) return chunk_scan(a, seqs, n_seqs, st);
+  int rpt, groups;
+  if (max_len == 1 && step_shape(a, rpt, groups)) {
+    StateScan b = a;
+    if (!normed || !a.out) b.norm_w = nullptr;
+    if (normed) *normed = b.norm_w != nullptr;
+    if (a.mode == kScanDelta)
+      return a.f32 ? launch_step<float, kScanDelta>(b, seqs, n_seqs, rpt, groups, st) : launch_step<bf16, kScanDelta>(b, seqs, n_seqs, rpt, groups, st);
+    return a.f32 ? launch_step<float, kScanDecay>(b, seqs, n_seqs, rpt, groups, st) : launch_step<bf16, kScanDecay>(b, seqs, n_seqs, rpt, groups, st);
+  }
   return scan_any(a, seqs, n_seqs, false, st);
 }
+
+namespace {
+template <typename T>
+int launch_gated_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, void* out, long long ldout, int T_rows,
+                      int cols, int group_size, float eps, float scale, cudaStream_t st) {
+  const T* g = static_cast<const T*>(gate);
+  T* y = static_cast<T*>(out);
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) |
+                          reinterpret_cast<uintptr_t>(out);
+  const bool vec = (bases & 15) == 0 && ((ldo | ldg | ldout | cols) & 3) == 0 && static_cast<long long>(T_rows) * cols < (1ll << 32);
+  const dim3 block(256);
+#define TEENY_GRN(LPG, VPT, GRID) \
+  launch_kernel(gated_rms_norm_vec_kernel<T, LPG, VPT>, dim3(GRID), block, 0, st, 1, o, ldo, g, ldg, w, y, ldout, T_rows, cols, eps, scale)
+  if (vec && (group_size == 16 || group_size == 32 || group_size == 64 || group_size == 128)) {
+    const long long vectors = static_cast<long long>(T_rows) * (cols / 4);
+    const unsigned grid = static_cast<unsigned>((vectors + 511) / 512);
+    if (group_size == 16) TEENY_GRN(4, 2, grid);
+    else if (group_size == 32) TEENY_GRN(8, 2, grid);
+    else if (group_size == 64) TEENY_GRN(16, 2, grid);
+    else TEENY_GRN(32, 2, grid);
+  } else if (vec && group_size == cols && cols <= 8 * 1024) {
+    if (cols <= 1024) TEENY_GRN(0, 1, T_rows);
+    else if (cols <= 2048) TEENY_GRN(0, 2, T_rows);
+    else if (cols <= 4096) TEENY_GRN(0, 4, T_rows);
+    else TEENY_GRN(0, 8, T_rows);
+  } else {
+    const int groups = cols / group_size;
+    const long long blocks = (static_cast<long long>(T_rows) * groups + 7) / 8;
+    if (blocks > 0x7fffffffLL) return TEENY_ERR_BAD_ARG;
+    launch_kernel(gated_rms_norm_kernel<T>, dim3(static_cast<unsigned>(blocks)), block, 0, st, 1, o, ldo, g, ldg, w, y, ldout, T_rows, groups,
+                  group_size, eps, scale);
+  }
+#undef TEENY_GRN
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int launch_min_gru(const MinGru& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
+  constexpr int TS = 8;
+  const dim3 grid((a.W + 63) / 64, n_seqs);
+  const bool vec = ((a.W | a.off_z | a.off_x | a.off_g) & 1) == 0 && ((a.ld | a.ldout) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 7) == 0;
+  int warps = (max_len + TS - 1) / TS;
+  if (warps > 8) warps = 8;
+#define TEENY_GRU(N) \
+  vec ? launch_kernel(min_gru_kernel<T, N, true>, grid, dim3(32 * warps), 0, st, 1, a, seqs) \
+      : launch_kernel(min_gru_kernel<T, N, false>, grid, dim3(32 * warps), 0, st, 1, a, seqs)
+  if (max_len == 1) TEENY_GRU(1);
+  else TEENY_GRU(TS);
+#undef TEENY_GRU
+  return static_cast<int>(cudaGetLastError());
+}
+}  // namespace
 
 int gated_rms_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, void* out, long long ldout,
                    int T, int cols, int group_size, float eps, float scale, bool f32, cudaStream_t st) {
   if (!o || !gate || !w || !out || T <= 0 || cols <= 0 || group_size <= 0 || cols % group_size) return TEENY_ERR_BAD_ARG;
-  const int groups = cols / group_size;
-  const bool cta = group_size > 512;
-  const long long units = static_cast<long long>(T) * groups;
-  const long long blocks = cta ? units : (units + 7) / 8;
-  if (blocks > 0x7fffffffLL) return TEENY_ERR_BAD_ARG;
-  const dim3 grid(static_cast<unsigned>(blocks)), block(256);
-#define TEENY_GRN(TT, C)                                                                                                     \
-  launch_kernel(gated_rms_norm_kernel<TT, C>, grid, block, 0, st, 1, o, ldo, static_cast<const TT*>(gate), ldg, w,           \
-                static_cast<TT*>(out), ldout, T, groups, group_size, eps, scale)
-  if (f32) { if (cta) TEENY_GRN(float, true); else TEENY_GRN(float, false); }
-  else { if (cta) TEENY_GRN(bf16, true); else TEENY_GRN(bf16, false); }
-#undef TEENY_GRN
-  return static_cast<int>(cudaGetLastError());
+  return f32 ? launch_gated_norm<float>(o, ldo, gate, ldg, w, out, ldout, T, cols, group_size, eps, scale, st)
+             : launch_gated_norm<bf16>(o, ldo, gate, ldg, w, out, ldout, T, cols, group_size, eps, scale, st);
 }
 
 int min_gru(const MinGru& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
   if (!a.proj || !a.z_bias || !a.x_bias || !a.state || !a.out || !seqs || n_seqs <= 0 || n_seqs > 65535 || max_len <= 0 || a.W <= 0)
     return TEENY_ERR_BAD_ARG;
-  const dim3 grid((a.W + 31) / 32, n_seqs);
-  constexpr int TS = 16;
-  if (max_len == 1) {
-    if (a.f32) launch_kernel(min_gru_kernel<float, 1>, grid, dim3(32), 0, st, 1, a, seqs);
-    else launch_kernel(min_gru_kernel<bf16, 1>, grid, dim3(32), 0, st, 1, a, seqs);
-  } else {
-    int warps = (max_len + TS - 1) / TS;
-    if (warps > 8) warps = 8;
-    if (a.f32) launch_kernel(min_gru_kernel<float, TS>, grid, dim3(32 * warps), 0, st, 1, a, seqs);
-    else launch_kernel(min_gru_kernel<bf16, TS>, grid, dim3(32 * warps), 0, st, 1, a, seqs);
-  }
-  return static_cast<int>(cudaGetLastError());
+  return a.f32 ? launch_min_gru<float>(a, seqs, n_seqs, max_len, st) : launch_min_gru<bf16>(a, seqs, n_seqs, max_len, st);
 }
 
 }  // namespace teeny

@@ -6,11 +6,12 @@
 //   o_t = r_t^T S_t     = R_t X_0 + sum_{s<=t} (R_t . Ka_s) p_s + (R_t . Kk_s) v_s     R_t = W_t o r_t
 //   S_16 = diag(W_16) (X_0 + sum_s Ka_s p_s + Kk_s v_s)                                Ka_s = -a_s u_s / W_s, Kk_s = k_s / W_s
 // so a chunk is four 16 x 16 matrices, one triangular inverse T = (1 - U Ka^T)^{-1} and products with the state.
-// Scalar decay.  o_t = d^{t+1} q_t^T S_0 + sum_{s<=t} d^{t-s} (q_t . k_s) v_s, S_n = d^n S_0 + sum_s d^{n-1-s} k_s v_s; no
-// division by a power of d, however small d is.
+// Scalar decay.  o_t = d^{t+1} q_t^T S_0 + sum_{s<=t} d^{t-s} (q_t . k_s) v_s, S_n = d^n S_0 + sum_s k_s (d^{n-1-s} v_s); no
+// division by a power of d, however small d is.  q, k, v are the activated projections, bf16 tensors.
 //
-// 32-bit accuracy from bf16 tensor cores: every f32 operand goes in as hi + lo (2^-17), a product as hi hi + hi lo +
-// lo hi with f32 accumulation; the carried state itself is never rounded (f32 accumulators from chunk to chunk).
+// 32-bit accuracy from bf16 tensor cores: every f32 operand goes in as hi + lo (2^-17), a product of two as hi hi + hi lo
+// + lo hi with f32 accumulation, projections as they are (one term); the carried state itself is never rounded (f32
+// accumulators from chunk to chunk).
 //
 // One CTA per (head, sequence).  Warps 0 .. n-1, the consumers, own 16 value columns each and keep S^T [16, DK] as C
 // fragments: those are, packed, the A operand of S^T U^T and S^T R^T, whose results (P^T, O^T) are in turn the A operand
@@ -51,8 +52,8 @@ __device__ __forceinline__ void buffer_arrive(int buf, int nthreads) {
 }
 __device__ __forceinline__ void group_sync(int group) { buffer_sync<kBarProducers>(group, kGroup); }
 
-// Shared memory of one buffer, byte offsets.  Delta: rows are U, R, Ka, Kk; decay: q, R, k, Kk (q and k without powers of d
-// are the producers' own).  Each as hi then lo, [16][DKP + 8] bf16.
+// Shared memory of one buffer, byte offsets.  Row tiles [16][DKP + 8] bf16: delta U, R, Ka, Kk, each as hi then lo; decay q
+// (in the place of R hi) and k (of Kk hi).  V: delta v; decay v, then d^{n-1-s} v as hi and lo.
 template <int DKP>
 struct Lay {
   static constexpr int kLd = DKP + 8;
@@ -62,22 +63,21 @@ struct Lay {
   static constexpr int mat(int which, int lo) { return kMats + (2 * which + lo) * kC * kMatLd * 2; }
   static constexpr int kScale = kMats + 8 * kC * kMatLd * 2;   // f32 [DKP]: decay of the chunk per key channel
   static constexpr int kV = kScale + DKP * 4;                  // V hi, then lo: [16][DVP + 8] bf16
-  static __host__ __device__ constexpr int bytes(int dvp) { return kV + 2 * kC * (dvp + 8) * 2; }
+  static __host__ __device__ constexpr int bytes(int dvp) { return kV + 3 * kC * (dvp + 8) * 2; }
 };
 constexpr int kU = 0, kR = 1, kKa = 2, kKk = 3;
 constexpr int kT = 0, kA2 = 1, kB1 = 2, kB2 = 3;
 
-// Two neighbouring elements of a bf16 row as loaded; zero beyond n.  VEC: the pair is 4-byte aligned and n even; the load is
-// unconditional (element 0 where i is beyond).
+// Two neighbouring elements of a bf16 row of n as loaded, unconditionally; what lies beyond n is any element of the row (the
+// caller clears it when it uses the pair: a select here would wait for the load).  VEC: the pair is 4-byte aligned, n even.
 template <bool VEC>
 __device__ __forceinline__ uint32_t ld_pair(const bf16* p, int i, int n) {
-  if (VEC) {
-    const uint32_t v = *reinterpret_cast<const uint32_t*>(p + (i < n ? i : 0));
-    return i < n ? v : 0u;
-  }
+  if (VEC) return *reinterpret_cast<const uint32_t*>(p + (i < n ? i : 0));
   const uint16_t* q = reinterpret_cast<const uint16_t*>(p);
-  const uint32_t lo = q[i < n ? i : 0], hi = q[i + 1 < n ? i + 1 : 0];
-  return (i < n ? lo : 0u) | (i + 1 < n ? hi << 16 : 0u);
+  return q[i < n ? i : 0] | (static_cast<uint32_t>(q[i + 1 < n ? i + 1 : 0]) << 16);
+}
+__device__ __forceinline__ uint32_t keep_pair(uint32_t v, int i, int n) {
+  return i + 1 < n ? v : (i < n ? v & 0xffffu : 0u);
 }
 __device__ __forceinline__ float2 f2(uint32_t v) { return make_float2(bf16_lo(v), bf16_hi(v)); }
 
@@ -89,23 +89,33 @@ __device__ __forceinline__ void st_split(uint8_t* tile_hi, uint8_t* tile_lo, int
 }
 
 // acc[2][4] (16 rows x 16 columns) += A B^T for row tiles A, B [16][LD] given as hi / lo, over NK 16-deep steps.
-template <int NK, int LD>
+template <int NK, int LD, bool SPLIT>
 __device__ __forceinline__ void rows_product(float (&acc)[2][4], uint32_t a_hi, uint32_t a_lo, uint32_t b_hi, uint32_t b_lo, int lane) {
   const uint32_t ao = static_cast<uint32_t>(((lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8) * 2;
   const uint32_t bo = static_cast<uint32_t>(((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2;
+  float acc2[2][4] = {};
 #pragma unroll
   for (int k = 0; k < NK; ++k) {
     uint32_t ah[4], al[4], bh[4], bl[4];
     ldsm_x4(ah, a_hi + ao + k * 32);
-    ldsm_x4(al, a_lo + ao + k * 32);
     ldsm_x4(bh, b_hi + bo + k * 32);
-    ldsm_x4(bl, b_lo + bo + k * 32);
+    if (SPLIT) {
+      ldsm_x4(al, a_lo + ao + k * 32);
+      ldsm_x4(bl, b_lo + bo + k * 32);
+    }
 #pragma unroll
     for (int n = 0; n < 2; ++n) {
       mma_bf16_16816(acc[n], ah[0], ah[1], ah[2], ah[3], bh[2 * n], bh[2 * n + 1]);
-      mma_bf16_16816(acc[n], ah[0], ah[1], ah[2], ah[3], bl[2 * n], bl[2 * n + 1]);
-      mma_bf16_16816(acc[n], al[0], al[1], al[2], al[3], bh[2 * n], bh[2 * n + 1]);
+      if (!SPLIT) continue;
+      mma_bf16_16816(acc2[n], ah[0], ah[1], ah[2], ah[3], bl[2 * n], bl[2 * n + 1]);
+      mma_bf16_16816(acc2[n], al[0], al[1], al[2], al[3], bh[2 * n], bh[2 * n + 1]);
     }
+  }
+  if (SPLIT) {
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[n][e] += acc2[n][e];
   }
 }
 
@@ -130,14 +140,15 @@ __device__ __forceinline__ void split_frag(const float (&x)[4], const float (&y)
   split_bf16x2(y[2], y[3], hi[3], lo[3]);
 }
 
-template <int MODE, int NK, bool VEC, int THREADS, int BLOCKS>
+template <int MODE, int NK, int NV, bool VEC, int THREADS, int BLOCKS>  // NV = value columns / 64, rounded up
 __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const StateScan a, const SeqDesc* __restrict__ seqs, int dvp) {
   constexpr int DKP = 16 * NK, NP = DKP / 64, LD = DKP + 8;
   constexpr bool DELTA = MODE == kScanDelta;
   using L = Lay<DKP>;
   extern __shared__ __align__(128) uint8_t chunk_smem[];
   __shared__ float sh_tot[2][4][DELTA ? DKP : 1];   // producer groups: log-decay sums of each warp's four tokens
-  __shared__ float sh_a1[2][kC][kC + 1];  // producer groups: U Ka^T, strictly lower
+  __shared__ float sh_a1[2][kC][kC + 1];  // producer groups: U Ka^T, strictly lower, ...
+  __shared__ float sh_inv[2][kC][kC + 1]; // ... and the diagonal blocks of the inverse, with the product between them
   __shared__ float sh_pow[kC + 1];
   const int buf_bytes = L::bytes(dvp), ldv = dvp + 8;
   const int n_cons = blockDim.x - kProducers;
@@ -157,7 +168,6 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
     const bf16* proj = static_cast<const bf16*>(a.proj);
     const bf16* wzp = static_cast<const bf16*>(a.wz);
     const int hk = h * a.DK, hv = h * a.DV;
-    constexpr int NV = kMaxDV / 64;  // value pairs per lane and token
     float2 wb[NP], ab[NP];
     if (DELTA) {
 #pragma unroll
@@ -167,7 +177,7 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
         ab[i] = make_float2(c < a.DK ? a.a_bias[hk + c] : 0.0f, c + 1 < a.DK ? a.a_bias[hk + c + 1] : 0.0f);
       }
     }
-    uint32_t rk[4][NP], rq[4][NP], rw[4][NP], ra[4][NP];  // raw projections of the chunk, bf16 pairs; zero for absent tokens
+    uint32_t rk[4][NP], rq[4][NP], rw[4][NP], ra[4][NP];  // raw projections of the chunk, bf16 pairs
     auto fetch = [&](int c) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
@@ -175,15 +185,14 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
         const bool in = t < seq.len;
         const size_t row = static_cast<size_t>(seq.row0) + (in ? t : 0);
         const bf16* pr = proj + row * a.ld + hk;
-        const int n = in ? a.DK : 0;
 #pragma unroll
         for (int i = 0; i < NP; ++i) {
           const int ch = 2 * lane + 64 * i;
-          rk[j][i] = ld_pair<VEC>(pr + a.off_k, ch, n);
-          rq[j][i] = ld_pair<VEC>(pr + a.off_q, ch, n);
+          rk[j][i] = ld_pair<VEC>(pr + a.off_k, ch, a.DK);
+          rq[j][i] = ld_pair<VEC>(pr + a.off_q, ch, a.DK);
           if (DELTA) {
-            rw[j][i] = ld_pair<VEC>(wzp + row * a.ld_wz + hk, ch, n);
-            ra[j][i] = ld_pair<VEC>(pr + a.off_a, ch, n);
+            rw[j][i] = ld_pair<VEC>(wzp + row * a.ld_wz + hk, ch, a.DK);
+            ra[j][i] = ld_pair<VEC>(pr + a.off_a, ch, a.DK);
           }
         }
       }
@@ -199,9 +208,16 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
         const int t = 4 * pw + j;
         const bf16* pr = proj + (static_cast<size_t>(seq.row0) + c * kC + (t < n ? t : 0)) * a.ld + a.off_v + hv;
 #pragma unroll
-        for (int i = 0; i < NV; ++i)
-          if (64 * i < dvp) rv[j][i] = ld_pair<VEC>(pr, 2 * lane + 64 * i, t < n ? a.DV : 0);
+        for (int i = 0; i < NV; ++i) rv[j][i] = ld_pair<VEC>(pr, 2 * lane + 64 * i, a.DV);
       }
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int ch = 2 * lane + 64 * i, m = 4 * pw + j < n ? a.DK : 0;
+          rk[j][i] = keep_pair(rk[j][i], ch, m);
+          rq[j][i] = keep_pair(rq[j][i], ch, m);
+        }
       float2 lw[4][NP];  // delta: running log decay over the warp's four tokens
       float inv[4];
       if (DELTA) {
@@ -262,32 +278,32 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int t = 4 * pw + j;
-          const float dr = sh_pow[t + 1], dk = t < n ? sh_pow[n - 1 - t] : 0.0f;
 #pragma unroll
           for (int i = 0; i < NP; ++i) {
             const float2 qr = f2(rq[j][i]), kr = f2(rk[j][i]);
-            const float2 q = make_float2(silu_f(qr.x), silu_f(qr.y)), k = make_float2(silu_f(kr.x), silu_f(kr.y));
             const int off = (t * LD + 2 * lane + 64 * i) * 2;
-            st_split(sb + L::tile(kU, 0), sb + L::tile(kU, 1), off, q.x, q.y);
-            st_split(sb + L::tile(kR, 0), sb + L::tile(kR, 1), off, q.x * dr, q.y * dr);
-            st_split(sb + L::tile(kKa, 0), sb + L::tile(kKa, 1), off, k.x, k.y);
-            st_split(sb + L::tile(kKk, 0), sb + L::tile(kKk, 1), off, k.x * dk, k.y * dk);
+            *reinterpret_cast<uint32_t*>(sb + L::tile(kR, 0) + off) = pack_bf16x2(silu_f(qr.x), silu_f(qr.y));
+            *reinterpret_cast<uint32_t*>(sb + L::tile(kKk, 0) + off) = pack_bf16x2(silu_f(kr.x), silu_f(kr.y));
           }
         }
       }
-      // V: copied (delta) or silu, split (decay)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        uint8_t* v_hi = sb + L::kV + (4 * pw + j) * ldv * 2;
+        const int t = 4 * pw + j;
+        uint8_t* v_row = sb + L::kV + t * ldv * 2;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
           const int x = 2 * lane + 64 * i;
           if (x >= dvp) continue;
+          const uint32_t raw = keep_pair(rv[j][i], x, t < n ? a.DV : 0);
           if (DELTA) {
-            *reinterpret_cast<uint32_t*>(v_hi + 2 * x) = rv[j][i];
+            *reinterpret_cast<uint32_t*>(v_row + 2 * x) = raw;
           } else {
-            const float2 v = f2(rv[j][i]);
-            st_split(v_hi, v_hi + kC * ldv * 2, 2 * x, silu_f(v.x), silu_f(v.y));
+            const float2 v = f2(raw);
+            const uint32_t act = pack_bf16x2(silu_f(v.x), silu_f(v.y));
+            const float w = t < n ? sh_pow[n - 1 - t] : 0.0f;
+            *reinterpret_cast<uint32_t*>(v_row + 2 * x) = act;
+            st_split(v_row + kC * ldv * 2, v_row + 2 * kC * ldv * 2, 2 * x, bf16_lo(act) * w, bf16_hi(act) * w);
           }
         }
       }
@@ -297,8 +313,8 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
       const int g = lane >> 2, cc = lane & 3;
       if (DELTA || pw == 3) {
         float acc[2][4] = {};
-        const int ta = DELTA ? (pw < 2 ? kU : kR) : kU, tb = DELTA ? ((pw & 1) ? kKk : kKa) : kKa;
-        rows_product<NK, LD>(acc, sa + L::tile(ta, 0), sa + L::tile(ta, 1), sa + L::tile(tb, 0), sa + L::tile(tb, 1), lane);
+        const int ta = DELTA && pw < 2 ? kU : kR, tb = DELTA && !(pw & 1) ? kKa : kKk;
+        rows_product<NK, LD, DELTA>(acc, sa + L::tile(ta, 0), sa + L::tile(ta, 1), sa + L::tile(tb, 0), sa + L::tile(tb, 1), lane);
 #pragma unroll
         for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
@@ -322,25 +338,45 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
           }
         if (DELTA && pw == 0) {
           __syncwarp();
-          // column (lane % 16) of the inverse of a unit lower triangular matrix, row by row
-          const int col = lane & 15;
-          float T[kC];
+          // T = [T1 0; X T2] with the inverses T1, T2 of the two unit lower triangular 8 x 8 blocks (a half-warp each, a lane
+          // per column, row by row) and X = T2 (A21 T1)
+          const int blk = lane >> 4, col = lane & 7;
+          float T[8];
 #pragma unroll
-          for (int t = 0; t < kC; ++t) {
+          for (int t = 0; t < 8; ++t) {
             float v = t == col ? 1.0f : 0.0f, v2 = 0.0f;
 #pragma unroll
             for (int s = 0; s < t; ++s) {
-              if (s & 1) v2 = fmaf(sh_a1[grp][t][s], T[s], v2);
-              else v = fmaf(sh_a1[grp][t][s], T[s], v);
+              const float m = sh_a1[grp][8 * blk + t][8 * blk + s];
+              if (s & 1) v2 = fmaf(m, T[s], v2);
+              else v = fmaf(m, T[s], v);
             }
             T[t] = v + v2;
           }
 #pragma unroll
-          for (int t = 0; t < kC; ++t) {
-            const bf16 hi = __float2bfloat16_rn(T[t]);
-            bf16* dst = reinterpret_cast<bf16*>(sb + L::mat(kT, lane < 16 ? 0 : 1)) + t * kMatLd + col;
-            *dst = lane < 16 ? hi : __float2bfloat16_rn(T[t] - __bfloat162float(hi));
+          for (int t = 0; t < 8; ++t) sh_inv[grp][8 * blk + t][8 * blk + col] = T[t];  // (two lanes, the same value)
+          __syncwarp();
+          const int xi = lane >> 2, xc = 2 * (lane & 3);
+          float2 x = make_float2(0.0f, 0.0f);
+#pragma unroll
+          for (int s = 0; s < 8; ++s) {
+            const float m = sh_a1[grp][8 + xi][s];
+            x = make_float2(fmaf(m, sh_inv[grp][s][xc], x.x), fmaf(m, sh_inv[grp][s][xc + 1], x.y));
           }
+          sh_inv[grp][8 + xi][xc] = x.x;
+          sh_inv[grp][8 + xi][xc + 1] = x.y;
+          __syncwarp();
+          float2 y = make_float2(0.0f, 0.0f);
+#pragma unroll
+          for (int s = 0; s < 8; ++s) {
+            const float m = sh_inv[grp][8 + xi][8 + s];
+            y = make_float2(fmaf(m, sh_inv[grp][8 + s][xc], y.x), fmaf(m, sh_inv[grp][8 + s][xc + 1], y.y));
+          }
+          uint8_t *hi = sb + L::mat(kT, 0), *lo = sb + L::mat(kT, 1);
+          st_split(hi, lo, (xi * kMatLd + xc) * 2, sh_inv[grp][xi][xc], sh_inv[grp][xi][xc + 1]);
+          st_split(hi, lo, (xi * kMatLd + 8 + xc) * 2, 0.0f, 0.0f);
+          st_split(hi, lo, ((8 + xi) * kMatLd + xc) * 2, y.x, y.y);
+          st_split(hi, lo, ((8 + xi) * kMatLd + 8 + xc) * 2, sh_inv[grp][8 + xi][8 + xc], sh_inv[grp][8 + xi][8 + xc + 1]);
         }
       }
       buffer_arrive<kBarFull>(grp, n_cons + kGroup);
@@ -366,6 +402,10 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
   const uint32_t to = (row_t * LD + static_cast<uint32_t>(lane >> 4) * 8) * 2;
   const uint32_t vo = (row_b * static_cast<uint32_t>(ldv) + v0 + col_b) * 2;
 
+  const bool in0 = v0 + g < a.DV, in1 = v0 + g + 8 < a.DV;
+  const int ldo = static_cast<int>(a.ldo);
+  float* orow = a.o + (static_cast<size_t>(seq.row0) + 2 * cc) * a.ldo + h * a.DV + v0 + g;
+
   for (int c = 0; c < n_chunks; ++c) {
     const int buf = c & 1, n = min(kC, seq.len - c * kC);
     const uint32_t sa = smem_u32(chunk_smem) + buf * buf_bytes;
@@ -387,13 +427,23 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
         }
       }
       ldsm_x4(bh, sa + L::tile(kR, 0) + bo + k * 32);
-      ldsm_x4(bl, sa + L::tile(kR, 1) + bo + k * 32);
+      if (DELTA) ldsm_x4(bl, sa + L::tile(kR, 1) + bo + k * 32);
 #pragma unroll
       for (int nb = 0; nb < 2; ++nb) {
         mma_bf16_16816(O[nb], sh[0], sh[1], sh[2], sh[3], bh[2 * nb], bh[2 * nb + 1]);
-        mma_bf16_16816(O2[nb], sh[0], sh[1], sh[2], sh[3], bl[2 * nb], bl[2 * nb + 1]);
+        if (DELTA) mma_bf16_16816(O2[nb], sh[0], sh[1], sh[2], sh[3], bl[2 * nb], bl[2 * nb + 1]);
         mma_bf16_16816(O2[nb], sl[0], sl[1], sl[2], sl[3], bh[2 * nb], bh[2 * nb + 1]);
       }
+    }
+    if (!DELTA) {  // the state's decay up to token t = 8 nb + 2 cc + (e & 1)
+#pragma unroll
+      for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float d = sh_pow[8 * nb + 2 * cc + (e & 1) + 1];
+          O[nb][e] *= d;
+          O2[nb][e] *= d;
+        }
     }
     uint32_t vh[4], vl[4] = {};
     ldsm_x4_trans(vh, sa + L::kV + vo);
@@ -409,19 +459,21 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
       frag_mat(Q, ph, pl, true, sa + L::mat(kT, 0), sa + L::mat(kT, 1), mo);
       split_frag(Q[0], Q[1], ph, pl);
       frag_mat(O, ph, pl, true, sa + L::mat(kB1, 0), sa + L::mat(kB1, 1), mo);
-    } else {
-      ldsm_x4_trans(vl, sa + L::kV + kC * ldv * 2 + vo);
     }
-    frag_mat(O2, vh, vl, !DELTA, sa + L::mat(kB2, 0), sa + L::mat(kB2, 1), mo);
+    frag_mat(O2, vh, vl, false, sa + L::mat(kB2, 0), sa + L::mat(kB2, 1), mo);
+    if (!DELTA) {  // from here on the values that enter the state: d^{n-1-s} v_s
+      ldsm_x4_trans(vh, sa + L::kV + kC * ldv * 2 + vo);
+      ldsm_x4_trans(vl, sa + L::kV + 2 * kC * ldv * 2 + vo);
+    }
     // ---- output: token 8 nb + 2 cc + (e & 1), value column v0 + g + 8 (e >> 1) ----
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int t = 8 * nb + 2 * cc + (e & 1), v = v0 + g + 8 * (e >> 1);
-        if (t < n && v < a.DV)
-          a.o[(static_cast<size_t>(seq.row0) + c * kC + t) * a.ldo + h * a.DV + v] = O[nb][e] + O2[nb][e];
+        const int t = 8 * nb + (e & 1);
+        if (t + 2 * cc < n && ((e >> 1) ? in1 : in0)) orow[t * ldo + 8 * (e >> 1)] = O[nb][e] + O2[nb][e];
       }
+    orow += kC * ldo;
     // ---- state ----
     const float dn = DELTA ? 1.0f : sh_pow[n];
 #pragma unroll
@@ -443,12 +495,12 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
           for (int f = 0; f < 4; ++f) S[j + e][f] *= dn;
       }
       ldsm_x4_trans(kh, sa + L::tile(kKk, 0) + to + j * 16);
-      ldsm_x4_trans(kl, sa + L::tile(kKk, 1) + to + j * 16);
+      if (DELTA) ldsm_x4_trans(kl, sa + L::tile(kKk, 1) + to + j * 16);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         mma_bf16_16816(S[j + e], vh[0], vh[1], vh[2], vh[3], kh[2 * e], kh[2 * e + 1]);
-        mma_bf16_16816(S[j + e], vh[0], vh[1], vh[2], vh[3], kl[2 * e], kl[2 * e + 1]);
-        if (!DELTA) mma_bf16_16816(S[j + e], vl[0], vl[1], vl[2], vl[3], kh[2 * e], kh[2 * e + 1]);
+        if (DELTA) mma_bf16_16816(S[j + e], vh[0], vh[1], vh[2], vh[3], kl[2 * e], kl[2 * e + 1]);
+        else mma_bf16_16816(S[j + e], vl[0], vl[1], vl[2], vl[3], kh[2 * e], kh[2 * e + 1]);
       }
       if (DELTA) {
 #pragma unroll
@@ -470,14 +522,14 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) chunk_scan_kernel(const State
     }
 }
 
-template <int MODE, int NK, bool VEC, int THREADS, int BLOCKS>
+template <int MODE, int NK, int NV, bool VEC, int THREADS, int BLOCKS>
 int launch_chunk(const StateScan& a, const SeqDesc* seqs, int n_seqs, int dvp, bool prepare_only, cudaStream_t st) {
   static std::atomic<unsigned long long> done{0};  // one bit per device; threads may race to set it
   int dev = 0;
   cudaGetDevice(&dev);
-  const auto kernel = chunk_scan_kernel<MODE, NK, VEC, THREADS, BLOCKS>;
+  const auto kernel = chunk_scan_kernel<MODE, NK, NV, VEC, THREADS, BLOCKS>;
   if (!(dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull)) {
-    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * Lay<16 * NK>::bytes(kMaxDV));
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * Lay<16 * NK>::bytes(64 * NV));
     if (e != cudaSuccess) return static_cast<int>(e);
     if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
   }
@@ -493,14 +545,15 @@ int dispatch_chunk(const StateScan& a, const SeqDesc* seqs, int n_seqs, bool pre
   const bool vec = ((a.DK | a.DV | a.off_q | a.off_k | a.off_v) & 1) == 0 && (a.ld & 1) == 0 &&
                    (a.mode != kScanDelta || ((a.off_a & 1) == 0 && (a.ld_wz & 1) == 0));
   const int dvp = (a.DV + 15) / 16 * 16;
-#define TEENY_CHUNK(NK, T, B) \
-  return vec ? launch_chunk<MODE, NK, true, T, B>(a, seqs, n_seqs, dvp, prep, st) : launch_chunk<MODE, NK, false, T, B>(a, seqs, n_seqs, dvp, prep, st)
+#define TEENY_CHUNK(NK, NV, T, B)                                                          \
+  return vec ? launch_chunk<MODE, NK, NV, true, T, B>(a, seqs, n_seqs, dvp, prep, st)      \
+             : launch_chunk<MODE, NK, NV, false, T, B>(a, seqs, n_seqs, dvp, prep, st)
   if (a.DK <= 64) {
-    if (dvp <= 64) TEENY_CHUNK(4, 384, 2);
-    TEENY_CHUNK(4, 640, 1);
+    if (dvp <= 64) TEENY_CHUNK(4, 1, 384, 2);
+    TEENY_CHUNK(4, 3, 640, 1);
   }
-  if (dvp <= 128) TEENY_CHUNK(8, 512, 1);
-  TEENY_CHUNK(8, 640, 1);
+  if (dvp <= 128) TEENY_CHUNK(8, 2, 512, 1);
+  TEENY_CHUNK(8, 3, 640, 1);
 #undef TEENY_CHUNK
 }
 
