@@ -6,6 +6,7 @@
         bench.py --gpus N --steps K --warmup W
     python bench.py --config 1|2|3|4                             # the other BASELINE configs (one GPU)
     python bench.py --impl reference ...                         # CPU arm: what the reference runs for the path
+    python bench.py --model fiferax [--size 1k|4k]               # the Fiferax decoder beside a Qwen3 of equal size (one GPU)
 
 Config 5 (default) and 4: Qwen3-8B / Qwen3-0.6B shaped greedy generation; a "step" is one full generation (prefill,
 then CUDA-graph decode steps; the first new token comes out of the prefill); value = tokens (prompt + generated) per
@@ -67,6 +68,10 @@ def parse_args():
     p.add_argument("--weights", default="bf16", choices=["bf16", "fp8"],
                    help="config 4/5 only: fp8 = projections and LM head as FP8 E4M3 with per-channel scales (weight-only; "
                         "the arithmetic stays bf16 x bf16 -> f32).  A variant beside the headline, not the headline.")
+    p.add_argument("--model", default="qwen3", choices=["qwen3", "fiferax"],
+                   help="fiferax: prefill and decode of the Fiferax decoder and its kernels beside a Qwen3 of equal size (one GPU); "
+                        "--size picks the layer sizes, --config does not apply")
+    p.add_argument("--size", default="4k", choices=["1k", "4k"])
     p.add_argument("--no-cpu-baseline", action="store_true")
     p.add_argument("--no-verify", action="store_true", help="skip the CPU-oracle check of sequence 0 after the timing")
     return p.parse_args()
@@ -727,6 +732,254 @@ def generation_config(args):
         raise SystemExit(f"parity check failed: {parity}")
 
 
+# ------------------------------------------------------------------------------------------------ the Fiferax decoder
+# Layer sizes of real models: every layer has the feed-forward of the Qwen3 it is compared with (same width, layers, heads,
+# feed-forward and vocabulary); layers cycle through delta, parallel, delta, mingru.
+FIFERAX_SIZES = {"1k": dict(width=1024, layers=24, ff=3072, heads=16, kv_heads=8, vocab=32768),
+                 "4k": dict(width=4096, layers=8, ff=12288, heads=32, kv_heads=8, vocab=32768)}
+FIFERAX_WINDOW, FIFERAX_NEW = 1024, 128
+FIFERAX_WORKLOADS = [(16, 2048), (1, 2048)]
+
+
+def fiferax_config_of(size):
+    z = FIFERAX_SIZES[size]
+    W, H = z["width"], z["heads"]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    delta = {"type": "general_delta", "mixer": {"heads": W // 64, "dim": 64}, "mlp": mlp}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": H, "kv_heads": z["kv_heads"], "dim": 128, "vdim": 128, "mask": {"size": FIFERAX_WINDOW},
+                 "rot": {"dims": 128, "base": 1e6}, "scale": 128 ** -0.5},
+        "right": {"heads": W // 128, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1 - 9.0 * i / (W // 128)) for i in range(W // 128)]},
+        "left_scale": 1.0, "right_scale": 1.0}}
+    gru = {"type": "mingru", "mixer": {"width": W}, "mlp": mlp}
+    return {"architecture": "Fiferax", "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "vocab": z["vocab"], "width": W,
+            "layers": [[delta, par, delta, gru][i % 4] for i in range(z["layers"])]}
+
+
+def fiferax_kernels(size, peaks, timed, graph_timed):
+    """The new design's kernels and the like ones of Qwen3, each alone at this size: (rows of the table)."""
+    import torch
+    from teenygrad_b200 import ops
+    from teenygrad_b200._lib import lib
+    z = FIFERAX_SIZES[size]
+    W, H, G, win = z["width"], z["heads"], z["kv_heads"], FIFERAX_WINDOW
+    B, S = FIFERAX_WORKLOADS[0]
+    T, H64, H128, D = B * S, W // 64, W // 128, 128
+    g = torch.Generator(device="cuda").manual_seed(3)
+    rnd = lambda *s: torch.randn(*s, generator=g, device="cuda")  # noqa: E731
+    bf = lambda *s: rnd(*s).bfloat16()  # noqa: E731
+    rows = []
+
+    def row(kernel, ms, bound, amount, like=None):
+        peak = peaks["hbm_gbs"] if bound == "hbm" else peaks["bf16_tflops"]
+        ach = amount / ms / (1e6 if bound == "hbm" else 1e9)
+        rows.append({"kernel": kernel, "us": ms * 1e3, "bound": bound, "achieved": ach, "unit": "GB/s" if bound == "hbm" else "TFLOP/s",
+                     "frac": ach / peak, **({"like": like} if like else {})})
+
+    whole = ops.seq_table([(b, 0, b * S, S) for b in range(B)])
+    proj = bf(T, 6 * W)
+    wz = bf(T, W)
+    bias = rnd(W)
+    offs = (0, W, 2 * W, 3 * W)
+    st64 = torch.zeros(B, H64, 64, 64, device="cuda")
+    row("state scan, delta rule (prefill)", timed(lambda: ops.state_scan_delta(proj, offs, wz, bias, bias, 0.6, 1e-6, st64, whole, S)), "hbm",
+        T * W * (5 * 2 + 4), "attention, prefill")
+    st128 = torch.zeros(B, H128, 128, 128, device="cuda")
+    decay = torch.full((H128,), 0.99, device="cuda")
+    row("state scan, scalar decay (prefill)", timed(lambda: ops.state_scan_decay(proj, offs[:3], decay, st128, whole, S)), "hbm",
+        T * W * (3 * 2 + 4), "attention, prefill")
+    o32, w32 = rnd(T, W), torch.ones(W, device="cuda")
+    row("gated norm per head", timed(lambda: ops.gated_rms_norm(o32, wz, w32, 64, 1e-5)), "hbm", T * W * 8, "residual add + norm, bf16")
+    row("gated norm over all heads", timed(lambda: ops.gated_rms_norm(o32, wz, w32, W, 1e-5)), "hbm", T * W * 8, "residual add + norm, bf16")
+    gs = torch.zeros(B, W, device="cuda")
+    row("minimal GRU scan (prefill)", timed(lambda: ops.min_gru(proj, offs[:3], bias, bias, gs, whole, S)), "hbm", T * W * 8,
+        "residual add + norm, bf16")
+    q, k = proj[:, :H * D].view(T, H, D), proj[:, H * D:(H + G) * D].view(T, G, D)
+    inv, nw = torch.rand(D // 2, device="cuda", generator=g), torch.ones(D, device="cuda")
+    row("head norm + rotary, f32 angles", timed(lambda: ops.head_norm_rope(q, k, nw, nw, inv, D, 1e-5, whole, S)), "hbm",
+        2 * 2 * T * (H + G) * D, "head norm + rotary + cache, bf16 tables")
+    kr, vr = (torch.zeros(B, G, win, D, dtype=torch.bfloat16, device="cuda") for _ in range(2))
+    kc = k.contiguous()
+    seen = sum(min(i + 1, win) for i in range(S))
+    row("windowed attention (prefill) + ring append", timed(lambda: ops.window_attention(q, kc, k, kr, vr, win, D ** -0.5, whole, S,
+                                                                                         uniform_fresh=True)),
+        "tensor", 4.0 * B * H * D * seen, "attention, prefill")
+    x32, delta = rnd(T, W), bf(T, W)
+    row("residual add + norm, f32 residual", timed(lambda: ops.residual_rms_norm(x32, delta, w32, 1e-5)), "hbm", T * W * 12,
+        "residual add + norm, bf16")
+    # one token per sequence, batch 32, states / caches rotated beyond L2
+    n, copies = 32, 8
+    one = ops.seq_table([(b, S, b, 1) for b in range(n)])
+    p1, z1 = proj[:n], wz[:n]
+    s64 = [torch.zeros(n, H64, 64, 64, device="cuda") for _ in range(copies)]
+    row("state step, delta rule (decode)", graph_timed([(lambda s=s: ops.state_scan_delta(p1, offs, z1, bias, bias, 0.6, 1e-6, s, one, 1))
+                                                        for s in s64]), "hbm", 2.0 * n * H64 * 64 * 64 * 4, "attention, decode")
+    del s64
+    s128 = [torch.zeros(n, H128, 128, 128, device="cuda") for _ in range(copies)]
+    row("state step, scalar decay (decode)", graph_timed([(lambda s=s: ops.state_scan_decay(p1, offs[:3], decay, s, one, 1)) for s in s128]),
+        "hbm", 2.0 * n * H128 * 128 * 128 * 4, "attention, decode")
+    del s128
+    # decode attention over full rings: min(pos + 1, window) keys
+    from teenygrad_b200.ops import flash_attn_decode, flash_attn_fwd
+    for length, name in ((win, "attention, decode (ring of the window)"), (S, "attention, decode")):
+        kvs = [(bf(n, G, length, D), bf(n, G, length, D)) for _ in range(6)]
+        q1 = bf(n, H, 1, D)
+        o1 = torch.empty_like(q1)
+        sc = torch.empty(lib.teeny_attn_decode_scratch_bytes(n, H, D, length), dtype=torch.uint8, device="cuda")
+        row(name, graph_timed([(lambda kk=kk, vv=vv: flash_attn_decode(q1, kk, vv, length, D ** -0.5, out=o1, scratch=sc)) for kk, vv in kvs]),
+            "hbm", 2.0 * n * G * length * D * 2, "attention, decode" if length == win else None)
+        del kvs
+    # Qwen3's like kernels
+    qa, ka = bf(B, H, S, D), bf(B, G, S, D)
+    row("attention, prefill", timed(lambda: flash_attn_fwd(qa, ka, ka, D ** -0.5, causal=True)), "tensor", 0.5 * 4 * B * H * S * S * D)
+    xr, w16 = bf(T, W), torch.ones(W, dtype=torch.bfloat16, device="cuda")
+    row("residual add + norm, bf16", timed(lambda: ops.add_rms_norm(delta, xr, w16, 1e-5)), "hbm", T * W * 8)
+    cos, sin = ops.rope_table(inv, S)
+    qkv, n16 = bf(T, (H + 2 * G) * D), torch.ones(D, dtype=torch.bfloat16, device="cuda")
+    kk, vv = (torch.zeros(B, G, S, D, dtype=torch.bfloat16, device="cuda") for _ in range(2))
+    row("head norm + rotary + cache, bf16 tables", timed(lambda: ops.qk_norm_rope_kv(qkv, n16, n16, cos, sin, kk, vv, S, H, G, 0, 1e-6)), "hbm",
+        2.0 * T * D * (2 * H + 4 * G))
+    return rows
+
+
+def fiferax_bench(args):
+    import torch
+    from teenygrad_b200 import fiferax, qwen3
+    from teenygrad_b200._lib import lib
+    if args.gpus != 1 or args.impl != "ours":
+        raise SystemExit("--model fiferax runs on one GPU")
+    torch.cuda.set_device(0)
+    peaks, z, NEW = measured_peaks(), FIFERAX_SIZES[args.size], FIFERAX_NEW
+    cfg = fiferax_config_of(args.size)
+    warm = max(args.warmup, 3)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def timed(fn, steps=5):
+        for _ in range(3):
+            fn()
+        total = 0.0
+        for _ in range(steps):
+            flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            total += a.elapsed_time(b)
+        return total / steps
+
+    def graph_timed(fns, reps=5):
+        st = torch.cuda.Stream()
+        with torch.cuda.stream(st):
+            for f in fns:
+                f()
+            torch.cuda.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph, stream=st):
+                for f in fns:
+                    f()
+            for _ in range(3):
+                graph.replay()
+            torch.cuda.synchronize()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            for _ in range(reps):
+                graph.replay()
+            b.record()
+            torch.cuda.synchronize()
+        return a.elapsed_time(b) / reps / len(fns)
+
+    def phases(prefill, decode, steps):
+        for _ in range(warm):
+            prefill()
+            for _ in range(3):
+                decode()
+        ev = [[torch.cuda.Event(enable_timing=True) for _ in range(3)] for _ in range(steps)]
+        torch.cuda.synchronize()
+        for e in ev:
+            e[0].record()
+            prefill()
+            e[1].record()
+            for _ in range(NEW - 1):
+                decode()
+            e[2].record()
+        torch.cuda.synchronize()
+        return [sum(e[i].elapsed_time(e[i + 1]) for e in ev) / steps for i in range(2)]
+
+    def matmul_params(model):
+        if model == "qwen3":
+            return z["layers"] * (z["width"] * (2 * z["heads"] + 2 * z["kv_heads"]) * 128 + 3 * z["width"] * z["ff"]) + z["vocab"] * z["width"]
+        shapes = fiferax.tensor_shapes(cfg, z["width"] // 32)
+        return sum(s[0] * s[1] for n, s in shapes.items() if len(s) == 2 and n != "embed")
+
+    sampler = ClockSampler(0)
+    sampler.start()
+    results, launches, e2e = [], 0, None
+    for B, S in FIFERAX_WORKLOADS:
+        g = torch.Generator().manual_seed(6)
+        host = torch.randint(0, z["vocab"], (B, S), generator=g, dtype=torch.int32).pin_memory()
+        dev = host.cuda()
+        entry = {"batch": B, "prefill": S, "new_tokens": NEW}
+        for model in ("fiferax", "qwen3"):
+            if model == "fiferax":
+                r = fiferax.build(cfg, fiferax.RandomTensors(cfg, 7, "cuda", z["width"] // 32), max_batch=B, max_len=S + NEW, max_tokens=B * S,
+                                  max_new_tokens=NEW)
+                seqs = [r.open() for _ in range(B)]
+
+                def prefill():
+                    for s in seqs:
+                        s.pos = 0
+                    r.prefill(dev, seqs)
+            else:
+                r = qwen3.Qwen3Runner(qwen3.Qwen3Config(z["layers"], z["width"], z["heads"], z["kv_heads"], 128, z["ff"], z["vocab"]), max_batch=B,
+                                      max_len=S + NEW, max_tokens=B * S, max_new_tokens=NEW)
+                qwen3.load_random_weights(r, 7)
+
+                def prefill():
+                    r.prefill(dev)
+            lib.teeny_launch_count(1)
+            pre, dec = phases(prefill, lambda: r.decode_step(graph=True), args.steps)
+            if model == "fiferax":
+                launches += int(lib.teeny_launch_count(1))
+            entry[model] = {"prefill_ms": pre, "decode_ms_per_step": dec / (NEW - 1), "prefill_tok_s": B * S / pre * 1e3,
+                            "decode_tok_s": B * (NEW - 1) / dec * 1e3, "tok_s": B * (S + NEW) / (pre + dec) * 1e3,
+                            "matmul_params": matmul_params(model),
+                            "prefill_matmul_tflops": 2.0 * matmul_params(model) * B * S / pre / 1e9,
+                            "decode_weight_gbs": 2.0 * matmul_params(model) / (dec / (NEW - 1)) / 1e6}
+            if model == "fiferax" and e2e is None:
+                for s in seqs:
+                    r.close(s)
+                out = torch.empty(B, NEW, dtype=torch.int32).pin_memory()
+
+                def once():
+                    out.copy_(r.generate(host.to("cuda", non_blocking=True), NEW), non_blocking=True)
+                    torch.cuda.current_stream().synchronize()
+                once()
+                t0 = time.perf_counter()
+                for _ in range(args.steps):
+                    once()
+                e2e = {"value": B * (S + NEW) * args.steps / (time.perf_counter() - t0), "unit": "tok/s", "h2d_bytes_per_step": host.numel() * 4,
+                       "d2h_bytes_per_step": out.numel() * 4}
+            if r.device_error():
+                raise SystemExit("device error word set")
+            del r
+            torch.cuda.empty_cache()
+        results.append(entry)
+    clocks = sampler.stop()
+    kernels = fiferax_kernels(args.size, peaks, timed, graph_timed)
+    first = results[0]
+    emit({"metric": "fiferax_tokens_per_s", "value": first["fiferax"]["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+          "warmup": args.warmup, "warmup_run": warm,
+          "ms_per_step": first["fiferax"]["prefill_ms"] + first["fiferax"]["decode_ms_per_step"] * (NEW - 1), "higher_is_better": True,
+          "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+          "config": {"workload": f"Fiferax {args.size}: width {z['width']}, {z['layers']} layers (delta, parallel, delta, mingru), window "
+                                 f"{FIFERAX_WINDOW}, feed-forward {z['ff']}, vocabulary {z['vocab']}, random weights; beside a Qwen3 of the same "
+                                 "width, layers, heads, feed-forward and vocabulary", "parallelism": "1 GPU",
+                     "l2": "inputs larger than L2; kernels alone: L2 flushed before every timed launch, one-token kernels replayed from a graph "
+                           "over state copies larger than L2"},
+          "workloads": results, "kernels": kernels, "e2e": e2e, "gpu_launches": launches, "clocks": clocks})
+
+
 def main():
     args = parse_args()
     # Keep stdout to the one JSON line: libraries write there at the file-descriptor level (NCCL prints its version
@@ -736,7 +989,9 @@ def main():
     sys.stdout.flush()
     _JSON_OUT = os.fdopen(os.dup(1), "w")
     os.dup2(2, 1)
-    if args.impl == "reference":
+    if args.model == "fiferax":
+        fiferax_bench(args)
+    elif args.impl == "reference":
         reference_arm(args)
     elif args.config in (4, 5):
         generation_config(args)

@@ -114,6 +114,40 @@ int teeny_hybrid_capture_decode(teeny_hybrid* model, teeny_stream_t stream);
 int teeny_hybrid_decode_replay(teeny_hybrid* model, teeny_stream_t stream);
 void* teeny_hybrid_buffer(teeny_hybrid* model, int which);
 
+/* The runner's kernels on their own.  seqs: device int32 [n_seqs][4] = {slot, position of the first token, first row, tokens}
+ * per entry; max_len: the longest entry.  f32: element type of the void pointers (0 bf16, 1 f32).  Row strides and column
+ * offsets are in elements.
+ *
+ * Matrix-state recurrences over [slots, heads, dk, dv] f32 states; o [rows, ldo] f32, head h at column h * dv.  mode 0:
+ * generalized delta rule (proj columns off_q, off_k, off_v, off_a; wz the decay's low-rank product; w_bias, a_bias [heads * dk]);
+ * mode 1: scalar decay per head with silu on q, k, v. */
+int teeny_state_scan(int mode, int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, int off_a, const void* wz,
+                     long long ld_wz, const float* w_bias, const float* a_bias, const float* decay, float decay_coef,
+                     float unit_eps, float* state, float* o, long long ldo, int heads, int dk, int dv, const int* seqs,
+                     int n_seqs, int max_len, teeny_stream_t stream);
+/* out = o / rms(groups of group_size columns) * weight * sigmoid(gate) * scale */
+int teeny_gated_rms_norm(int f32, const float* o, long long ldo, const void* gate, long long ldg, const float* weight, void* out,
+                         long long ldout, int rows, int cols, int group_size, float eps, float scale, teeny_stream_t stream);
+/* Element-wise gated recurrence with the z, x and gate columns of proj; state [slots, width] f32. */
+int teeny_min_gru(int f32, const void* proj, long long ld, int off_z, int off_x, int off_g, const float* z_bias, const float* x_bias,
+                  float* state, void* out, long long ldout, int width, float scale, const int* seqs, int n_seqs, int max_len,
+                  teeny_stream_t stream);
+/* Per-head RMS norm (q_weight / k_weight [dim] f32, or null for none) and rotate-half positions on the first rot_dims
+ * dimensions: q [rows, ldq] in place, k_raw -> k_out; angles position * inv_freq[i] in f32. */
+int teeny_head_norm_rope(int f32, void* q, long long ldq, const void* k_raw, long long ldkr, void* k_out, long long ldk,
+                         const float* q_weight, const float* k_weight, const float* inv_freq, int heads, int kv_heads, int dim,
+                         int rot_dims, float eps, const int* seqs, int n_seqs, int max_len, teeny_stream_t stream);
+/* Sliding-window attention of every entry's tokens over the ring caches [slots, kv_heads, ring, dim] (keys older than the
+ * entry) and the entry's own k_new / v_new rows, which are then appended to the rings.  uniform_fresh: the entries are whole
+ * prompts of one length from position 0, rows in order (a faster kernel for head size 128). */
+int teeny_window_attention(int f32, const void* q, long long ldq, const void* k_new, long long ldk, const void* v_new, long long ldv,
+                           void* k_ring, void* v_ring, int slots, int ring, int window, void* out, long long ldo, int heads,
+                           int kv_heads, int dim, int vdim, float score_scale, float out_scale, int uniform_fresh,
+                           const int* seqs, int n_seqs, int max_len, teeny_stream_t stream);
+/* x [rows, n] f32 += delta (or null); y = rms_norm(x) * weight. */
+int teeny_residual_rms_norm(int f32, float* x, const void* delta, long long ldd, void* y, long long ldy, const float* weight, int rows,
+                            int n, float eps, teeny_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

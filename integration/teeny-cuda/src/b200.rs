@@ -258,6 +258,12 @@ extern "C" {
     pub fn teeny_hybrid_capture_decode(model: *mut TeenyHybrid, stream: CUstream) -> c_int;
     pub fn teeny_hybrid_decode_replay(model: *mut TeenyHybrid, stream: CUstream) -> c_int;
     pub fn teeny_hybrid_buffer(model: *mut TeenyHybrid, which: c_int) -> *mut c_void;
+    pub fn teeny_state_scan(mode: c_int, f32: c_int, proj: *const c_void, ld: c_longlong, off_q: c_int, off_k: c_int, off_v: c_int, off_a: c_int, wz: *const c_void, ld_wz: c_longlong, w_bias: *const f32, a_bias: *const f32, decay: *const f32, decay_coef: f32, unit_eps: f32, state: *mut f32, o: *mut f32, ldo: c_longlong, heads: c_int, dk: c_int, dv: c_int, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_gated_rms_norm(f32: c_int, o: *const f32, ldo: c_longlong, gate: *const c_void, ldg: c_longlong, weight: *const f32, out: *mut c_void, ldout: c_longlong, rows: c_int, cols: c_int, group_size: c_int, eps: f32, scale: f32, stream: CUstream) -> c_int;
+    pub fn teeny_min_gru(f32: c_int, proj: *const c_void, ld: c_longlong, off_z: c_int, off_x: c_int, off_g: c_int, z_bias: *const f32, x_bias: *const f32, state: *mut f32, out: *mut c_void, ldout: c_longlong, width: c_int, scale: f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_head_norm_rope(f32: c_int, q: *mut c_void, ldq: c_longlong, k_raw: *const c_void, ldkr: c_longlong, k_out: *mut c_void, ldk: c_longlong, q_weight: *const f32, k_weight: *const f32, inv_freq: *const f32, heads: c_int, kv_heads: c_int, dim: c_int, rot_dims: c_int, eps: f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_window_attention(f32: c_int, q: *const c_void, ldq: c_longlong, k_new: *const c_void, ldk: c_longlong, v_new: *const c_void, ldv: c_longlong, k_ring: *mut c_void, v_ring: *mut c_void, slots: c_int, ring: c_int, window: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, kv_heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, out_scale: f32, uniform_fresh: c_int, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_residual_rms_norm(f32: c_int, x: *mut f32, delta: *const c_void, ldd: c_longlong, y: *mut c_void, ldy: c_longlong, weight: *const f32, rows: c_int, n: c_int, eps: f32, stream: CUstream) -> c_int;
 }
 // ---- generated from include/*.h: end ----
 

@@ -67,6 +67,14 @@ SIGNATURES = {
     "teeny_argmax_combine": (i32, [vp, vp, vp, i32, i32, vp]),
     "teeny_sample_top_k_top_p_bf16": (i32, [vp, i64, i32, i32, f32, i32, f32, vp, vp, vp, vp]),
     "teeny_sample_candidates_bf16": (i32, [vp, i64, i32, i32, i32, i32, vp, vp]),
+    # kernels of the hybrid decoders (include/teeny_hybrid.h)
+    "teeny_state_scan": (i32, [i32, i32, vp, i64] + [i32] * 4 + [vp, i64, vp, vp, vp, f32, f32, vp, vp, i64] + [i32] * 3 + [vp, i32, i32, vp]),
+    "teeny_gated_rms_norm": (i32, [i32, vp, i64, vp, i64, vp, vp, i64, i32, i32, i32, f32, f32, vp]),
+    "teeny_min_gru": (i32, [i32, vp, i64, i32, i32, i32, vp, vp, vp, vp, i64, i32, f32, vp, i32, i32, vp]),
+    "teeny_head_norm_rope": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, f32, vp, i32, i32, vp]),
+    "teeny_window_attention": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i32, i32, i32, vp, i64, i32, i32, i32, i32, f32, f32, i32,
+                                     vp, i32, i32, vp]),
+    "teeny_residual_rms_norm": (i32, [i32, vp, vp, i64, vp, i64, vp, i32, i32, f32, vp]),
     "teeny_sample_merge": (i32, [vp, i32, sz, i32, f32, i32, f32, vp, vp, vp, vp]),
 }
 

@@ -589,4 +589,79 @@ void* teeny_hybrid_buffer(teeny_hybrid* m, int which) {
   }
 }
 
+// ---- the kernels on their own ----
+int teeny_state_scan(int mode, int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, int off_a, const void* wz,
+                     long long ld_wz, const float* w_bias, const float* a_bias, const float* decay, float decay_coef,
+                     float unit_eps, float* state, float* o, long long ldo, int heads, int dk, int dv, const int* seqs,
+                     int n_seqs, int max_len, teeny_stream_t stream) {
+  if (mode != kScanDelta && mode != kScanDecay) return TEENY_ERR_BAD_ARG;
+  TEENY_TRY(state_scan_prepare());
+  StateScan a{};
+  a.mode = mode; a.f32 = f32;
+  a.proj = proj; a.ld = ld;
+  a.off_q = off_q; a.off_k = off_k; a.off_v = off_v; a.off_a = off_a;
+  a.wz = wz; a.ld_wz = ld_wz;
+  a.w_bias = w_bias; a.a_bias = a_bias; a.decay = decay;
+  a.decay_coef = decay_coef; a.unit_eps = unit_eps;
+  a.state = state;
+  a.o = o; a.ldo = ldo;
+  a.H = heads; a.DK = dk; a.DV = dv;
+  return state_scan(a, reinterpret_cast<const SeqDesc*>(seqs), n_seqs, max_len, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int teeny_gated_rms_norm(int f32, const float* o, long long ldo, const void* gate, long long ldg, const float* weight, void* out,
+                         long long ldout, int rows, int cols, int group_size, float eps, float scale, teeny_stream_t stream) {
+  return gated_rms_norm(o, ldo, gate, ldg, weight, out, ldout, rows, cols, group_size, eps, scale, f32 != 0,
+                        reinterpret_cast<cudaStream_t>(stream));
+}
+
+int teeny_min_gru(int f32, const void* proj, long long ld, int off_z, int off_x, int off_g, const float* z_bias, const float* x_bias,
+                  float* state, void* out, long long ldout, int width, float scale, const int* seqs, int n_seqs, int max_len,
+                  teeny_stream_t stream) {
+  const MinGru a{f32, proj, ld, off_z, off_x, off_g, z_bias, x_bias, state, out, ldout, width, scale};
+  return min_gru(a, reinterpret_cast<const SeqDesc*>(seqs), n_seqs, max_len, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int teeny_head_norm_rope(int f32, void* q, long long ldq, const void* k_raw, long long ldkr, void* k_out, long long ldk,
+                         const float* q_weight, const float* k_weight, const float* inv_freq, int heads, int kv_heads, int dim,
+                         int rot_dims, float eps, const int* seqs, int n_seqs, int max_len, teeny_stream_t stream) {
+  HeadNormRope a{};
+  a.f32 = f32;
+  a.q = q; a.ldq = ldq;
+  a.k_raw = k_raw; a.ldkr = ldkr;
+  a.k_out = k_out; a.ldk = ldk;
+  a.q_w = q_weight; a.k_w = k_weight; a.inv_freq = inv_freq;
+  a.Hq = heads; a.Hkv = kv_heads; a.D = dim; a.rot_dims = rot_dims;
+  a.eps = eps;
+  return head_norm_rope_rows(a, reinterpret_cast<const SeqDesc*>(seqs), n_seqs, max_len, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int teeny_window_attention(int f32, const void* q, long long ldq, const void* k_new, long long ldk, const void* v_new, long long ldv,
+                           void* k_ring, void* v_ring, int slots, int ring, int window, void* out, long long ldo, int heads,
+                           int kv_heads, int dim, int vdim, float score_scale, float out_scale, int uniform_fresh,
+                           const int* seqs, int n_seqs, int max_len, teeny_stream_t stream) {
+  if (slots <= 0) return TEENY_ERR_BAD_ARG;
+  WindowAttn a{};
+  a.f32 = f32;
+  a.q = q; a.ldq = ldq;
+  a.k_new = k_new; a.ldk = ldk;
+  a.v_new = v_new; a.ldv = ldv;
+  a.k_ring = k_ring; a.v_ring = v_ring;
+  a.ring = ring; a.window = window;
+  a.out = out; a.ldo = ldo;
+  a.Hq = heads; a.Hkv = kv_heads; a.D = dim; a.DV = vdim;
+  a.scale = score_scale; a.out_scale = out_scale;
+  a.slots = slots;
+  a.uniform_fresh = uniform_fresh;
+  const SeqDesc* sq = reinterpret_cast<const SeqDesc*>(seqs);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  TEENY_TRY(window_attention(a, sq, n_seqs, max_len, st));
+  return ring_append(a, sq, n_seqs, max_len, st);
+}
+
+int teeny_residual_rms_norm(int f32, float* x, const void* delta, long long ldd, void* y, long long ldy, const float* weight, int rows,
+                            int n, float eps, teeny_stream_t stream) {
+  return residual_rms_norm(x, delta, ldd, y, ldy, weight, rows, n, eps, nullptr, f32 != 0, reinterpret_cast<cudaStream_t>(stream));
+}
+
 }  // extern "C"

@@ -378,18 +378,20 @@ __global__ void gated_rms_norm_kernel(const float* __restrict__ o, long long ldo
 // a CTA takes TS consecutive tokens of 64 channels (a pair per lane), composes their maps, the compositions meet in shared
 // memory, and every warp finishes its own tokens from the state that enters them.  The raw projections of the next tile are
 // requested before the exchange. ----
+// Two neighbouring elements as loaded: converted where they are used, not where they are requested.
+template <typename T> struct Pair;
+template <> struct Pair<float> { typedef float2 raw; static __device__ float2 f(raw v) { return v; } };
+template <> struct Pair<bf16> { typedef uint32_t raw; static __device__ float2 f(raw v) { return make_float2(bf16_lo(v), bf16_hi(v)); } };
 template <bool VEC>
 __device__ __forceinline__ float2 ld_two(const float* p, bool second) {
   if (VEC) return *reinterpret_cast<const float2*>(p);
   return make_float2(p[0], second ? p[1] : 0.0f);
 }
 template <bool VEC>
-__device__ __forceinline__ float2 ld_two(const bf16* p, bool second) {
-  if (VEC) {
-    const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
-    return make_float2(bf16_lo(v), bf16_hi(v));
-  }
-  return make_float2(__bfloat162float(p[0]), second ? __bfloat162float(p[1]) : 0.0f);
+__device__ __forceinline__ uint32_t ld_two(const bf16* p, bool second) {
+  if (VEC) return *reinterpret_cast<const uint32_t*>(p);
+  const uint16_t* q = reinterpret_cast<const uint16_t*>(p);
+  return q[0] | (second ? static_cast<uint32_t>(q[1]) << 16 : 0u);
 }
 template <bool VEC>
 __device__ __forceinline__ void st_two(float* p, float2 v, bool second) {
@@ -404,11 +406,15 @@ __device__ __forceinline__ void st_two(bf16* p, float2 v, bool second) {
   if (second) p[1] = __float2bfloat16_rn(v.y);
 }
 
-__device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_f(u); }
+// sigmoid at the accuracy the element type calls for: f32 models get the full-precision functions
+template <typename T> __device__ __forceinline__ float sigmoid_as(float x);
+template <> __device__ __forceinline__ float sigmoid_as<float>(float x) { return sigmoid_f(x); }
+template <> __device__ __forceinline__ float sigmoid_as<bf16>(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+template <typename T> __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_as<T>(u); }
 
 template <typename T, int TS, bool VEC>
-__global__ void __launch_bounds__(256) min_gru_kernel(const MinGru a, const SeqDesc* __restrict__ seqs) {
-  __shared__ float2 sA[2][8][32], sB[2][8][32];
+__global__ void __launch_bounds__(512) min_gru_kernel(const MinGru a, const SeqDesc* __restrict__ seqs) {
+  __shared__ float2 sA[2][16][32], sB[2][16][32];
   const SeqDesc seq = seqs[blockIdx.y];  // written well before the kernel in front of this one
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const int ch = blockIdx.x * 64 + 2 * lane;
@@ -422,7 +428,7 @@ __global__ void __launch_bounds__(256) min_gru_kernel(const MinGru a, const SeqD
   float2 S = make_float2(0.0f, 0.0f);
   if (seq.pos > 0) S = make_float2(st[0], second ? st[1] : 0.0f);
   const int tile = warps * TS;
-  float2 z[TS], u[TS], g[TS];
+  typename Pair<T>::raw z[TS], u[TS], g[TS];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < TS; ++i) {
@@ -440,11 +446,12 @@ __global__ void __launch_bounds__(256) min_gru_kernel(const MinGru a, const SeqD
     float2 A[TS], B[TS], G[TS], pa = make_float2(1.0f, 1.0f), pb = make_float2(0.0f, 0.0f);
 #pragma unroll
     for (int i = 0; i < TS; ++i) {
-      const float2 zz = make_float2(sigmoid_f(z[i].x + zb.x), sigmoid_f(z[i].y + zb.y));
+      const float2 zr = Pair<T>::f(z[i]), ur = Pair<T>::f(u[i]), gr = Pair<T>::f(g[i]);
+      const float2 zz = make_float2(sigmoid_as<T>(zr.x + zb.x), sigmoid_as<T>(zr.y + zb.y));
       const bool on = first + i < seq.len;
       A[i] = on ? make_float2(1.0f - zz.x, 1.0f - zz.y) : make_float2(1.0f, 1.0f);
-      B[i] = on ? make_float2(zz.x * gru_candidate(u[i].x + xb.x), zz.y * gru_candidate(u[i].y + xb.y)) : make_float2(0.0f, 0.0f);
-      G[i] = make_float2(silu_f(g[i].x) * a.scale, silu_f(g[i].y) * a.scale);
+      B[i] = on ? make_float2(zz.x * gru_candidate<T>(ur.x + xb.x), zz.y * gru_candidate<T>(ur.y + xb.y)) : make_float2(0.0f, 0.0f);
+      G[i] = make_float2(gr.x * sigmoid_as<T>(gr.x) * a.scale, gr.y * sigmoid_as<T>(gr.y) * a.scale);
       pa = make_float2(pa.x * A[i].x, pa.y * A[i].y);
       pb = make_float2(fmaf(A[i].x, pb.x, B[i].x), fmaf(A[i].y, pb.y, B[i].y));
     }
@@ -706,7 +713,7 @@ int launch_min_gru(const MinGru& a, const SeqDesc* seqs, int n_seqs, int max_len
   const dim3 grid((a.W + 63) / 64, n_seqs);
   const bool vec = ((a.W | a.off_z | a.off_x | a.off_g) & 1) == 0 && ((a.ld | a.ldout) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 7) == 0;
   int warps = (max_len + TS - 1) / TS;
-  if (warps > 8) warps = 8;
+  if (warps > 16) warps = 16;
 #define TEENY_GRU(N) \
   vec ? launch_kernel(min_gru_kernel<T, N, true>, grid, dim3(32 * warps), 0, st, 1, a, seqs) \
       : launch_kernel(min_gru_kernel<T, N, false>, grid, dim3(32 * warps), 0, st, 1, a, seqs)

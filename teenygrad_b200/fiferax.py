@@ -5,6 +5,7 @@ Three token mixers in any order, each behind a pre-norm and optionally followed 
 scalar-decay linear attention) and ``mingru``.
 """
 import math
+import zlib
 
 import torch
 
@@ -78,3 +79,46 @@ def build(config, tensors, dtype=torch.bfloat16, **sizes):
     runner = hybrid.HybridRunner(cfg, dtype=dtype, **sizes)
     load_weights(runner, config, tensors)
     return runner
+
+
+def tensor_shapes(config, rank):
+    """name -> shape of every tensor of a checkpoint; ``rank``: rows of the decay factors ``w1``."""
+    d = config["width"]
+    out = {"embed": (config["vocab"], d), "final.norm": (d,), "head": (config["vocab"], d)}
+    for i, layer in enumerate(config["layers"]):
+        out[f"l{i}.norm1"] = (d,)
+        for b, side in zip(_branches(layer, rank), ("left.", "right.") if layer["type"] == "parallel" else ("",)):
+            p = f"l{i}.mix.{side}"
+            names = {hybrid.ATTENTION: "qk", hybrid.DELTA: "rkvag", hybrid.DECAY: "qkvg", hybrid.MIN_GRU: "zxg"}[b.kind]
+            out.update({p + n: (rows, d) for n, rows in zip(names, b.input_sizes())})
+            out[p + "o"] = (d, b.output_size())
+            n = b.heads * b.dim
+            if b.kind == hybrid.ATTENTION:
+                out.update({p + "q.norm": (b.dim,), p + "k.norm": (b.dim,)})
+            elif b.kind == hybrid.MIN_GRU:
+                out.update({p + "z.b": (n,), p + "x.b": (n,)})
+            else:
+                out[p + "norm"] = (b.output_size(),)
+            if b.kind == hybrid.DELTA:
+                out.update({p + "w1": (rank, d), p + "w2": (n, rank), p + "w0": (n,), p + "a.b": (n,)})
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            out.update({f"l{i}.norm2": (d,), f"l{i}.mlp.gate": (ff, d), f"l{i}.mlp.up": (ff, d), f"l{i}.mlp.down": (d, ff)})
+    return out
+
+
+class RandomTensors:
+    """Seeded random bf16 checkpoint tensors, made on ``device`` when asked for: matrices of unit gain, norms around 1."""
+
+    def __init__(self, config, seed, device, rank):
+        self.shapes, self.seed, self.device = tensor_shapes(config, rank), seed, device
+
+    def __getitem__(self, name):
+        shape = self.shapes[name]
+        g = torch.Generator(device=self.device).manual_seed(self.seed * 1000003 + zlib.crc32(name.encode()))
+        t = torch.randn(*shape, generator=g, device=self.device)
+        if len(shape) == 2:
+            t *= shape[1] ** -0.5
+        elif "norm" in name:
+            t = 1.0 + 0.1 * t
+        return t.to(torch.bfloat16)

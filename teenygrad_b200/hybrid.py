@@ -126,7 +126,7 @@ def pad_to(n, m):
 def fuse_rows(parts, dtype):
     """Matrices stacked with every part starting at a multiple of 8 rows, rows padded to a multiple of 8 columns."""
     k = parts[0].shape[1]
-    out = torch.zeros(sum(pad_to(p.shape[0], 8) for p in parts), pad_to(k, 8), dtype=dtype)
+    out = torch.zeros(sum(pad_to(p.shape[0], 8) for p in parts), pad_to(k, 8), dtype=dtype, device=parts[0].device)
     r = 0
     for p in parts:
         out[r:r + p.shape[0], :k] = p
@@ -136,7 +136,7 @@ def fuse_rows(parts, dtype):
 
 def fuse_columns(parts, dtype):
     """Matrices side by side with every part starting at a multiple of 8 columns."""
-    out = torch.zeros(parts[0].shape[0], sum(pad_to(p.shape[1], 8) for p in parts), dtype=dtype)
+    out = torch.zeros(parts[0].shape[0], sum(pad_to(p.shape[1], 8) for p in parts), dtype=dtype, device=parts[0].device)
     c = 0
     for p in parts:
         out[:, c:c + p.shape[1]] = p
@@ -148,13 +148,13 @@ def interleave_glu(gate, up, dtype):
     """Gate and up rows in alternating blocks of 64, zero rows beyond the feed-forward size; columns padded to 8."""
     ff, k = gate.shape
     f = pad_to(ff, 64)
-    both = torch.zeros(2, f, pad_to(k, 8), dtype=dtype)
+    both = torch.zeros(2, f, pad_to(k, 8), dtype=dtype, device=gate.device)
     both[0, :ff, :k], both[1, :ff, :k] = gate, up
     return both.view(2, f // 64, 64, -1).transpose(0, 1).reshape(2 * f, -1).contiguous()
 
 
 def pad_columns(w, multiple, dtype):
-    out = torch.zeros(w.shape[0], pad_to(w.shape[1], multiple), dtype=dtype)
+    out = torch.zeros(w.shape[0], pad_to(w.shape[1], multiple), dtype=dtype, device=w.device)
     out[:, :w.shape[1]] = w
     return out
 
