@@ -782,27 +782,28 @@ def fiferax_kernels(size, peaks, timed, graph_timed):
     bias = rnd(W)
     offs = (0, W, 2 * W, 3 * W)
     st64 = torch.zeros(B, H64, 64, 64, device="cuda")
-    row("state scan, delta rule (prefill)", timed(lambda: ops.state_scan_delta(proj, offs, wz, bias, bias, 0.6, 1e-6, st64, whole, S)), "hbm",
+    o32, o16 = rnd(T, W), bf(T, W)
+    row("state scan, delta rule (prefill)", timed(lambda: ops.state_scan_delta(proj, offs, wz, bias, bias, 0.6, 1e-6, st64, whole, S, out=o32)), "hbm",
         T * W * (5 * 2 + 4), "attention, prefill")
     st128 = torch.zeros(B, H128, 128, 128, device="cuda")
     decay = torch.full((H128,), 0.99, device="cuda")
-    row("state scan, scalar decay (prefill)", timed(lambda: ops.state_scan_decay(proj, offs[:3], decay, st128, whole, S)), "hbm",
+    row("state scan, scalar decay (prefill)", timed(lambda: ops.state_scan_decay(proj, offs[:3], decay, st128, whole, S, out=o32)), "hbm",
         T * W * (3 * 2 + 4), "attention, prefill")
-    o32, w32 = rnd(T, W), torch.ones(W, device="cuda")
-    row("gated norm per head", timed(lambda: ops.gated_rms_norm(o32, wz, w32, 64, 1e-5)), "hbm", T * W * 8, "residual add + norm, bf16")
-    row("gated norm over all heads", timed(lambda: ops.gated_rms_norm(o32, wz, w32, W, 1e-5)), "hbm", T * W * 8, "residual add + norm, bf16")
+    w32 = torch.ones(W, device="cuda")
+    row("gated norm per head", timed(lambda: ops.gated_rms_norm(o32, wz, w32, 64, 1e-5, out=o16)), "hbm", T * W * 8, "residual add + norm, bf16")
+    row("gated norm over all heads", timed(lambda: ops.gated_rms_norm(o32, wz, w32, W, 1e-5, out=o16)), "hbm", T * W * 8, "residual add + norm, bf16")
     gs = torch.zeros(B, W, device="cuda")
-    row("minimal GRU scan (prefill)", timed(lambda: ops.min_gru(proj, offs[:3], bias, bias, gs, whole, S)), "hbm", T * W * 8,
+    row("minimal GRU scan (prefill)", timed(lambda: ops.min_gru(proj, offs[:3], bias, bias, gs, whole, S, out=o16)), "hbm", T * W * 8,
         "residual add + norm, bf16")
     q, k = proj[:, :H * D].view(T, H, D), proj[:, H * D:(H + G) * D].view(T, G, D)
     inv, nw = torch.rand(D // 2, device="cuda", generator=g), torch.ones(D, device="cuda")
-    row("head norm + rotary, f32 angles", timed(lambda: ops.head_norm_rope(q, k, nw, nw, inv, D, 1e-5, whole, S)), "hbm",
+    kc, oa = k.contiguous(), bf(T, H, D)
+    row("head norm + rotary, f32 angles", timed(lambda: ops.head_norm_rope(q, k, nw, nw, inv, D, 1e-5, whole, S, out=kc)), "hbm",
         2 * 2 * T * (H + G) * D, "head norm + rotary + cache, bf16 tables")
     kr, vr = (torch.zeros(B, G, win, D, dtype=torch.bfloat16, device="cuda") for _ in range(2))
-    kc = k.contiguous()
     seen = sum(min(i + 1, win) for i in range(S))
     row("windowed attention (prefill) + ring append", timed(lambda: ops.window_attention(q, kc, k, kr, vr, win, D ** -0.5, whole, S,
-                                                                                         uniform_fresh=True)),
+                                                                                         uniform_fresh=True, out=oa)),
         "tensor", 4.0 * B * H * D * seen, "attention, prefill")
     x32, delta = rnd(T, W), bf(T, W)
     row("residual add + norm, f32 residual", timed(lambda: ops.residual_rms_norm(x32, delta, w32, 1e-5)), "hbm", T * W * 12,
@@ -810,13 +811,13 @@ def fiferax_kernels(size, peaks, timed, graph_timed):
     # one token per sequence, batch 32, states / caches rotated beyond L2
     n, copies = 32, 8
     one = ops.seq_table([(b, S, b, 1) for b in range(n)])
-    p1, z1 = proj[:n], wz[:n]
+    p1, z1, o1 = proj[:n], wz[:n], o32[:n]
     s64 = [torch.zeros(n, H64, 64, 64, device="cuda") for _ in range(copies)]
-    row("state step, delta rule (decode)", graph_timed([(lambda s=s: ops.state_scan_delta(p1, offs, z1, bias, bias, 0.6, 1e-6, s, one, 1))
+    row("state step, delta rule (decode)", graph_timed([(lambda s=s: ops.state_scan_delta(p1, offs, z1, bias, bias, 0.6, 1e-6, s, one, 1, out=o1))
                                                         for s in s64]), "hbm", 2.0 * n * H64 * 64 * 64 * 4, "attention, decode")
     del s64
     s128 = [torch.zeros(n, H128, 128, 128, device="cuda") for _ in range(copies)]
-    row("state step, scalar decay (decode)", graph_timed([(lambda s=s: ops.state_scan_decay(p1, offs[:3], decay, s, one, 1)) for s in s128]),
+    row("state step, scalar decay (decode)", graph_timed([(lambda s=s: ops.state_scan_decay(p1, offs[:3], decay, s, one, 1, out=o1)) for s in s128]),
         "hbm", 2.0 * n * H128 * 128 * 128 * 4, "attention, decode")
     del s128
     # decode attention over full rings: min(pos + 1, window) keys

@@ -377,61 +377,61 @@ def _f32_flag(t):
     return int(_sfx(t) == "f32")
 
 
-def state_scan_delta(proj, offs, wz, w_bias, a_bias, decay_coef, unit_eps, state, seqs, max_len):
+def state_scan_delta(proj, offs, wz, w_bias, a_bias, decay_coef, unit_eps, state, seqs, max_len, out=None):
     """Generalized delta rule over ``state`` f32 [slots, heads, dk, dv] (updated); ``proj`` [rows, .] with r, k, v and the raw
     removal rates at columns ``offs`` = (r, k, v, a).  Returns o f32 [rows, heads * dv]."""
     _req(proj, name="proj"); _req(wz, proj.dtype, "wz"); _req(state, _F32, "state")
     _, H, DK, DV = state.shape
-    o = torch.zeros(proj.shape[0], H * DV, dtype=_F32, device=proj.device)
+    o = torch.zeros(proj.shape[0], H * DV, dtype=_F32, device=proj.device) if out is None else out
     check(lib.teeny_state_scan(0, _f32_flag(proj), _ptr(proj), proj.stride(0), *offs, _ptr(wz), wz.stride(0), _ptr(w_bias), _ptr(a_bias),
                                None, float(decay_coef), float(unit_eps), _ptr(state), _ptr(o), o.stride(0), H, DK, DV, _ptr(seqs),
                                seqs.shape[0], max_len, _stream()), "state_scan")
     return o
 
 
-def state_scan_decay(proj, offs, decay, state, seqs, max_len):
+def state_scan_decay(proj, offs, decay, state, seqs, max_len, out=None):
     """Scalar-decay state with silu on q, k, v at columns ``offs`` of ``proj``; state and result as in state_scan_delta."""
     _req(proj, name="proj"); _req(decay, _F32, "decay"); _req(state, _F32, "state")
     _, H, DK, DV = state.shape
-    o = torch.zeros(proj.shape[0], H * DV, dtype=_F32, device=proj.device)
+    o = torch.zeros(proj.shape[0], H * DV, dtype=_F32, device=proj.device) if out is None else out
     check(lib.teeny_state_scan(1, _f32_flag(proj), _ptr(proj), proj.stride(0), *offs, 0, None, 0, None, None, _ptr(decay), 0.0, 0.0,
                                _ptr(state), _ptr(o), o.stride(0), H, DK, DV, _ptr(seqs), seqs.shape[0], max_len, _stream()),
           "state_scan")
     return o
 
 
-def gated_rms_norm(o, gate, weight, group_size, eps, scale=1.0):
+def gated_rms_norm(o, gate, weight, group_size, eps, scale=1.0, out=None):
     _req(o, _F32, "o"); _req(gate, name="gate"); _req(weight, _F32, "weight")
-    out = torch.empty(o.shape, dtype=gate.dtype, device=o.device)
+    out = torch.empty(o.shape, dtype=gate.dtype, device=o.device) if out is None else out
     check(lib.teeny_gated_rms_norm(_f32_flag(gate), _ptr(o), o.stride(0), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(out),
                                    out.stride(0), o.shape[0], o.shape[1], group_size, float(eps), float(scale), _stream()),
           "gated_rms_norm")
     return out
 
 
-def min_gru(proj, offs, z_bias, x_bias, state, seqs, max_len, scale=1.0):
+def min_gru(proj, offs, z_bias, x_bias, state, seqs, max_len, scale=1.0, out=None):
     """``proj`` [rows, .] with z, x and gate at columns ``offs``; ``state`` f32 [slots, width] (updated)."""
     _req(proj, name="proj"); _req(state, _F32, "state")
-    out = torch.zeros(proj.shape[0], state.shape[1], dtype=proj.dtype, device=proj.device)
+    out = torch.zeros(proj.shape[0], state.shape[1], dtype=proj.dtype, device=proj.device) if out is None else out
     check(lib.teeny_min_gru(_f32_flag(proj), _ptr(proj), proj.stride(0), *offs, _ptr(z_bias), _ptr(x_bias), _ptr(state), _ptr(out),
                             out.stride(0), state.shape[1], float(scale), _ptr(seqs), seqs.shape[0], max_len, _stream()), "min_gru")
     return out
 
 
-def head_norm_rope(q, k, q_weight, k_weight, inv_freq, rot_dims, eps, seqs, max_len):
+def head_norm_rope(q, k, q_weight, k_weight, inv_freq, rot_dims, eps, seqs, max_len, out=None):
     """q [rows, heads, dim] (in place) and k [rows, kv_heads, dim] as views with contiguous heads; returns the rotated k."""
     _req(q, name="q"); _req(k, q.dtype, "k")
-    out = torch.zeros(k.shape, dtype=k.dtype, device=k.device)
+    out = torch.zeros(k.shape, dtype=k.dtype, device=k.device) if out is None else out
     check(lib.teeny_head_norm_rope(_f32_flag(q), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(out), out.stride(0), _ptr(q_weight),
                                    _ptr(k_weight), _ptr(inv_freq), q.shape[1], k.shape[1], q.shape[2], rot_dims, float(eps), _ptr(seqs),
                                    seqs.shape[0], max_len, _stream()), "head_norm_rope")
     return out
 
 
-def window_attention(q, k, v, k_ring, v_ring, window, score_scale, seqs, max_len, out_scale=1.0, uniform_fresh=False):
+def window_attention(q, k, v, k_ring, v_ring, window, score_scale, seqs, max_len, out_scale=1.0, uniform_fresh=False, out=None):
     """q [rows, heads, dim], k / v [rows, kv_heads, dim]; rings [slots, kv_heads, ring, dim] (updated)."""
     _req(q, name="q"); _req(k, q.dtype, "k"); _req(v, q.dtype, "v"); _req(k_ring, q.dtype, "k_ring"); _req(v_ring, q.dtype, "v_ring")
-    out = torch.zeros(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype, device=q.device)
+    out = torch.zeros(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype, device=q.device) if out is None else out
     check(lib.teeny_window_attention(_f32_flag(q), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(k_ring),
                                      _ptr(v_ring), k_ring.shape[0], k_ring.shape[2], window, _ptr(out), out.stride(0), q.shape[1],
                                      k.shape[1], q.shape[2], v.shape[2], float(score_scale), float(out_scale), int(uniform_fresh),
