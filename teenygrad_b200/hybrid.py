@@ -302,7 +302,7 @@ class HybridRunner(DecoderRunner):
                 row0 += c
             self._run(ids, [entries[e][0] for e, _, _, _ in portion], [c for _, _, c, _ in portion], rows)
             if rows:
-                got, r = self.logits().float(), 0
+                got, r = self.logits().to(torch.float32, copy=True), 0  # the next step rewrites the buffer
                 for e, _, _, want in portion:
                     out[e].append(got[r:r + len(want)])
                     r += len(want)
