@@ -76,6 +76,7 @@ pub struct TeenyHybridConfig {
     pub vocab: c_int,
     pub eps: f32,
     pub embed_scale: f32,
+    pub residual_mult: f32,
     pub f32: c_int,
     pub max_batch: c_int,
     pub max_len: c_int,
@@ -90,6 +91,7 @@ pub struct TeenyHybridLayer {
     pub num_branches: c_int,
     pub ff: c_int,
     pub act: c_int,
+    pub flags: c_int,
 }
 #[repr(C)]
 #[derive(Clone, Copy, Debug, Default)]
@@ -100,6 +102,7 @@ pub struct TeenyHybridBranch {
     pub dim: c_int,
     pub vdim: c_int,
     pub rank: c_int,
+    pub q_rank: c_int,
     pub window: c_int,
     pub rot_dims: c_int,
     pub flags: c_int,
@@ -107,6 +110,8 @@ pub struct TeenyHybridBranch {
     pub out_scale: f32,
     pub decay_coef: f32,
     pub unit_eps: f32,
+    pub softcap: f32,
+    pub rot_scale: f32,
 }
 /// Opaque runner handle (`teeny_qwen3`).
 #[repr(C)]
@@ -151,8 +156,14 @@ pub const TEENY_HYBRID_ATTENTION: c_int = 0;
 pub const TEENY_HYBRID_DELTA: c_int = 1;
 pub const TEENY_HYBRID_DECAY: c_int = 2;
 pub const TEENY_HYBRID_MIN_GRU: c_int = 3;
+pub const TEENY_HYBRID_LATENT: c_int = 4;
 pub const TEENY_HYBRID_QK_NORM: c_int = 1;
 pub const TEENY_HYBRID_KEYS_ARE_VALUES: c_int = 2;
+pub const TEENY_HYBRID_SINK: c_int = 4;
+pub const TEENY_HYBRID_OUT_GATE: c_int = 8;
+pub const TEENY_HYBRID_VALUE_MIX: c_int = 16;
+pub const TEENY_HYBRID_IN_BIAS: c_int = 1;
+pub const TEENY_HYBRID_POST_NORM: c_int = 2;
 pub const TEENY_HYBRID_ACT_SILU: c_int = 1;
 pub const TEENY_HYBRID_ACT_GELU_TANH: c_int = 2;
 pub const TEENY_HYBRID_W_NORM1: c_int = 0;
@@ -161,6 +172,9 @@ pub const TEENY_HYBRID_W_IN: c_int = 2;
 pub const TEENY_HYBRID_W_OUT: c_int = 3;
 pub const TEENY_HYBRID_W_GATE_UP: c_int = 4;
 pub const TEENY_HYBRID_W_DOWN: c_int = 5;
+pub const TEENY_HYBRID_W_IN_BIAS: c_int = 6;
+pub const TEENY_HYBRID_W_NORM1_POST: c_int = 7;
+pub const TEENY_HYBRID_W_NORM2_POST: c_int = 8;
 pub const TEENY_HYBRID_W_Q_NORM: c_int = 50;
 pub const TEENY_HYBRID_W_K_NORM: c_int = 51;
 pub const TEENY_HYBRID_W_O_NORM: c_int = 52;
@@ -171,6 +185,12 @@ pub const TEENY_HYBRID_W_Z_BIAS: c_int = 56;
 pub const TEENY_HYBRID_W_X_BIAS: c_int = 57;
 pub const TEENY_HYBRID_W_DECAY: c_int = 58;
 pub const TEENY_HYBRID_W_INV_FREQ: c_int = 59;
+pub const TEENY_HYBRID_W_SINK: c_int = 60;
+pub const TEENY_HYBRID_W_VALUE_MIX: c_int = 61;
+pub const TEENY_HYBRID_W_UQ: c_int = 62;
+pub const TEENY_HYBRID_W_EXPAND: c_int = 63;
+pub const TEENY_HYBRID_W_ABSORB: c_int = 64;
+pub const TEENY_HYBRID_W_VALUE_UP: c_int = 65;
 pub const TEENY_HYBRID_W_EMBED: c_int = 100;
 pub const TEENY_HYBRID_W_FINAL_NORM: c_int = 101;
 pub const TEENY_HYBRID_W_LM_HEAD: c_int = 102;
@@ -263,7 +283,12 @@ extern "C" {
     pub fn teeny_min_gru(f32: c_int, proj: *const c_void, ld: c_longlong, off_z: c_int, off_x: c_int, off_g: c_int, z_bias: *const f32, x_bias: *const f32, state: *mut f32, out: *mut c_void, ldout: c_longlong, width: c_int, scale: f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
     pub fn teeny_head_norm_rope(f32: c_int, q: *mut c_void, ldq: c_longlong, k_raw: *const c_void, ldkr: c_longlong, k_out: *mut c_void, ldk: c_longlong, q_weight: *const f32, k_weight: *const f32, inv_freq: *const f32, heads: c_int, kv_heads: c_int, dim: c_int, rot_dims: c_int, eps: f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
     pub fn teeny_window_attention(f32: c_int, q: *const c_void, ldq: c_longlong, k_new: *const c_void, ldk: c_longlong, v_new: *const c_void, ldv: c_longlong, k_ring: *mut c_void, v_ring: *mut c_void, slots: c_int, ring: c_int, window: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, kv_heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, out_scale: f32, uniform_fresh: c_int, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
-    pub fn teeny_residual_rms_norm(f32: c_int, x: *mut f32, delta: *const c_void, ldd: c_longlong, y: *mut c_void, ldy: c_longlong, weight: *const f32, rows: c_int, n: c_int, eps: f32, stream: CUstream) -> c_int;
+    pub fn teeny_residual_rms_norm(f32: c_int, x: *mut f32, delta: *const c_void, ldd: c_longlong, y: *mut c_void, ldy: c_longlong, weight: *const f32, rows: c_int, n: c_int, eps: f32, post: *const f32, mult: f32, stream: CUstream) -> c_int;
+    pub fn teeny_rope_cache(f32: c_int, q: *mut c_void, ldq: c_longlong, k: *const c_void, ldk: c_longlong, v: *const c_void, ldv: c_longlong, k_cache: *mut c_void, v_cache: *mut c_void, max_cached: c_int, inv_freq: *const f32, rot_scale: f32, heads: c_int, kv_heads: c_int, dim: c_int, vdim: c_int, rot_dims: c_int, mix_mode: c_int, v_first: *mut c_void, mix: *const f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_cached_attention(f32: c_int, q: *const c_void, ldq: c_longlong, k_cache: *mut c_void, v_cache: *mut c_void, slots: c_int, max_cached: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, kv_heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, softcap: f32, sink: *const f32, gate: *const c_void, ldg: c_longlong, scratch: *mut c_void, scratch_bytes: usize, counters: *mut c_uint, seqs: *const c_int, host_seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_latent_prepare(f32: c_int, proj: *const c_void, ld: c_longlong, off_q: c_int, off_c: c_int, off_r: c_int, q_rank: c_int, rank: c_int, rot_dims: c_int, q_weight: *const f32, c_weight: *const f32, inv_freq: *const f32, eps: f32, rot_scale: f32, cq: *mut c_void, ldcq: c_longlong, latents: *mut c_void, cache: *mut c_void, max_cached: c_int, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_head_linear(f32: c_int, x: *const c_void, ldx: c_longlong, x_head: c_longlong, w: *const c_void, y: *mut c_void, ldy: c_longlong, y_head: c_longlong, heads: c_int, n: c_int, k: c_int, rows: c_int, rot_dims: c_int, rot_off: c_int, inv_freq: *const f32, rot_scale: f32, seqs: *const c_int, n_seqs: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_latent_attention(f32: c_int, q: *const c_void, ldq: c_longlong, cache: *const c_void, max_cached: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
 }
 // ---- generated from include/*.h: end ----
 

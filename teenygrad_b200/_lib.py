@@ -74,7 +74,13 @@ SIGNATURES = {
     "teeny_head_norm_rope": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, f32, vp, i32, i32, vp]),
     "teeny_window_attention": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i32, i32, i32, vp, i64, i32, i32, i32, i32, f32, f32, i32,
                                      vp, i32, i32, vp]),
-    "teeny_residual_rms_norm": (i32, [i32, vp, vp, i64, vp, i64, vp, i32, i32, f32, vp]),
+    "teeny_residual_rms_norm": (i32, [i32, vp, vp, i64, vp, i64, vp, i32, i32, f32, vp, f32, vp]),
+    "teeny_rope_cache": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i32, vp, f32] + [i32] * 6 + [vp, vp, vp, i32, i32, vp]),
+    "teeny_cached_attention": (i32, [i32, vp, i64, vp, vp, i32, i32, vp, i64, i32, i32, i32, i32, f32, f32, vp, vp, i64, vp, sz, vp, vp, vp,
+                                     i32, i32, vp]),
+    "teeny_latent_prepare": (i32, [i32, vp, i64] + [i32] * 6 + [vp, vp, vp, f32, f32, vp, i64, vp, vp, i32, vp, i32, i32, vp]),
+    "teeny_head_linear": (i32, [i32, vp, i64, i64, vp, vp, i64, i64] + [i32] * 6 + [vp, f32, vp, i32, vp]),
+    "teeny_latent_attention": (i32, [i32, vp, i64, vp, i32, vp, i64, i32, i32, i32, f32, vp, i32, i32, vp]),
     "teeny_sample_merge": (i32, [vp, i32, sz, i32, f32, i32, f32, vp, vp, vp, vp]),
 }
 

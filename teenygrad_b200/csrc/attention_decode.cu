@@ -54,6 +54,11 @@ struct DecodeArgs {
   const SeqDesc* seqs;  // ring caches: per-sequence slot and position (kv_len / kv_len_dev unused), ring rows
   int ring;
   float out_scale;
+  int D, DV;           // query/key and value sizes, at most the kernel's HD (the copies zero-fill the rest)
+  float two_y, cap_l2; // soft cap of the scores (cap_l2 = 0: none), see softcap_log2
+  const float* sink;
+  const bf16* gate;
+  long long gate_sb;
   DecodeRope rope;  // rope.k_new == nullptr: q is final and the caches already hold the new rows
   long long kc_sb, kc_sh, kc_ss, vc_sb, vc_sh, vc_ss;  // cache strides for the append
 };
@@ -206,10 +211,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       const bf16* qp = fused ? &sm_q[warp][g < G ? g : 0][0] : a.q + b * a.q_sb + (hk * G + (g < G ? g : 0)) * a.q_sh;
 #pragma unroll
       for (int ks = 0; ks < HD / 16; ++ks) {
-        const uint32_t lo = *reinterpret_cast<const uint32_t*>(qp + 16 * ks + 2 * c);
-        const uint32_t hi = *reinterpret_cast<const uint32_t*>(qp + 16 * ks + 8 + 2 * c);
-        qa[ks][0] = g < G ? lo : 0u;
-        qa[ks][1] = g < G ? hi : 0u;
+        const int d0 = 16 * ks + 2 * c, d1 = d0 + 8;
+        qa[ks][0] = g < G && d0 < a.D ? *reinterpret_cast<const uint32_t*>(qp + d0) : 0u;
+        qa[ks][1] = g < G && d1 < a.D ? *reinterpret_cast<const uint32_t*>(qp + d1) : 0u;
       }
     }
     const int row_k = 16 * warp + (lane & 7);  // ldmatrix row this lane addresses for K: + 8 * n-block
@@ -255,7 +259,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int key = kb + nb * 8 + 2 * c + e;
-            s[nb][e] = key < key_end ? s[nb][e] * a.scale_log2 : -INFINITY;
+            const float x = a.cap_l2 > 0.0f ? softcap_log2(s[nb][e], a.two_y, a.cap_l2) : s[nb][e] * a.scale_log2;
+            s[nb][e] = key < key_end ? x : -INFINITY;
             tmax = fmaxf(tmax, s[nb][e]);
           }
         tmax = fmaxf(tmax, __shfl_xor_sync(0xffffffffu, tmax, 1));
@@ -314,6 +319,14 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
     }
   }
   __syncthreads();
+  // output element of the group's head gg: row sum ll relative to the maximum mm (log2 domain), oo unnormalised
+  auto finish = [&](int gg, int d, float mm, float ll, float oo) {
+    if (d >= a.DV) return;
+    if (a.sink) ll += ex2(fmaf(a.sink[hk * G + gg], 1.4426950408889634f, -mm));
+    oo = oo / ll * a.out_scale;
+    if (a.gate) oo *= sigmoid_f(__bfloat162float(a.gate[b * a.gate_sb + (hk * G + gg) * a.DV + d]));
+    a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo);
+  };
   const size_t slot = (static_cast<size_t>(b) * a.Hkv + hk) * a.max_chunks + chunk;
   for (int idx = threadIdx.x; idx < G * HD; idx += kDecThreads) {
     const int gg = idx / HD, d = idx - gg * HD;
@@ -329,7 +342,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       oo += sm_o[w][gg][d] * sc;
     }
     if (gridDim.x == 1) {  // whole sequence in this CTA: finish here, no partials
-      a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo / ll * a.out_scale);
+      finish(gg, d, mm, ll, oo);
       continue;
     }
     a.part_o[(slot * G + gg) * HD + d] = oo;
@@ -365,7 +378,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
           ll += __ldcg(a.part_ml + sl * 2 + 1) * sc;
           oo += __ldcg(a.part_o + sl * HD + d) * sc;
         }
-        a.o[b * a.o_sb + (hk * G + gg) * a.o_sh + d] = __float2bfloat16_rn(oo / ll * a.out_scale);
+        finish(gg, d, mm, ll, oo);
       }
     }
   }
@@ -490,7 +503,10 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
                           const int* kv_len_dev, void* scratch, size_t scratch_bytes, cudaStream_t stream,
                           int fresh_rows, const DecodeRope* rope, unsigned* counters, const DecodeRing* ring) {
   if (!q || !k || !v || !o || !scratch || s.B <= 0 || s.Hq <= 0 || s.Hkv <= 0 || s.Skv <= 0) return TEENY_ERR_BAD_ARG;
-  if ((s.D != kHD && !(s.D == 64 && ring)) || s.Hq % s.Hkv != 0 || s.Sq != 1) return TEENY_ERR_BAD_ARG;
+  const int DV = s.DV ? s.DV : s.D;
+  const int HD = s.D <= 64 && DV <= 64 ? 64 : kHD;  // size class of the kernel
+  if (s.D <= 0 || s.D > kHD || DV <= 0 || DV > kHD || s.D % 8 || DV % 8 || s.Hq % s.Hkv != 0 || s.Sq != 1) return TEENY_ERR_BAD_ARG;
+  if (!ring && (s.D != kHD || DV != kHD || s.softcap > 0.0f || s.sink || s.gate)) return TEENY_ERR_BAD_ARG;
   if (ring && (!ring->seqs || ring->slots <= 0 || rope || !counters)) return TEENY_ERR_BAD_ARG;
   if (!ring && !kv_len_dev && (kv_len <= 0 || kv_len > s.Skv)) return TEENY_ERR_BAD_ARG;
   const int G = s.Hq / s.Hkv;
@@ -501,7 +517,7 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15)
     return TEENY_ERR_ALIGNMENT;
   // s.Skv is the cache capacity the grid is sized for; the live length comes from kv_len / kv_len_dev
-  if (scratch_bytes < attention_decode_scratch_bytes(s.B, s.Hq, s.D, s.Skv)) return TEENY_ERR_SCRATCH;
+  if (scratch_bytes < attention_decode_scratch_bytes(s.B, s.Hq, HD, s.Skv)) return TEENY_ERR_SCRATCH;
   const int max_chunks = (s.Skv + kDecChunk - 1) / kDecChunk;
   if (s.Hkv > 65535 || s.B > 65535) return TEENY_ERR_BAD_ARG;
 
@@ -516,7 +532,8 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
     const uint64_t vs[3] = {static_cast<uint64_t>(s.v_ss) * 2, nz(s.v_sh, s.v_ss), nz(s.v_sb, s.v_ss)};
     int rc = encode_tensor_map_bf16(&mk, k, 4, dims, ks, box);
     if (rc) return rc;
-    rc = encode_tensor_map_bf16(&mv, v, 4, dims, vs, box);
+    const uint64_t vdims[4] = {static_cast<uint64_t>(DV), dims[1], dims[2], dims[3]};
+    rc = encode_tensor_map_bf16(&mv, v, 4, vdims, vs, box);
     if (rc) return rc;
   }
   {
@@ -526,7 +543,7 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
   DecodeArgs a{};
   a.q = q;
   a.part_o = static_cast<float*>(scratch);
-  a.part_ml = a.part_o + static_cast<size_t>(s.B) * s.Hq * max_chunks * s.D;
+  a.part_ml = a.part_o + static_cast<size_t>(s.B) * s.Hq * max_chunks * HD;
   a.q_sb = s.q_sb; a.q_sh = s.q_sh;
   a.o = o; a.o_sb = s.o_sb; a.o_sh = s.o_sh;
   a.Hkv = s.Hkv; a.G = G; a.max_chunks = max_chunks;
@@ -535,6 +552,14 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
   a.seqs = ring ? ring->seqs : nullptr;
   a.ring = s.Skv;
   a.out_scale = s.out_scale;
+  a.D = s.D; a.DV = DV;
+  if (s.softcap > 0.0f) {
+    a.cap_l2 = s.softcap * 1.4426950408889634f;
+    a.two_y = 2.0f * 1.4426950408889634f * s.scale / s.softcap;
+  }
+  a.sink = s.sink;
+  a.gate = s.gate;
+  a.gate_sb = s.gate_sb;
   if (rope) {
     if (!rope->k_new || !rope->v_new || !rope->k_cache || !rope->v_cache || !rope->q_w || !rope->k_w || !rope->cos_t ||
         !rope->sin_t || rope->max_len <= 0)
@@ -565,10 +590,10 @@ int attention_decode_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, 
     if (n_split < 1) n_split = 1;
   }
   a.counters = n_split > 1 ? counters : nullptr;
-  const int smem = dec_smem_bytes(a.stages, s.D);
+  const int smem = dec_smem_bytes(a.stages, HD);
   dim3 grid(n_split, s.Hkv, s.B);
 #define TEENY_DEC(GG)                                                                                                     \
-  if (s.D == 64) launch_kernel(attention_decode_kernel<GG, 64>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a);      \
+  if (HD == 64) launch_kernel(attention_decode_kernel<GG, 64>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a);      \
   else launch_kernel(attention_decode_kernel<GG, 128>, grid, dim3(kDecThreads), smem, stream, 1, mk, mv, a)
   switch (G) {
     case 1: TEENY_DEC(1); break;

@@ -48,6 +48,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "mma.cuh"
 
 namespace teeny {
 
@@ -79,6 +80,9 @@ struct PrefillArgs {  // (Q, K, V and O travel as tensor maps)
   int causal;
   int window;        // > 0: query i sees only the last `window` keys up to its own (causal only)
   float out_scale;
+  float two_y, cap_l2;  // CAP: soft cap of the scores (softcap_log2); scale_log2 is then 1
+  const float* sink;    // [Hq] or null: exp(sink) joins the row sum
+  int two_out_boxes;    // values are wider than one 64-column box
   int n_pair_tiles;  // 256-row query tiles per (batch, head)
   int n_items;       // n_pair_tiles * Hq * B work items; CTA pair p takes items p, p + pairs, ...
   int* err;
@@ -166,6 +170,7 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
       : "memory");
 }
 
+template <bool CAP>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                          const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_o,
@@ -459,6 +464,10 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         }
         tc_fence_before();
         mbar_arrive_cluster(s_empty_leader);  // the buffer can take QK^T of tile g + 2 (once the peer's group is here too)
+        if (CAP) {  // monotonic: the maximum below may follow it
+#pragma unroll
+          for (int e = 0; e < 128; ++e) s[e] = softcap_log2(s[e], args.two_y, args.cap_l2);
+        }
         const int k0 = (it.t0 + j) * kKT;
         const int first = args.window > 0 ? qi + off - args.window + 1 : 0;  // first visible key
         const bool need_mask = (k0 + kKT > args.Skv) || (args.causal && (k0 + kKT - 1 > q0 + off)) ||
@@ -581,6 +590,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         if (ok) ok = mbar_wait(bar(PV_DONE + (glast & 1)), (glast >> 1) & 1, err, DEVERR_ATTN_SOFTMAX);
         if (ok) {
           tc_fence_after();
+          if (args.sink) l += fast_exp2(fmaf(args.sink[it.h], 1.4426950408889634f, -m_fin));
           float inv;
           asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(inv) : "f"(l));  // l >= 1 (the row's maximum contributes 2^0); 1 ulp
           inv *= args.out_scale;
@@ -618,7 +628,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
           if (lane == 0 && y < args.Sq) {  // rows past the end are clipped by the copy
             const uint32_t src = base + kSmemO + quarter * (32 * 256);
             tma_store_4d(&tmap_o, src, 0, y, it.h, it.b);
-            tma_store_4d(&tmap_o, src + 32 * 128, 64, y, it.h, it.b);
+            if (args.two_out_boxes) tma_store_4d(&tmap_o, src + 32 * 128, 64, y, it.h, it.b);
             bulk_commit();
           }
           if (valid && args.lse)
@@ -658,8 +668,9 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
   }
 }
 
-int make_map(CUtensorMap* m, const bf16* p, int S, int H, int B, long long ss, long long sh, long long sb, int box_rows) {
-  const uint64_t dims[4] = {kHD, static_cast<uint64_t>(S), static_cast<uint64_t>(H), static_cast<uint64_t>(B)};
+// `d` < 128: the copies fill the columns beyond with zeros (loads) or leave them out (stores)
+int make_map(CUtensorMap* m, const bf16* p, int d, int S, int H, int B, long long ss, long long sh, long long sb, int box_rows) {
+  const uint64_t dims[4] = {static_cast<uint64_t>(d), static_cast<uint64_t>(S), static_cast<uint64_t>(H), static_cast<uint64_t>(B)};
   const uint64_t strides[3] = {static_cast<uint64_t>(ss) * 2, static_cast<uint64_t>(sh) * 2,
                                static_cast<uint64_t>(sb) * 2};
   const uint32_t box[4] = {64, static_cast<uint32_t>(box_rows), 1, 1};
@@ -673,7 +684,8 @@ int attention_prefill_prepare() {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull) return 0;
-  cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemTotal);
+  cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemTotal);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemTotal);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
   return 0;
@@ -682,7 +694,8 @@ int attention_prefill_prepare() {
 int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, float* lse, const AttnShape& s,
                            cudaStream_t stream) {
   if (!q || !k || !v || !o || s.B <= 0 || s.Hq <= 0 || s.Hkv <= 0 || s.Sq <= 0 || s.Skv <= 0) return TEENY_ERR_BAD_ARG;
-  if (s.D != kHD || s.Hq % s.Hkv != 0) return TEENY_ERR_BAD_ARG;
+  const int DV = s.DV ? s.DV : s.D;
+  if (s.D <= 0 || s.D > kHD || s.D % 8 || DV <= 0 || DV > kHD || DV % 8 || s.Hq % s.Hkv != 0 || s.gate) return TEENY_ERR_BAD_ARG;
   if (s.causal && s.Skv < s.Sq) return TEENY_ERR_BAD_ARG;
   if (s.window < 0 || (s.window > 0 && !s.causal)) return TEENY_ERR_BAD_ARG;
   const long long strides[] = {s.q_sb, s.q_sh, s.q_ss, s.k_sb, s.k_sh, s.k_ss, s.v_sb, s.v_sh, s.v_ss, s.o_ss, s.o_sh, s.o_sb};
@@ -696,10 +709,10 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   int rc;
   // a dimension of extent 1 still needs a legal (multiple-of-16-byte, non-zero) stride
   auto fix = [](long long st, long long fallback) { return st > 0 ? st : fallback; };
-  if ((rc = make_map(&mk, k, s.Skv, s.Hkv, s.B, s.k_ss, fix(s.k_sh, s.k_ss), fix(s.k_sb, s.k_ss), 64))) return rc;
-  if ((rc = make_map(&mv, v, s.Skv, s.Hkv, s.B, s.v_ss, fix(s.v_sh, s.v_ss), fix(s.v_sb, s.v_ss), 128))) return rc;
-  if ((rc = make_map(&mq, q, s.Sq, s.Hq, s.B, s.q_ss, fix(s.q_sh, s.q_ss), fix(s.q_sb, s.q_ss), kQT))) return rc;
-  if ((rc = make_map(&mo, o, s.Sq, s.Hq, s.B, s.o_ss, fix(s.o_sh, s.o_ss), fix(s.o_sb, s.o_ss), 32))) return rc;
+  if ((rc = make_map(&mk, k, s.D, s.Skv, s.Hkv, s.B, s.k_ss, fix(s.k_sh, s.k_ss), fix(s.k_sb, s.k_ss), 64))) return rc;
+  if ((rc = make_map(&mv, v, DV, s.Skv, s.Hkv, s.B, s.v_ss, fix(s.v_sh, s.v_ss), fix(s.v_sb, s.v_ss), 128))) return rc;
+  if ((rc = make_map(&mq, q, s.D, s.Sq, s.Hq, s.B, s.q_ss, fix(s.q_sh, s.q_ss), fix(s.q_sb, s.q_ss), kQT))) return rc;
+  if ((rc = make_map(&mo, o, DV, s.Sq, s.Hq, s.B, s.o_ss, fix(s.o_sh, s.o_ss), fix(s.o_sb, s.o_ss), 32))) return rc;
 
   PrefillArgs a{};
   a.lse = lse; a.B = s.B; a.Hq = s.Hq; a.Hkv = s.Hkv; a.Sq = s.Sq; a.Skv = s.Skv;
@@ -707,6 +720,13 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   a.causal = s.causal;
   a.window = s.window;
   a.out_scale = s.out_scale;
+  if (s.softcap > 0.0f) {
+    a.cap_l2 = s.softcap * 1.4426950408889634f;
+    a.two_y = 2.0f * a.scale_log2 / s.softcap;
+    a.scale_log2 = 1.0f;
+  }
+  a.sink = s.sink;
+  a.two_out_boxes = DV > 64;
   a.err = device_error_word();
   if (!a.err) return TEENY_ERR_DRIVER;  // kernels report expired waits through this word: no launch without it
 
@@ -726,7 +746,8 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   if (pairs > items) pairs = items;
   if (pairs < 1) pairs = 1;
   if (pairs > 0x3fffffffLL) return TEENY_ERR_BAD_ARG;
-  launch_kernel(attention_prefill_kernel, dim3(static_cast<unsigned>(2 * pairs)), dim3(kThreads), kSmemTotal, stream, 2, mk, mv, mq, mo, a);
+  auto kernel = s.softcap > 0.0f ? attention_prefill_kernel<true> : attention_prefill_kernel<false>;
+  launch_kernel(kernel, dim3(static_cast<unsigned>(2 * pairs)), dim3(kThreads), kSmemTotal, stream, 2, mk, mv, mq, mo, a);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -4,9 +4,13 @@
 // ring and its own tokens' keys from the step's activations, and leaves its last `ring` keys in the ring afterwards,
 // so portions may be cut anywhere and a long prompt never overwrites a key that one of its own queries still needs.
 //
+// A cache as long as a sequence can get is a ring that never wraps: a step's keys and values then go into it first
+// (kKeysInRing) and every kernel reads all keys from there.
+//
 // window_attention chooses among
-//   attention_prefill_bf16   whole prompts of one length, head size 128 (tcgen05 on CTA pairs, attention_prefill.cu)
-//   attention_decode_bf16    single tokens, head size 64 or 128 (TMA-streamed ring, attention_decode.cu)
+//   attention_prefill_bf16   whole prompts of one length, head size 128 (tcgen05 on CTA pairs, attention_prefill.cu); over a
+//                            cache that never wraps, any long entry, head sizes up to 128
+//   attention_decode_bf16    single tokens, head sizes up to 128 (TMA-streamed ring, attention_decode.cu)
 //   window_attention_mma_kernel   any other bf16 step, head sizes up to 256 in multiples of 8 (mma.sync tiles, cp.async rows
 //                            from ring and step): portions, unequal prompts, other head sizes
 //   window_attention_rows_kernel<T>   anything, f32 included: one or eight warps per (token, query head)
@@ -27,6 +31,13 @@ __device__ __forceinline__ void stf(float* p, float v) { *p = v; }
 __device__ __forceinline__ void stf(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 
 constexpr int kMaxHead = 256;
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ void rope_angle(const HeadNormRope& a, int pos, int d, float* sn, float* cs) {
+  sincosf(static_cast<float>(pos) * a.inv_freq[d], &sn[d], &cs[d]);
+  sn[d] *= a.rot_scale;
+  cs[d] *= a.rot_scale;
+}
 
 // One CTA per (token, entry): the token's cos / sin once, then a warp per head (q heads, then k heads).
 template <typename T>
@@ -41,18 +52,30 @@ __global__ void head_norm_rope_rows_kernel(const HeadNormRope a, const SeqDesc* 
   const size_t row = static_cast<size_t>(seq.row0) + i;
   const int half = a.rot_dims >> 1;
   for (int d = threadIdx.x; d < half; d += blockDim.x)
-    sincosf(static_cast<float>(seq.pos + i) * a.inv_freq[d], &sn[d], &cs[d]);
+    rope_angle(a, seq.pos + i, d, sn, cs);
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int at = a.ring ? (seq.pos + i) % a.ring : 0;
+  if (a.v) {
+    const float lam = a.v_mode == kMixWith ? *a.mix : 0.0f;
+    for (int c = threadIdx.x; c < a.Hkv * a.DV; c += blockDim.x) {
+      float v = ldf(static_cast<const T*>(a.v) + row * a.ldv + c);
+      T* first = static_cast<T*>(a.v_first) + row * a.ldvf + c;
+      if (a.v_mode == kMixKeep) stf(first, v);
+      else if (a.v_mode == kMixWith) v = (1.0f - lam) * v + lam * ldf(first);
+      const int hd = c / a.DV;
+      stf(static_cast<T*>(a.v_ring) + ((static_cast<size_t>(seq.slot) * a.Hkv + hd) * a.ring + at) * a.DV + (c - hd * a.DV), v);
+    }
+  }
   for (int u = warp; u < a.Hq + a.Hkv; u += warps) {
     const bool is_q = u < a.Hq;
     const int hd = is_q ? u : u - a.Hq;
     const T* src = is_q ? static_cast<const T*>(a.q) + row * a.ldq + hd * a.D : static_cast<const T*>(a.k_raw) + row * a.ldkr + hd * a.D;
-    T* dst = is_q ? static_cast<T*>(a.q) + row * a.ldq + hd * a.D : static_cast<T*>(a.k_out) + row * a.ldk + hd * a.D;
-    // single tokens: the rotated key (and, where the values are the raw keys, the value) straight into the ring as well
-    const size_t rr0 = ((static_cast<size_t>(seq.slot) * a.Hkv + hd) * a.ring + (a.ring ? seq.pos % a.ring : 0)) * a.D;
+    T* dst = is_q ? static_cast<T*>(a.q) + row * a.ldq + hd * a.D : (a.k_out ? static_cast<T*>(a.k_out) + row * a.ldk + hd * a.D : nullptr);
+    // the rotated key (and, where the values are the raw keys, the value) straight into the ring as well
+    const size_t rr0 = ((static_cast<size_t>(seq.slot) * a.Hkv + hd) * a.ring + at) * a.D;
     T* kring = !is_q && a.ring ? static_cast<T*>(a.k_ring) + rr0 : nullptr;
-    T* vring = !is_q && a.ring && a.v_ring ? static_cast<T*>(a.v_ring) + rr0 : nullptr;
+    T* vring = !is_q && a.ring && a.v_ring && !a.v ? static_cast<T*>(a.v_ring) + rr0 : nullptr;
     const float* w = is_q ? a.q_w : a.k_w;
     float* buf = rowbuf[warp];
     float sq = 0.0f;
@@ -72,7 +95,7 @@ __global__ void head_norm_rope_rows_kernel(const HeadNormRope a, const SeqDesc* 
       float v = buf[d];
       if (d < half) v = v * cs[d] - buf[d + half] * sn[d];
       else if (d < 2 * half) v = v * cs[d - half] + buf[d - half] * sn[d - half];
-      stf(dst + d, v);
+      if (dst) stf(dst + d, v);
       if (kring) stf(kring + d, v);
     }
     __syncwarp();
@@ -89,7 +112,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormR
   const int half = a.rot_dims >> 1;
   if (i < seq.len)
     for (int d = threadIdx.x; d < half; d += blockDim.x)
-      sincosf(static_cast<float>(seq.pos + i) * a.inv_freq[d], &sn[d], &cs[d]);
+      rope_angle(a, seq.pos + i, d, sn, cs);
   pdl_wait();
   pdl_trigger();
   if (i >= seq.len) return;
@@ -99,6 +122,24 @@ __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormR
   const int lane = threadIdx.x & 31, sub = lane & (lph - 1), d0 = sub * 8;
   const int per = 256 / lph, heads = a.Hq + a.Hkv, h0 = threadIdx.x / lph;
   const int step = half >> 3;
+  const int at = a.ring ? (seq.pos + i) % a.ring : 0;
+  if (a.v) {
+    const float lam = a.v_mode == kMixWith ? *a.mix : 0.0f, keep = 1.0f - lam;
+    for (int c = threadIdx.x * 8; c < a.Hkv * a.DV; c += 256 * 8) {
+      uint4 v = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(a.v) + row * a.ldv + c);
+      bf16* first = static_cast<bf16*>(a.v_first) + row * a.ldvf + c;
+      if (a.v_mode == kMixKeep) *reinterpret_cast<uint4*>(first) = v;
+      else if (a.v_mode == kMixWith) {
+        const uint4 f = *reinterpret_cast<const uint4*>(first);
+        auto mix = [&](uint32_t p, uint32_t q) {
+          return pack_bf16x2(fmaf(lam, bf16_lo(q), keep * bf16_lo(p)), fmaf(lam, bf16_hi(q), keep * bf16_hi(p)));
+        };
+        v = make_uint4(mix(v.x, f.x), mix(v.y, f.y), mix(v.z, f.z), mix(v.w, f.w));
+      }
+      const int hd = c / a.DV;
+      *reinterpret_cast<uint4*>(static_cast<bf16*>(a.v_ring) + ((static_cast<size_t>(seq.slot) * a.Hkv + hd) * a.ring + at) * a.DV + (c - hd * a.DV)) = v;
+    }
+  }
   const int partner = (lane - sub) + (sub < step ? sub + step : (sub < 2 * step ? sub - step : sub));
   const bool in_head = d0 < a.D;
   for (int base = 0; base < heads; base += per * kRopeTasks) {
@@ -144,11 +185,11 @@ __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormR
         *reinterpret_cast<uint4*>(static_cast<bf16*>(a.q) + row * a.ldq + u * a.D + d0) = out;
       } else {
         const int hk = u - a.Hq;
-        *reinterpret_cast<uint4*>(static_cast<bf16*>(a.k_out) + row * a.ldk + hk * a.D + d0) = out;
+        if (a.k_out) *reinterpret_cast<uint4*>(static_cast<bf16*>(a.k_out) + row * a.ldk + hk * a.D + d0) = out;
         if (a.ring) {
-          const size_t r = ((static_cast<size_t>(seq.slot) * a.Hkv + hk) * a.ring + seq.pos % a.ring) * a.D + d0;
+          const size_t r = ((static_cast<size_t>(seq.slot) * a.Hkv + hk) * a.ring + at) * a.D + d0;
           *reinterpret_cast<uint4*>(static_cast<bf16*>(a.k_ring) + r) = out;
-          if (a.v_ring) *reinterpret_cast<uint4*>(static_cast<bf16*>(a.v_ring) + r) = raw[t];
+          if (a.v_ring && !a.v) *reinterpret_cast<uint4*>(static_cast<bf16*>(a.v_ring) + r) = raw[t];
         }
       }
     }
@@ -168,6 +209,10 @@ __global__ void ring_append_kernel(const WindowAttn a, const SeqDesc* __restrict
     static_cast<T*>(a.k_ring)[((dst + c / a.D) * a.ring + r) * a.D + c % a.D] = static_cast<const T*>(a.k_new)[row * a.ldk + c];
   for (int c = threadIdx.x; c < a.Hkv * a.DV; c += blockDim.x)
     static_cast<T*>(a.v_ring)[((dst + c / a.DV) * a.ring + r) * a.DV + c % a.DV] = static_cast<const T*>(a.v_new)[row * a.ldv + c];
+}
+
+__device__ __forceinline__ bool from_new(const WindowAttn& a, const SeqDesc& seq, int j) {
+  return a.keys == kKeysSplit ? j >= seq.pos : a.keys == kKeysInNew;
 }
 
 // WPU warps share a (token, query head): each takes every WPU-th key with an online softmax, merged through shared memory.
@@ -198,9 +243,9 @@ __global__ void __launch_bounds__(WPU > 1 ? 32 * WPU : 128) window_attention_row
   }
   float m = -INFINITY, l = 0.0f;
   for (int j = max(0, pos - a.window + 1) + (WPU > 1 ? warp : 0); j <= pos; j += WPU) {
-    const bool fresh = j >= seq.pos;
-    const T* kp = fresh ? kn + static_cast<size_t>(j - seq.pos) * a.ldk : kr + static_cast<size_t>(j % a.ring) * a.D;
-    const T* vp = fresh ? vn + static_cast<size_t>(j - seq.pos) * a.ldv : vr + static_cast<size_t>(j % a.ring) * a.DV;
+    const bool fresh = from_new(a, seq, j);
+    const T* kp = fresh ? kn + static_cast<long long>(j - seq.pos) * a.ldk : kr + static_cast<size_t>(j % a.ring) * a.D;
+    const T* vp = fresh ? vn + static_cast<long long>(j - seq.pos) * a.ldv : vr + static_cast<size_t>(j % a.ring) * a.DV;
     float dot = 0.0f;
 #pragma unroll
     for (int e = 0; e < kMaxHead / 32; ++e) {
@@ -208,6 +253,7 @@ __global__ void __launch_bounds__(WPU > 1 ? 32 * WPU : 128) window_attention_row
       if (d < a.D) dot = fmaf(qv[e], ldf(kp + d), dot);
     }
     dot = warp_sum(dot);
+    if (a.softcap > 0.0f) dot = a.softcap * tanhf(dot / a.softcap);
     const float m_new = fmaxf(m, dot);
     const float corr = expf(m - m_new), p = expf(dot - m_new);
     l = fmaf(corr, l, p);
@@ -219,12 +265,14 @@ __global__ void __launch_bounds__(WPU > 1 ? 32 * WPU : 128) window_attention_row
     m = m_new;
   }
   T* orow = static_cast<T*>(a.out) + row * a.ldo + h * a.DV;
+  const T* grow = a.gate ? static_cast<const T*>(a.gate) + row * a.ldg + h * a.DV : nullptr;
   if (WPU == 1) {
+    if (a.sink) l += expf(a.sink[h] - m);
     const float inv = a.out_scale / l;
 #pragma unroll
     for (int e = 0; e < kMaxHead / 32; ++e) {
       const int d = lane + 32 * e;
-      if (d < a.DV) stf(orow + d, acc[e] * inv);
+      if (d < a.DV) stf(orow + d, acc[e] * inv * (grow ? sigmoid_f(ldf(grow + d)) : 1.0f));
     }
     return;
   }
@@ -247,7 +295,8 @@ __global__ void __launch_bounds__(WPU > 1 ? 32 * WPU : 128) window_attention_row
       ll = fmaf(sm_ml[w][1], sc, ll);
       o = fmaf(sm_o[WPU > 1 ? w : 0][d], sc, o);
     }
-    stf(orow + d, o / ll * a.out_scale);
+    if (a.sink) ll += expf(a.sink[h] - mm);
+    stf(orow + d, o / ll * a.out_scale * (grow ? sigmoid_f(ldf(grow + d)) : 1.0f));
   }
 }
 
@@ -262,6 +311,7 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+constexpr int kPrefillLen = 128;  // shortest entry for the tcgen05 kernel
 constexpr int kQRows = 64, kKeys = 64;
 constexpr int mma_smem_bytes(int nd) { return (kQRows + 4 * kKeys) * (16 * nd + 8) * 2; }
 
@@ -295,12 +345,12 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const WindowA
     for (int idx = threadIdx.x; idx < kKeys * CH; idx += 128) {
       const int r = idx / CH, ch = idx % CH, j = key_lo + t * kKeys + r;
       const uint32_t off = static_cast<uint32_t>(r * LD + ch * 8) * 2;
-      const bool in = j <= key_hi, fresh = j >= seq.pos;
+      const bool in = j <= key_hi, fresh = from_new(a, seq, j);
       if (in && ch * 8 < a.D)
-        cp_async16(kt + off, (fresh ? kn + static_cast<size_t>(j - seq.pos) * a.ldk : kr + static_cast<size_t>(j % a.ring) * a.D) + ch * 8);
+        cp_async16(kt + off, (fresh ? kn + static_cast<long long>(j - seq.pos) * a.ldk : kr + static_cast<size_t>(j % a.ring) * a.D) + ch * 8);
       else zero16(kt + off);
       if (in && ch * 8 < a.DV)
-        cp_async16(vt + off, (fresh ? vn + static_cast<size_t>(j - seq.pos) * a.ldv : vr + static_cast<size_t>(j % a.ring) * a.DV) + ch * 8);
+        cp_async16(vt + off, (fresh ? vn + static_cast<long long>(j - seq.pos) * a.ldv : vr + static_cast<size_t>(j % a.ring) * a.DV) + ch * 8);
       else zero16(vt + off);
     }
     cp_async_commit();
@@ -321,7 +371,9 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const WindowA
 #pragma unroll
   for (int n = 0; n < 2 * ND; ++n) O[n][0] = O[n][1] = O[n][2] = O[n][3] = 0.0f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
-  const float sc = a.scale * 1.4426950408889634f;
+  const float sc = a.scale * kLog2e;
+  const bool capped = a.softcap > 0.0f;
+  const float two_y = capped ? 2.0f * sc / a.softcap : 0.0f, cap_l2 = a.softcap * kLog2e;
   const int p_lo = seq.pos + i0 + warp * 16;  // position of the warp's first row; rows g and g + 8
   for (int t = 0; t < n_tiles; ++t) {
     if (t + 1 < n_tiles) {
@@ -365,7 +417,8 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const WindowA
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int p = p_lo + g + 8 * (e >> 1), j = j0 + 8 * n + 2 * c + (e & 1);
-          s[n][e] = mask && (j > p || j <= p - a.window) ? -INFINITY : s[n][e] * sc;
+          const float x = capped ? softcap_log2(s[n][e], two_y, cap_l2) : s[n][e] * sc;
+          s[n][e] = mask && (j > p || j <= p - a.window) ? -INFINITY : x;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
         }
       float alpha[2], base[2];
@@ -413,32 +466,66 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const WindowA
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     const int i = i0 + warp * 16 + g + 8 * r;
     if (i > last_i) continue;
+    if (a.sink) l[r] += ex2(fmaf(a.sink[h], kLog2e, -m[r]));
     const float inv = a.out_scale / l[r];
-    bf16* orow = static_cast<bf16*>(a.out) + (static_cast<size_t>(seq.row0) + i) * a.ldo + h * a.DV;
+    const size_t row = static_cast<size_t>(seq.row0) + i;
+    bf16* orow = static_cast<bf16*>(a.out) + row * a.ldo + h * a.DV;
+    const bf16* grow = a.gate ? static_cast<const bf16*>(a.gate) + row * a.ldg + h * a.DV : nullptr;
 #pragma unroll
     for (int n = 0; n < 2 * ND; ++n) {
       const int d = 8 * n + 2 * c;
-      if (d < a.DV) *reinterpret_cast<uint32_t*>(orow + d) = pack_bf16x2(O[n][2 * r] * inv, O[n][2 * r + 1] * inv);
+      if (d >= a.DV) continue;
+      float o0 = O[n][2 * r] * inv, o1 = O[n][2 * r + 1] * inv;
+      if (grow) {
+        const uint32_t g2 = *reinterpret_cast<const uint32_t*>(grow + d);
+        o0 *= sigmoid_f(bf16_lo(g2));
+        o1 *= sigmoid_f(bf16_hi(g2));
+      }
+      *reinterpret_cast<uint32_t*>(orow + d) = pack_bf16x2(o0, o1);
     }
   }
 }
 
+// out *= sigmoid(gate), eight columns per thread
+__global__ void sigmoid_gate_kernel(bf16* __restrict__ out, long long ldo, const bf16* __restrict__ gate, long long ldg, long long rows, int vecs) {
+  pdl_wait();
+  pdl_trigger();
+  const long long total = rows * vecs;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / vecs;
+    const int c = static_cast<int>(i - r * vecs) * 8;
+    const uint4 o = *reinterpret_cast<const uint4*>(out + r * ldo + c), g = *reinterpret_cast<const uint4*>(gate + r * ldg + c);
+    auto mul = [](uint32_t x, uint32_t y) { return pack_bf16x2(bf16_lo(x) * sigmoid_f(bf16_lo(y)), bf16_hi(x) * sigmoid_f(bf16_hi(y))); };
+    *reinterpret_cast<uint4*>(out + r * ldo + c) = make_uint4(mul(o.x, g.x), mul(o.y, g.y), mul(o.z, g.z), mul(o.w, g.w));
+  }
+}
+
+int sigmoid_gate_rows(bf16* out, long long ldo, const bf16* gate, long long ldg, long long rows, int cols, cudaStream_t st) {
+  const long long blocks = (rows * (cols / 8) + 255) / 256;
+  launch_kernel(sigmoid_gate_kernel, dim3(static_cast<unsigned>(blocks < 16LL * sm_count() ? blocks : 16LL * sm_count())), dim3(256), 0, st, 1, out, ldo,
+                gate, ldg, rows, cols / 8);
+  return static_cast<int>(cudaGetLastError());
+}
+
 bool valid(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len) {
-  return a.k_new && a.v_new && a.k_ring && a.v_ring && seqs && n_seqs > 0 && n_seqs <= 65535 && max_len > 0 && a.ring > 0 &&
+  return (a.keys == kKeysInRing || (a.k_new && a.v_new)) && (a.keys == kKeysInNew || (a.k_ring && a.v_ring)) && seqs && n_seqs > 0 && n_seqs <= 65535 && max_len > 0 && a.ring > 0 &&
          a.window > 0 && a.Hq > 0 && a.Hkv > 0 && a.Hq % a.Hkv == 0 && a.D > 0 && a.D <= kMaxHead && a.DV > 0 && a.DV <= kMaxHead;
 }
 
 }  // namespace
 
 int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st) {
-  if (!a.q || !a.k_raw || !a.k_out || !seqs || n_seqs <= 0 || n_seqs > 65535 || max_len <= 0 || a.D <= 0 || a.D > kMaxHead ||
-      a.rot_dims < 0 || a.rot_dims > a.D || (a.rot_dims & 1) || (a.rot_dims && !a.inv_freq))
+  if (!a.q || (a.Hkv > 0 && (!a.k_raw || (!a.k_out && !a.ring))) || !seqs || n_seqs <= 0 || n_seqs > 65535 || max_len <= 0 || a.D <= 0 ||
+      a.D > kMaxHead || a.rot_dims < 0 || a.rot_dims > a.D || (a.rot_dims & 1) || (a.rot_dims && !a.inv_freq) || a.ring < 0 ||
+      (a.ring && !a.k_ring))
+    return TEENY_ERR_BAD_ARG;
+  if (a.v && (!a.ring || !a.v_ring || a.DV <= 0 || (a.v_mode != kMixNone && !a.v_first) || (a.v_mode == kMixWith && !a.mix)))
     return TEENY_ERR_BAD_ARG;
   const dim3 grid(max_len, n_seqs), block(256);
   const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k_raw) | reinterpret_cast<uintptr_t>(a.k_out) |
                           reinterpret_cast<uintptr_t>(a.k_ring) | reinterpret_cast<uintptr_t>(a.v_ring) | reinterpret_cast<uintptr_t>(a.q_w) |
-                          reinterpret_cast<uintptr_t>(a.k_w);
-  if (!a.f32 && a.D % 8 == 0 && a.rot_dims % 16 == 0 && ((a.ldq | a.ldkr | a.ldk) & 7) == 0 && (bases & 15) == 0) {
+                          reinterpret_cast<uintptr_t>(a.k_w) | reinterpret_cast<uintptr_t>(a.v) | reinterpret_cast<uintptr_t>(a.v_first);
+  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && a.rot_dims % 16 == 0 && ((a.ldq | a.ldkr | a.ldk | a.ldv | a.ldvf) & 7) == 0 && (bases & 15) == 0) {
     int lph = 1;
     while (lph * 8 < a.D) lph *= 2;
     launch_kernel(head_norm_rope_vec_kernel, grid, block, 0, st, 1, a, seqs, lph);
@@ -474,37 +561,78 @@ int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int m
   // 16-byte rows everywhere
   const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k_new) | reinterpret_cast<uintptr_t>(a.v_new) |
                           reinterpret_cast<uintptr_t>(a.k_ring) | reinterpret_cast<uintptr_t>(a.v_ring) | reinterpret_cast<uintptr_t>(a.out);
-  const bool rows16 = !a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && ((a.ldq | a.ldk | a.ldv | a.ldo) & 7) == 0 && (bases & 15) == 0;
+  const bool rows16 = !a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && ((a.ldq | a.ldk | a.ldv | a.ldo | a.ldg) & 7) == 0 && (bases & 15) == 0;
+  const int head = a.D > a.DV ? a.D : a.DV;
   AttnShape s{};
-  s.Hq = a.Hq; s.Hkv = a.Hkv; s.D = a.D; s.scale = a.scale; s.out_scale = a.out_scale;
-  if (rows16 && max_len == 1 && a.in_ring && a.D == a.DV && (a.D == 64 || a.D == 128) && (G == 1 || G == 2 || G == 4 || G == 8) && a.scratch &&
-      a.scratch_bytes >= attention_decode_scratch_bytes(n_seqs, a.Hq, a.D, a.ring)) {
+  s.Hq = a.Hq; s.Hkv = a.Hkv; s.D = a.D; s.DV = a.DV; s.scale = a.scale; s.out_scale = a.out_scale;
+  s.softcap = a.softcap; s.sink = a.sink;
+  s.q_sb = a.ldq; s.q_sh = a.D; s.q_ss = a.ldq;
+  s.o_sb = a.ldo; s.o_sh = a.DV; s.o_ss = a.ldo;
+  // the ring as a tensor [slot, kv head, row, d]
+  s.k_ss = a.D; s.k_sh = static_cast<long long>(a.ring) * a.D; s.k_sb = s.k_sh * a.Hkv;
+  s.v_ss = a.DV; s.v_sh = static_cast<long long>(a.ring) * a.DV; s.v_sb = s.v_sh * a.Hkv;
+  if (rows16 && max_len == 1 && a.keys == kKeysInRing && head <= 128 && (G == 1 || G == 2 || G == 4 || G == 8) && a.scratch &&
+      a.scratch_bytes >= attention_decode_scratch_bytes(n_seqs, a.Hq, head <= 64 ? 64 : 128, a.ring)) {
     s.B = n_seqs; s.Sq = 1; s.Skv = a.ring;
-    s.q_sb = a.ldq; s.q_sh = a.D; s.q_ss = a.ldq;
-    s.k_ss = s.v_ss = a.D;
-    s.k_sh = s.v_sh = static_cast<long long>(a.ring) * a.D;
-    s.k_sb = s.v_sb = s.k_sh * a.Hkv;
-    s.o_sb = a.ldo; s.o_sh = a.D; s.o_ss = a.ldo;
+    s.gate = static_cast<const bf16*>(a.gate); s.gate_sb = a.ldg;
     const DecodeRing ring{seqs, a.slots};
     // (the kernel before this one, head_norm_rope_rows, wrote q and each sequence's newest ring row)
     return attention_decode_bf16(static_cast<const bf16*>(a.q), static_cast<const bf16*>(a.k_ring), static_cast<const bf16*>(a.v_ring),
                                  static_cast<bf16*>(a.out), s, 0, nullptr, a.scratch, a.scratch_bytes, st, 1, nullptr, a.counters, &ring);
   }
-  if (rows16 && a.uniform_fresh && a.D == 128 && a.DV == 128 && max_len >= 128 && a.scale > 0.0f) {
-    s.B = n_seqs; s.Sq = s.Skv = max_len; s.causal = 1;
-    s.window = a.window < max_len ? a.window : 0;
-    s.q_sb = max_len * a.ldq; s.q_sh = a.D; s.q_ss = a.ldq;
+  const bool prefill = rows16 && head <= 128 && a.scale > 0.0f;
+  if (prefill && a.keys == kKeysInRing && a.host && a.window >= a.ring && max_len >= kPrefillLen) {
+    // Entries of equal length and position in neighbouring slots make one launch over the cache; short ones in between go
+    // to the other kernels together.
+    WindowAttn rest = a;
+    rest.host = nullptr;
+    for (int e = 0; e < n_seqs;) {
+      const SeqDesc f = a.host[e];
+      int n = 1;
+      if (f.len < kPrefillLen) {
+        int most = f.len;
+        for (; e + n < n_seqs && a.host[e + n].len < kPrefillLen; ++n) most = a.host[e + n].len > most ? a.host[e + n].len : most;
+        const int rc = window_attention(rest, seqs + e, n, most, st);
+        if (rc) return rc;
+      } else {
+        while (e + n < n_seqs && a.host[e + n].len == f.len && a.host[e + n].pos == f.pos && a.host[e + n].slot == f.slot + n &&
+               a.host[e + n].row0 == f.row0 + n * f.len)
+          ++n;
+        s.B = n; s.Sq = f.len; s.Skv = f.pos + f.len; s.causal = 1;
+        s.q_sb = f.len * a.ldq; s.o_sb = f.len * a.ldo;
+        bf16* out = static_cast<bf16*>(a.out) + static_cast<size_t>(f.row0) * a.ldo;
+        int rc = attention_prefill_bf16(static_cast<const bf16*>(a.q) + static_cast<size_t>(f.row0) * a.ldq,
+                                        static_cast<const bf16*>(a.k_ring) + static_cast<size_t>(f.slot) * s.k_sb,
+                                        static_cast<const bf16*>(a.v_ring) + static_cast<size_t>(f.slot) * s.v_sb, out, nullptr, s, st);
+        if (rc == 0 && a.gate)
+          rc = sigmoid_gate_rows(out, a.ldo, static_cast<const bf16*>(a.gate) + static_cast<size_t>(f.row0) * a.ldg, a.ldg,
+                                 static_cast<long long>(n) * f.len, a.Hq * a.DV, st);
+        if (rc) return rc;
+      }
+      e += n;
+    }
+    return 0;
+  }
+  // whole prompts of one length, or one entry with its keys all in k_new
+  const bool alone = a.keys == kKeysInNew && a.host && n_seqs == 1;
+  if (prefill && ((a.uniform_fresh && a.keys != kKeysInRing) || alone) && max_len >= kPrefillLen) {
+    const long long first = alone ? a.host->row0 : 0, pos = alone ? a.host->pos : 0;
+    s.B = n_seqs; s.Sq = max_len; s.Skv = max_len + static_cast<int>(pos); s.causal = 1;
+    s.window = a.window < s.Skv ? a.window : 0;
+    s.q_sb = max_len * a.ldq; s.o_sb = max_len * a.ldo;
     s.k_sb = max_len * a.ldk; s.k_sh = a.D; s.k_ss = a.ldk;
-    s.v_sb = max_len * a.ldv; s.v_sh = a.D; s.v_ss = a.ldv;
-    s.o_sb = max_len * a.ldo; s.o_sh = a.D; s.o_ss = a.ldo;
-    return attention_prefill_bf16(static_cast<const bf16*>(a.q), static_cast<const bf16*>(a.k_new), static_cast<const bf16*>(a.v_new),
-                                  static_cast<bf16*>(a.out), nullptr, s, st);
+    s.v_sb = max_len * a.ldv; s.v_sh = a.DV; s.v_ss = a.ldv;
+    bf16* out = static_cast<bf16*>(a.out) + first * a.ldo;
+    const int rc = attention_prefill_bf16(static_cast<const bf16*>(a.q) + first * a.ldq, static_cast<const bf16*>(a.k_new) + (first - pos) * a.ldk,
+                                          static_cast<const bf16*>(a.v_new) + (first - pos) * a.ldv, out, nullptr, s, st);
+    if (rc || !a.gate) return rc;
+    return sigmoid_gate_rows(out, a.ldo, static_cast<const bf16*>(a.gate) + first * a.ldg, a.ldg, static_cast<long long>(n_seqs) * max_len,
+                             a.Hq * a.DV, st);
   }
   if (rows16 && max_len >= 8) {
     const dim3 grid((max_len + kQRows - 1) / kQRows, a.Hq, n_seqs), block(128);
-    const int d = a.D > a.DV ? a.D : a.DV;
-    if (d <= 64) launch_kernel(window_attention_mma_kernel<4>, grid, block, mma_smem_bytes(4), st, 1, a, seqs);
-    else if (d <= 128) launch_kernel(window_attention_mma_kernel<8>, grid, block, mma_smem_bytes(8), st, 1, a, seqs);
+    if (head <= 64) launch_kernel(window_attention_mma_kernel<4>, grid, block, mma_smem_bytes(4), st, 1, a, seqs);
+    else if (head <= 128) launch_kernel(window_attention_mma_kernel<8>, grid, block, mma_smem_bytes(8), st, 1, a, seqs);
     else launch_kernel(window_attention_mma_kernel<16>, grid, block, mma_smem_bytes(16), st, 1, a, seqs);
     return static_cast<int>(cudaGetLastError());
   }

@@ -843,15 +843,18 @@ __global__ void embedding_scaled_kernel(const int* __restrict__ ids, const T* __
 }
 
 // One CTA per row, the row held in registers (VPT vectors of four per thread) between the statistics and the scaling.
-template <typename T, int VPT>
+// POST: the added vector is rms_norm(delta) * post * mult.
+template <typename T, int VPT, bool POST>
 __global__ void residual_rms_norm_kernel(float* __restrict__ x, const T* __restrict__ delta, long long ldd, T* __restrict__ y,
-                                         long long ldy, const float* __restrict__ w, int N, float eps, const int* __restrict__ rows) {
+                                         long long ldy, const float* __restrict__ w, int N, float eps, const int* __restrict__ rows,
+                                         const float* __restrict__ post, float mult) {
   const int nv = N >> 2;
-  float4 g[VPT];
+  float4 g[VPT], p[POST ? VPT : 1];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int idx = threadIdx.x + i * blockDim.x;
     g[i] = idx < nv ? __ldg(reinterpret_cast<const float4*>(w) + idx) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (POST) p[i] = idx < nv ? __ldg(reinterpret_cast<const float4*>(post) + idx) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   }
   pdl_wait();
   pdl_trigger();
@@ -866,6 +869,18 @@ __global__ void residual_rms_norm_kernel(float* __restrict__ x, const T* __restr
     if (idx < nv) {
       v[i] = ld4(xr + 4 * idx);
       if (delta) d[i] = ld4(delta + row * ldd + 4 * idx);
+    }
+  }
+  if (POST) {
+    __shared__ float red2[32];
+    float dq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) dq = fmaf(d[i].x, d[i].x, fmaf(d[i].y, d[i].y, fmaf(d[i].z, d[i].z, fmaf(d[i].w, d[i].w, dq))));
+    const float dr = mult / sqrtf(block_sum(dq, red2) / static_cast<float>(N) + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const float4 w2 = p[POST ? i : 0];
+      d[i] = make_float4(d[i].x * dr * w2.x, d[i].y * dr * w2.y, d[i].z * dr * w2.z, d[i].w * dr * w2.w);
     }
   }
   float sq = 0.0f;
@@ -890,21 +905,31 @@ __global__ void residual_rms_norm_kernel(float* __restrict__ x, const T* __restr
 template <typename T>
 __global__ void residual_rms_norm_scalar_kernel(float* __restrict__ x, const T* __restrict__ delta, long long ldd, T* __restrict__ y,
                                                 long long ldy, const float* __restrict__ w, int N, float eps,
-                                                const int* __restrict__ rows) {
+                                                const int* __restrict__ rows, const float* __restrict__ post, float mult) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[32];
+  __shared__ float red[32], red2[32];
   const size_t row = rows ? rows[blockIdx.x] : blockIdx.x;
   float* xr = x + row * N;
+  float dr = 1.0f;
+  if (post) {
+    float dq = 0.0f;
+    for (int c = threadIdx.x; c < N; c += blockDim.x) {
+      const float d = ldf<T>(delta + row * ldd + c);
+      dq = fmaf(d, d, dq);
+    }
+    dr = mult / sqrtf(block_sum(dq, red2) / static_cast<float>(N) + eps);
+  }
+  auto sum = [&](int c) { return xr[c] + (delta ? ldf<T>(delta + row * ldd + c) * (post ? dr * post[c] : 1.0f) : 0.0f); };
   float sq = 0.0f;
   for (int c = threadIdx.x; c < N; c += blockDim.x) {
-    const float v = xr[c] + (delta ? ldf<T>(delta + row * ldd + c) : 0.0f);
+    const float v = sum(c);
     sq = fmaf(v, v, sq);
   }
   sq = block_sum(sq, red);
   const float rr = 1.0f / sqrtf(sq / static_cast<float>(N) + eps);
   for (int c = threadIdx.x; c < N; c += blockDim.x) {
-    const float v = xr[c] + (delta ? ldf<T>(delta + row * ldd + c) : 0.0f);
+    const float v = sum(c);
     if (delta && !rows) xr[c] = v;
     st_as(y + static_cast<size_t>(blockIdx.x) * ldy + c, v * rr * w[c]);
   }
@@ -1121,14 +1146,14 @@ int embedding_scaled(const int* ids, const void* table, float* x, int T, int wid
 namespace {
 template <typename T>
 int launch_residual_norm(float* x, const void* delta, long long ldd, void* y, long long ldy, const float* w, int M, int N, float eps,
-                         const int* rows, cudaStream_t st) {
+                         const int* rows, const float* post, float mult, cudaStream_t st) {
   const T* d = static_cast<const T*>(delta);
   T* yo = static_cast<T*>(y);
   const int nv = N / 4;
   const bool vec = N % 4 == 0 && ldy % 4 == 0 && (!delta || ldd % 4 == 0) && aligned16(x) && aligned16(y) && aligned16(w) &&
-                   (!delta || aligned16(delta)) && nv <= 8 * 512;
+                   (!delta || aligned16(delta)) && (!post || aligned16(post)) && nv <= 8 * 512;
   if (!vec) {
-    launch_kernel(residual_rms_norm_scalar_kernel<T>, dim3(M), dim3(256), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps, rows);
+    launch_kernel(residual_rms_norm_scalar_kernel<T>, dim3(M), dim3(256), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps, rows, post, mult);
     return static_cast<int>(cudaGetLastError());
   }
   // a few rows (decode) are one chain of latencies: one vector per thread
@@ -1137,7 +1162,13 @@ int launch_residual_norm(float* x, const void* delta, long long ldd, void* y, lo
   if (threads > most) threads = most;
   if (nv > 8 * threads) threads = 512;
   const int vpt = (nv + threads - 1) / threads;
-#define TEENY_RRN(V) launch_kernel(residual_rms_norm_kernel<T, V>, dim3(M), dim3(threads), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps, rows)
+#define TEENY_RRN(V)                                                                                                                \
+  do {                                                                                                                             \
+    if (post) launch_kernel(residual_rms_norm_kernel<T, V, true>, dim3(M), dim3(threads), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps, \
+                            rows, post, mult);                                                                                     \
+    else launch_kernel(residual_rms_norm_kernel<T, V, false>, dim3(M), dim3(threads), 0, st, 1, x, d, ldd, yo, ldy, w, N, eps,     \
+                       rows, post, mult);                                                                                          \
+  } while (0)
   if (vpt <= 1) TEENY_RRN(1);
   else if (vpt <= 2) TEENY_RRN(2);
   else if (vpt <= 4) TEENY_RRN(4);
@@ -1148,10 +1179,11 @@ int launch_residual_norm(float* x, const void* delta, long long ldd, void* y, lo
 }  // namespace
 
 int residual_rms_norm(float* x, const void* delta, long long ldd, void* y, long long ldy, const float* w, int M, int N, float eps,
-                      const int* rows, bool f32, cudaStream_t st) {
+                      const int* rows, bool f32, cudaStream_t st, const float* post, float mult) {
   if (!x || !y || !w || M <= 0 || N <= 0) return TEENY_ERR_BAD_ARG;
-  return f32 ? launch_residual_norm<float>(x, delta, ldd, y, ldy, w, M, N, eps, rows, st)
-             : launch_residual_norm<bf16>(x, delta, ldd, y, ldy, w, M, N, eps, rows, st);
+  if (!delta) post = nullptr;
+  return f32 ? launch_residual_norm<float>(x, delta, ldd, y, ldy, w, M, N, eps, rows, post, mult, st)
+             : launch_residual_norm<bf16>(x, delta, ldd, y, ldy, w, M, N, eps, rows, post, mult, st);
 }
 
 int tanh_rows(const void* x, long long ldx, void* y, long long ldy, int M, int N, bool f32, cudaStream_t st) {

@@ -136,6 +136,11 @@ struct AttnShape {
   int causal;
   int window = 0;           // attention_prefill_bf16, causal: query i sees only its last `window` keys (0 = all)
   float out_scale = 1.0f;   // factor of the output (attention_prefill_bf16, attention_decode_bf16)
+  int DV = 0;               // value size (0: D); attention_prefill_bf16 and ring decode take any D, DV <= 128, multiples of 8
+  float softcap = 0.0f;     // > 0: scores s * scale are capped, softcap * tanh(s * scale / softcap)
+  const float* sink = nullptr;   // [Hq]: exp(sink) joins the softmax denominator of the head
+  const bf16* gate = nullptr;    // attention_decode_bf16: output times sigmoid(gate); batch stride gate_sb, heads DV apart
+  long long gate_sb = 0;
 };
 int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, float* lse, const AttnShape& s,
                            cudaStream_t stream);
@@ -160,7 +165,7 @@ struct DecodeRope {
 };
 // Decode over ring caches with per-sequence positions: sequence b's cache is row seqs[b].slot of the cache tensors (`slots`
 // of them, s.Skv = ring rows), its new key is already in row pos % ring, and it attends over min(pos + 1, ring) rows.
-// Head size 64 or 128.
+// Head sizes up to 128, multiples of 8 (D and DV of the AttnShape).
 struct DecodeRing {
   const SeqDesc* seqs;
   int slots;
@@ -291,9 +296,14 @@ struct MinGru {
 };
 int min_gru(const MinGru& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
 
-// Sliding-window grouped-query attention over a ring cache.  Query i sees keys i - window + 1 .. i.  Keys of positions
-// below the entry's `pos` come from the ring (row position % ring of [slots, Hkv, ring, D]); those of the entry itself
-// from k_new / v_new (row of the token, head at column head * D).
+// Sliding-window grouped-query attention over a ring cache.  Query i sees keys i - window + 1 .. i.  Where they are:
+//   kKeysSplit   positions below the entry's `pos` in the ring (row position % ring of [slots, Hkv, ring, D]), the entry's own
+//                in k_new / v_new (row of the token, head at column head * D)
+//   kKeysInRing  all in the ring (head_norm_rope_rows put the entry's own there; k_new / v_new unused)
+//   kKeysInNew   all in k_new / v_new: position j in the row of the entry's first token + j - pos (the rings unused)
+// Scores q . k * scale are capped (softcap > 0), a head's sink joins its denominator, and the output is
+// multiplied by out_scale and by sigmoid(gate).
+constexpr int kKeysSplit = 0, kKeysInRing = 1, kKeysInNew = 2;
 struct WindowAttn {
   int f32;
   const void* q;             // [T, ldq], normed and rotated
@@ -311,42 +321,113 @@ struct WindowAttn {
   float scale, out_scale;
   int slots;                 // state slots: rows of the ring tensors
   int uniform_fresh;         // every entry starts at position 0 and has the step's longest length, rows in order
-  int in_ring;               // single tokens: k_new / v_new are in the ring already (head_norm_rope_rows)
-  void* scratch;             // attention_decode_scratch_bytes(entries, Hq, D, ring), or null
+  int keys;                  // kKeys*
+  void* scratch;             // attention_decode_scratch_bytes(entries, Hq, head size, ring), or null
   size_t scratch_bytes;
   unsigned* counters;        // entries * Hkv words, zero between calls
+  float softcap;
+  const float* sink;         // [Hq], or null
+  const void* gate;          // [T, ldg], heads DV apart, or null
+  long long ldg;
+  const SeqDesc* host;       // the entries in host memory, where the caller has them: with kKeysInRing groups of equal long entries,
+                             // with kKeysInNew a single long entry, then run on the tcgen05 kernel
 };
 // Per-head RMSNorm of q (in place) and k (k_raw -> k_out), then rotary positions on the first rot_dims dimensions
-// (i with i + rot_dims / 2), angles position * inv_freq[i] in f32.  q_w / k_w null: no norm.
+// (i with i + rot_dims / 2), angles position * inv_freq[i] in f32, cos and sin times rot_scale.  q_w / k_w null: no norm.
 struct HeadNormRope {
   int f32;
   void* q;
   long long ldq;
-  const void* k_raw;
+  const void* k_raw;         // null (Hkv = 0): q alone
   long long ldkr;
-  void* k_out;
+  void* k_out;               // null: the ring only
   long long ldk;
   const float *q_w, *k_w, *inv_freq;
   int Hq, Hkv, D, rot_dims;
   float eps;
-  // ring > 0 (single tokens): the rotated key also goes to its row of the ring, and with v_ring the raw key to the value ring
+  // ring > 0: the rotated key also goes to row position % ring of the ring (no two tokens of an entry may share a row), and
+  // with v_ring the raw key (v null) or the value to the value ring
   void* k_ring;
   void* v_ring;
   int ring;
+  float rot_scale;
+  // Values [T, ldv], Hkv heads of DV, on their way into the value ring: kMixKeep copies them to v_first, kMixWith replaces
+  // them by (1 - lambda) v + lambda v_first, lambda = *mix.
+  const void* v;
+  long long ldv;
+  int DV, v_mode;
+  void* v_first;
+  long long ldvf;
+  const float* mix;
 };
+constexpr int kMixNone = 0, kMixKeep = 1, kMixWith = 2;
 int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
 int window_attention_prepare();
 int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
 // The last min(len, ring) tokens of every entry into the ring.
 int ring_append(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
 
+// ---- latent attention (csrc/attention_latent.cu) ----
+// A cache row is one token's [latent c (KR = pad8(rank)) | rotated key part (RD)], shared by all heads.
+// latent_prepare: cq = rms_norm(proj[off_q .. + q_rank]) * q_w; c = rms_norm(proj[off_c .. + rank]) * c_w; the rotated part of
+// proj[off_r .. + RD] (rotate-half layout, cos and sin times rot_scale); the row goes to `rows` [T, KR + RD] and to the cache
+// [slots, max_len, KR + RD].
+struct LatentPrepare {
+  int f32;
+  const void* proj;
+  long long ld;
+  int off_q, off_c, off_r, q_rank, rank, RD;
+  const float *q_w, *c_w, *inv_freq;  // q_w, c_w padded to a multiple of 8
+  float eps, rot_scale;
+  void* cq;                  // [T, ldcq]
+  long long ldcq;
+  void* rows;                // [T, KR + RD], or null
+  void* cache;
+  int max_len;
+};
+int latent_prepare(const LatentPrepare& a, const SeqDesc* seqs, int n_seqs, int max_len, cudaStream_t st);
+// y[t, h * y_head + n] = sum_k x[t, h * x_head + k] w[h, n, k], one small product per head (w [H, N, K] contiguous, K and N
+// multiples of 8).  With RD > 0 the head's RD elements x[t, h * x_head + rot_off ..] are rotated by the token's position as in
+// head_norm_rope_rows and written behind the N columns.
+struct HeadLinear {
+  int f32;
+  const void* x;
+  long long ldx, x_head;
+  const void* w;
+  void* y;
+  long long ldy, y_head;
+  int H, N, K, T;            // T rows
+  int RD, rot_off;
+  const float* inv_freq;
+  float rot_scale;
+  const SeqDesc* seqs;       // RD > 0: the entries that hold the T rows (row0 of the first is row 0 of x and y)
+  int n_seqs;
+};
+int head_linear(const HeadLinear& a, cudaStream_t st);
+// Causal attention of H query heads over one shared key per token whose first DV elements are the value: q [T, ldq] with
+// heads D apart, cache [slots, max_len, D] holding the entries' own rows already, out [T, ldo] with heads DV apart.
+struct LatentAttn {
+  int f32;
+  const void* q;
+  long long ldq;
+  const void* cache;
+  int max_len;
+  void* out;
+  long long ldo;
+  int H, D, DV;
+  float scale;
+};
+int latent_attention_prepare();
+int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int longest, cudaStream_t st);
+
 // f32 residual stream: x = embed[id] * scale; x += delta, y = rms_norm(x) * w (y in the activation type).
 int embedding_scaled(const int* ids, const void* table, float* x, int T, int width, int vocab, float scale, bool f32,
                      cudaStream_t st);
 // delta null: nothing is added.  rows null: row i -> y row i, and x is updated; else y row i comes from x row rows[i] (plus
 // its delta) and x stays as it is.
+// post: what is added is rms_norm(delta) * post * mult (post null: delta as it is).
 int residual_rms_norm(float* x, const void* delta, long long ldd, void* y, long long ldy, const float* w, int M, int N, float eps,
-                      const int* rows, bool f32, cudaStream_t st);
+                      const int* rows, bool f32, cudaStream_t st, const float* post = nullptr, float mult = 1.0f);
 int tanh_rows(const void* x, long long ldx, void* y, long long ldy, int M, int N, bool f32, cudaStream_t st);
 // act(gate) * up from rows interleaved in blocks of 64 (kGlu* of common.cuh), f32
 int glu_interleaved_f32(const float* gu, long long ld, float* out, long long ldo, int T, int inter, int kind, cudaStream_t st);

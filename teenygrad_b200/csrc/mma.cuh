@@ -31,6 +31,15 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
+// Soft-capped score in the log2 domain: log2(e) cap tanh(s scale / cap), through tanh(y) = 1 - 2 / (1 + exp(2 y)).  `two_y` =
+// 2 log2(e) scale / cap, cap_l2 = log2(e) cap; absolute error about 1e-7 cap.
+__device__ __forceinline__ float softcap_log2(float s, float two_y, float cap_l2) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(ex2(s * two_y) + 1.0f));
+  return fmaf(-2.0f * cap_l2, r, cap_l2);
+}
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+
 // Two f32 values as bf16 pairs: x = hi + lo up to 2^-17 of |x|.
 __device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x, y);

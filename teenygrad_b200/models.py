@@ -26,7 +26,12 @@ def _fiferax(config, tensors, dtype, **sizes):
     return fiferax.build(config, tensors, dtype, **sizes)
 
 
-REGISTRY = {"Qwen3ForCausalLM": _qwen3, "Fiferax": _fiferax}
+def _molitar(config, tensors, dtype, **sizes):
+    from . import molitar
+    return molitar.build(config, tensors, dtype, **sizes)
+
+
+REGISTRY = {"Qwen3ForCausalLM": _qwen3, "Fiferax": _fiferax, "Molitar": _molitar}
 
 
 def architecture(config):

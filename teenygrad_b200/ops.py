@@ -439,10 +439,76 @@ def window_attention(q, k, v, k_ring, v_ring, window, score_scale, seqs, max_len
     return out
 
 
-def residual_rms_norm(x, delta, weight, eps):
-    """x f32 [rows, n] += delta (in place); returns rms_norm(x) * weight in delta's type."""
+def residual_rms_norm(x, delta, weight, eps, post=None, mult=1.0):
+    """x f32 [rows, n] += delta, or rms_norm(delta) * post * mult (in place); returns rms_norm(x) * weight in delta's type."""
     _req(x, _F32, "x"); _req(weight, _F32, "weight")
     y = torch.empty(x.shape, dtype=delta.dtype, device=x.device)
     check(lib.teeny_residual_rms_norm(_f32_flag(delta), _ptr(x), _ptr(delta), delta.stride(0), _ptr(y), y.stride(0), _ptr(weight),
-                                      x.shape[0], x.shape[1], float(eps), _stream()), "residual_rms_norm")
+                                      x.shape[0], x.shape[1], float(eps), _ptr(post), float(mult), _stream()), "residual_rms_norm")
     return y
+
+
+def rope_cache(q, k, v, k_cache, v_cache, inv_freq, rot_dims, seqs, max_len, rot_scale=1.0, v_first=None, mix=None):
+    """q [rows, heads, dim] rotated in place; the rotated k [rows, kv_heads, dim] and v [rows, kv_heads, vdim] into the caches
+    [slots, kv_heads, max_len, .].  ``v_first`` alone: receives v; with ``mix`` f32 [1]: v <- (1 - mix) v + mix v_first."""
+    _req(q, name="q"); _req(k, q.dtype, "k"); _req(v, q.dtype, "v"); _req(k_cache, q.dtype, "k_cache"); _req(v_cache, q.dtype, "v_cache")
+    mode = 0 if v_first is None else (1 if mix is None else 2)
+    check(lib.teeny_rope_cache(_f32_flag(q), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(k_cache), _ptr(v_cache),
+                               k_cache.shape[2], _ptr(inv_freq), float(rot_scale), q.shape[1], k.shape[1], q.shape[2], v.shape[2], rot_dims,
+                               mode, _ptr(v_first), _ptr(mix), _ptr(seqs), seqs.shape[0], max_len, _stream()), "rope_cache")
+
+
+def cached_attention(q, k_cache, v_cache, score_scale, entries, softcap=0.0, sink=None, gate=None, out=None, scratch=None):
+    """Causal attention of ``entries`` (see seq_table) over caches [slots, kv_heads, max_len, .] that hold their own tokens
+    already; q [rows, heads, dim], ``gate`` [rows, heads * vdim].  ``scratch``: (uint8 buffer, zeroed int32 counters) for single
+    tokens, made here when missing."""
+    _req(q, name="q"); _req(k_cache, q.dtype, "k_cache"); _req(v_cache, q.dtype, "v_cache")
+    slots, G, cap, V = v_cache.shape
+    H, D = q.shape[1:]
+    n, longest = len(entries), max(e[3] for e in entries)
+    out = torch.zeros(q.shape[0], H, V, dtype=q.dtype, device=q.device) if out is None else out
+    if scratch is None and longest == 1:
+        scratch = (torch.empty(lib.teeny_attn_decode_scratch_bytes(n, H, 128, cap), dtype=torch.uint8, device=q.device),
+                   torch.zeros(n * G, dtype=torch.int32, device=q.device))
+    seqs = seq_table(entries, q.device)
+    host = seq_table(entries, "cpu")
+    check(lib.teeny_cached_attention(_f32_flag(q), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), slots, cap, _ptr(out), out.stride(0), H, G,
+                                     D, V, float(score_scale), float(softcap), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                     _ptr(scratch[0]) if scratch else None, scratch[0].numel() if scratch else 0,
+                                     _ptr(scratch[1]) if scratch else None, _ptr(seqs), _ptr(host), n, longest, _stream()), "cached_attention")
+    return out
+
+
+def latent_prepare(proj, offs, q_rank, rank, q_weight, c_weight, inv_freq, eps, cache, seqs, max_len, rot_scale=1.0, latents=None):
+    """``proj`` [rows, .] with the query latent, the latent and the shared key part at columns ``offs``; weights zero-padded to
+    multiples of 8.  Fills ``cache`` [slots, max_len, pad8(rank) + rot_dims] (and ``latents`` [rows, ..]); returns the normed
+    query latent [rows, pad8(q_rank)]."""
+    _req(proj, name="proj"); _req(cache, proj.dtype, "cache")
+    cq = torch.zeros(proj.shape[0], (q_rank + 7) // 8 * 8, dtype=proj.dtype, device=proj.device)
+    rot = cache.shape[2] - (rank + 7) // 8 * 8
+    check(lib.teeny_latent_prepare(_f32_flag(proj), _ptr(proj), proj.stride(0), *offs, q_rank, rank, rot, _ptr(q_weight), _ptr(c_weight),
+                                   _ptr(inv_freq), float(eps), float(rot_scale), _ptr(cq), cq.stride(0), _ptr(latents), _ptr(cache),
+                                   cache.shape[1], _ptr(seqs), seqs.shape[0], max_len, _stream()), "latent_prepare")
+    return cq
+
+
+def head_linear(x, w, rot_dims=0, rot_off=0, inv_freq=None, rot_scale=1.0, seqs=None, out=None):
+    """Per-head product: x [rows, heads, .] (a view; its first k elements), w [heads, n, k] -> [rows, heads, n + rot_dims]; the
+    elements x[.., rot_off: rot_off + rot_dims] are rotated (rotate-half) by their token's position into the last columns."""
+    _req(x, name="x"); _req(w, x.dtype, "w")
+    H, N, K = w.shape
+    out = torch.zeros(x.shape[0], H, N + rot_dims, dtype=x.dtype, device=x.device) if out is None else out
+    check(lib.teeny_head_linear(_f32_flag(x), _ptr(x), x.stride(0), x.stride(1), _ptr(w), _ptr(out), out.stride(0), out.stride(1), H, N, K,
+                                x.shape[0], rot_dims, rot_off, _ptr(inv_freq), float(rot_scale), _ptr(seqs),
+                                0 if seqs is None else seqs.shape[0], _stream()), "head_linear")
+    return out
+
+
+def latent_attention(q, cache, vdim, score_scale, seqs, max_len, out=None):
+    """q [rows, heads, dim] over ``cache`` [slots, max_len, dim], whose rows' first ``vdim`` elements are the values; causal, the
+    entries' own rows are in the cache already.  Returns [rows, heads, vdim]."""
+    _req(q, name="q"); _req(cache, q.dtype, "cache")
+    out = torch.zeros(q.shape[0], q.shape[1], vdim, dtype=q.dtype, device=q.device) if out is None else out
+    check(lib.teeny_latent_attention(_f32_flag(q), _ptr(q), q.stride(0), _ptr(cache), cache.shape[1], _ptr(out), out.stride(0), q.shape[1],
+                                     q.shape[2], vdim, float(score_scale), _ptr(seqs), seqs.shape[0], max_len, _stream()), "latent_attention")
+    return out
