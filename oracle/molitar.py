@@ -217,7 +217,9 @@ def tensor_shapes(config):
         else:
             for n, rows in (("q", H * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
                 s.update({p + n: (rows, d), p + n + ".b": (rows,)})
-            s.update({p + "vmix": (), p + "sink": (H,), p + "g": (H * m["vdim"], d), p + "o": (d, H * m["vdim"])})
+            if m.get("v_mix"):
+                s[p + "vmix"] = ()
+            s.update({p + "sink": (H,), p + "g": (H * m["vdim"], d), p + "o": (d, H * m["vdim"])})
         if layer["mlp"] is not None:
             p, ff = f"l{i}.", layer["mlp"]["ff"]
             s.update({p + "norm2": (d,), p + "norm2b": (d,), p + "mlp.gate": (ff, d), p + "mlp.up": (ff, d), p + "mlp.down": (d, ff)})
@@ -230,7 +232,7 @@ def make_weights(config, seed):
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in sorted(tensor_shapes(config).items()):
-        t = torch.randn(*shape, generator=g)
+        t = torch.randn(shape, generator=g)
         if name.endswith("vmix"):
             t = 0.2 + 0.6 * torch.rand((), generator=g)
         elif len(shape) == 2:

@@ -88,7 +88,7 @@ def _branch_weights(layer, t):
     head, value = _heads(layer)
     return {"inputs": [head.place(t("q")), head.place(t("k")), value.place(t("v")), value.place(t("g"))],
             "biases": [head.place(t("q.b")), head.place(t("k.b")), value.place(t("v.b")), None],
-            "out": _columns(t("o"), value), "sink": t("sink"), "value_mix": t("vmix")}
+            "out": _columns(t("o"), value), "sink": t("sink"), **({"value_mix": t("vmix")} if m.get("v_mix") else {})}
 
 
 def _offset(w):
@@ -130,7 +130,7 @@ def tensor_shapes(config):
         else:
             rows = {"q": H * m["dim"], "k": m["kv_heads"] * m["dim"], "v": m["kv_heads"] * m["vdim"]}
             mats = {**{n: (r, d) for n, r in rows.items()}, **{n + ".b": (r,) for n, r in rows.items()}, "g": (H * m["vdim"], d),
-                    "sink": (H,), "vmix": ()}
+                    "sink": (H,), **({"vmix": ()} if m.get("v_mix") else {})}
         out.update({f"{p}mix.{n}": s for n, s in mats.items()})
         out.update({p + "mix.o": (d, H * m["vdim"]), p + "norm1": (d,), p + "norm1b": (d,)})
         if layer["mlp"] is not None:
@@ -148,7 +148,7 @@ class RandomTensors:
     def __getitem__(self, name):
         shape = self.shapes[name]
         g = torch.Generator(device=self.device).manual_seed(self.seed * 1000003 + zlib.crc32(name.encode()))
-        t = torch.randn(*shape, generator=g, device=self.device)
+        t = torch.randn(shape, generator=g, device=self.device)
         if len(shape) == 2:
             t *= shape[1] ** -0.5
         elif name.endswith(("dq.norm", "dkv.norm")):
