@@ -6,7 +6,7 @@
         bench.py --gpus N --steps K --warmup W
     python bench.py --config 1|2|3|4                             # the other BASELINE configs (one GPU)
     python bench.py --impl reference ...                         # CPU arm: what the reference runs for the path
-    python bench.py --model fiferax [--size 1k|4k]               # the Fiferax decoder beside a Qwen3 of equal size (one GPU)
+    python bench.py --model fiferax|molitar [--size 1k|4k]       # a hybrid decoder beside a Qwen3 of equal size (one GPU)
 
 Config 5 (default) and 4: Qwen3-8B / Qwen3-0.6B shaped greedy generation; a "step" is one full generation (prefill,
 then CUDA-graph decode steps; the first new token comes out of the prefill); value = tokens (prompt + generated) per
@@ -68,8 +68,8 @@ def parse_args():
     p.add_argument("--weights", default="bf16", choices=["bf16", "fp8"],
                    help="config 4/5 only: fp8 = projections and LM head as FP8 E4M3 with per-channel scales (weight-only; "
                         "the arithmetic stays bf16 x bf16 -> f32).  A variant beside the headline, not the headline.")
-    p.add_argument("--model", default="qwen3", choices=["qwen3", "fiferax"],
-                   help="fiferax: prefill and decode of the Fiferax decoder and its kernels beside a Qwen3 of equal size (one GPU); "
+    p.add_argument("--model", default="qwen3", choices=["qwen3", "fiferax", "molitar"],
+                   help="fiferax, molitar: prefill and decode of that decoder and its kernels beside a Qwen3 of equal size (one GPU); "
                         "--size picks the layer sizes, --config does not apply")
     p.add_argument("--size", default="4k", choices=["1k", "4k"])
     p.add_argument("--no-cpu-baseline", action="store_true")
@@ -732,17 +732,20 @@ def generation_config(args):
         raise SystemExit(f"parity check failed: {parity}")
 
 
-# ------------------------------------------------------------------------------------------------ the Fiferax decoder
+# ------------------------------------------------------------------------------------------------ the hybrid decoders
 # Layer sizes of real models: every layer has the feed-forward of the Qwen3 it is compared with (same width, layers, heads,
-# feed-forward and vocabulary); layers cycle through delta, parallel, delta, mingru.
-FIFERAX_SIZES = {"1k": dict(width=1024, layers=24, ff=3072, heads=16, kv_heads=8, vocab=32768),
-                 "4k": dict(width=4096, layers=8, ff=12288, heads=32, kv_heads=8, vocab=32768)}
-FIFERAX_WINDOW, FIFERAX_NEW = 1024, 128
-FIFERAX_WORKLOADS = [(16, 2048), (1, 2048)]
+# feed-forward and vocabulary).  Fiferax layers cycle through delta, parallel, delta, mingru; Molitar's through latent
+# attention and full attention.
+HYBRID_SIZES = {"1k": dict(width=1024, layers=24, ff=3072, heads=16, kv_heads=8, vocab=32768,
+                           latent=dict(dim=64, rot_dim=32, vdim=64, q_rank=512, kv_rank=256)),
+                "4k": dict(width=4096, layers=8, ff=12288, heads=32, kv_heads=8, vocab=32768,
+                           latent=dict(dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512))}
+FIFERAX_WINDOW, HYBRID_NEW = 1024, 128
+HYBRID_WORKLOADS = [(16, 2048), (1, 2048)]
 
 
 def fiferax_config_of(size):
-    z = FIFERAX_SIZES[size]
+    z = HYBRID_SIZES[size]
     W, H = z["width"], z["heads"]
     mlp = {"kind": "dense", "ff": z["ff"]}
     delta = {"type": "general_delta", "mixer": {"heads": W // 64, "dim": 64}, "mlp": mlp}
@@ -756,18 +759,9 @@ def fiferax_config_of(size):
             "layers": [[delta, par, delta, gru][i % 4] for i in range(z["layers"])]}
 
 
-def fiferax_kernels(size, peaks, timed, graph_timed):
-    """The new design's kernels and the like ones of Qwen3, each alone at this size: (rows of the table)."""
-    import torch
-    from teenygrad_b200 import ops
-    from teenygrad_b200._lib import lib
-    z = FIFERAX_SIZES[size]
-    W, H, G, win = z["width"], z["heads"], z["kv_heads"], FIFERAX_WINDOW
-    B, S = FIFERAX_WORKLOADS[0]
-    T, H64, H128, D = B * S, W // 64, W // 128, 128
-    g = torch.Generator(device="cuda").manual_seed(3)
-    rnd = lambda *s: torch.randn(*s, generator=g, device="cuda")  # noqa: E731
-    bf = lambda *s: rnd(*s).bfloat16()  # noqa: E731
+def kernel_rows(peaks):
+    """A table of kernels and the function that adds a row: achieved rate (bytes or FLOPs per launch over its time) and its
+    fraction of the measured peak."""
     rows = []
 
     def row(kernel, ms, bound, amount, like=None):
@@ -776,6 +770,22 @@ def fiferax_kernels(size, peaks, timed, graph_timed):
         rows.append({"kernel": kernel, "us": ms * 1e3, "bound": bound, "achieved": ach, "unit": "GB/s" if bound == "hbm" else "TFLOP/s",
                      "frac": ach / peak, **({"like": like} if like else {})})
 
+    return rows, row
+
+
+def fiferax_kernels(size, peaks, timed, graph_timed):
+    """The new design's kernels and the like ones of Qwen3, each alone at this size: (rows of the table)."""
+    import torch
+    from teenygrad_b200 import ops
+    from teenygrad_b200._lib import lib
+    z = HYBRID_SIZES[size]
+    W, H, G, win = z["width"], z["heads"], z["kv_heads"], FIFERAX_WINDOW
+    B, S = HYBRID_WORKLOADS[0]
+    T, H64, H128, D = B * S, W // 64, W // 128, 128
+    g = torch.Generator(device="cuda").manual_seed(3)
+    rnd = lambda *s: torch.randn(*s, generator=g, device="cuda")  # noqa: E731
+    bf = lambda *s: rnd(*s).bfloat16()  # noqa: E731
+    rows, row = kernel_rows(peaks)
     whole = ops.seq_table([(b, 0, b * S, S) for b in range(B)])
     proj = bf(T, 6 * W)
     wz = bf(T, W)
@@ -821,7 +831,7 @@ def fiferax_kernels(size, peaks, timed, graph_timed):
         "hbm", 2.0 * n * H128 * 128 * 128 * 4, "attention, decode")
     del s128
     # decode attention over full rings: min(pos + 1, window) keys
-    from teenygrad_b200.ops import flash_attn_decode, flash_attn_fwd
+    from teenygrad_b200.ops import flash_attn_decode
     for length, name in ((win, "attention, decode (ring of the window)"), (S, "attention, decode")):
         kvs = [(bf(n, G, length, D), bf(n, G, length, D)) for _ in range(6)]
         q1 = bf(n, H, 1, D)
@@ -830,28 +840,142 @@ def fiferax_kernels(size, peaks, timed, graph_timed):
         row(name, graph_timed([(lambda kk=kk, vv=vv: flash_attn_decode(q1, kk, vv, length, D ** -0.5, out=o1, scratch=sc)) for kk, vv in kvs]),
             "hbm", 2.0 * n * G * length * D * 2, "attention, decode" if length == win else None)
         del kvs
-    # Qwen3's like kernels
+    qwen3_kernels(z, B, S, row, timed)
+    return rows
+
+
+def molitar_config_of(size):
+    z = HYBRID_SIZES[size]
+    H, lat = z["heads"], z["latent"]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": H, **lat, "scale": (lat["dim"] + lat["rot_dim"]) ** -0.5,
+        "rot": {"dims": lat["rot_dim"], "base": 1e6, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    full = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": H, "kv_heads": z["kv_heads"], "dim": 128, "vdim": 128, "rot": {"dims": 64, "base": 1e6}, "scale": 128 ** -0.5,
+        "softcap": 30.0, "v_mix": True}}
+    return {"architecture": "Molitar", "logit_scale": 0.25, "norm": {"eps": 1e-6}, "residual_mult": 0.7, "vocab": z["vocab"],
+            "width": z["width"], "layers": [[latent, full][i % 2] for i in range(z["layers"])]}
+
+
+def molitar_kernels(size, peaks, timed, graph_timed):
+    """The design's kernels and the like ones of Qwen3, each alone at this size."""
+    import torch
+    from teenygrad_b200 import ops
+    z = HYBRID_SIZES[size]
+    W, H, G, D, lat = z["width"], z["heads"], z["kv_heads"], 128, z["latent"]
+    B, S = HYBRID_WORKLOADS[0]
+    T = B * S
+    g = torch.Generator(device="cuda").manual_seed(3)
+    rnd = lambda *s: torch.randn(*s, generator=g, device="cuda")  # noqa: E731
+    bf = lambda *s: rnd(*s).bfloat16()  # noqa: E731
+    rows, row = kernel_rows(peaks)
+    table = lambda entries: (ops.seq_table(entries), ops.seq_table(entries, "cpu"))  # noqa: E731
+    whole = table([(b, 0, b * S, S) for b in range(B)])
+    causal = lambda d: 2.0 * B * H * d * S * (S + 1) / 2  # noqa: E731  (FLOPs of one product per visible pair)
+    # ---- prompts
+    sink, inv = rnd(H), torch.rand(D // 2, device="cuda", generator=g)
+    q, out, gate = bf(T, H, D), bf(T, H, D), bf(T, H * D)
+    kc, vc = bf(B, G, S, D), bf(B, G, S, D)
+    row("full attention (cap, sink) + output gate, prefill", timed(lambda: ops.cached_attention(q, kc, vc, D ** -0.5, whole, softcap=30.0, sink=sink,
+                                                                                             gate=gate, out=out)),
+        "tensor", causal(2 * D), "attention, prefill")
+    proj, first, lam = bf(T, (H + 2 * G) * D), bf(T, G * D), torch.full((1,), 0.5, device="cuda")
+    qp, kp, vp = (proj[:, a * D:b * D].view(T, -1, D) for a, b in ((0, H), (H, H + G), (H + G, H + 2 * G)))
+    row("rotary + value mixing + cache", timed(lambda: ops.rope_cache(qp, kp, vp, kc, vc, inv, 64, whole[0], S, v_first=first, mix=lam)), "hbm",
+        2.0 * T * D * (2 * H + 5 * G), "head norm + rotary + cache, bf16 tables")
+    del proj, first
+    KD, V, R, RD, QR = lat["dim"] + lat["rot_dim"], lat["vdim"], lat["kv_rank"], lat["rot_dim"], lat["q_rank"]
+    ql, ol = bf(T, H, KD), bf(T, H, V)
+    kl, vl = bf(B, H, S, KD), bf(B, H, S, V)
+    row("latent attention, expanded, prefill", timed(lambda: ops.cached_attention(ql, kl, vl, KD ** -0.5, whole, out=ol)), "tensor", causal(KD + V),
+        "attention, prefill")
+    del kl, vl, ql, ol, q, out, gate
+    down, cache, latents = bf(T, QR + R + RD), bf(B, S, R + RD), bf(T, R + RD)
+    qw, cw = torch.ones(QR, device="cuda"), torch.ones(R, device="cuda")
+    row("latent norms + rotary + cache", timed(lambda: ops.latent_prepare(down, (0, QR, QR + R), QR, R, qw, cw, inv, 1e-6, cache, whole[0], S,
+                                                                       latents=latents)), "hbm",
+        2.0 * T * (2 * QR + 3 * (R + RD)), "head norm + rotary + cache, bf16 tables")
+    del down, cache, latents
+    x32, delta, w32 = rnd(T, W), bf(T, W), torch.ones(W, device="cuda")
+    row("norm + residual add + norm, f32 residual", timed(lambda: ops.residual_rms_norm(x32, delta, w32, 1e-6, w32, 0.7)), "hbm", T * W * 12,
+        "residual add + norm, bf16")
+    del x32, delta
+    # ---- one token per sequence, weights and caches rotated beyond L2
+    n, copies = B, 6
+    one = table([(b, S - 1, b, 1) for b in range(n)])
+    q1, o1, g1 = bf(n, H, D), bf(n, H, D), bf(n, H * D)
+    from teenygrad_b200._lib import lib
+    scratch = (torch.empty(lib.teeny_attn_decode_scratch_bytes(n, H, 128, S), dtype=torch.uint8, device="cuda"),
+               torch.zeros(n * G, dtype=torch.int32, device="cuda"))
+    kvs = [(bf(n, G, S, D), bf(n, G, S, D)) for _ in range(copies)]
+    row("full attention (cap, sink, gate), decode", graph_timed([(lambda k=k, v=v: ops.cached_attention(
+        q1, k, v, D ** -0.5, one, softcap=30.0, sink=sink, gate=g1, out=o1, scratch=scratch)) for k, v in kvs]), "hbm", 2.0 * n * G * S * D * 2,
+        "attention, decode")
+    del kvs
+    caches = [bf(n, S, R + RD) for _ in range(copies + 2)]
+    ql, ol = bf(n, H, R + RD), bf(n, H, R)
+    row("latent attention, absorbed, decode", graph_timed([(lambda c=c: ops.latent_attention(ql, c, R, KD ** -0.5, one[0], 1, out=ol)) for c in caches]),
+        "hbm", 2.0 * n * S * (R + RD), "attention, decode")
+    del caches
+    qh, vo = bf(n, H, KD), bf(n, H, V)
+    many = max(8, (300 << 20) // (2 * H * R * lat["dim"]))
+    ws = [bf(H, R, lat["dim"]) for _ in range(many)]
+    row("queries into the latent space + rotary, decode", graph_timed([(lambda w=w: ops.head_linear(
+        qh[:, :, RD:], w, RD, -RD, inv, 1.0, one[0], out=ql)) for w in ws]), "hbm", 2.0 * H * R * lat["dim"], "matrix product, decode")
+    ws = [bf(H, V, R) for _ in range(many)]
+    row("values out of the latent space, decode", graph_timed([(lambda w=w: ops.head_linear(ol, w, out=vo)) for w in ws]), "hbm", 2.0 * H * R * V,
+        "matrix product, decode")
+    ws = [bf(H * V, R) for _ in range(many)]
+    x1 = bf(n, R)
+    row("matrix product, decode", graph_timed([(lambda w=w: ops.linear_forward(x1, w)) for w in ws]), "hbm", 2.0 * H * R * V)
+    del ws
+    qwen3_kernels(z, B, S, row, timed)
+    from teenygrad_b200.ops import flash_attn_decode
+    kvs = [(bf(n, G, S, D), bf(n, G, S, D)) for _ in range(copies)]
+    qd = bf(n, H, 1, D)
+    od = torch.empty_like(qd)
+    row("attention, decode", graph_timed([(lambda k=k, v=v: flash_attn_decode(qd, k, v, S, D ** -0.5, out=od, scratch=scratch[0])) for k, v in kvs]),
+        "hbm", 2.0 * n * G * S * D * 2)
+    return rows
+
+
+def qwen3_kernels(z, B, S, row, timed):
+    """The like kernels of the Qwen3 runner over prompts."""
+    import torch
+    from teenygrad_b200 import ops
+    from teenygrad_b200.ops import flash_attn_fwd
+    W, H, G, D, T = z["width"], z["heads"], z["kv_heads"], 128, B * S
+    bf = lambda *s: torch.randn(*s, device="cuda").bfloat16()  # noqa: E731
     qa, ka = bf(B, H, S, D), bf(B, G, S, D)
     row("attention, prefill", timed(lambda: flash_attn_fwd(qa, ka, ka, D ** -0.5, causal=True)), "tensor", 0.5 * 4 * B * H * S * S * D)
-    xr, w16 = bf(T, W), torch.ones(W, dtype=torch.bfloat16, device="cuda")
+    delta, xr, w16 = bf(T, W), bf(T, W), torch.ones(W, dtype=torch.bfloat16, device="cuda")
     row("residual add + norm, bf16", timed(lambda: ops.add_rms_norm(delta, xr, w16, 1e-5)), "hbm", T * W * 8)
-    cos, sin = ops.rope_table(inv, S)
+    cos, sin = ops.rope_table(torch.rand(D // 2, device="cuda"), S)
     qkv, n16 = bf(T, (H + 2 * G) * D), torch.ones(D, dtype=torch.bfloat16, device="cuda")
     kk, vv = (torch.zeros(B, G, S, D, dtype=torch.bfloat16, device="cuda") for _ in range(2))
     row("head norm + rotary + cache, bf16 tables", timed(lambda: ops.qk_norm_rope_kv(qkv, n16, n16, cos, sin, kk, vv, S, H, G, 0, 1e-6)), "hbm",
         2.0 * T * D * (2 * H + 4 * G))
-    return rows
 
 
-def fiferax_bench(args):
+def hybrid_bench(args):
     import torch
-    from teenygrad_b200 import fiferax, qwen3
+    from teenygrad_b200 import fiferax, molitar, qwen3
     from teenygrad_b200._lib import lib
+    name = args.model
     if args.gpus != 1 or args.impl != "ours":
-        raise SystemExit("--model fiferax runs on one GPU")
+        raise SystemExit(f"--model {name} runs on one GPU")
     torch.cuda.set_device(0)
-    peaks, z, NEW = measured_peaks(), FIFERAX_SIZES[args.size], FIFERAX_NEW
-    cfg = fiferax_config_of(args.size)
+    peaks, z, NEW = measured_peaks(), HYBRID_SIZES[args.size], HYBRID_NEW
+    if name == "fiferax":
+        rank = z["width"] // 32
+        cfg, kernel_table = fiferax_config_of(args.size), fiferax_kernels
+        shapes, tensors, module = fiferax.tensor_shapes(cfg, rank), fiferax.RandomTensors(cfg, 7, "cuda", rank), fiferax
+        layers = f"delta, parallel, delta, mingru), window {FIFERAX_WINDOW}"
+    else:
+        cfg, kernel_table = molitar_config_of(args.size), molitar_kernels
+        shapes, tensors, module = molitar.tensor_shapes(cfg), molitar.RandomTensors(cfg, 7, "cuda"), molitar
+        layers = f"latent attention, full attention), latents {z['latent']}"
     warm = max(args.warmup, 3)
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
 
@@ -910,21 +1034,19 @@ def fiferax_bench(args):
     def matmul_params(model):
         if model == "qwen3":
             return z["layers"] * (z["width"] * (2 * z["heads"] + 2 * z["kv_heads"]) * 128 + 3 * z["width"] * z["ff"]) + z["vocab"] * z["width"]
-        shapes = fiferax.tensor_shapes(cfg, z["width"] // 32)
-        return sum(s[0] * s[1] for n, s in shapes.items() if len(s) == 2 and n != "embed")
+        return sum(s[0] * s[1] for n, s in shapes.items() if len(s) == 2 and (n != "embed" or "head" not in shapes))
 
     sampler = ClockSampler(0)
     sampler.start()
     results, launches, e2e = [], 0, None
-    for B, S in FIFERAX_WORKLOADS:
+    for B, S in HYBRID_WORKLOADS:
         g = torch.Generator().manual_seed(6)
         host = torch.randint(0, z["vocab"], (B, S), generator=g, dtype=torch.int32).pin_memory()
         dev = host.cuda()
         entry = {"batch": B, "prefill": S, "new_tokens": NEW}
-        for model in ("fiferax", "qwen3"):
-            if model == "fiferax":
-                r = fiferax.build(cfg, fiferax.RandomTensors(cfg, 7, "cuda", z["width"] // 32), max_batch=B, max_len=S + NEW, max_tokens=B * S,
-                                  max_new_tokens=NEW)
+        for model in (name, "qwen3"):
+            if model == name:
+                r = module.build(cfg, tensors, max_batch=B, max_len=S + NEW, max_tokens=B * S, max_new_tokens=NEW)
                 seqs = [r.open() for _ in range(B)]
 
                 def prefill():
@@ -940,14 +1062,14 @@ def fiferax_bench(args):
                     r.prefill(dev)
             lib.teeny_launch_count(1)
             pre, dec = phases(prefill, lambda: r.decode_step(graph=True), args.steps)
-            if model == "fiferax":
+            if model == name:
                 launches += int(lib.teeny_launch_count(1))
             entry[model] = {"prefill_ms": pre, "decode_ms_per_step": dec / (NEW - 1), "prefill_tok_s": B * S / pre * 1e3,
                             "decode_tok_s": B * (NEW - 1) / dec * 1e3, "tok_s": B * (S + NEW) / (pre + dec) * 1e3,
                             "matmul_params": matmul_params(model),
                             "prefill_matmul_tflops": 2.0 * matmul_params(model) * B * S / pre / 1e9,
                             "decode_weight_gbs": 2.0 * matmul_params(model) / (dec / (NEW - 1)) / 1e6}
-            if model == "fiferax" and e2e is None:
+            if model == name and e2e is None:
                 for s in seqs:
                     r.close(s)
                 out = torch.empty(B, NEW, dtype=torch.int32).pin_memory()
@@ -967,14 +1089,14 @@ def fiferax_bench(args):
             torch.cuda.empty_cache()
         results.append(entry)
     clocks = sampler.stop()
-    kernels = fiferax_kernels(args.size, peaks, timed, graph_timed)
+    kernels = kernel_table(args.size, peaks, timed, graph_timed)
     first = results[0]
-    emit({"metric": "fiferax_tokens_per_s", "value": first["fiferax"]["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+    emit({"metric": f"{name}_tokens_per_s", "value": first[name]["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
           "warmup": args.warmup, "warmup_run": warm,
-          "ms_per_step": first["fiferax"]["prefill_ms"] + first["fiferax"]["decode_ms_per_step"] * (NEW - 1), "higher_is_better": True,
+          "ms_per_step": first[name]["prefill_ms"] + first[name]["decode_ms_per_step"] * (NEW - 1), "higher_is_better": True,
           "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-          "config": {"workload": f"Fiferax {args.size}: width {z['width']}, {z['layers']} layers (delta, parallel, delta, mingru), window "
-                                 f"{FIFERAX_WINDOW}, feed-forward {z['ff']}, vocabulary {z['vocab']}, random weights; beside a Qwen3 of the same "
+          "config": {"workload": f"{name.capitalize()} {args.size}: width {z['width']}, {z['layers']} layers ({layers}, "
+                                 f"feed-forward {z['ff']}, vocabulary {z['vocab']}, random weights; beside a Qwen3 of the same "
                                  "width, layers, heads, feed-forward and vocabulary", "parallelism": "1 GPU",
                      "l2": "inputs larger than L2; kernels alone: L2 flushed before every timed launch, one-token kernels replayed from a graph "
                            "over state copies larger than L2"},
@@ -990,8 +1112,8 @@ def main():
     sys.stdout.flush()
     _JSON_OUT = os.fdopen(os.dup(1), "w")
     os.dup2(2, 1)
-    if args.model == "fiferax":
-        fiferax_bench(args)
+    if args.model != "qwen3":
+        hybrid_bench(args)
     elif args.impl == "reference":
         reference_arm(args)
     elif args.config in (4, 5):

@@ -199,8 +199,9 @@ int teeny_head_linear(int f32, const void* x, long long ldx, long long x_head, c
                       int n_seqs, teeny_stream_t stream);
 /* Causal attention of `heads` query heads over one cached row per token (its first vdim elements are the value): q [rows, ldq]
  * with heads dim apart, cache [slots, max_cached, dim], out with heads vdim apart. */
-int teeny_latent_attention(int f32, const void* q, long long ldq, const void* cache, int max_cached, void* out, long long ldo, int heads,
-                           int dim, int vdim, float score_scale, const int* seqs, int n_seqs, int max_len, teeny_stream_t stream);
+int teeny_latent_attention(int f32, const void* q, long long ldq, int rows, const void* cache, int slots, int max_cached, void* out,
+                           long long ldo, int heads, int dim, int vdim, float score_scale, const int* seqs, int n_seqs, int max_len,
+                           teeny_stream_t stream);
 
 #ifdef __cplusplus
 }

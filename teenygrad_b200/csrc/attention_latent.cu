@@ -9,8 +9,8 @@
 //   latent_prepare_kernel<T>          norms of the query latent and the latent, rotation of the shared key part, cache append
 //   head_linear_mma_kernel<MT>        the small per-head products, bf16 (mma.sync; weights fetched ahead of the dependency wait)
 //   head_linear_rows_kernel<T>        the same, anything
-//   latent_attention_mma_kernel       absorbed attention, bf16 (mma.sync tiles over cp.async stages; the key range is split over
-//                                     a cluster whose CTAs merge through distributed shared memory)
+//   latent_attention_kernel<N>        absorbed attention, bf16 (tcgen05; the key range is split over a cluster whose CTAs merge
+//                                     through distributed shared memory)
 //   latent_attention_rows_kernel<T>   the same, anything: eight warps per (token, head)
 #include <atomic>
 #include <type_traits>
@@ -293,7 +293,7 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int i = blockIdx.x / a.H, h = blockIdx.x % a.H;
   if (i >= seq.len) return;
-  const size_t row = static_cast<size_t>(seq.row0) + i;
+  const size_t row = static_cast<size_t>(seq.row0) - a.row_base + i;
   const T* qr = static_cast<const T*>(a.q) + row * a.ldq + h * a.D;
   const T* kr = static_cast<const T*>(a.cache) + static_cast<size_t>(seq.slot) * a.max_len * a.D;
   float qv[NE], acc[NE];
@@ -346,20 +346,51 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
   }
 }
 
-// CTA = 16 MT consecutive (token, head) rows of one entry x one share of the keys; the CTAs of a cluster hold the shares of
-// one row tile.  Keys come in tiles of 64 cache rows through two cp.async stages.  Eight warps; per tile
-//   scores   warp (kq, kh) multiplies a quarter of the row's dimensions (its queries stay in registers for the whole walk) for
-//            32 of the keys; the four partial sums meet in shared memory, where each row belongs to 256 / rows threads that
-//            keep its running maximum and sum and write the weights as bf16;
-//   values   warp w owns 16 NV columns of the value and multiplies the weights with them, the same cache rows transposed on
-//            the way out of shared memory.
-// At the end the shares are scaled to the cluster's maximum and summed through distributed shared memory, every CTA a slice
-// of the columns.  Columns between D and 64 NK are zero in shared memory.
-constexpr int kLatKeys = 64;
-constexpr int lat_ld(int nk) { return 64 * nk + 8; }
-constexpr int kLatSLd = kLatKeys + 2, kLatPLd = kLatKeys + 8;
-constexpr int lat_smem_bytes(int mt, int nk) {
-  return 2 * kLatKeys * lat_ld(nk) * 2 + 4 * 16 * mt * kLatSLd * 4 + 16 * mt * kLatPLd * 2 + 3 * 16 * mt * 4;
+// Absorbed attention on the tensor cores (tcgen05).  CTA = N consecutive (token, head) rows of one entry x one share of its keys;
+// the CTAs of a cluster hold the shares of one row tile.  The rows are the N side of both products, so a few query heads waste
+// nothing, and the cache rows, loaded once per 128-key tile, are the A operand of both:
+//   S^T [128 keys, N]   = C [128 keys, D] Q^T          C K-major, Q in shared memory for the whole walk
+//   O^T [DV, N]        += C^T [DV, 128 keys] P^T       the same shared memory read MN-major; one M = 128 product per 128 values
+// Tensor memory: O^T in ceil(DV / 128) blocks of N columns, two S^T buffers of N columns.
+//   warp 4   TMA producer: ring of 32 KB slots, each 128 keys x 128 value dimensions (two [128 keys][64 d] boxes); the dimensions
+//            behind the values (the rotated part) travel in a ring of single boxes.  A slot is free again when its product with P
+//            has completed, so the next tile's loads follow the current one's products block by block.  Starts before the
+//            dependency wait: only the queries come from the kernel in front of this one.
+//   warp 5   allocates tensor memory, loads the queries, issues the MMAs (one thread); S of tile t + 1 goes ahead of P V of tile t
+//            where the ring holds two tiles.
+//   warps 0-3  thread = key in a tile: its N scores out of tensor memory, mask, weights against the rows' running maxima (shared
+//            memory), sums in registers, weights as bf16 into shared memory ([row][key], the B operand).  The maxima only move when
+//            some score exceeds its row's by more than 2^8 (one vote per tile); then the tile's maxima are reduced across the
+//            lanes and O^T is rescaled.
+// At the end the shares meet in distributed shared memory: every CTA sums a slice of the columns, scaled to the common maximum.
+constexpr int kLatTile = 128, kLatPair = 32768, kLatBox = 16384, kLatMaxSlots = 12, kLatThreads = 192;
+constexpr float kLatGrow = 8.0f;  // log2 units
+
+struct LatTcArgs {
+  bf16* out;
+  long long ldo;
+  int row_base;        // step row that row 0 of q and out stands for
+  int H, D, DV;
+  int pairs, rests;    // 128-dimension slots of a tile that hold values; single boxes behind them
+  int slots, rest_slots, ahead;
+  int o_ld;            // row stride (floats) of the output staging
+  uint32_t tmem_cols;
+  float scale_log2;
+  int* err;
+};
+
+struct LatSmem {  // byte offsets
+  int rest, q, p, bars, stats, total;
+};
+__host__ __device__ inline LatSmem lat_smem(int n, int pairs, int rests, int slots, int rest_slots) {
+  LatSmem s;
+  s.rest = slots * kLatPair;
+  s.q = s.rest + rest_slots * kLatBox;
+  s.p = s.q + (2 * pairs + rests) * n * 128;
+  s.bars = s.p + 2 * n * 128;
+  s.stats = s.bars + 8 * (2 * kLatMaxSlots + 2 * kLatMaxSlots + 8);
+  s.total = s.stats + 4 * 9 * n + 1024;
+  return s;
 }
 
 __device__ __forceinline__ void cluster_sync() {
@@ -379,237 +410,454 @@ __device__ __forceinline__ float2 ld_cluster2(uint32_t local_addr, uint32_t rank
   asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(r) : "memory");
   return v;
 }
+// whether `v` holds in any of the 128 softmax threads (barrier 1)
+__device__ __forceinline__ bool any128(bool v) {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbar.red.or.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+               : "=r"(r) : "r"(static_cast<uint32_t>(v)) : "memory");
+  return r != 0;
+}
+// N consecutive tensor-memory columns of this warp's lanes
+template <int N>
+__device__ __forceinline__ void tmem_ld_cols(uint32_t addr, float (&v)[N]) {
+  if constexpr (N == 16) {
+    uint32_t t[16];
+    tmem_ld_32x16(addr, t);
+    tmem_wait_ld();
+#pragma unroll
+    for (int e = 0; e < 16; ++e) v[e] = __uint_as_float(t[e]);
+  } else {
+    uint32_t t[N / 32][32];
+#pragma unroll
+    for (int i = 0; i < N / 32; ++i) tmem_ld_32x32(addr + 32 * i, t[i]);
+    tmem_wait_ld();
+#pragma unroll
+    for (int i = 0; i < N / 32; ++i)
+#pragma unroll
+      for (int e = 0; e < 32; ++e) v[32 * i + e] = __uint_as_float(t[i][e]);
+  }
+}
+template <int N>
+__device__ __forceinline__ void tmem_st_cols(uint32_t addr, const float (&v)[N]) {
+  if constexpr (N == 16) {
+    uint32_t t[16];
+#pragma unroll
+    for (int e = 0; e < 16; ++e) t[e] = __float_as_uint(v[e]);
+    tmem_st_32x16(addr, t);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N / 32; ++i) {
+      uint32_t t[32];
+#pragma unroll
+      for (int e = 0; e < 32; ++e) t[e] = __float_as_uint(v[32 * i + e]);
+      tmem_st_32x32(addr + 32 * i, t);
+    }
+  }
+}
+// Reduction of W columns over the warp's lanes, halving the columns a lane holds at every step; lane i ends with column i % W.
+template <int W, bool MAX>
+__device__ __forceinline__ float reduce_columns(float (&v)[W]) {
+  const int lane = threadIdx.x & 31;
+  auto op = [](float a, float b) { return MAX ? fmaxf(a, b) : a + b; };
+  if (W == 16) {
+#pragma unroll
+    for (int i = 0; i < 16; ++i) v[i] = op(v[i], __shfl_xor_sync(0xffffffffu, v[i], 16));
+  }
+#pragma unroll
+  for (int w = W / 2; w > 0; w >>= 1)
+#pragma unroll
+    for (int i = 0; i < w; ++i) {
+      const bool hi = (lane & w) != 0;
+      const float keep = hi ? v[i + w] : v[i], send = hi ? v[i] : v[i + w];
+      v[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, w));
+    }
+  return v[0];
+}
+// ... of all N columns, into dst[N] of this warp
+template <int N, bool MAX>
+__device__ __forceinline__ void reduce_to(const float (&v)[N], float* dst) {
+  constexpr int W = N < 32 ? N : 32;
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int i = 0; i < N / W; ++i) {
+    float t[W];
+#pragma unroll
+    for (int e = 0; e < W; ++e) t[e] = v[W * i + e];
+    const float r = reduce_columns<W, MAX>(t);
+    if (lane < W) dst[W * i + lane] = r;
+  }
+}
 
-template <int MT, int NK, int NV>
-__global__ void __launch_bounds__(256) latent_attention_mma_kernel(const LatentAttn a, const SeqDesc* __restrict__ seqs) {
-  constexpr int R = 16 * MT, LD = lat_ld(NK), CH = 8 * NK, TPR = 256 / R, KPT = kLatKeys / TPR;  // threads per row, keys per thread
-  extern __shared__ __align__(16) uint8_t lat_smem[];
-  bf16* stage0 = reinterpret_cast<bf16*>(lat_smem);
-  float* sp = reinterpret_cast<float*>(lat_smem + 2 * kLatKeys * LD * 2);   // [4][R][kLatSLd] partial scores
-  bf16* pb = reinterpret_cast<bf16*>(sp + 4 * R * kLatSLd);                 // [R][kLatPLd] weights
-  float* row_f = reinterpret_cast<float*>(pb + R * kLatPLd);                // [3][R]: rescale factor of the tile; final maximum, sum
+template <int N>
+__global__ void __launch_bounds__(kLatThreads, 1)
+latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid_constant__ CUtensorMap tmap_q, const LatTcArgs a,
+                        const SeqDesc* __restrict__ seqs) {
+  extern __shared__ uint8_t lat_raw[];
   const SeqDesc seq = seqs[blockIdx.z];  // written well before the kernel in front of this one
-  const int row0 = blockIdx.y * R, n_rows = min(R, seq.len * a.H - row0);
-  if (n_rows <= 0) {                     // the whole cluster
+  const int row0 = blockIdx.y * N, n_rows = min(N, seq.len * a.H - row0);
+  if (n_rows <= 0) {  // the whole cluster
     pdl_wait();
     return;
   }
+  const uint32_t base = (smem_u32(lat_raw) + 1023u) & ~1023u;
+  uint8_t* gen = lat_raw + (base - smem_u32(lat_raw));
+  const LatSmem lay = lat_smem(N, a.pairs, a.rests, a.slots, a.rest_slots);
+  const uint32_t bar0 = base + lay.bars;
+  auto full = [&](int i) { return bar0 + 8u * i; };
+  auto empty = [&](int i) { return bar0 + 8u * (kLatMaxSlots + i); };
+  auto rfull = [&](int i) { return bar0 + 8u * (2 * kLatMaxSlots + i); };
+  auto rempty = [&](int i) { return bar0 + 8u * (3 * kLatMaxSlots + i); };
+  const uint32_t misc = bar0 + 8u * 4 * kLatMaxSlots;
+  const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40;  // two s_full
+  float* m_sh = reinterpret_cast<float*>(gen + lay.stats);  // [N] running maxima, log2 domain
+  float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally the row sums
+  float* red = alpha_sh + N;                                // [4][N]
+  int* lim = reinterpret_cast<int*>(red + 4 * N);           // [N] last key each row sees
+
   const int splits = gridDim.x, split = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int L = seq.pos + (row0 + n_rows - 1) / a.H + 1;  // keys the tile's last row sees
-  const int span = ((L + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
+  const int span = ((L + splits - 1) / splits + kLatTile - 1) / kLatTile * kLatTile;
   const int key0 = split * span, key_end = min(L, key0 + span);
-  const int n_tiles = key0 < key_end ? (key_end - key0 + kLatKeys - 1) / kLatKeys : 0;
-  const bf16* cache = static_cast<const bf16*>(a.cache) + static_cast<size_t>(seq.slot) * a.max_len * a.D;
-  const uint32_t st_a = smem_u32(stage0);
+  const int n_tiles = key0 < key_end ? (key_end - key0 + kLatTile - 1) / kLatTile : 0;
 
-  for (int idx = threadIdx.x; idx < 2 * kLatKeys * (CH - a.D / 8); idx += 256) {  // columns that no copy fills
-    const int r = idx / (CH - a.D / 8), ch = a.D / 8 + idx % (CH - a.D / 8);
-    zero16(st_a + static_cast<uint32_t>(r * LD + ch * 8) * 2);
+  if (threadIdx.x == 128) {
+    tma_prefetch_desc(&tmap_c);
+    tma_prefetch_desc(&tmap_q);
+    for (int i = 0; i < a.slots; ++i) {
+      mbar_init(full(i), 1);
+      mbar_init(empty(i), 1);
+    }
+    for (int i = 0; i < a.rest_slots; ++i) {
+      mbar_init(rfull(i), 1);
+      mbar_init(rempty(i), 1);
+    }
+    mbar_init(q_full, 1);
+    mbar_init(s_full, 1);
+    mbar_init(s_full + 8, 1);
+    mbar_init(p_ready, 128);
+    mbar_init(pv_done, 1);
+    mbar_fence_init();
   }
-  pdl_wait();
-  auto load_tile = [&](int t) {
-    const uint32_t dst0 = st_a + static_cast<uint32_t>((t & 1) * kLatKeys * LD) * 2;
-    const int n = a.D / 8;
-    for (int idx = threadIdx.x; idx < kLatKeys * n; idx += 256) {
-      const int r = idx / n, ch = idx - r * n, j = key0 + t * kLatKeys + r;
-      const uint32_t dst = dst0 + static_cast<uint32_t>(r * LD + ch * 8) * 2;
-      if (j < key_end) cp_async16(dst, cache + static_cast<size_t>(j) * a.D + ch * 8);
-      else zero16(dst);
-    }
-    cp_async_commit();
-  };
-  if (n_tiles > 0) load_tile(0);
+  if (warp == 5) {
+    tmem_alloc(tmem_slot, a.tmem_cols);
+    tmem_relinquish();
+  }
+  if (threadIdx.x < N) {
+    m_sh[threadIdx.x] = -INFINITY;
+    lim[threadIdx.x] = seq.pos + min(row0 + static_cast<int>(threadIdx.x), row0 + n_rows - 1) / a.H;
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(gen + lay.bars + 8 * 4 * kLatMaxSlots + 40);
+  const uint32_t t_s = tmem + a.pairs * N;
+  bool ok = true;
 
-  // query fragments of this warp's quarter of the dimensions
-  const int kq = warp & 3, kh = warp >> 2;
-  uint32_t qf[MT][NK][4];
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = row0 + mt * 16 + g + 8 * e, tok = r / a.H, h = r - tok * a.H;
-      const bool in = r < row0 + n_rows;
-      const bf16* q = static_cast<const bf16*>(a.q) + (static_cast<size_t>(seq.row0) + (in ? tok : 0)) * a.ldq + (in ? h : 0) * a.D;
-#pragma unroll
-      for (int k = 0; k < NK; ++k) {
-        const int d = (kq * NK + k) * 16 + 2 * c;
-        qf[mt][k][e] = in && d < a.D ? *reinterpret_cast<const uint32_t*>(q + d) : 0u;
-        qf[mt][k][2 + e] = in && d + 8 < a.D ? *reinterpret_cast<const uint32_t*>(q + d + 8) : 0u;
+  if (warp == 4) {
+    // ---------------- producer ----------------
+    if (lane == 0) {
+      bool waited = false;
+      for (int t = 0, g = 0, r = 0; ok && t < n_tiles; ++t) {
+        const int key = key0 + t * kLatTile;
+        for (int p = 0; p < a.pairs + a.rests; ++p) {
+          const bool pair = p < a.pairs;
+          const int idx = pair ? g++ : r++, n = pair ? a.slots : a.rest_slots, slot = idx % n;
+          if (idx >= n && !waited) {  // the rings are full: the queries' kernel has to be done by now anyway
+            pdl_wait();
+            waited = true;
+          }
+          if (!mbar_wait(pair ? empty(slot) : rempty(slot), ((idx / n) & 1) ^ 1, a.err, DEVERR_ATTN_PRODUCER)) { ok = false; break; }
+          if (pair) {
+            mbar_expect_tx(full(slot), kLatPair);
+            tma_load_3d(base + slot * kLatPair, &tmap_c, full(slot), 128 * p, key, seq.slot);
+            tma_load_3d(base + slot * kLatPair + kLatBox, &tmap_c, full(slot), 128 * p + 64, key, seq.slot);
+          } else {
+            mbar_expect_tx(rfull(slot), kLatBox);
+            tma_load_3d(base + lay.rest + slot * kLatBox, &tmap_c, rfull(slot), 128 * a.pairs + 64 * (p - a.pairs), key, seq.slot);
+          }
+        }
       }
-    }
-  float O[MT][2 * NV][4];
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int n = 0; n < 2 * NV; ++n) O[mt][n][0] = O[mt][n][1] = O[mt][n][2] = O[mt][n][3] = 0.0f;
-  // softmax: thread = (row sr, keys KPT * sub ..)
-  const int sr = threadIdx.x / TPR, sub = threadIdx.x % TPR;
-  const int s_pos = seq.pos + min(row0 + sr, row0 + n_rows - 1) / a.H;  // last key this row sees
-  float m = -INFINITY, l = 0.0f;
-  const float sc = a.scale * 1.4426950408889634f;
-  const int v0 = warp * 16 * NV;  // value columns of this warp
-  for (int t = 0; t < n_tiles; ++t) {
-    if (t + 1 < n_tiles) {
-      load_tile(t + 1);
-      cp_async_wait<1>();
+      if (!waited) pdl_wait();
     } else {
-      cp_async_wait<0>();
+      pdl_wait();
     }
-    __syncthreads();
-    const uint32_t kt = st_a + static_cast<uint32_t>((t & 1) * kLatKeys * LD) * 2;
-    {
-      float s[MT][4][4];
+  } else if (warp == 5) {
+    // ---------------- MMA issuer ----------------
+    pdl_wait();
+    if (lane == 0 && n_tiles > 0) {
+      const int boxes = 2 * a.pairs + a.rests;
+      mbar_expect_tx(q_full, boxes * N * 128);
+      for (int b = 0; b < boxes; ++b) tma_load_2d(base + lay.q + b * N * 128, &tmap_q, q_full, 64 * b, (seq.row0 - a.row_base) * a.H + row0);
+      constexpr uint32_t idesc_s = make_idesc_bf16(128, N, false, false), idesc_pv = make_idesc_bf16(128, N, true, false);
+      const uint64_t q_desc = make_smem_desc_sw128(base + lay.q, 16, 1024), p_desc = make_smem_desc_sw128(base + lay.p, 16, 1024);
+      ok = mbar_wait(q_full, 0, a.err, DEVERR_ATTN_MMA);
+      // one 64-dimension box of cache rows times the queries' box
+      auto box_products = [&](uint32_t smem, int box, uint32_t d, bool first) {
+        const uint64_t c_desc = make_smem_desc_sw128(smem, 16, 1024);
+        const int steps = min(4, (a.D - 64 * box + 15) / 16);  // 16 dimensions = 32 bytes along the rows
+        for (int k = 0; k < steps; ++k)
+          umma_bf16_ss(d, c_desc + 2 * k, q_desc + static_cast<uint64_t>(box * N * 8 + 2 * k), idesc_s, first && k == 0 ? 0u : 1u);
+      };
+      auto scores = [&](int t) {
+        const uint32_t d = t_s + (t & 1) * N;
+        for (int p = 0; ok && p < a.pairs; ++p) {
+          const int g = t * a.pairs + p, slot = g % a.slots;
+          ok = mbar_wait(full(slot), (g / a.slots) & 1, a.err, DEVERR_ATTN_MMA);
+          tc_fence_after();
+          box_products(base + slot * kLatPair, 2 * p, d, p == 0);
+          if (128 * p + 64 < a.D) box_products(base + slot * kLatPair + kLatBox, 2 * p + 1, d, false);
+        }
+        for (int r = 0; ok && r < a.rests; ++r) {
+          const int g = t * a.rests + r, slot = g % a.rest_slots;
+          ok = mbar_wait(rfull(slot), (g / a.rest_slots) & 1, a.err, DEVERR_ATTN_MMA);
+          tc_fence_after();
+          box_products(base + lay.rest + slot * kLatBox, 2 * a.pairs + r, d, false);
+          umma_commit(rempty(slot));
+        }
+        umma_commit(s_full + 8 * (t & 1));
+      };
+      auto values = [&](int t) {
+        if (ok) ok = mbar_wait(p_ready, t & 1, a.err, DEVERR_ATTN_MMA);
+        tc_fence_after();
+        for (int i = 0; ok && i < a.pairs; ++i) {
+          const int slot = (t * a.pairs + i) % a.slots;
+          // MN-major: 64 values contiguous per key row, 8 keys 1 KB apart, the second 64 values one box further on; 16 keys = 2 KB
+          const uint64_t v_desc = make_smem_desc_sw128(base + slot * kLatPair, kLatBox, 1024);
+          for (int k = 0; k < kLatTile / 16; ++k)
+            umma_bf16_ss(tmem + i * N, v_desc + 128 * k, p_desc + static_cast<uint64_t>((k >> 2) * N * 8 + 2 * (k & 3)), idesc_pv,
+                         t > 0 || k > 0 ? 1u : 0u);
+          umma_commit(empty(slot));
+        }
+        umma_commit(pv_done);
+      };
+      if (ok) scores(0);
+      for (int t = 0; ok && t < n_tiles; ++t) {
+        if (a.ahead && t + 1 < n_tiles) scores(t + 1);
+        values(t);
+        if (!a.ahead && ok && t + 1 < n_tiles) scores(t + 1);
+      }
+    }
+    __syncwarp();
+  } else {
+    // ---------------- softmax: thread = key of the tile (tensor-memory lane) ----------------
+    pdl_wait();
+    const int r = threadIdx.x;
+    const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
+    const int min_lim = lim[0];  // rows are in token order
+    float l[N];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
+    for (int n = 0; n < N; ++n) l[n] = 0.0f;
+    uint8_t* pw = gen + lay.p + (r >> 6) * (N * 128) + (r & 7) * 2;  // this key's column of the weights
+    const int pc = (r & 63) >> 3;
+    for (int t = 0; t < n_tiles; ++t) {
+      const int k0 = key0 + t * kLatTile, j = k0 + r;
+      if (ok) ok = mbar_wait(s_full + 8 * (t & 1), (t >> 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
+      __syncwarp();
+      tc_fence_after();
+      float s[N];
+      tmem_ld_cols<N>(t_s + lane_addr + (t & 1) * N, s);
+      tc_fence_before();
+      if (k0 + kLatTile > key_end || k0 + kLatTile - 1 > min_lim) {
+        const bool live = j < key_end;
 #pragma unroll
-        for (int n = 0; n < 4; ++n) s[mt][n][0] = s[mt][n][1] = s[mt][n][2] = s[mt][n][3] = 0.0f;
-      const uint32_t ka = kt + static_cast<uint32_t>((kh * 32 + (lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8 + kq * NK * 16) * 2;
+        for (int n = 0; n < N; ++n) s[n] = live && j <= lim[n] ? s[n] : -INFINITY;
+        if (k0 + kLatTile > key_end && !live)
+          // rows past the live length hold whatever the cache had; their weights are zero, but 0 * NaN is NaN inside the product
+          for (int i = 0; i < a.pairs; ++i) {
+            uint8_t* row = gen + ((t * a.pairs + i) % a.slots) * kLatPair + r * 128;
 #pragma unroll
-      for (int k = 0; k < NK; ++k)
-#pragma unroll
-        for (int n = 0; n < 4; n += 2) {
-          uint32_t b[4];
-          ldsm_x4(b, ka + static_cast<uint32_t>(n * 8 * LD) * 2 + k * 32);
-#pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
-            mma_bf16_16816(s[mt][n], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[0], b[1]);
-            mma_bf16_16816(s[mt][n + 1], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[2], b[3]);
+            for (int c = 0; c < 8; ++c) {
+              *reinterpret_cast<uint4*>(row + c * 16) = make_uint4(0, 0, 0, 0);
+              *reinterpret_cast<uint4*>(row + kLatBox + c * 16) = make_uint4(0, 0, 0, 0);
+            }
           }
-        }
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int n = 0; n < 4; ++n)
-#pragma unroll
-          for (int e = 0; e < 2; ++e)
-            *reinterpret_cast<float2*>(sp + (kq * R + mt * 16 + g + 8 * e) * kLatSLd + kh * 32 + 8 * n + 2 * c) =
-                make_float2(s[mt][n][2 * e], s[mt][n][2 * e + 1]);
-    }
-    __syncthreads();
-    {
-      float x[KPT], mx = m;
-      const int j0 = key0 + t * kLatKeys + sub * KPT;
-#pragma unroll
-      for (int e = 0; e < KPT; e += 2) {
-        float2 v = make_float2(0.0f, 0.0f);
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const float2 p = *reinterpret_cast<const float2*>(sp + (q * R + sr) * kLatSLd + sub * KPT + e);
-          v.x += p.x;
-          v.y += p.y;
-        }
-        x[e] = j0 + e <= s_pos && j0 + e < key_end ? v.x * sc : -INFINITY;
-        x[e + 1] = j0 + e + 1 <= s_pos && j0 + e + 1 < key_end ? v.y * sc : -INFINITY;
-        mx = fmaxf(mx, fmaxf(x[e], x[e + 1]));
       }
+      bool grow = t == 0;
+      if (t > 0) {
+        bool mine = false;
 #pragma unroll
-      for (int o = TPR >> 1; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float base = mx == -INFINITY ? 0.0f : mx;  // a row that has seen no key yet
-      const float alpha = ex2(m - base);
-      m = mx;
-      l *= alpha;
-#pragma unroll
-      for (int e = 0; e < KPT; e += 2) {
-        const float p0 = ex2(x[e] - base), p1 = ex2(x[e + 1] - base);
-        l += p0 + p1;
-        *reinterpret_cast<uint32_t*>(pb + sr * kLatPLd + sub * KPT + e) = pack_bf16x2(p0, p1);
+        for (int n = 0; n < N; ++n) mine = mine || s[n] * a.scale_log2 > m_sh[n] + kLatGrow;
+        grow = any128(mine);
       }
-      if (sub == 0) row_f[sr] = alpha;
-    }
-    __syncthreads();
-    if (v0 < a.DV) {
-      float al[MT][2];
+      if (grow) {
+        {
+          float x[N];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        al[mt][0] = row_f[mt * 16 + g];
-        al[mt][1] = row_f[mt * 16 + g + 8];
-#pragma unroll
-        for (int n = 0; n < 2 * NV; ++n) {
-          O[mt][n][0] *= al[mt][0]; O[mt][n][1] *= al[mt][0];
-          O[mt][n][2] *= al[mt][1]; O[mt][n][3] *= al[mt][1];
+          for (int n = 0; n < N; ++n) x[n] = s[n] * a.scale_log2;
+          reduce_to<N, true>(x, red + warp * N);
         }
-      }
-      const uint32_t pa = smem_u32(pb) + static_cast<uint32_t>(((lane & 7) + ((lane >> 3) & 1) * 8) * kLatPLd + (lane >> 4) * 8) * 2;
-      const uint32_t va = kt + static_cast<uint32_t>(((lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8 + v0) * 2;
+        named_barrier_sync(1, 128);
+        if (r < N) {
+          const float old = m_sh[r];
+          // finite from here on, also for rows that see none of this share's keys
+          const float now = fmaxf(fmaxf(fmaxf(old, -1e30f), fmaxf(red[r], red[N + r])), fmaxf(red[2 * N + r], red[3 * N + r]));
+          m_sh[r] = now;
+          alpha_sh[r] = ex2(old - now);
+        }
+        named_barrier_sync(1, 128);
+        if (t > 0) {
+          if (ok) ok = mbar_wait(pv_done, (t - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);  // O^T is final for the tiles before
+          __syncwarp();
+          tc_fence_after();
+          for (int i = 0; i < a.pairs; ++i) {
+            float o[N];
+            tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
 #pragma unroll
-      for (int k = 0; k < kLatKeys / 16; ++k) {
-        uint32_t pf[MT][4];
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt) ldsm_x4(pf[mt], pa + static_cast<uint32_t>(mt * 16 * kLatPLd + k * 16) * 2);
-#pragma unroll
-        for (int n = 0; n < NV; ++n) {
-          uint32_t b[4];
-          ldsm_x4_trans(b, va + static_cast<uint32_t>(k * 16 * LD + n * 16) * 2);
-#pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
-            mma_bf16_16816(O[mt][2 * n], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], b[0], b[1]);
-            mma_bf16_16816(O[mt][2 * n + 1], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], b[2], b[3]);
+            for (int n = 0; n < N; ++n) o[n] *= alpha_sh[n];
+            tmem_st_cols<N>(tmem + lane_addr + i * N, o);
           }
+          tmem_wait_st();
+          tc_fence_before();
         }
+#pragma unroll
+        for (int n = 0; n < N; ++n) l[n] *= alpha_sh[n];
       }
+      uint32_t pk[N / 2];
+#pragma unroll
+      for (int n = 0; n < N; n += 2) {
+        const float p0 = ex2(fmaf(s[n], a.scale_log2, -m_sh[n])), p1 = ex2(fmaf(s[n + 1], a.scale_log2, -m_sh[n + 1]));
+        l[n] += p0;
+        l[n + 1] += p1;
+        pk[n / 2] = pack_bf16x2(p0, p1);
+      }
+      if (t > 0) {
+        if (ok) ok = mbar_wait(pv_done, (t - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);  // the weights of the tile before have been read
+      }
+#pragma unroll
+      for (int n = 0; n < N; ++n)
+        *reinterpret_cast<uint16_t*>(pw + n * 128 + ((pc ^ (n & 7)) << 4)) = static_cast<uint16_t>(n & 1 ? pk[n / 2] >> 16 : pk[n / 2] & 0xffffu);
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(p_ready);
     }
-    __syncthreads();  // the stage, the scores and the weights may be written again
+    // ---- this share's sums and output ----
+    reduce_to<N, false>(l, red + warp * N);
+    if (n_tiles > 0 && ok) ok = mbar_wait(pv_done, (n_tiles - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
+    tc_fence_after();
+    named_barrier_sync(1, 128);
+    if (r < N) alpha_sh[r] = (red[r] + red[N + r]) + (red[2 * N + r] + red[3 * N + r]);
+    float* ob = reinterpret_cast<float*>(gen);  // [N][o_ld] over the slots, which no copy or product uses any more
+    for (int i = 0; i < a.pairs; ++i) {
+      float o[N];
+      if (n_tiles > 0) {
+        tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
+      } else {
+#pragma unroll
+        for (int n = 0; n < N; ++n) o[n] = 0.0f;
+      }
+#pragma unroll
+      for (int n = 0; n < N; ++n) ob[n * a.o_ld + i * 128 + r] = o[n];
+    }
+    tc_fence_before();
   }
   pdl_trigger();
-  // ---- merge ----
-#pragma unroll
-  for (int o = TPR >> 1; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-  if (sub == 0) {
-    row_f[R + sr] = m;
-    row_f[2 * R + sr] = l;
+  __syncthreads();
+  if (warp == 5) {
+    if (*reinterpret_cast<volatile int*>(a.err) != 0) {  // a wait was given up: let copies and products in flight finish
+      const uint64_t t0 = global_timer_ns();
+      while (global_timer_ns() - t0 < 2000000ull) __nanosleep(1000);
+    }
+    tc_fence_after();
+    tmem_dealloc(tmem, a.tmem_cols);
   }
-  float* ob = reinterpret_cast<float*>(lat_smem);  // [R][16 NV * 8] this share's output, over the stages
-  constexpr int OLD = 128 * NV + 2;
-  static_assert(R * OLD * 4 <= 2 * kLatKeys * LD * 2, "the output fits into the stages");
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int n = 0; n < 2 * NV; ++n)
-#pragma unroll
-      for (int e = 0; e < 2; ++e)
-        *reinterpret_cast<float2*>(ob + (mt * 16 + g + 8 * e) * OLD + v0 + 8 * n + 2 * c) = make_float2(O[mt][n][2 * e], O[mt][n][2 * e + 1]);
   if (splits > 1) cluster_sync();
-  else __syncthreads();
-  // this CTA's share of the columns, in pairs
-  const int pairs = a.DV / 2, per = (pairs + splits - 1) / splits, p0 = split * per, p1 = min(pairs, p0 + per);
-  const uint32_t ob_a = smem_u32(ob), rf_a = smem_u32(row_f);
-  for (int r = warp; r < n_rows; r += 8) {
-    float w = 0.0f, mm = -INFINITY;  // lane s: weight of share s (at most 32 shares)
+  // ---- merge: this CTA's slice of the columns, in pairs ----
+  const int cols = a.DV / 2, per = (cols + splits - 1) / splits, c0 = split * per, c1 = min(cols, c0 + per);
+  const uint32_t ob_a = base, m_a = smem_u32(m_sh), l_a = smem_u32(alpha_sh);
+  for (int r = warp; r < n_rows; r += kLatThreads / 32) {
+    float w;  // lane s: weight of share s (at most eight)
     if (splits > 1) {
-      const float ms = lane < splits ? ld_cluster(rf_a + (R + r) * 4, lane) : -INFINITY;
-      const float ls = lane < splits ? ld_cluster(rf_a + (2 * R + r) * 4, lane) : 0.0f;
-      mm = warp_max(ms);
-      w = ex2(ms - mm);  // shares without keys hold -inf: 0
+      const float ms = lane < splits ? ld_cluster(m_a + r * 4, lane) : -INFINITY;
+      const float ls = lane < splits ? ld_cluster(l_a + r * 4, lane) : 0.0f;
+      w = ex2(ms - warp_max(ms));  // shares without keys hold -inf: 0
       w /= warp_sum(w * ls);
     } else {
-      w = 1.0f / row_f[2 * R + r];
+      w = 1.0f / alpha_sh[r];
     }
     const int rr = row0 + r, tok = rr / a.H, h = rr - tok * a.H;
-    bf16* orow = static_cast<bf16*>(a.out) + (static_cast<size_t>(seq.row0) + tok) * a.ldo + h * a.DV;
-    for (int pp = p0; pp < p1; pp += 32) {  // (whole warps: shuffles)
-      const int p = pp + lane;
+    bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV;
+    for (int cc = c0; cc < c1; cc += 32) {  // (whole warps: shuffles)
+      const int c = min(cc + lane, c1 - 1);
+      const uint32_t addr = ob_a + static_cast<uint32_t>(r * a.o_ld + 2 * c) * 4;
       float2 o = make_float2(0.0f, 0.0f);
-      for (int s = 0; s < splits; ++s) {
-        const float ws = __shfl_sync(0xffffffffu, w, s);
-        if (p >= p1) continue;
-        const float2 v = splits > 1 ? ld_cluster2(ob_a + (r * OLD + 2 * p) * 4, s) : *reinterpret_cast<const float2*>(ob + r * OLD + 2 * p);
-        o.x = fmaf(ws, v.x, o.x);
-        o.y = fmaf(ws, v.y, o.y);
+      if (splits > 1) {
+        float2 v[8];
+#pragma unroll
+        for (int s = 0; s < 8; ++s) v[s] = s < splits ? ld_cluster2(addr, s) : make_float2(0.0f, 0.0f);
+#pragma unroll
+        for (int s = 0; s < 8; ++s) {
+          const float ws = __shfl_sync(0xffffffffu, w, s);
+          if (s < splits) {
+            o.x = fmaf(ws, v[s].x, o.x);
+            o.y = fmaf(ws, v[s].y, o.y);
+          }
+        }
+      } else {
+        const float2 v = *reinterpret_cast<const float2*>(gen + (addr - base));
+        o = make_float2(w * v.x, w * v.y);
       }
-      if (p < p1) *reinterpret_cast<uint32_t*>(orow + 2 * p) = pack_bf16x2(o.x, o.y);
+      if (cc + lane < c1) *reinterpret_cast<uint32_t*>(orow + 2 * c) = pack_bf16x2(o.x, o.y);
     }
   }
   if (splits > 1) cluster_sync();  // no CTA leaves while others read its shared memory
 }
 
-// Size classes of the mma kernel: cache rows up to 64 NK elements (each a quarter of 16 NK), values up to 128 NV.
+constexpr int kLatSmemLimit = 232448;
+
 template <typename F>
-int for_class(int d, int dv, F&& f) {
-  if (d <= 192 && dv <= 128) return f(std::integral_constant<int, 3>(), std::integral_constant<int, 1>());
-  if (d <= 320 && dv <= 256) return f(std::integral_constant<int, 5>(), std::integral_constant<int, 2>());
-  if (d <= 576 && dv <= 512) return f(std::integral_constant<int, 9>(), std::integral_constant<int, 4>());
-  return TEENY_ERR_BAD_ARG;
+int for_rows(int n, F&& f) {
+  if (n <= 16) return f(std::integral_constant<int, 16>());
+  if (n <= 32) return f(std::integral_constant<int, 32>());
+  return f(std::integral_constant<int, 64>());
+}
+
+// Ring sizes for row tiles of n; false if the sizes do not fit.
+bool plan_tc(int n, int d, int dv, LatTcArgs& a, int& smem) {
+  a.pairs = (dv + 127) / 128;
+  a.rests = d > 128 * a.pairs ? (d - 128 * a.pairs + 63) / 64 : 0;
+  uint32_t cols = 32;
+  while (static_cast<int>(cols) < (a.pairs + 2) * n) cols *= 2;
+  a.tmem_cols = cols;
+  a.o_ld = 128 * a.pairs + 2;
+  if (cols > 512) return false;
+  for (int tiles = 2; tiles >= 1; --tiles) {  // two whole tiles in flight, or one and what else fits
+    a.rest_slots = tiles * a.rests;
+    a.slots = (kLatSmemLimit - lat_smem(n, a.pairs, a.rests, 0, a.rest_slots).total) / kLatPair;
+    if (a.slots > kLatMaxSlots) a.slots = kLatMaxSlots;
+    if (a.slots > 3 * a.pairs) a.slots = 3 * a.pairs;
+    a.ahead = tiles == 2;
+    if (a.slots >= tiles * a.pairs && a.rest_slots <= kLatMaxSlots && a.slots * kLatPair >= n * a.o_ld * 4) {
+      smem = lat_smem(n, a.pairs, a.rests, a.slots, a.rest_slots).total;
+      return true;
+    }
+  }
+  return false;
+}
+
+// Clusters of `size` CTAs that can be resident at once (per device, worked out once).
+template <int N>
+int max_clusters(int size, int smem) {
+  static std::atomic<int> known[9][64];  // [size][shared memory in 4 KB steps]
+  std::atomic<int>& k = known[size][(smem >> 12) & 63];
+  int v = k.load(std::memory_order_relaxed);
+  if (v > 0) return v;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(size, 1, 1);
+  cfg.blockDim = dim3(kLatThreads);
+  cfg.dynamicSmemBytes = smem;
+  cudaLaunchAttribute attr;
+  attr.id = cudaLaunchAttributeClusterDimension;
+  attr.val.clusterDim.x = size;
+  attr.val.clusterDim.y = attr.val.clusterDim.z = 1;
+  cfg.attrs = &attr;
+  cfg.numAttrs = 1;
+  if (cudaOccupancyMaxActiveClusters(&v, latent_attention_kernel<N>, &cfg) != cudaSuccess || v < 1) {
+    cudaGetLastError();
+    v = 1;
+  }
+  k.store(v, std::memory_order_relaxed);
+  return v;
 }
 
 }  // namespace
@@ -661,14 +909,10 @@ int latent_attention_prepare() {
   if (dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull) return 0;
   cudaError_t e = cudaFuncSetAttribute(head_linear_mma_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, hl_smem_bytes(1, kLatMax));
   if (e == cudaSuccess) e = cudaFuncSetAttribute(head_linear_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, hl_smem_bytes(4, kLatMax));
-  const int sizes[][2] = {{192, 128}, {320, 256}, {576, 512}};
-  for (const auto& s : sizes)
-    for_class(s[0], s[1], [&](auto nk, auto nv) {
-      constexpr int NK = decltype(nk)::value, NV = decltype(nv)::value;
+  for (int n : {16, 32, 64})
+    for_rows(n, [&](auto nn) {
       if (e == cudaSuccess)
-        e = cudaFuncSetAttribute(latent_attention_mma_kernel<1, NK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, lat_smem_bytes(1, NK));
-      if (e == cudaSuccess)
-        e = cudaFuncSetAttribute(latent_attention_mma_kernel<2, NK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, lat_smem_bytes(2, NK));
+        e = cudaFuncSetAttribute(latent_attention_kernel<decltype(nn)::value>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLatSmemLimit);
       return 0;
     });
   if (e != cudaSuccess) return static_cast<int>(e);
@@ -684,24 +928,53 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
     const int rc = latent_attention_prepare();
     if (rc) return rc;
   }
-  const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache) | reinterpret_cast<uintptr_t>(a.out);
-  const bool vec = !a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && ((a.ldq | a.ldo) & 7) == 0 && (bases & 15) == 0;
-  const int rows = longest * a.H, mt = rows <= 16 ? 1 : 2, tiles = (rows + 16 * mt - 1) / (16 * mt);
-  if (vec && tiles <= 65535) {
-    // shares of the keys: as many as still leave every SM at most about one CTA
-    int splits = 1;
-    const long long ctas = static_cast<long long>(tiles) * n_seqs;
-    while (splits < 8 && ctas * splits * 2 <= sm_count() && splits * 2 * kLatKeys <= a.max_len) splits *= 2;
-    const dim3 grid(splits, tiles, n_seqs);
-    const int rc = for_class(a.D, a.DV, [&](auto nk, auto nv) {
-      constexpr int NK = decltype(nk)::value, NV = decltype(nv)::value;
-      if (mt == 1)
-        launch_kernel(latent_attention_mma_kernel<1, NK, NV>, grid, dim3(256), lat_smem_bytes(1, NK), st, static_cast<unsigned>(splits), a, seqs);
-      else
-        launch_kernel(latent_attention_mma_kernel<2, NK, NV>, grid, dim3(256), lat_smem_bytes(2, NK), st, static_cast<unsigned>(splits), a, seqs);
-      return static_cast<int>(cudaGetLastError());
-    });
-    if (rc != TEENY_ERR_BAD_ARG) return rc;
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache);
+  const int rows = longest * a.H;
+  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (a.ldo & 1) == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 3) == 0 &&
+      a.ldq == static_cast<long long>(a.H) * a.D) {
+    LatTcArgs t{};
+    int smem = 0, n = rows <= 16 ? 16 : (rows <= 32 ? 32 : 64);
+    while (n >= 16 && !plan_tc(n, a.D, a.DV, t, smem)) n /= 2;
+    const int tiles = n >= 16 ? (rows + n - 1) / n : 0;
+    if (n >= 16 && tiles <= 65535) {
+      t.out = static_cast<bf16*>(a.out);
+      t.ldo = a.ldo;
+      t.row_base = a.row_base;
+      t.H = a.H; t.D = a.D; t.DV = a.DV;
+      t.scale_log2 = a.scale * 1.4426950408889634f;
+      t.err = device_error_word();
+      if (!t.err) return TEENY_ERR_DRIVER;  // kernels report expired waits through this word: no launch without it
+      CUtensorMap mc, mq;
+      const uint64_t cd[3] = {static_cast<uint64_t>(a.D), static_cast<uint64_t>(a.max_len), static_cast<uint64_t>(a.slots)};
+      const uint64_t cs[2] = {static_cast<uint64_t>(a.D) * 2, static_cast<uint64_t>(a.D) * 2 * a.max_len};
+      const uint32_t cb[3] = {64, kLatTile, 1};
+      int rc = encode_tensor_map_bf16(&mc, a.cache, 3, cd, cs, cb);
+      if (rc) return rc;
+      const uint64_t qd[2] = {static_cast<uint64_t>(a.D), static_cast<uint64_t>(a.q_rows) * a.H};
+      const uint64_t qs[1] = {static_cast<uint64_t>(a.D) * 2};
+      const uint32_t qb[2] = {64, static_cast<uint32_t>(n)};
+      rc = encode_tensor_map_bf16(&mq, a.q, 2, qd, qs, qb);
+      if (rc) return rc;
+      return for_rows(n, [&](auto nn) {
+        constexpr int N = decltype(nn)::value;
+        // shares of the keys per row tile: fewest rounds of tiles over all waves of clusters
+        const long long work = static_cast<long long>(tiles) * n_seqs;
+        const int key_tiles = (a.max_len + kLatTile - 1) / kLatTile;
+        int splits = 1;
+        long long best = -1;
+        for (int c = 1; c <= 8 && c <= key_tiles; ++c) {
+          const long long waves = (work + max_clusters<N>(c, smem) - 1) / max_clusters<N>(c, smem);
+          const long long cost = waves * ((key_tiles + c - 1) / c);
+          if (best < 0 || cost < best) {
+            best = cost;
+            splits = c;
+          }
+        }
+        launch_kernel(latent_attention_kernel<N>, dim3(splits, tiles, n_seqs), dim3(kLatThreads), smem, st, static_cast<unsigned>(splits), mc, mq, t,
+                      seqs);
+        return static_cast<int>(cudaGetLastError());
+      });
+    }
   }
   const dim3 grid(static_cast<unsigned>(rows), n_seqs);
   if (a.f32) launch_kernel(latent_attention_rows_kernel<float>, grid, dim3(256), 0, st, 1, a, seqs);

@@ -355,10 +355,12 @@ int run_latent_absorbed(teeny_hybrid* m, const Layer& L, const Branch& b, int e0
   TEENY_TRY(head_linear(in, st));
   LatentAttn a{};
   a.f32 = m->cfg.f32;
-  a.q = element(m, p.lat_qa, -r0, H * DL); a.ldq = H * DL;
+  a.q = in.y; a.ldq = H * DL;
+  a.q_rows = rows; a.row_base = r0;
   a.cache = m->at<void>(b.state);
+  a.slots = m->cfg.max_batch;
   a.max_len = m->cfg.max_len;
-  a.out = element(m, p.lat_oa, -r0, H * KR); a.ldo = H * KR;
+  a.out = m->at<void>(p.lat_oa); a.ldo = H * KR;
   a.H = H; a.D = DL; a.DV = KR;
   a.scale = c.score_scale;
   TEENY_TRY(latent_attention(a, seqs, n, longest, st));
@@ -972,9 +974,10 @@ int teeny_head_linear(int f32, const void* x, long long ldx, long long x_head, c
   return head_linear(a, reinterpret_cast<cudaStream_t>(stream));
 }
 
-int teeny_latent_attention(int f32, const void* q, long long ldq, const void* cache, int max_cached, void* out, long long ldo, int heads,
-                           int dim, int vdim, float score_scale, const int* seqs, int n_seqs, int max_len, teeny_stream_t stream) {
-  const LatentAttn a{f32, q, ldq, cache, max_cached, out, ldo, heads, dim, vdim, score_scale};
+int teeny_latent_attention(int f32, const void* q, long long ldq, int rows, const void* cache, int slots, int max_cached, void* out,
+                           long long ldo, int heads, int dim, int vdim, float score_scale, const int* seqs, int n_seqs, int max_len,
+                           teeny_stream_t stream) {
+  const LatentAttn a{f32, q, ldq, rows, 0, cache, slots, max_cached, out, ldo, heads, dim, vdim, score_scale};
   return latent_attention(a, reinterpret_cast<const SeqDesc*>(seqs), n_seqs, max_len, reinterpret_cast<cudaStream_t>(stream));
 }
 

@@ -404,14 +404,16 @@ struct HeadLinear {
   int n_seqs;
 };
 int head_linear(const HeadLinear& a, cudaStream_t st);
-// Causal attention of H query heads over one shared key per token whose first DV elements are the value: q [T, ldq] with
-// heads D apart, cache [slots, max_len, D] holding the entries' own rows already, out [T, ldo] with heads DV apart.
+// Causal attention of H query heads over one shared key per token whose first DV elements are the value: q [q_rows, ldq] with
+// heads D apart, cache [slots, max_len, D] holding the entries' own rows already, out [q_rows, ldo] with heads DV apart; row 0
+// of q and out is the step's row row_base.
 struct LatentAttn {
   int f32;
   const void* q;
   long long ldq;
+  int q_rows, row_base;
   const void* cache;
-  int max_len;
+  int slots, max_len;
   void* out;
   long long ldo;
   int H, D, DV;

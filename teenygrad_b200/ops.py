@@ -460,18 +460,17 @@ def rope_cache(q, k, v, k_cache, v_cache, inv_freq, rot_dims, seqs, max_len, rot
 
 def cached_attention(q, k_cache, v_cache, score_scale, entries, softcap=0.0, sink=None, gate=None, out=None, scratch=None):
     """Causal attention of ``entries`` (see seq_table) over caches [slots, kv_heads, max_len, .] that hold their own tokens
-    already; q [rows, heads, dim], ``gate`` [rows, heads * vdim].  ``scratch``: (uint8 buffer, zeroed int32 counters) for single
-    tokens, made here when missing."""
+    already; q [rows, heads, dim], ``gate`` [rows, heads * vdim].  ``entries``: a list, or its device and host tables.
+    ``scratch``: (uint8 buffer, zeroed int32 counters) for single tokens, made here when missing."""
     _req(q, name="q"); _req(k_cache, q.dtype, "k_cache"); _req(v_cache, q.dtype, "v_cache")
     slots, G, cap, V = v_cache.shape
     H, D = q.shape[1:]
-    n, longest = len(entries), max(e[3] for e in entries)
+    seqs, host = entries if isinstance(entries, tuple) else (seq_table(entries, q.device), seq_table(entries, "cpu"))
+    n, longest = host.shape[0], int(host[:, 3].max())
     out = torch.zeros(q.shape[0], H, V, dtype=q.dtype, device=q.device) if out is None else out
     if scratch is None and longest == 1:
         scratch = (torch.empty(lib.teeny_attn_decode_scratch_bytes(n, H, 128, cap), dtype=torch.uint8, device=q.device),
                    torch.zeros(n * G, dtype=torch.int32, device=q.device))
-    seqs = seq_table(entries, q.device)
-    host = seq_table(entries, "cpu")
     check(lib.teeny_cached_attention(_f32_flag(q), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), slots, cap, _ptr(out), out.stride(0), H, G,
                                      D, V, float(score_scale), float(softcap), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
                                      _ptr(scratch[0]) if scratch else None, scratch[0].numel() if scratch else 0,
@@ -509,6 +508,6 @@ def latent_attention(q, cache, vdim, score_scale, seqs, max_len, out=None):
     entries' own rows are in the cache already.  Returns [rows, heads, vdim]."""
     _req(q, name="q"); _req(cache, q.dtype, "cache")
     out = torch.zeros(q.shape[0], q.shape[1], vdim, dtype=q.dtype, device=q.device) if out is None else out
-    check(lib.teeny_latent_attention(_f32_flag(q), _ptr(q), q.stride(0), _ptr(cache), cache.shape[1], _ptr(out), out.stride(0), q.shape[1],
-                                     q.shape[2], vdim, float(score_scale), _ptr(seqs), seqs.shape[0], max_len, _stream()), "latent_attention")
+    check(lib.teeny_latent_attention(_f32_flag(q), _ptr(q), q.stride(0), q.shape[0], _ptr(cache), cache.shape[0], cache.shape[1], _ptr(out),
+                                     out.stride(0), q.shape[1], q.shape[2], vdim, float(score_scale), _ptr(seqs), seqs.shape[0], max_len, _stream()), "latent_attention")
     return out
