@@ -389,7 +389,7 @@ __host__ __device__ inline LatSmem lat_smem(int n, int pairs, int rests, int slo
   s.p = s.q + (2 * pairs + rests) * n * 128;
   s.bars = s.p + 2 * n * 128;
   s.stats = s.bars + 8 * (2 * kLatMaxSlots + 2 * kLatMaxSlots + 8);
-  s.total = s.stats + 4 * 9 * n + 1024;
+  s.total = s.stats + 4 * (8 + 16) * n + 1024;
   return s;
 }
 
@@ -403,11 +403,11 @@ __device__ __forceinline__ float ld_cluster(uint32_t local_addr, uint32_t rank) 
   asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
   return v;
 }
-__device__ __forceinline__ float2 ld_cluster2(uint32_t local_addr, uint32_t rank) {
+__device__ __forceinline__ float4 ld_cluster4(uint32_t local_addr, uint32_t rank) {
   uint32_t r;
-  float2 v;
+  float4 v;
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(local_addr), "r"(rank));
-  asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(r) : "memory");
+  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(r) : "memory");
   return v;
 }
 // whether `v` holds in any of the 128 softmax threads (barrier 1)
@@ -488,6 +488,37 @@ __device__ __forceinline__ void reduce_to(const float (&v)[N], float* dst) {
   }
 }
 
+// Straight-line runs of products: a lone thread with address arithmetic in between issues a product only every ~100 cycles.
+// Four K-steps over one K-major box of each operand (32 bytes along the rows per step).
+__device__ __forceinline__ void umma_box(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate_first) {
+  asm volatile(
+      "{\n\t.reg .pred p, t;\n\t.reg .b64 x, y;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t setp.eq.b32 t, %3, %3;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
+      "add.u64 x, %1, 2;\n\t add.u64 y, %2, 2;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 4;\n\t add.u64 y, %2, 4;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 6;\n\t add.u64 y, %2, 6;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate_first)
+      : "memory");
+}
+// The eight K-steps of 128 keys: A MN-major (2 KB per 16 keys), B K-major in two boxes BOX 16-byte units apart.
+template <int BOX>
+__device__ __forceinline__ void umma_keys(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate_first) {
+  asm volatile(
+      "{\n\t.reg .pred p, t;\n\t.reg .b64 x, y;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t setp.eq.b32 t, %3, %3;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
+      "add.u64 x, %1, 128;\n\t add.u64 y, %2, 2;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 256;\n\t add.u64 y, %2, 4;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 384;\n\t add.u64 y, %2, 6;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 512;\n\t add.u64 y, %2, %5;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 640;\n\t add.u64 y, %2, %6;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 768;\n\t add.u64 y, %2, %7;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, 896;\n\t add.u64 y, %2, %8;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate_first), "n"(BOX), "n"(BOX + 2), "n"(BOX + 4), "n"(BOX + 6)
+      : "memory");
+}
+
 template <int N>
 __global__ void __launch_bounds__(kLatThreads, 1)
 latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid_constant__ CUtensorMap tmap_q, const LatTcArgs a,
@@ -511,8 +542,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40;  // two s_full
   float* m_sh = reinterpret_cast<float*>(gen + lay.stats);  // [N] running maxima, log2 domain
   float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally the row sums
-  float* red = alpha_sh + N;                                // [4][N]
+  float* up_sh = alpha_sh + N;                              // [N] by how much the maxima just rose
+  float* red = up_sh + N;                                   // [4][N]
   int* lim = reinterpret_cast<int*>(red + 4 * N);           // [N] last key each row sees
+  float2* share = reinterpret_cast<float2*>(lim + N);       // [N][8] maximum and sum of every share; then its weight
 
   const int splits = gridDim.x, split = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -544,7 +577,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tmem_relinquish();
   }
   if (threadIdx.x < N) {
-    m_sh[threadIdx.x] = -INFINITY;
+    m_sh[threadIdx.x] = 0.0f;
     lim[threadIdx.x] = seq.pos + min(row0 + static_cast<int>(threadIdx.x), row0 + n_rows - 1) / a.H;
   }
   tc_fence_before();
@@ -592,12 +625,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       constexpr uint32_t idesc_s = make_idesc_bf16(128, N, false, false), idesc_pv = make_idesc_bf16(128, N, true, false);
       const uint64_t q_desc = make_smem_desc_sw128(base + lay.q, 16, 1024), p_desc = make_smem_desc_sw128(base + lay.p, 16, 1024);
       ok = mbar_wait(q_full, 0, a.err, DEVERR_ATTN_MMA);
-      // one 64-dimension box of cache rows times the queries' box
-      auto box_products = [&](uint32_t smem, int box, uint32_t d, bool first) {
-        const uint64_t c_desc = make_smem_desc_sw128(smem, 16, 1024);
-        const int steps = min(4, (a.D - 64 * box + 15) / 16);  // 16 dimensions = 32 bytes along the rows
-        for (int k = 0; k < steps; ++k)
-          umma_bf16_ss(d, c_desc + 2 * k, q_desc + static_cast<uint64_t>(box * N * 8 + 2 * k), idesc_s, first && k == 0 ? 0u : 1u);
+      // one 64-dimension box of cache rows times the queries' box (dimensions beyond D are zero in both)
+      const uint64_t c_desc0 = make_smem_desc_sw128(base, 16, 1024), v_desc0 = make_smem_desc_sw128(base, kLatBox, 1024);
+      auto box_products = [&](int offset, int box, uint32_t d, bool first) {
+        umma_box(d, c_desc0 + (offset >> 4), q_desc + static_cast<uint64_t>(box * N * 8), idesc_s, first ? 0u : 1u);
       };
       auto scores = [&](int t) {
         const uint32_t d = t_s + (t & 1) * N;
@@ -605,14 +636,14 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
           const int g = t * a.pairs + p, slot = g % a.slots;
           ok = mbar_wait(full(slot), (g / a.slots) & 1, a.err, DEVERR_ATTN_MMA);
           tc_fence_after();
-          box_products(base + slot * kLatPair, 2 * p, d, p == 0);
-          if (128 * p + 64 < a.D) box_products(base + slot * kLatPair + kLatBox, 2 * p + 1, d, false);
+          box_products(slot * kLatPair, 2 * p, d, p == 0);
+          if (128 * p + 64 < a.D) box_products(slot * kLatPair + kLatBox, 2 * p + 1, d, false);
         }
         for (int r = 0; ok && r < a.rests; ++r) {
           const int g = t * a.rests + r, slot = g % a.rest_slots;
           ok = mbar_wait(rfull(slot), (g / a.rest_slots) & 1, a.err, DEVERR_ATTN_MMA);
           tc_fence_after();
-          box_products(base + lay.rest + slot * kLatBox, 2 * a.pairs + r, d, false);
+          box_products(lay.rest + slot * kLatBox, 2 * a.pairs + r, d, false);
           umma_commit(rempty(slot));
         }
         umma_commit(s_full + 8 * (t & 1));
@@ -623,10 +654,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
         for (int i = 0; ok && i < a.pairs; ++i) {
           const int slot = (t * a.pairs + i) % a.slots;
           // MN-major: 64 values contiguous per key row, 8 keys 1 KB apart, the second 64 values one box further on; 16 keys = 2 KB
-          const uint64_t v_desc = make_smem_desc_sw128(base + slot * kLatPair, kLatBox, 1024);
-          for (int k = 0; k < kLatTile / 16; ++k)
-            umma_bf16_ss(tmem + i * N, v_desc + 128 * k, p_desc + static_cast<uint64_t>((k >> 2) * N * 8 + 2 * (k & 3)), idesc_pv,
-                         t > 0 || k > 0 ? 1u : 0u);
+          umma_keys<N * 8>(tmem + i * N, v_desc0 + static_cast<uint64_t>(slot * (kLatPair >> 4)), p_desc, idesc_pv, t > 0 ? 1u : 0u);
           umma_commit(empty(slot));
         }
         umma_commit(pv_done);
@@ -673,27 +701,26 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
             }
           }
       }
+      // scores relative to the running maxima (first tile: to zero)
       bool grow = t == 0;
-      if (t > 0) {
-        bool mine = false;
 #pragma unroll
-        for (int n = 0; n < N; ++n) mine = mine || s[n] * a.scale_log2 > m_sh[n] + kLatGrow;
-        grow = any128(mine);
+      for (int n = 0; n < N; n += 4) {
+        const float4 m4 = *reinterpret_cast<const float4*>(m_sh + n);
+        s[n] = fmaf(s[n], a.scale_log2, -m4.x);
+        s[n + 1] = fmaf(s[n + 1], a.scale_log2, -m4.y);
+        s[n + 2] = fmaf(s[n + 2], a.scale_log2, -m4.z);
+        s[n + 3] = fmaf(s[n + 3], a.scale_log2, -m4.w);
+        grow = grow || fmaxf(fmaxf(s[n], s[n + 1]), fmaxf(s[n + 2], s[n + 3])) > kLatGrow;
       }
-      if (grow) {
-        {
-          float x[N];
-#pragma unroll
-          for (int n = 0; n < N; ++n) x[n] = s[n] * a.scale_log2;
-          reduce_to<N, true>(x, red + warp * N);
-        }
+      if (any128(grow)) {
+        reduce_to<N, true>(s, red + warp * N);
         named_barrier_sync(1, 128);
         if (r < N) {
-          const float old = m_sh[r];
-          // finite from here on, also for rows that see none of this share's keys
-          const float now = fmaxf(fmaxf(fmaxf(old, -1e30f), fmaxf(red[r], red[N + r])), fmaxf(red[2 * N + r], red[3 * N + r]));
-          m_sh[r] = now;
-          alpha_sh[r] = ex2(old - now);
+          float up = fmaxf(fmaxf(red[r], red[N + r]), fmaxf(red[2 * N + r], red[3 * N + r]));
+          up = t == 0 ? fmaxf(up, -1e30f) : fmaxf(up, 0.0f);  // finite also for rows that see none of this share's keys
+          m_sh[r] += up;
+          up_sh[r] = up;
+          alpha_sh[r] = t == 0 ? 0.0f : ex2(-up);
         }
         named_barrier_sync(1, 128);
         if (t > 0) {
@@ -711,12 +738,15 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
           tc_fence_before();
         }
 #pragma unroll
-        for (int n = 0; n < N; ++n) l[n] *= alpha_sh[n];
+        for (int n = 0; n < N; ++n) {
+          l[n] *= alpha_sh[n];
+          s[n] -= up_sh[n];
+        }
       }
       uint32_t pk[N / 2];
 #pragma unroll
       for (int n = 0; n < N; n += 2) {
-        const float p0 = ex2(fmaf(s[n], a.scale_log2, -m_sh[n])), p1 = ex2(fmaf(s[n + 1], a.scale_log2, -m_sh[n + 1]));
+        const float p0 = ex2(s[n]), p1 = ex2(s[n + 1]);
         l[n] += p0;
         l[n + 1] += p1;
         pk[n / 2] = pack_bf16x2(p0, p1);
@@ -736,6 +766,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     if (n_tiles > 0 && ok) ok = mbar_wait(pv_done, (n_tiles - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
     tc_fence_after();
     named_barrier_sync(1, 128);
+    if (r < N && n_tiles == 0) m_sh[r] = -INFINITY;
     if (r < N) alpha_sh[r] = (red[r] + red[N + r]) + (red[2 * N + r] + red[3 * N + r]);
     float* ob = reinterpret_cast<float*>(gen);  // [N][o_ld] over the slots, which no copy or product uses any more
     for (int i = 0; i < a.pairs; ++i) {
@@ -762,43 +793,45 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tmem_dealloc(tmem, a.tmem_cols);
   }
   if (splits > 1) cluster_sync();
-  // ---- merge: this CTA's slice of the columns, in pairs ----
-  const int cols = a.DV / 2, per = (cols + splits - 1) / splits, c0 = split * per, c1 = min(cols, c0 + per);
+  // ---- merge: this CTA's slice of the columns, in fours ----
   const uint32_t ob_a = base, m_a = smem_u32(m_sh), l_a = smem_u32(alpha_sh);
-  for (int r = warp; r < n_rows; r += kLatThreads / 32) {
-    float w;  // lane s: weight of share s (at most eight)
-    if (splits > 1) {
-      const float ms = lane < splits ? ld_cluster(m_a + r * 4, lane) : -INFINITY;
-      const float ls = lane < splits ? ld_cluster(l_a + r * 4, lane) : 0.0f;
-      w = ex2(ms - warp_max(ms));  // shares without keys hold -inf: 0
-      w /= warp_sum(w * ls);
-    } else {
-      w = 1.0f / alpha_sh[r];
+  for (int i = threadIdx.x; i < n_rows * splits; i += kLatThreads) {
+    const int r = i / splits, sh = i - r * splits;
+    share[r * 8 + sh] = splits > 1 ? make_float2(ld_cluster(m_a + r * 4, sh), ld_cluster(l_a + r * 4, sh)) : make_float2(m_sh[r], alpha_sh[r]);
+  }
+  __syncthreads();
+  if (threadIdx.x < n_rows) {
+    float2* mine = share + threadIdx.x * 8;
+    float mm = -INFINITY, sum = 0.0f;
+    for (int i = 0; i < splits; ++i) mm = fmaxf(mm, mine[i].x);
+    for (int i = 0; i < splits; ++i) {
+      mine[i].x = ex2(mine[i].x - mm);  // shares without keys hold -inf: 0
+      sum = fmaf(mine[i].x, mine[i].y, sum);
     }
+    for (int i = 0; i < splits; ++i) mine[i].x /= sum;
+  }
+  __syncthreads();
+  const int cols = a.DV / 4, per = (cols + splits - 1) / splits, c0 = split * per, width = min(per, cols - c0);
+  for (int i = threadIdx.x; i < n_rows * width; i += kLatThreads) {
+    const int r = i / width, c = c0 + (i - r * width);
+    const uint32_t addr = ob_a + static_cast<uint32_t>(r * a.o_ld + 4 * c) * 4;
+    float4 v[8];
+#pragma unroll
+    for (int sh = 0; sh < 8; ++sh)
+      if (sh < splits) v[sh] = splits > 1 ? ld_cluster4(addr, sh) : *reinterpret_cast<const float4*>(gen + (addr - base));
+    float4 o = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int sh = 0; sh < 8; ++sh)
+      if (sh < splits) {
+        const float w = share[r * 8 + sh].x;
+        o.x = fmaf(w, v[sh].x, o.x);
+        o.y = fmaf(w, v[sh].y, o.y);
+        o.z = fmaf(w, v[sh].z, o.z);
+        o.w = fmaf(w, v[sh].w, o.w);
+      }
     const int rr = row0 + r, tok = rr / a.H, h = rr - tok * a.H;
     bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV;
-    for (int cc = c0; cc < c1; cc += 32) {  // (whole warps: shuffles)
-      const int c = min(cc + lane, c1 - 1);
-      const uint32_t addr = ob_a + static_cast<uint32_t>(r * a.o_ld + 2 * c) * 4;
-      float2 o = make_float2(0.0f, 0.0f);
-      if (splits > 1) {
-        float2 v[8];
-#pragma unroll
-        for (int s = 0; s < 8; ++s) v[s] = s < splits ? ld_cluster2(addr, s) : make_float2(0.0f, 0.0f);
-#pragma unroll
-        for (int s = 0; s < 8; ++s) {
-          const float ws = __shfl_sync(0xffffffffu, w, s);
-          if (s < splits) {
-            o.x = fmaf(ws, v[s].x, o.x);
-            o.y = fmaf(ws, v[s].y, o.y);
-          }
-        }
-      } else {
-        const float2 v = *reinterpret_cast<const float2*>(gen + (addr - base));
-        o = make_float2(w * v.x, w * v.y);
-      }
-      if (cc + lane < c1) *reinterpret_cast<uint32_t*>(orow + 2 * c) = pack_bf16x2(o.x, o.y);
-    }
+    *reinterpret_cast<uint2*>(orow + 4 * c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
   }
   if (splits > 1) cluster_sync();  // no CTA leaves while others read its shared memory
 }
@@ -819,7 +852,7 @@ bool plan_tc(int n, int d, int dv, LatTcArgs& a, int& smem) {
   uint32_t cols = 32;
   while (static_cast<int>(cols) < (a.pairs + 2) * n) cols *= 2;
   a.tmem_cols = cols;
-  a.o_ld = 128 * a.pairs + 2;
+  a.o_ld = 128 * a.pairs + 4;
   if (cols > 512) return false;
   for (int tiles = 2; tiles >= 1; --tiles) {  // two whole tiles in flight, or one and what else fits
     a.rest_slots = tiles * a.rests;
@@ -930,7 +963,7 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
   }
   const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache);
   const int rows = longest * a.H;
-  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (a.ldo & 1) == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 3) == 0 &&
+  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (a.ldo & 3) == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 7) == 0 &&
       a.ldq == static_cast<long long>(a.H) * a.D) {
     LatTcArgs t{};
     int smem = 0, n = rows <= 16 ? 16 : (rows <= 32 ? 32 : 64);

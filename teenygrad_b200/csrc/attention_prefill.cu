@@ -1,4 +1,6 @@
-// Causal grouped-query flash-attention forward for sm_100a, head_dim 128, bf16 in/out, f32 softmax, on CTA pairs.
+// Causal grouped-query flash-attention forward for sm_100a, query / key size up to 192, value size up to 128, bf16 in/out, f32
+// softmax, on CTA pairs.  (Smaller heads run as 128 with columns that the copies fill with zeros; where numbers below depend on
+// the head size they are for 128.)
 //
 // A cluster of two CTAs (two neighbouring SMs) takes 256 queries of one (head, batch): CTA r owns query rows
 // [q0 + 128 r, q0 + 128 r + 128).  Keys / values stream through in tiles of 128 keys.  Every tcgen05.mma is issued by
@@ -43,6 +45,15 @@
 // tile.  Values the groups exchange (running maximum, row sums) and the barriers that guard them alternate with the
 // item, because the opener is up to one item ahead of the closer.  (Plain 16-byte-per-row loads of Q and stores of O
 // kept the load/store unit busy for ~2000 cycles per item each: a warp instruction touched 32 lines.)
+// Options (template parameters, so that the plain kernel carries none of it):
+//   WIDE   query / key sizes 129 .. 192: tensor memory holds the first 128 dimensions of Q as always, the other 64 stay in shared
+//          memory (two boxes, alternating with the item) and join S as four more K-steps with both operands from there; K stages
+//          grow by a third box and the rings are three deep.
+//   OPT 1  a sink (exp(sink) in the row sum) and a gate (output times sigmoid(gate), its rows fetched by TMA into the boxes the
+//          output leaves from), at an item's end.
+//   OPT 2  soft-capped scores as well: cap tanh(s / cap) by an odd polynomial while a warp's scores are all within half the cap
+//          (the multiply pipes have room beside the exponentials; two more special-function operations per score have not), by
+//          exponential and reciprocal otherwise.  In tiles without a mask the polynomial runs inside the exponential's loop.
 // Tensor memory columns per CTA: S0 0-127, S1 128-255 (f32 scores), O 256-383 (f32), Q 384-447, P 448-511 (bf16 pairs).
 #include <atomic>
 
@@ -60,16 +71,22 @@ constexpr int kHD = 128;
 constexpr int kThreads = 384;                   // TMA K, MMA QK, MMA PV + TMEM, TMA V; two softmax warpgroups
 constexpr int kHalfBytes = 64 * kHD * 2;        // 16 KB: this CTA's half of a K tile (64 keys) or of a V tile (64 d)
 constexpr int kKBoxBytes = 64 * 64 * 2;         // 8 KB: [64 keys][64 d]
-constexpr int kKV = 4;                          // stages of the K ring and of the V ring
-constexpr int kSmemK = 0;
-constexpr int kSmemV = kSmemK + kKV * kHalfBytes;
-constexpr int kSmemQ = kSmemV + kKV * kHalfBytes;   // 32 KB: the next item's Q rows of this CTA, two [128 rows][64 d] boxes
-constexpr int kSmemO = kSmemQ + 2 * kQT * 128;      // 32 KB: output rows on their way out, per warp quarter two [32 rows][64 d] boxes
-constexpr int kSmemBar = kSmemO + 2 * kQT * 128;
-constexpr int kSmemXch = kSmemBar + 512;        // per item parity: running maximum per row, and the row sum / maximum the
-                                                // group that leaves an item first hands to the one that finishes it
-constexpr int kSmemTotal = kSmemXch + 2 * 3 * 128 * 4 + 1024;
-static_assert(kSmemTotal <= 232448, "exceeds the 227 KB of shared memory a CTA can have");
+// Shared memory of a variant.
+template <bool WIDE>
+struct Smem {
+  static constexpr int kKV = WIDE ? 3 : 4;                      // stages of the K ring and of the V ring
+  static constexpr int kStageK = (WIDE ? 3 : 2) * kKBoxBytes;   // this CTA's 64 keys
+  static constexpr int kSmemK = 0;
+  static constexpr int kSmemV = kSmemK + kKV * kStageK;
+  static constexpr int kSmemQ = kSmemV + kKV * kHalfBytes;      // 32 KB: the next item's Q rows of this CTA, two [128 rows][64 d] boxes
+  static constexpr int kSmemQX = kSmemQ + 2 * kQT * 128;        // WIDE: columns 128.. of the current and the next item's Q rows
+  static constexpr int kSmemO = kSmemQX + (WIDE ? 2 * kQT * 128 : 0);  // 32 KB: output rows on their way out, per warp quarter two [32 rows][64 d] boxes
+  static constexpr int kSmemBar = kSmemO + 2 * kQT * 128;
+  static constexpr int kSmemXch = kSmemBar + 512;               // per item parity: running maximum per row, and the row sum / maximum the
+                                                                // group that leaves an item first hands to the one that finishes it
+  static constexpr int kSmemTotal = kSmemXch + 2 * 3 * 128 * 4 + 1024;
+  static_assert(kSmemTotal <= 232448, "exceeds the 227 KB of shared memory a CTA can have");
+};
 constexpr float kRescaleThreshold = 8.0f;       // log2 units
 constexpr uint32_t kPeerBitMask = 0xFEFFFFFFu;  // clears the CTA-rank bit of a shared::cluster address -> leader
 
@@ -81,6 +98,8 @@ struct PrefillArgs {  // (Q, K, V and O travel as tensor maps)
   int window;        // > 0: query i sees only the last `window` keys up to its own (causal only)
   float out_scale;
   float two_y, cap_l2;  // CAP: soft cap of the scores (softcap_log2); scale_log2 is then 1
+  float small, cap_c[4];  // ... and as a polynomial of the scores up to `small` (half the cap)
+  int gate;             // the gate's tensor map is valid
   const float* sink;    // [Hq] or null: exp(sink) joins the row sum
   int two_out_boxes;    // values are wider than one 64-column box
   int n_pair_tiles;  // 256-row query tiles per (batch, head)
@@ -92,6 +111,19 @@ __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// Sigmoids of four bf16 values, one reciprocal between them: 1 / a = b c d / (a b c d) with a = 1 + exp(-x); x below -20 counts as
+// -20 (2e-9), which keeps the product in range.
+__device__ __forceinline__ void sigmoid_x4(uint32_t x01, uint32_t x23, uint32_t& y01, uint32_t& y23) {
+  constexpr float k = -1.4426950408889634f, top = 20.0f * 1.4426950408889634f;
+  const float a = 1.0f + fast_exp2(fminf(bf16_lo(x01) * k, top)), b = 1.0f + fast_exp2(fminf(bf16_hi(x01) * k, top));
+  const float c = 1.0f + fast_exp2(fminf(bf16_lo(x23) * k, top)), d = 1.0f + fast_exp2(fminf(bf16_hi(x23) * k, top));
+  const float ab = a * b, cd = c * d;
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(ab * cd));
+  const float rab = r * cd, rcd = r * ab;  // 1 / (a b), 1 / (c d)
+  y01 = pack_bf16x2(rab * b, rab * a);
+  y23 = pack_bf16x2(rcd * d, rcd * c);
 }
 // Development builds: clock of event `id` at key tile g of CTA 0, for a window of twenty tiles in the middle of its list
 // (kept in shared memory and written out when the CTA is done, so that the stamps cost a store each;
@@ -162,6 +194,45 @@ __device__ __forceinline__ void umma_bf16_ts_pair_x8(uint32_t d_tmem, uint32_t a
         "n"(O6), "n"(O7)
       : "memory");
 }
+// Four more K-steps with A from shared memory too (each CTA's own 128 rows at the same offset).
+__device__ __forceinline__ void umma_bf16_ss_pair_x4(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc) {
+  asm volatile(
+      "{\n\t.reg .pred t;\n\t.reg .b64 a, b;\n\t"
+      "setp.eq.b32 t, %3, %3;\n\t"
+      "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, t;\n\t"
+      "add.u64 a, %1, 2;\n\t add.u64 b, %2, 2;\n\t tcgen05.mma.cta_group::2.kind::f16 [%0], a, b, %3, t;\n\t"
+      "add.u64 a, %1, 4;\n\t add.u64 b, %2, 4;\n\t tcgen05.mma.cta_group::2.kind::f16 [%0], a, b, %3, t;\n\t"
+      "add.u64 a, %1, 6;\n\t add.u64 b, %2, 6;\n\t tcgen05.mma.cta_group::2.kind::f16 [%0], a, b, %3, t;\n\t}"
+      ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc)
+      : "memory");
+}
+// s (c0 + c1 s^2 + c2 s^4 + c3 s^6) for two scores, plus `add`
+__device__ __forceinline__ float2 cap_poly(float2 s, const float (&c)[4], float2 add) {
+  const float2 u = __fmul2_rn(s, s);
+  float2 p = __ffma2_rn(u, make_float2(c[3], c[3]), make_float2(c[2], c[2]));
+  p = __ffma2_rn(p, u, make_float2(c[1], c[1]));
+  p = __ffma2_rn(p, u, make_float2(c[0], c[0]));
+  return __ffma2_rn(p, s, add);
+}
+__device__ __forceinline__ float fmin3(float a, float b, float c) {
+  float y;
+  asm("min.f32 %0, %1, %2, %3;" : "=f"(y) : "f"(a), "f"(b), "f"(c));
+  return y;
+}
+// maximum of a row: four independent chains of three-input maxima
+__device__ __forceinline__ float row_max(const float (&s)[128]) {
+  float tm[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+  for (int e = 4; e + 8 <= 128; e += 8) {
+    tm[0] = fmax3(tm[0], s[e], s[e + 1]);
+    tm[1] = fmax3(tm[1], s[e + 2], s[e + 3]);
+    tm[2] = fmax3(tm[2], s[e + 4], s[e + 5]);
+    tm[3] = fmax3(tm[3], s[e + 6], s[e + 7]);
+  }
+  tm[0] = fmax3(tm[0], s[124], s[125]);
+  tm[1] = fmax3(tm[1], s[126], s[127]);
+  return fmaxf(fmax3(tm[0], tm[1], tm[2]), tm[3]);
+}
 // Arrives on the barrier at this offset in BOTH CTAs of the pair once all MMAs issued so far have completed.
 __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
   asm volatile(
@@ -170,11 +241,15 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
       : "memory");
 }
 
-template <bool CAP>
+template <int OPT, bool WIDE>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                          const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_o,
-                         const PrefillArgs args) {
+                         const __grid_constant__ CUtensorMap tmap_g, const PrefillArgs args) {
+  using L = Smem<WIDE>;
+  constexpr bool CAP = OPT == 2;
+  constexpr int kKV = L::kKV, kSmemK = L::kSmemK, kSmemV = L::kSmemV, kSmemQ = L::kSmemQ, kSmemO = L::kSmemO, kSmemBar = L::kSmemBar,
+                kSmemXch = L::kSmemXch;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* gen = smem_raw + (base - smem_u32(smem_raw));
@@ -185,7 +260,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
   constexpr int Q_READY = 0, K_FULL = 1, K_EMPTY = K_FULL + kKV, V_FULL = K_EMPTY + kKV, V_EMPTY = V_FULL + kKV,
                 S_FULL = V_EMPTY + kKV, S_EMPTY = S_FULL + 2, P_FULL = S_EMPTY + 2, PV_DONE = P_FULL + 1,
                 M_READY = PV_DONE + 2, O_FREE = M_READY + 4, L_READY = O_FREE + 1, QS_FULL = L_READY + 2,
-                QS_FREE = QS_FULL + 1, kNumBars = QS_FREE + 1;
+                QS_FREE = QS_FULL + 1, G_FULL = QS_FREE + 1, O_BOX = G_FULL + 4, kNumBars = O_BOX + 4;
   static_assert(8 * kNumBars + 8 <= 512, "barrier block");
   const uint32_t tmem_slot = bar0 + 8u * kNumBars;
   volatile uint32_t* tmem_slot_ptr = reinterpret_cast<volatile uint32_t*>(gen + kSmemBar + 8 * kNumBars);
@@ -259,11 +334,12 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
           const int st = g % kKV;
           const uint32_t ph = (g / kKV) & 1;
           if (!mbar_wait(bar(K_EMPTY + st), ph ^ 1, err, DEVERR_ATTN_PRODUCER)) { ok = false; break; }
-          if (leader) mbar_expect_tx(bar(K_FULL + st), 2 * kHalfBytes);  // both CTAs' halves
-          const uint32_t dst = base + kSmemK + st * kHalfBytes;
+          if (leader) mbar_expect_tx(bar(K_FULL + st), 2 * L::kStageK);  // both CTAs' halves
+          const uint32_t dst = base + kSmemK + st * L::kStageK;
           const int key0 = (it.t0 + j) * kKT + static_cast<int>(rank) * 64;
           tma_load_4d_pair(dst, &tmap_k, bar(K_FULL + st), 0, key0, it.hk, it.b);
           tma_load_4d_pair(dst + kKBoxBytes, &tmap_k, bar(K_FULL + st), 64, key0, it.hk, it.b);
+          if (WIDE) tma_load_4d_pair(dst + 2 * kKBoxBytes, &tmap_k, bar(K_FULL + st), 128, key0, it.hk, it.b);
         }
       }
     }
@@ -288,8 +364,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
     // neither waits for the other's barriers, and together they keep the tensor pipe fed.
     if (leader && lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc_bf16(2 * kQT, kKT, false, false);
-      // K-major B: 8-row groups 1 KB apart; ring stage s is kHalfBytes further on
-      const uint64_t kdesc0 = make_smem_desc_sw128(base + kSmemK, 16, 1024);
+      // K-major B: 8-row groups 1 KB apart; ring stage s is kStageK further on
+      const uint64_t kdesc0 = make_smem_desc_sw128(base + kSmemK, 16, 1024), qxdesc0 = make_smem_desc_sw128(base + L::kSmemQX, 16, 1024);
       // development builds: cycles this thread spends waiting for K and for a free S buffer (summed over the tiles)
       TRACE_ONLY(long long w_k = 0, w_se = 0, c0; const long long c_begin = clock64();)
       bool ok = true;
@@ -311,8 +387,11 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
           // 16 d per step: 8 tensor-memory columns of Q; 32 bytes along a K box row, the second box 8 KB further on
           constexpr int B2 = kKBoxBytes >> 4;
           umma_bf16_ts_pair_x8<2, 4, 6, B2, B2 + 2, B2 + 4, B2 + 6>(tmem_s0 + sb * 128, tmem_q,
-                                                                     kdesc0 + static_cast<uint64_t>(kst * (kHalfBytes >> 4)),
+                                                                     kdesc0 + static_cast<uint64_t>(kst * (L::kStageK >> 4)),
                                                                      idesc_qk, 0u);
+          if (WIDE)
+            umma_bf16_ss_pair_x4(tmem_s0 + sb * 128, qxdesc0 + static_cast<uint64_t>((seq & 1) * (kQT * 128 >> 4)),
+                                 kdesc0 + static_cast<uint64_t>((kst * L::kStageK + 2 * kKBoxBytes) >> 4), idesc_qk);
           umma_commit_pair(bar(K_EMPTY + kst));
           umma_commit_pair(bar(S_FULL + sb));
           TL(1, g, true);
@@ -373,9 +452,10 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
 
     // All 128 d columns of this thread's Q row of an item, global -> tensor memory (by the ONE group that opens the item)
     // An item's Q rows of this CTA, global -> the staging boxes in shared memory (one thread; an item ahead of their use)
-    auto fetch_q = [&](const Item& it) {
+    auto fetch_q = [&](const Item& it, int n) {  // n-th item of this pair
       const int y = it.pt * 2 * kQT + static_cast<int>(rank) * kQT;
-      mbar_expect_tx(bar(QS_FULL), 2 * kQT * 128);
+      mbar_expect_tx(bar(QS_FULL), (WIDE ? 3 : 2) * kQT * 128);
+      if (WIDE) tma_load_4d(base + L::kSmemQX + (n & 1) * (kQT * 128), &tmap_q, bar(QS_FULL), 128, y, it.h, it.b);
       tma_load_4d(base + kSmemQ, &tmap_q, bar(QS_FULL), 0, y, it.h, it.b);
       tma_load_4d(base + kSmemQ + kQT * 128, &tmap_q, bar(QS_FULL), 64, y, it.h, it.b);
     };
@@ -399,9 +479,22 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
       tc_fence_before();
       mbar_arrive_cluster(map_to_leader(bar(Q_READY)));
     };
+    // Gate (lane 0 of a warp): the closing group fetches the gate's rows into its output boxes while it works on
+    // the item's last tile.  The boxes are free once the item before has left them: its closer says so (O_BOX) at its next tile.
+    bool leaving = false;     // this thread's last output may still be in its boxes
+    int gated_items = 0;      // items so far with rows in this quarter, whichever group closed them: G_FULL and O_BOX complete once for each
+    auto fetch_gate = [&](const Item& it, int q0) {
+      if (gated_items > 0 && ok) ok = mbar_wait(bar(O_BOX + quarter), (gated_items - 1) & 1, err, DEVERR_ATTN_SOFTMAX);
+      if (!ok) return;
+      const uint32_t box = base + kSmemO + quarter * (32 * 256), full = bar(G_FULL + quarter);
+      const int y = q0 + quarter * 32;
+      mbar_expect_tx(full, args.two_out_boxes ? 32 * 256 : 32 * 128);
+      tma_load_4d(box, &tmap_g, full, 0, y, it.h, it.b);
+      if (args.two_out_boxes) tma_load_4d(box + 32 * 128, &tmap_g, full, 64, y, it.h, it.b);
+    };
     // The first item: group 1 brings Q in while group 0, which takes tile 0, has nothing else to do either.
     if (wg == 1 && pair_id < args.n_items) {
-      if (r == 0) fetch_q(item_at(pair_id));
+      if (r == 0) fetch_q(item_at(pair_id), 0);
       put_q(0);
     }
 
@@ -421,6 +514,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
       float* mu_sh = m_sh + 256;            // ... and the maximum it is relative to, of the group that leaves first
       float m_used = -INFINITY, l = 0.0f;   // the maximum this group's sums are relative to
       const int glast = g0 + n_tiles - 1;
+      const float sink = OPT > 0 && args.sink ? args.sink[it.h] : -INFINITY;  // (needed an item from now)
       const bool closer = (glast & 1) == wg;  // this group takes the item's last tile and writes its output
       // The "maximum decided" barriers alternate with the item like the values they guard: the group that opens the
       // next item decides its first tile before the other group has looked at this item's last decision, and one
@@ -430,16 +524,27 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
       const int j_other = (wg ^ 1) ^ (g0 & 1);
       const uint32_t m_seen = (seq & 1) ? m_seen1 : m_seen0;
       const bool more = item + n_pairs < args.n_items;
+      const bool has_rows = q0 + quarter * 32 < args.Sq;  // this warp's rows of the item
       if (!closer && more && r == 0) {
         // this group brings the next item's Q in, an item from now: fetch it as soon as this item's has left the boxes
         if (ok) ok = mbar_wait(bar(QS_FREE), seq & 1, err, DEVERR_ATTN_SOFTMAX);
-        if (ok) fetch_q(item_at(item + n_pairs));
+        // (WIDE: its columns 128.. take the box of the item before this one, whose products are complete)
+        if (ok) fetch_q(item_at(item + n_pairs), seq + 1);
       }
       // this group takes the pair's tiles of parity wg (S buffer wg), whichever items they belong to
 #pragma unroll 1
       for (int j = (wg ^ (g0 & 1)); ok && j < n_tiles; j += 2) {
         const int g = g0 + j;
         const uint32_t ph = (g >> 1) & 1;
+        if (OPT > 0 && args.gate && lane == 0) {
+          if (leaving) {
+            bulk_wait_read();
+            mbar_arrive(bar(O_BOX + quarter));
+            leaving = false;
+          }
+          if (g == glast && has_rows) fetch_gate(it, q0);
+        }
+        __syncwarp();
         TRACE_ONLY(c0 = clock64();)
         if (!mbar_wait(bar(S_FULL + wg), ph, err, DEVERR_ATTN_SOFTMAX)) { ok = false; break; }
         TRACE_ONLY(w_s += clock64() - c0; if (j < 2) w_s0 += clock64() - c0; c0 = clock64();)
@@ -464,32 +569,41 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         }
         tc_fence_before();
         mbar_arrive_cluster(s_empty_leader);  // the buffer can take QK^T of tile g + 2 (once the peer's group is here too)
-        if (CAP) {  // monotonic: the maximum below may follow it
-#pragma unroll
-          for (int e = 0; e < 128; ++e) s[e] = softcap_log2(s[e], args.two_y, args.cap_l2);
-        }
         const int k0 = (it.t0 + j) * kKT;
         const int first = args.window > 0 ? qi + off - args.window + 1 : 0;  // first visible key
         const bool need_mask = (k0 + kKT > args.Skv) || (args.causal && (k0 + kKT - 1 > q0 + off)) ||
                                (args.window > 0 && k0 < q0 + kQT + off - args.window);
+        bool raw = false;  // the scores go uncapped into the exponential's loop
+        float tmax = 0.0f;
+        if (CAP) {
+          tmax = row_max(s);
+          float tn[2] = {s[0], s[1]};
+#pragma unroll
+          for (int e = 2; e + 4 <= 128; e += 4) {
+            tn[0] = fmin3(tn[0], s[e], s[e + 1]);
+            tn[1] = fmin3(tn[1], s[e + 2], s[e + 3]);
+          }
+          tn[0] = fmin3(tn[0], s[126], s[127]);
+          const bool small = __all_sync(0xffffffffu, tmax <= args.small && fminf(tn[0], tn[1]) >= -args.small);
+          raw = small;
+          if (!small) {
+#pragma unroll
+            for (int e = 0; e < 128; ++e) s[e] = softcap_log2(s[e], args.two_y, args.cap_l2);
+          }
+        }
         if (need_mask) {
           const int limit = args.causal ? min(args.Skv - 1, qi + off) : args.Skv - 1;  // last visible key
 #pragma unroll
           for (int e = 0; e < 128; ++e)
             if (k0 + e > limit || k0 + e < first) s[e] = -INFINITY;
         }
-        // row maximum: four independent chains of three-input maxima
-        float tm[4] = {s[0], s[1], s[2], s[3]};
-#pragma unroll
-        for (int e = 4; e + 8 <= 128; e += 8) {
-          tm[0] = fmax3(tm[0], s[e], s[e + 1]);
-          tm[1] = fmax3(tm[1], s[e + 2], s[e + 3]);
-          tm[2] = fmax3(tm[2], s[e + 4], s[e + 5]);
-          tm[3] = fmax3(tm[3], s[e + 6], s[e + 7]);
+        if (!CAP) {
+          tmax = row_max(s) * args.scale_log2;  // log2 domain (scale > 0)
+        } else {
+          if (!raw || need_mask) tmax = row_max(s);
+          // (the cap is monotonic)
+          if (raw && tmax != -INFINITY) tmax = cap_poly(make_float2(tmax, tmax), args.cap_c, make_float2(0.0f, 0.0f)).x;
         }
-        tm[0] = fmax3(tm[0], s[124], s[125]);
-        tm[1] = fmax3(tm[1], s[126], s[127]);
-        const float tmax = fmaxf(fmax3(tm[0], tm[1], tm[2]), tm[3]) * args.scale_log2;  // log2 domain (scale > 0)
         TRACE_ONLY(t_ld += clock64() - c0; c0 = clock64();)
         TL(4, g, r == 0);
         // ---- the running maximum: tile j's decision follows tile j-1's (made by the other group) ----
@@ -537,12 +651,31 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         float2 ls[2] = {{0.0f, 0.0f}, {0.0f, 0.0f}};
         const float2 sc2 = {args.scale_log2, args.scale_log2}, neg_m2 = {-m, -m};
         uint32_t pk[64];
+        if (CAP && raw && !need_mask) {
 #pragma unroll
-        for (int e = 0; e < 64; ++e) {
-          const float2 x = __ffma2_rn(make_float2(s[2 * e], s[2 * e + 1]), sc2, neg_m2);  // masked scores are -inf -> 0
-          const float2 pr = {fast_exp2(x.x), fast_exp2(x.y)};
-          ls[e & 1] = __fadd2_rn(ls[e & 1], pr);
-          pk[e] = pack_bf16x2(pr.x, pr.y);
+          for (int e = 0; e < 64; ++e) {
+            const float2 x = cap_poly(make_float2(s[2 * e], s[2 * e + 1]), args.cap_c, neg_m2);
+            const float2 pr = {fast_exp2(x.x), fast_exp2(x.y)};
+            ls[e & 1] = __fadd2_rn(ls[e & 1], pr);
+            pk[e] = pack_bf16x2(pr.x, pr.y);
+          }
+        } else if (CAP && raw) {
+#pragma unroll
+          for (int e = 0; e < 64; ++e) {
+            const float2 x = cap_poly(make_float2(s[2 * e], s[2 * e + 1]), args.cap_c, neg_m2);  // (nothing of value for a masked score)
+            const float2 pr = {s[2 * e] == -INFINITY ? 0.0f : fast_exp2(x.x), s[2 * e + 1] == -INFINITY ? 0.0f : fast_exp2(x.y)};
+            ls[e & 1] = __fadd2_rn(ls[e & 1], pr);
+            pk[e] = pack_bf16x2(pr.x, pr.y);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 64; ++e) {
+            const float2 s2 = make_float2(s[2 * e], s[2 * e + 1]);
+            const float2 x = CAP ? __fadd2_rn(s2, neg_m2) : __ffma2_rn(s2, sc2, neg_m2);  // masked scores are -inf -> 0
+            const float2 pr = {fast_exp2(x.x), fast_exp2(x.y)};
+            ls[e & 1] = __fadd2_rn(ls[e & 1], pr);
+            pk[e] = pack_bf16x2(pr.x, pr.y);
+          }
         }
         TRACE_ONLY(t_exp += clock64() - c0; c0 = clock64();)
         TL(6, g, r == 0);
@@ -570,6 +703,11 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
       // has been free since its own last tile: it hands over its row sum and moves on -- it opens the next item (Q into
       // tensor memory as soon as the last Q K^T of this item is complete) and takes that item's first tile, while the
       // first group is still on this item's last tile and output. ----
+      if (OPT > 0 && args.gate && lane == 0 && leaving) {
+        bulk_wait_read();
+        mbar_arrive(bar(O_BOX + quarter));
+        leaving = false;
+      }
       bulk_wait_read();  // this thread's last output rows have left shared memory: whichever group writes there next has
       __syncwarp();      // waited for this point, here or through L_READY
       if (!closer) {
@@ -587,10 +725,25 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         if (more) next_it = item_at(item + n_pairs);  // (the last P V is still running)
         if (ok) ok = mbar_wait(bar(L_READY + (seq & 1)), (seq >> 1) & 1, err, DEVERR_ATTN_SOFTMAX);
         l += l_sh[r] * fast_exp2(mu_sh[r] - m_fin);  // 0 * 2^-inf = 0 for a group without tiles
+        const int y = q0 + quarter * 32;
+        const uint32_t o_box = base + kSmemO + quarter * (32 * 256);
+        const bool gated = OPT > 0 && args.gate && has_rows;
+        uint32_t sig[OPT > 0 ? 64 : 1];  // sigmoid of the gate's row as bf16 pairs, while the last product runs
+        if (gated) {
+          if (ok) ok = mbar_wait(bar(G_FULL + quarter), gated_items & 1, err, DEVERR_ATTN_SOFTMAX);
+          const uint8_t* grow = gen + kSmemO + quarter * (32 * 256) + lane * 128;
+#pragma unroll
+          for (int ch = 0; ch < 16; ++ch) {  // (without a second box its columns are nobody's)
+            const uint4 g4 = *reinterpret_cast<const uint4*>(grow + (ch >> 3) * (32 * 128) + (((ch & 7) ^ (lane & 7)) << 4));
+            sigmoid_x4(g4.x, g4.y, sig[OPT > 0 ? 4 * ch : 0], sig[OPT > 0 ? 4 * ch + 1 : 0]);
+            sigmoid_x4(g4.z, g4.w, sig[OPT > 0 ? 4 * ch + 2 : 0], sig[OPT > 0 ? 4 * ch + 3 : 0]);
+          }
+          __syncwarp();
+        }
         if (ok) ok = mbar_wait(bar(PV_DONE + (glast & 1)), (glast >> 1) & 1, err, DEVERR_ATTN_SOFTMAX);
         if (ok) {
           tc_fence_after();
-          if (args.sink) l += fast_exp2(fmaf(args.sink[it.h], 1.4426950408889634f, -m_fin));
+          if (OPT > 0) l += fast_exp2(fmaf(sink, 1.4426950408889634f, -m_fin));
           float inv;
           asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(inv) : "f"(l));  // l >= 1 (the row's maximum contributes 2^0); 1 ulp
           inv *= args.out_scale;
@@ -610,6 +763,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
               uint4 o4;
+              const int ch = (c & 1) * 4 + v;  // chunk of the box's 128-byte row; columns 64.. are the second box
+              uint4* place = reinterpret_cast<uint4*>(orow + (c >> 1) * (32 * 128) + ((ch ^ (lane & 7)) << 4));
               const float2 a0 = __fmul2_rn(make_float2(__uint_as_float(t[c][v * 8 + 0]), __uint_as_float(t[c][v * 8 + 1])), inv2);
               const float2 a1 = __fmul2_rn(make_float2(__uint_as_float(t[c][v * 8 + 2]), __uint_as_float(t[c][v * 8 + 3])), inv2);
               const float2 a2 = __fmul2_rn(make_float2(__uint_as_float(t[c][v * 8 + 4]), __uint_as_float(t[c][v * 8 + 5])), inv2);
@@ -618,18 +773,22 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
               o4.y = pack_bf16x2(a1.x, a1.y);
               o4.z = pack_bf16x2(a2.x, a2.y);
               o4.w = pack_bf16x2(a3.x, a3.y);
-              const int ch = (c & 1) * 4 + v;  // chunk of the box's 128-byte row; columns 64.. are the second box
-              *reinterpret_cast<uint4*>(orow + (c >> 1) * (32 * 128) + ((ch ^ (lane & 7)) << 4)) = o4;
+              if (gated) {
+                o4.x = bf16x2_mul(o4.x, sig[OPT > 0 ? 16 * c + 4 * v : 0]);
+                o4.y = bf16x2_mul(o4.y, sig[OPT > 0 ? 16 * c + 4 * v + 1 : 0]);
+                o4.z = bf16x2_mul(o4.z, sig[OPT > 0 ? 16 * c + 4 * v + 2 : 0]);
+                o4.w = bf16x2_mul(o4.w, sig[OPT > 0 ? 16 * c + 4 * v + 3 : 0]);
+              }
+              *place = o4;
             }
           }
           fence_proxy_async_smem();
           __syncwarp();
-          const int y = q0 + quarter * 32;
           if (lane == 0 && y < args.Sq) {  // rows past the end are clipped by the copy
-            const uint32_t src = base + kSmemO + quarter * (32 * 256);
-            tma_store_4d(&tmap_o, src, 0, y, it.h, it.b);
-            if (args.two_out_boxes) tma_store_4d(&tmap_o, src + 32 * 128, 64, y, it.h, it.b);
+            tma_store_4d(&tmap_o, o_box, 0, y, it.h, it.b);
+            if (args.two_out_boxes) tma_store_4d(&tmap_o, o_box + 32 * 128, 64, y, it.h, it.b);
             bulk_commit();
+            leaving = true;
           }
           if (valid && args.lse)
             args.lse[(static_cast<long long>(it.b) * args.Hq + it.h) * args.Sq + qi] = 0.6931471805599453f * (m_fin + log2f(l));
@@ -639,6 +798,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
       }
       TRACE_ONLY(t_end += clock64() - c0; if (closer) t_close += clock64() - c0;)
       TL(closer ? 10 : 11, glast, r == 0);
+      if (has_rows) ++gated_items;
       if (seq & 1) m_seen1 += (n_tiles - j_other + 1) >> 1; else m_seen0 += (n_tiles - j_other + 1) >> 1;
       g0 += n_tiles;
     }
@@ -684,8 +844,16 @@ int attention_prefill_prepare() {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 64 && (done.load(std::memory_order_acquire) >> dev) & 1ull) return 0;
-  cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemTotal);
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemTotal);
+  cudaError_t e = cudaSuccess;
+  auto raise = [&](auto kernel, int bytes) {
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+  };
+  raise(attention_prefill_kernel<1, false>, Smem<false>::kSmemTotal);
+  raise(attention_prefill_kernel<1, true>, Smem<true>::kSmemTotal);
+  raise(attention_prefill_kernel<0, false>, Smem<false>::kSmemTotal);
+  raise(attention_prefill_kernel<2, false>, Smem<false>::kSmemTotal);
+  raise(attention_prefill_kernel<0, true>, Smem<true>::kSmemTotal);
+  raise(attention_prefill_kernel<2, true>, Smem<true>::kSmemTotal);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (dev < 64) done.fetch_or(1ull << dev, std::memory_order_release);
   return 0;
@@ -695,17 +863,17 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
                            cudaStream_t stream) {
   if (!q || !k || !v || !o || s.B <= 0 || s.Hq <= 0 || s.Hkv <= 0 || s.Sq <= 0 || s.Skv <= 0) return TEENY_ERR_BAD_ARG;
   const int DV = s.DV ? s.DV : s.D;
-  if (s.D <= 0 || s.D > kHD || s.D % 8 || DV <= 0 || DV > kHD || DV % 8 || s.Hq % s.Hkv != 0 || s.gate) return TEENY_ERR_BAD_ARG;
+  if (s.D <= 0 || s.D > kHD + 64 || s.D % 8 || DV <= 0 || DV > kHD || DV % 8 || s.Hq % s.Hkv != 0) return TEENY_ERR_BAD_ARG;
   if (s.causal && s.Skv < s.Sq) return TEENY_ERR_BAD_ARG;
   if (s.window < 0 || (s.window > 0 && !s.causal)) return TEENY_ERR_BAD_ARG;
-  const long long strides[] = {s.q_sb, s.q_sh, s.q_ss, s.k_sb, s.k_sh, s.k_ss, s.v_sb, s.v_sh, s.v_ss, s.o_ss, s.o_sh, s.o_sb};
+  const long long strides[] = {s.q_sb, s.q_sh, s.q_ss, s.k_sb, s.k_sh, s.k_ss, s.v_sb, s.v_sh, s.v_ss, s.o_ss, s.o_sh, s.o_sb, s.gate_sb, s.gate_ss};
   for (long long st : strides)
     if (st % 8 != 0) return TEENY_ERR_ALIGNMENT;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
-       reinterpret_cast<uintptr_t>(o)) & 15)
+       reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(s.gate)) & 15)
     return TEENY_ERR_ALIGNMENT;
   if (s.Hq > 65535 || s.B > 65535) return TEENY_ERR_BAD_ARG;
-  CUtensorMap mk, mv, mq, mo;
+  CUtensorMap mk, mv, mq, mo, mg;
   int rc;
   // a dimension of extent 1 still needs a legal (multiple-of-16-byte, non-zero) stride
   auto fix = [](long long st, long long fallback) { return st > 0 ? st : fallback; };
@@ -713,8 +881,11 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   if ((rc = make_map(&mv, v, DV, s.Skv, s.Hkv, s.B, s.v_ss, fix(s.v_sh, s.v_ss), fix(s.v_sb, s.v_ss), 128))) return rc;
   if ((rc = make_map(&mq, q, s.D, s.Sq, s.Hq, s.B, s.q_ss, fix(s.q_sh, s.q_ss), fix(s.q_sb, s.q_ss), kQT))) return rc;
   if ((rc = make_map(&mo, o, DV, s.Sq, s.Hq, s.B, s.o_ss, fix(s.o_sh, s.o_ss), fix(s.o_sb, s.o_ss), 32))) return rc;
+  if (!s.gate) mg = mo;
+  else if ((rc = make_map(&mg, s.gate, DV, s.Sq, s.Hq, s.B, s.gate_ss, DV, fix(s.gate_sb, s.gate_ss), 32))) return rc;
 
   PrefillArgs a{};
+  a.gate = s.gate != nullptr;
   a.lse = lse; a.B = s.B; a.Hq = s.Hq; a.Hkv = s.Hkv; a.Sq = s.Sq; a.Skv = s.Skv;
   a.scale_log2 = s.scale * 1.4426950408889634f;
   a.causal = s.causal;
@@ -724,6 +895,12 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
     a.cap_l2 = s.softcap * 1.4426950408889634f;
     a.two_y = 2.0f * a.scale_log2 / s.softcap;
     a.scale_log2 = 1.0f;
+    // tanh(x) = x P(x^2) on [-1/2, 1/2]: minimax fit of the relative error (6e-7 in f32)
+    static const float kTanh[4] = {0.99999946f, -0.33326319f, 0.13190296f, -0.044402227f};
+    const float x = s.scale / s.softcap;
+    float power = x * a.cap_l2;
+    for (int i = 0; i < 4; ++i, power *= x * x) a.cap_c[i] = kTanh[i] * power;
+    a.small = a.cap_c[3] < -1e-30f ? 0.5f / x : -1.0f;  // (coefficients near the end of f32's range: exponential and reciprocal only)
   }
   a.sink = s.sink;
   a.two_out_boxes = DV > 64;
@@ -746,8 +923,12 @@ int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o,
   if (pairs > items) pairs = items;
   if (pairs < 1) pairs = 1;
   if (pairs > 0x3fffffffLL) return TEENY_ERR_BAD_ARG;
-  auto kernel = s.softcap > 0.0f ? attention_prefill_kernel<true> : attention_prefill_kernel<false>;
-  launch_kernel(kernel, dim3(static_cast<unsigned>(2 * pairs)), dim3(kThreads), kSmemTotal, stream, 2, mk, mv, mq, mo, a);
+  const dim3 grid(static_cast<unsigned>(2 * pairs));
+  const bool wide = s.D > kHD;
+  auto kernel = s.softcap > 0.0f     ? (wide ? attention_prefill_kernel<2, true> : attention_prefill_kernel<2, false>)
+                : s.gate || s.sink ? (wide ? attention_prefill_kernel<1, true> : attention_prefill_kernel<1, false>)
+                                   : (wide ? attention_prefill_kernel<0, true> : attention_prefill_kernel<0, false>);
+  launch_kernel(kernel, grid, dim3(kThreads), wide ? Smem<true>::kSmemTotal : Smem<false>::kSmemTotal, stream, 2, mk, mv, mq, mo, mg, a);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -8,8 +8,8 @@
 // (kKeysInRing) and every kernel reads all keys from there.
 //
 // window_attention chooses among
-//   attention_prefill_bf16   whole prompts of one length, head size 128 (tcgen05 on CTA pairs, attention_prefill.cu); over a
-//                            cache that never wraps, any long entry, head sizes up to 128
+//   attention_prefill_bf16   whole prompts of one length, and long entries whose keys lie in order (a cache that never wraps, or
+//                            all in k_new); keys up to 192, values up to 128 (tcgen05 on CTA pairs, attention_prefill.cu)
 //   attention_decode_bf16    single tokens, head sizes up to 128 (TMA-streamed ring, attention_decode.cu)
 //   window_attention_mma_kernel   any other bf16 step, head sizes up to 256 in multiples of 8 (mma.sync tiles, cp.async rows
 //                            from ring and step): portions, unequal prompts, other head sizes
@@ -486,27 +486,6 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const WindowA
   }
 }
 
-// out *= sigmoid(gate), eight columns per thread
-__global__ void sigmoid_gate_kernel(bf16* __restrict__ out, long long ldo, const bf16* __restrict__ gate, long long ldg, long long rows, int vecs) {
-  pdl_wait();
-  pdl_trigger();
-  const long long total = rows * vecs;
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / vecs;
-    const int c = static_cast<int>(i - r * vecs) * 8;
-    const uint4 o = *reinterpret_cast<const uint4*>(out + r * ldo + c), g = *reinterpret_cast<const uint4*>(gate + r * ldg + c);
-    auto mul = [](uint32_t x, uint32_t y) { return pack_bf16x2(bf16_lo(x) * sigmoid_f(bf16_lo(y)), bf16_hi(x) * sigmoid_f(bf16_hi(y))); };
-    *reinterpret_cast<uint4*>(out + r * ldo + c) = make_uint4(mul(o.x, g.x), mul(o.y, g.y), mul(o.z, g.z), mul(o.w, g.w));
-  }
-}
-
-int sigmoid_gate_rows(bf16* out, long long ldo, const bf16* gate, long long ldg, long long rows, int cols, cudaStream_t st) {
-  const long long blocks = (rows * (cols / 8) + 255) / 256;
-  launch_kernel(sigmoid_gate_kernel, dim3(static_cast<unsigned>(blocks < 16LL * sm_count() ? blocks : 16LL * sm_count())), dim3(256), 0, st, 1, out, ldo,
-                gate, ldg, rows, cols / 8);
-  return static_cast<int>(cudaGetLastError());
-}
-
 bool valid(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int max_len) {
   return (a.keys == kKeysInRing || (a.k_new && a.v_new)) && (a.keys == kKeysInNew || (a.k_ring && a.v_ring)) && seqs && n_seqs > 0 && n_seqs <= 65535 && max_len > 0 && a.ring > 0 &&
          a.window > 0 && a.Hq > 0 && a.Hkv > 0 && a.Hq % a.Hkv == 0 && a.D > 0 && a.D <= kMaxHead && a.DV > 0 && a.DV <= kMaxHead;
@@ -580,7 +559,7 @@ int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int m
     return attention_decode_bf16(static_cast<const bf16*>(a.q), static_cast<const bf16*>(a.k_ring), static_cast<const bf16*>(a.v_ring),
                                  static_cast<bf16*>(a.out), s, 0, nullptr, a.scratch, a.scratch_bytes, st, 1, nullptr, a.counters, &ring);
   }
-  const bool prefill = rows16 && head <= 128 && a.scale > 0.0f;
+  const bool prefill = rows16 && a.D <= 192 && a.DV <= 128 && a.scale > 0.0f;
   if (prefill && a.keys == kKeysInRing && a.host && a.window >= a.ring && max_len >= kPrefillLen) {
     // Entries of equal length and position in neighbouring slots make one launch over the cache; short ones in between go
     // to the other kernels together.
@@ -601,12 +580,14 @@ int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int m
         s.B = n; s.Sq = f.len; s.Skv = f.pos + f.len; s.causal = 1;
         s.q_sb = f.len * a.ldq; s.o_sb = f.len * a.ldo;
         bf16* out = static_cast<bf16*>(a.out) + static_cast<size_t>(f.row0) * a.ldo;
-        int rc = attention_prefill_bf16(static_cast<const bf16*>(a.q) + static_cast<size_t>(f.row0) * a.ldq,
-                                        static_cast<const bf16*>(a.k_ring) + static_cast<size_t>(f.slot) * s.k_sb,
-                                        static_cast<const bf16*>(a.v_ring) + static_cast<size_t>(f.slot) * s.v_sb, out, nullptr, s, st);
-        if (rc == 0 && a.gate)
-          rc = sigmoid_gate_rows(out, a.ldo, static_cast<const bf16*>(a.gate) + static_cast<size_t>(f.row0) * a.ldg, a.ldg,
-                                 static_cast<long long>(n) * f.len, a.Hq * a.DV, st);
+        if (a.gate) {
+          s.gate = static_cast<const bf16*>(a.gate) + static_cast<size_t>(f.row0) * a.ldg;
+          s.gate_sb = f.len * a.ldg;
+          s.gate_ss = a.ldg;
+        }
+        const int rc = attention_prefill_bf16(static_cast<const bf16*>(a.q) + static_cast<size_t>(f.row0) * a.ldq,
+                                              static_cast<const bf16*>(a.k_ring) + static_cast<size_t>(f.slot) * s.k_sb,
+                                              static_cast<const bf16*>(a.v_ring) + static_cast<size_t>(f.slot) * s.v_sb, out, nullptr, s, st);
         if (rc) return rc;
       }
       e += n;
@@ -623,11 +604,13 @@ int window_attention(const WindowAttn& a, const SeqDesc* seqs, int n_seqs, int m
     s.k_sb = max_len * a.ldk; s.k_sh = a.D; s.k_ss = a.ldk;
     s.v_sb = max_len * a.ldv; s.v_sh = a.DV; s.v_ss = a.ldv;
     bf16* out = static_cast<bf16*>(a.out) + first * a.ldo;
-    const int rc = attention_prefill_bf16(static_cast<const bf16*>(a.q) + first * a.ldq, static_cast<const bf16*>(a.k_new) + (first - pos) * a.ldk,
-                                          static_cast<const bf16*>(a.v_new) + (first - pos) * a.ldv, out, nullptr, s, st);
-    if (rc || !a.gate) return rc;
-    return sigmoid_gate_rows(out, a.ldo, static_cast<const bf16*>(a.gate) + first * a.ldg, a.ldg, static_cast<long long>(n_seqs) * max_len,
-                             a.Hq * a.DV, st);
+    if (a.gate) {
+      s.gate = static_cast<const bf16*>(a.gate) + first * a.ldg;
+      s.gate_sb = max_len * a.ldg;
+      s.gate_ss = a.ldg;
+    }
+    return attention_prefill_bf16(static_cast<const bf16*>(a.q) + first * a.ldq, static_cast<const bf16*>(a.k_new) + (first - pos) * a.ldk,
+                                  static_cast<const bf16*>(a.v_new) + (first - pos) * a.ldv, out, nullptr, s, st);
   }
   if (rows16 && max_len >= 8) {
     const dim3 grid((max_len + kQRows - 1) / kQRows, a.Hq, n_seqs), block(128);

@@ -136,11 +136,11 @@ struct AttnShape {
   int causal;
   int window = 0;           // attention_prefill_bf16, causal: query i sees only its last `window` keys (0 = all)
   float out_scale = 1.0f;   // factor of the output (attention_prefill_bf16, attention_decode_bf16)
-  int DV = 0;               // value size (0: D); attention_prefill_bf16 and ring decode take any D, DV <= 128, multiples of 8
+  int DV = 0;               // value size (0: D).  Multiples of 8; attention_prefill_bf16: D <= 192, DV <= 128, ring decode: both <= 128
   float softcap = 0.0f;     // > 0: scores s * scale are capped, softcap * tanh(s * scale / softcap)
   const float* sink = nullptr;   // [Hq]: exp(sink) joins the softmax denominator of the head
-  const bf16* gate = nullptr;    // attention_decode_bf16: output times sigmoid(gate); batch stride gate_sb, heads DV apart
-  long long gate_sb = 0;
+  const bf16* gate = nullptr;    // output times sigmoid(gate); batch stride gate_sb, row stride gate_ss (prefill), heads DV apart
+  long long gate_sb = 0, gate_ss = 0;
 };
 int attention_prefill_bf16(const bf16* q, const bf16* k, const bf16* v, bf16* o, float* lse, const AttnShape& s,
                            cudaStream_t stream);

@@ -110,7 +110,8 @@ def planted(seed, T, heads, kv, dim, vdim):
     return q, k, v
 
 
-SHAPES = [(4, 1, 128, 128), (4, 2, 96, 64), (6, 2, 64, 64), (2, 2, 72, 120), (8, 1, 32, 48), (2, 1, 136, 24), (3, 3, 20, 12), (8, 2, 48, 128)]
+SHAPES = [(4, 1, 128, 128), (4, 2, 96, 64), (6, 2, 64, 64), (2, 2, 72, 120), (8, 1, 32, 48), (2, 1, 136, 24), (3, 3, 20, 12), (8, 2, 48, 128),
+          (4, 4, 192, 128), (2, 1, 144, 64)]
 
 
 @DTYPES
@@ -137,10 +138,11 @@ def test_full_attention(dtype, heads, kv, dim, vdim, cuts):
 
 
 @pytest.mark.parametrize("cap,sinks,gated", [(0.0, False, False), (50.0, False, True), (0.0, True, False), (4.0, True, True)])
-def test_full_attention_in_batches(cap, sinks, gated):
+@pytest.mark.parametrize("D,V", [(128, 128), (192, 128), (96, 56)])
+def test_full_attention_in_batches(cap, sinks, gated, D, V):
     """Unequal entries in one step: equal long ones in neighbouring slots, long ones with a past, short ones and single tokens."""
     from teenygrad_b200 import ops
-    H, G, D, V, C = 4, 2, 128, 128, 700
+    H, G, C = 4, 2, 700
     sink = torch.tensor([-1.0, 0.5, 2.0, 5.0]) if sinks else None
     full = {b: planted(20 * b + 1, C, H, G, D, V) for b in range(7)}
     full = {b: tuple(t.to(BF) for t in p) for b, p in full.items()}
@@ -156,6 +158,25 @@ def test_full_attention_in_batches(cap, sinks, gated):
         if gated:
             e = e * om.sigmoid(gate[s][p:p + n].double()).view(n, H, V)
         assert rel(got[r0:r0 + n], e) < 1.5e-2, (s, p)
+
+
+@pytest.mark.parametrize("D,V", [(128, 128), (192, 64)])
+@pytest.mark.parametrize("cap", [0.0, 2.0, 400.0])
+def test_full_attention_many_work_items(D, V, cap):
+    """More (query tile, head, sequence) items than the GPU has CTA pairs, unequal numbers of key tiles; soft caps on both sides of
+    the polynomial's range."""
+    from teenygrad_b200 import ops
+    B, H, S = 5, 12, 900
+    parts = [planted(50 * b, S, H, H, D, V) for b in range(B)]
+    q, k, v = (torch.cat([p[i] for p in parts]).to(BF) for i in range(3))
+    gate, sink = (3 * rnd(7, B * S, H * V)).to(BF), torch.linspace(-3.0, 3.0, H)
+    kc, vc = (t.view(B, S, H, -1).transpose(1, 2).contiguous().cuda() for t in (k, v))
+    got = ops.cached_attention(q.cuda(), kc, vc, 0.15, entries_of([S] * B, range(B)), softcap=cap, sink=sink.cuda(), gate=gate.cuda()).double()
+    g = om.sigmoid(gate.double()).view(-1, H, V)
+    for b in range(B):
+        s = slice(b * S, (b + 1) * S)
+        want = om.causal_attention_fast(q[s].double(), k[s].double(), v[s].double(), 0.15, cap or None, sink.double()) * g[s]
+        assert rel(got[s], want) < 1.5e-2, b
 
 
 @DTYPES
