@@ -728,18 +728,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
         const int y = q0 + quarter * 32;
         const uint32_t o_box = base + kSmemO + quarter * (32 * 256);
         const bool gated = OPT > 0 && args.gate && has_rows;
-        uint32_t sig[OPT > 0 ? 64 : 1];  // sigmoid of the gate's row as bf16 pairs, while the last product runs
-        if (gated) {
-          if (ok) ok = mbar_wait(bar(G_FULL + quarter), gated_items & 1, err, DEVERR_ATTN_SOFTMAX);
-          const uint8_t* grow = gen + kSmemO + quarter * (32 * 256) + lane * 128;
-#pragma unroll
-          for (int ch = 0; ch < 16; ++ch) {  // (without a second box its columns are nobody's)
-            const uint4 g4 = *reinterpret_cast<const uint4*>(grow + (ch >> 3) * (32 * 128) + (((ch & 7) ^ (lane & 7)) << 4));
-            sigmoid_x4(g4.x, g4.y, sig[OPT > 0 ? 4 * ch : 0], sig[OPT > 0 ? 4 * ch + 1 : 0]);
-            sigmoid_x4(g4.z, g4.w, sig[OPT > 0 ? 4 * ch + 2 : 0], sig[OPT > 0 ? 4 * ch + 3 : 0]);
-          }
-          __syncwarp();
-        }
+        if (gated && ok) ok = mbar_wait(bar(G_FULL + quarter), gated_items & 1, err, DEVERR_ATTN_SOFTMAX);
         if (ok) ok = mbar_wait(bar(PV_DONE + (glast & 1)), (glast >> 1) & 1, err, DEVERR_ATTN_SOFTMAX);
         if (ok) {
           tc_fence_after();
@@ -773,11 +762,11 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __gri
               o4.y = pack_bf16x2(a1.x, a1.y);
               o4.z = pack_bf16x2(a2.x, a2.y);
               o4.w = pack_bf16x2(a3.x, a3.y);
-              if (gated) {
-                o4.x = bf16x2_mul(o4.x, sig[OPT > 0 ? 16 * c + 4 * v : 0]);
-                o4.y = bf16x2_mul(o4.y, sig[OPT > 0 ? 16 * c + 4 * v + 1 : 0]);
-                o4.z = bf16x2_mul(o4.z, sig[OPT > 0 ? 16 * c + 4 * v + 2 : 0]);
-                o4.w = bf16x2_mul(o4.w, sig[OPT > 0 ? 16 * c + 4 * v + 3 : 0]);
+              if (gated) {  // (without a second box its columns are nobody's)
+                uint4 g4 = *place;
+                sigmoid_x4(g4.x, g4.y, g4.x, g4.y);
+                sigmoid_x4(g4.z, g4.w, g4.z, g4.w);
+                o4 = make_uint4(bf16x2_mul(o4.x, g4.x), bf16x2_mul(o4.y, g4.y), bf16x2_mul(o4.z, g4.z), bf16x2_mul(o4.w, g4.w));
               }
               *place = o4;
             }
