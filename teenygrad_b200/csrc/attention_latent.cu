@@ -346,23 +346,26 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
   }
 }
 
-// Absorbed attention on the tensor cores (tcgen05).  CTA = N consecutive (token, head) rows of one entry x one share of its keys;
-// the CTAs of a cluster hold the shares of one row tile.  The rows are the N side of both products, so a few query heads waste
-// nothing, and the cache rows, loaded once per 128-key tile, are the A operand of both:
+// Absorbed attention on the tensor cores (tcgen05).  A row tile is N consecutive (token, head) rows of one entry; a cluster shares
+// it: each CTA takes a share of the keys and, where there are 256 or more value dimensions, one of two halves of the dimensions,
+// so that two 128-key tiles fit into its shared memory.  The rows are the N side of both products (a few query heads waste
+// nothing), and the cache rows, loaded once per tile, are the A operand of both:
 //   S^T [128 keys, N]   = C [128 keys, D] Q^T          C K-major, Q in shared memory for the whole walk
 //   O^T [DV, N]        += C^T [DV, 128 keys] P^T       the same shared memory read MN-major; one M = 128 product per 128 values
-// Tensor memory: O^T in ceil(DV / 128) blocks of N columns, two S^T buffers of N columns.
+// Tensor memory: O^T in blocks of N columns per 128 values, two S^T buffers of N columns.
 //   warp 4   TMA producer: ring of 32 KB slots, each 128 keys x 128 value dimensions (two [128 keys][64 d] boxes); the dimensions
 //            behind the values (the rotated part) travel in a ring of single boxes.  A slot is free again when its product with P
 //            has completed, so the next tile's loads follow the current one's products block by block.  Starts before the
 //            dependency wait: only the queries come from the kernel in front of this one.
 //   warp 5   allocates tensor memory, loads the queries, issues the MMAs (one thread); S of tile t + 1 goes ahead of P V of tile t
 //            where the ring holds two tiles.
-//   warps 0-3  thread = key in a tile: its N scores out of tensor memory, mask, weights against the rows' running maxima (shared
-//            memory), sums in registers, weights as bf16 into shared memory ([row][key], the B operand).  The maxima only move when
-//            some score exceeds its row's by more than 2^8 (one vote per tile); then the tile's maxima are reduced across the
-//            lanes and O^T is rescaled.
-// At the end the shares meet in distributed shared memory: every CTA sums a slice of the columns, scaled to the common maximum.
+//   warps 0-3  thread = key in a tile: its N scores out of tensor memory -- with halved dimensions plus the partial scores of the
+//            other half's CTA, exchanged through distributed shared memory, after which both do the same --, mask, weights
+//            against the rows' running maxima (shared memory), sums in registers, weights as bf16 into shared memory ([row][key],
+//            the B operand).  The maxima only move when some score exceeds its row's by more than 2^8 (one vote per tile); then
+//            the tile's maxima are reduced across the lanes and O^T is rescaled.
+// At the end the shares tell one another their maxima and sums (while the last product runs), every CTA scales its O^T by its
+// weights and stores each column into the shared memory of the CTA that sums this column over the shares.
 constexpr int kLatTile = 128, kLatPair = 32768, kLatBox = 16384, kLatMaxSlots = 12, kLatThreads = 192;
 constexpr float kLatGrow = 8.0f;  // log2 units
 
@@ -371,44 +374,72 @@ struct LatTcArgs {
   long long ldo;
   int row_base;        // step row that row 0 of q and out stands for
   int H, D, DV;
-  int pairs, rests;    // 128-dimension slots of a tile that hold values; single boxes behind them
+  int halves;          // CTAs that share the dimensions: 1 or 2
+  int blocks;          // 128-dimension blocks that hold values
+  int pairs, rests;    // of a tile: slots with values of one CTA (at most); single boxes behind the values (the last half's)
   int slots, rest_slots, ahead;
-  int o_ld;            // row stride (floats) of the output staging
   uint32_t tmem_cols;
   float scale_log2;
   int* err;
 };
 
 struct LatSmem {  // byte offsets
-  int rest, q, p, bars, stats, total;
+  int rest, q, p, swap, bars, stats, total;
 };
-__host__ __device__ inline LatSmem lat_smem(int n, int pairs, int rests, int slots, int rest_slots) {
+__host__ __device__ inline LatSmem lat_smem(int n, int halves, int pairs, int rests, int slots, int rest_slots) {
   LatSmem s;
   s.rest = slots * kLatPair;
   s.q = s.rest + rest_slots * kLatBox;
   s.p = s.q + (2 * pairs + rests) * n * 128;
-  s.bars = s.p + 2 * n * 128;
-  s.stats = s.bars + 8 * (2 * kLatMaxSlots + 2 * kLatMaxSlots + 8);
+  // partial scores from the other half, two tiles of [n / 4][128 keys] float4; in the end the columns to be summed here
+  s.swap = s.p + 2 * n * 128;
+  const int scores = halves > 1 ? 2 * n * 128 * 4 : 0, sums = n * (128 * pairs + 32) * 4;
+  s.bars = s.swap + (scores > sums ? scores : sums);
+  s.stats = s.bars + 8 * (4 * kLatMaxSlots + 8);
   s.total = s.stats + 4 * (8 + 16) * n + 1024;
   return s;
 }
 
-__device__ __forceinline__ void cluster_sync() {
-  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-__device__ __forceinline__ float ld_cluster(uint32_t local_addr, uint32_t rank) {
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ uint32_t map_rank(uint32_t local_addr, uint32_t rank) {
   uint32_t r;
-  float v;
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(local_addr), "r"(rank));
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
-  return v;
+  return r;
 }
-__device__ __forceinline__ float4 ld_cluster4(uint32_t local_addr, uint32_t rank) {
-  uint32_t r;
-  float4 v;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(local_addr), "r"(rank));
-  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(r) : "memory");
-  return v;
+__device__ __forceinline__ void st_cluster(uint32_t addr, float v) { asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
+__device__ __forceinline__ void st_cluster2(uint32_t addr, float x, float y) {
+  asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(x), "f"(y) : "memory");
+}
+__device__ __forceinline__ void st_cluster4(uint32_t addr, float x, float y, float z, float w) {
+  asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(x), "f"(y), "f"(z), "f"(w) : "memory");
+}
+// This thread's stores to the other CTA's shared memory, then its arrival on a barrier there; mbar_wait_cluster sees them.
+__device__ __forceinline__ void mbar_arrive_remote(uint32_t addr) {
+  asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(addr) : "memory");
+}
+__device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity, int* err, int code) {
+  uint64_t t0 = 0;
+#pragma unroll 1
+  for (uint32_t it = 0;; ++it) {
+    uint32_t done;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(done) : "r"(bar), "r"(parity) : "memory");
+    if (done) return true;
+    if ((it & 0xff) == 0xff) {
+      if (*reinterpret_cast<volatile int*>(err) != 0) return false;
+      const uint64_t now = global_timer_ns();
+      if (t0 == 0) {
+        t0 = now;
+      } else if (now - t0 > kWaitLimitNs) {
+        atomicCAS(err, 0, code);
+        return false;
+      }
+    }
+  }
 }
 // whether `v` holds in any of the 128 softmax threads (barrier 1)
 __device__ __forceinline__ bool any128(bool v) {
@@ -532,22 +563,26 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   }
   const uint32_t base = (smem_u32(lat_raw) + 1023u) & ~1023u;
   uint8_t* gen = lat_raw + (base - smem_u32(lat_raw));
-  const LatSmem lay = lat_smem(N, a.pairs, a.rests, a.slots, a.rest_slots);
+  const LatSmem lay = lat_smem(N, a.halves, a.pairs, a.rests, a.slots, a.rest_slots);
   const uint32_t bar0 = base + lay.bars;
   auto full = [&](int i) { return bar0 + 8u * i; };
   auto empty = [&](int i) { return bar0 + 8u * (kLatMaxSlots + i); };
   auto rfull = [&](int i) { return bar0 + 8u * (2 * kLatMaxSlots + i); };
   auto rempty = [&](int i) { return bar0 + 8u * (3 * kLatMaxSlots + i); };
   const uint32_t misc = bar0 + 8u * 4 * kLatMaxSlots;
-  const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40;  // two s_full
+  const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40, x_full = misc + 48;  // two s_full, two x_full
   float* m_sh = reinterpret_cast<float*>(gen + lay.stats);  // [N] running maxima, log2 domain
-  float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally the row sums
+  float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally this share's weights
   float* up_sh = alpha_sh + N;                              // [N] by how much the maxima just rose
   float* red = up_sh + N;                                   // [4][N]
   int* lim = reinterpret_cast<int*>(red + 4 * N);           // [N] last key each row sees
-  float2* share = reinterpret_cast<float2*>(lim + N);       // [N][8] maximum and sum of every share; then its weight
+  float2* share = reinterpret_cast<float2*>(lim + N);       // [N][8] maximum and sum of every share
 
-  const int splits = gridDim.x, split = blockIdx.x;
+  const int rank = blockIdx.x, half = rank % a.halves, split = rank / a.halves, splits = gridDim.x / a.halves;
+  const bool clustered = gridDim.x > 1;
+  const int block0 = half * a.pairs;                                     // this CTA's blocks of 128 values ...
+  const int pairs = min(a.pairs, a.blocks - block0);
+  const int rests = half == a.halves - 1 ? a.rests : 0;                  // ... and single boxes behind the values
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int L = seq.pos + (row0 + n_rows - 1) / a.H + 1;  // keys the tile's last row sees
   const int span = ((L + splits - 1) / splits + kLatTile - 1) / kLatTile * kLatTile;
@@ -570,6 +605,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     mbar_init(s_full + 8, 1);
     mbar_init(p_ready, 128);
     mbar_init(pv_done, 1);
+    mbar_init(x_full, 128);
+    mbar_init(x_full + 8, 128);
     mbar_fence_init();
   }
   if (warp == 5) {
@@ -583,6 +620,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  if (clustered) cluster_arrive();  // [0] this CTA's barriers exist
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(gen + lay.bars + 8 * 4 * kLatMaxSlots + 40);
   const uint32_t t_s = tmem + a.pairs * N;
   bool ok = true;
@@ -593,8 +631,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       bool waited = false;
       for (int t = 0, g = 0, r = 0; ok && t < n_tiles; ++t) {
         const int key = key0 + t * kLatTile;
-        for (int p = 0; p < a.pairs + a.rests; ++p) {
-          const bool pair = p < a.pairs;
+        for (int p = 0; p < pairs + rests; ++p) {
+          const bool pair = p < pairs;
           const int idx = pair ? g++ : r++, n = pair ? a.slots : a.rest_slots, slot = idx % n;
           if (idx >= n && !waited) {  // the rings are full: the queries' kernel has to be done by now anyway
             pdl_wait();
@@ -603,11 +641,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
           if (!mbar_wait(pair ? empty(slot) : rempty(slot), ((idx / n) & 1) ^ 1, a.err, DEVERR_ATTN_PRODUCER)) { ok = false; break; }
           if (pair) {
             mbar_expect_tx(full(slot), kLatPair);
-            tma_load_3d(base + slot * kLatPair, &tmap_c, full(slot), 128 * p, key, seq.slot);
-            tma_load_3d(base + slot * kLatPair + kLatBox, &tmap_c, full(slot), 128 * p + 64, key, seq.slot);
+            tma_load_3d(base + slot * kLatPair, &tmap_c, full(slot), 128 * (block0 + p), key, seq.slot);
+            tma_load_3d(base + slot * kLatPair + kLatBox, &tmap_c, full(slot), 128 * (block0 + p) + 64, key, seq.slot);
           } else {
             mbar_expect_tx(rfull(slot), kLatBox);
-            tma_load_3d(base + lay.rest + slot * kLatBox, &tmap_c, rfull(slot), 128 * a.pairs + 64 * (p - a.pairs), key, seq.slot);
+            tma_load_3d(base + lay.rest + slot * kLatBox, &tmap_c, rfull(slot), 128 * a.blocks + 64 * (p - pairs), key, seq.slot);
           }
         }
       }
@@ -615,35 +653,38 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     } else {
       pdl_wait();
     }
+    __syncwarp();
   } else if (warp == 5) {
     // ---------------- MMA issuer ----------------
     pdl_wait();
     if (lane == 0 && n_tiles > 0) {
-      const int boxes = 2 * a.pairs + a.rests;
-      mbar_expect_tx(q_full, boxes * N * 128);
-      for (int b = 0; b < boxes; ++b) tma_load_2d(base + lay.q + b * N * 128, &tmap_q, q_full, 64 * b, (seq.row0 - a.row_base) * a.H + row0);
+      mbar_expect_tx(q_full, (2 * pairs + rests) * N * 128);
+      const int q_row = (seq.row0 - a.row_base) * a.H + row0;
+      for (int b = 0; b < 2 * pairs + rests; ++b)
+        tma_load_2d(base + lay.q + b * N * 128, &tmap_q, q_full, b < 2 * pairs ? 128 * block0 + 64 * b : 128 * a.blocks + 64 * (b - 2 * pairs), q_row);
       constexpr uint32_t idesc_s = make_idesc_bf16(128, N, false, false), idesc_pv = make_idesc_bf16(128, N, true, false);
       const uint64_t q_desc = make_smem_desc_sw128(base + lay.q, 16, 1024), p_desc = make_smem_desc_sw128(base + lay.p, 16, 1024);
+      // cache rows: K-major for the scores; MN-major (64 values contiguous per key, 8 keys 1 KB apart, the next 64 values a box on) for O
+      const uint64_t c_desc0 = make_smem_desc_sw128(base, 16, 1024), v_desc0 = make_smem_desc_sw128(base, kLatBox, 1024);
       ok = mbar_wait(q_full, 0, a.err, DEVERR_ATTN_MMA);
       // one 64-dimension box of cache rows times the queries' box (dimensions beyond D are zero in both)
-      const uint64_t c_desc0 = make_smem_desc_sw128(base, 16, 1024), v_desc0 = make_smem_desc_sw128(base, kLatBox, 1024);
       auto box_products = [&](int offset, int box, uint32_t d, bool first) {
         umma_box(d, c_desc0 + (offset >> 4), q_desc + static_cast<uint64_t>(box * N * 8), idesc_s, first ? 0u : 1u);
       };
       auto scores = [&](int t) {
         const uint32_t d = t_s + (t & 1) * N;
-        for (int p = 0; ok && p < a.pairs; ++p) {
-          const int g = t * a.pairs + p, slot = g % a.slots;
+        for (int p = 0; ok && p < pairs; ++p) {
+          const int g = t * pairs + p, slot = g % a.slots;
           ok = mbar_wait(full(slot), (g / a.slots) & 1, a.err, DEVERR_ATTN_MMA);
           tc_fence_after();
           box_products(slot * kLatPair, 2 * p, d, p == 0);
-          if (128 * p + 64 < a.D) box_products(slot * kLatPair + kLatBox, 2 * p + 1, d, false);
+          if (128 * (block0 + p) + 64 < a.D) box_products(slot * kLatPair + kLatBox, 2 * p + 1, d, false);
         }
-        for (int r = 0; ok && r < a.rests; ++r) {
-          const int g = t * a.rests + r, slot = g % a.rest_slots;
+        for (int r = 0; ok && r < rests; ++r) {
+          const int g = t * rests + r, slot = g % a.rest_slots;
           ok = mbar_wait(rfull(slot), (g / a.rest_slots) & 1, a.err, DEVERR_ATTN_MMA);
           tc_fence_after();
-          box_products(lay.rest + slot * kLatBox, 2 * a.pairs + r, d, false);
+          box_products(lay.rest + slot * kLatBox, 2 * pairs + r, d, false);
           umma_commit(rempty(slot));
         }
         umma_commit(s_full + 8 * (t & 1));
@@ -651,9 +692,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       auto values = [&](int t) {
         if (ok) ok = mbar_wait(p_ready, t & 1, a.err, DEVERR_ATTN_MMA);
         tc_fence_after();
-        for (int i = 0; ok && i < a.pairs; ++i) {
-          const int slot = (t * a.pairs + i) % a.slots;
-          // MN-major: 64 values contiguous per key row, 8 keys 1 KB apart, the second 64 values one box further on; 16 keys = 2 KB
+        for (int i = 0; ok && i < pairs; ++i) {
+          const int slot = (t * pairs + i) % a.slots;
           umma_keys<N * 8>(tmem + i * N, v_desc0 + static_cast<uint64_t>(slot * (kLatPair >> 4)), p_desc, idesc_pv, t > 0 ? 1u : 0u);
           umma_commit(empty(slot));
         }
@@ -667,11 +707,21 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       }
     }
     __syncwarp();
+  }
+  if (warp >= 4) {
+    if (clustered) {
+      cluster_wait();    // [0]
+      cluster_arrive();  // [1]
+      cluster_wait();
+    }
   } else {
     // ---------------- softmax: thread = key of the tile (tensor-memory lane) ----------------
     pdl_wait();
+    if (clustered) cluster_wait();  // [0]
     const int r = threadIdx.x;
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
+    const uint32_t swap_peer = a.halves > 1 ? map_rank(base + lay.swap, rank ^ 1) : 0u, x_peer = a.halves > 1 ? map_rank(x_full, rank ^ 1) : 0u;
+    const float4* swap = reinterpret_cast<const float4*>(gen + lay.swap);
     const int min_lim = lim[0];  // rows are in token order
     float l[N];
 #pragma unroll
@@ -686,18 +736,35 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       float s[N];
       tmem_ld_cols<N>(t_s + lane_addr + (t & 1) * N, s);
       tc_fence_before();
+      if (a.halves > 1) {
+        // A buffer is written again two tiles on, after this thread has seen the peer's arrivals of the tile in between, which
+        // follow the peer's reads.
+        const uint32_t buf = (t & 1) * (N * 512);
+#pragma unroll
+        for (int n = 0; n < N; n += 4) st_cluster4(swap_peer + buf + (n / 4 * 128 + r) * 16, s[n], s[n + 1], s[n + 2], s[n + 3]);
+        mbar_arrive_remote(x_peer + 8 * (t & 1));
+        if (ok) ok = mbar_wait_cluster(x_full + 8 * (t & 1), (t >> 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
+#pragma unroll
+        for (int n = 0; n < N; n += 4) {
+          const float4 o = swap[(buf >> 4) + n / 4 * 128 + r];
+          s[n] += o.x;
+          s[n + 1] += o.y;
+          s[n + 2] += o.z;
+          s[n + 3] += o.w;
+        }
+      }
       if (k0 + kLatTile > key_end || k0 + kLatTile - 1 > min_lim) {
         const bool live = j < key_end;
 #pragma unroll
         for (int n = 0; n < N; ++n) s[n] = live && j <= lim[n] ? s[n] : -INFINITY;
         if (k0 + kLatTile > key_end && !live)
           // rows past the live length hold whatever the cache had; their weights are zero, but 0 * NaN is NaN inside the product
-          for (int i = 0; i < a.pairs; ++i) {
-            uint8_t* row = gen + ((t * a.pairs + i) % a.slots) * kLatPair + r * 128;
+          for (int i = 0; i < pairs; ++i) {
+            uint8_t* row = gen + ((t * pairs + i) % a.slots) * kLatPair + r * 128;
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
-              *reinterpret_cast<uint4*>(row + c * 16) = make_uint4(0, 0, 0, 0);
-              *reinterpret_cast<uint4*>(row + kLatBox + c * 16) = make_uint4(0, 0, 0, 0);
+              *reinterpret_cast<uint4*>(row + ((c ^ (r & 7)) << 4)) = make_uint4(0, 0, 0, 0);
+              *reinterpret_cast<uint4*>(row + kLatBox + ((c ^ (r & 7)) << 4)) = make_uint4(0, 0, 0, 0);
             }
           }
       }
@@ -727,7 +794,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
           if (ok) ok = mbar_wait(pv_done, (t - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);  // O^T is final for the tiles before
           __syncwarp();
           tc_fence_after();
-          for (int i = 0; i < a.pairs; ++i) {
+          for (int i = 0; i < pairs; ++i) {
             float o[N];
             tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
 #pragma unroll
@@ -761,15 +828,38 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       tc_fence_before();
       mbar_arrive(p_ready);
     }
-    // ---- this share's sums and output ----
+    // ---- maxima and sums of all shares, while the last product runs ----
     reduce_to<N, false>(l, red + warp * N);
-    if (n_tiles > 0 && ok) ok = mbar_wait(pv_done, (n_tiles - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
-    tc_fence_after();
     named_barrier_sync(1, 128);
-    if (r < N && n_tiles == 0) m_sh[r] = -INFINITY;
-    if (r < N) alpha_sh[r] = (red[r] + red[N + r]) + (red[2 * N + r] + red[3 * N + r]);
-    float* ob = reinterpret_cast<float*>(gen);  // [N][o_ld] over the slots, which no copy or product uses any more
-    for (int i = 0; i < a.pairs; ++i) {
+    if (r < N) {
+      const float mine = n_tiles > 0 ? m_sh[r] : -INFINITY, sum = (red[r] + red[N + r]) + (red[2 * N + r] + red[3 * N + r]);
+      if (clustered) {
+        const uint32_t at = smem_u32(share + r * 8 + split);
+        for (int i = 0; i < splits; ++i) st_cluster2(map_rank(at, i * a.halves + half), mine, sum);
+      } else {
+        share[r * 8] = make_float2(mine, sum);
+      }
+    }
+    __syncwarp();
+    if (clustered) cluster_arrive();  // [1] maxima and sums are out; the partial scores here have been read
+    if (n_tiles > 0 && ok) ok = mbar_wait(pv_done, (n_tiles - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
+    __syncwarp();
+    tc_fence_after();
+    if (clustered) cluster_wait();
+    named_barrier_sync(1, 128);
+    if (r < N) {
+      float mm = -INFINITY, sum = 0.0f;
+      for (int i = 0; i < splits; ++i) mm = fmaxf(mm, share[r * 8 + i].x);
+      for (int i = 0; i < splits; ++i) sum = fmaf(ex2(share[r * 8 + i].x - mm), share[r * 8 + i].y, sum);  // shares without keys hold -inf: 0
+      alpha_sh[r] = ex2(share[r * 8 + split].x - mm) / sum;
+    }
+    named_barrier_sync(1, 128);
+  }
+  // ---- columns: this half's values, `per` of them summed by each of its CTAs, from [share][row][column] ----
+  const int col0 = 128 * block0, cols = min(a.DV, col0 + 128 * pairs) - col0, per = ((cols + splits - 1) / splits + 3) & ~3;
+  if (warp < 4) {
+    const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
+    for (int i = 0; i < pairs; ++i) {
       float o[N];
       if (n_tiles > 0) {
         tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
@@ -777,13 +867,24 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
 #pragma unroll
         for (int n = 0; n < N; ++n) o[n] = 0.0f;
       }
+      const int c = i * 128 + static_cast<int>(threadIdx.x), to = c / per;
+      if (c < cols) {
+        const uint32_t local = base + lay.swap + (static_cast<uint32_t>(split * N) * per + (c - to * per)) * 4;
+        if (clustered) {
+          const uint32_t at = map_rank(local, to * a.halves + half);
 #pragma unroll
-      for (int n = 0; n < N; ++n) ob[n * a.o_ld + i * 128 + r] = o[n];
+          for (int n = 0; n < N; ++n) st_cluster(at + n * per * 4, o[n] * alpha_sh[n]);
+        } else {
+#pragma unroll
+          for (int n = 0; n < N; ++n) *reinterpret_cast<float*>(gen + (local - base) + n * per * 4) = o[n] * alpha_sh[n];
+        }
+      }
     }
     tc_fence_before();
   }
   pdl_trigger();
   __syncthreads();
+  if (clustered) cluster_arrive();  // [2]
   if (warp == 5) {
     if (*reinterpret_cast<volatile int*>(a.err) != 0) {  // a wait was given up: let copies and products in flight finish
       const uint64_t t0 = global_timer_ns();
@@ -792,48 +893,23 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tc_fence_after();
     tmem_dealloc(tmem, a.tmem_cols);
   }
-  if (splits > 1) cluster_sync();
-  // ---- merge: this CTA's slice of the columns, in fours ----
-  const uint32_t ob_a = base, m_a = smem_u32(m_sh), l_a = smem_u32(alpha_sh);
-  for (int i = threadIdx.x; i < n_rows * splits; i += kLatThreads) {
-    const int r = i / splits, sh = i - r * splits;
-    share[r * 8 + sh] = splits > 1 ? make_float2(ld_cluster(m_a + r * 4, sh), ld_cluster(l_a + r * 4, sh)) : make_float2(m_sh[r], alpha_sh[r]);
-  }
-  __syncthreads();
-  if (threadIdx.x < n_rows) {
-    float2* mine = share + threadIdx.x * 8;
-    float mm = -INFINITY, sum = 0.0f;
-    for (int i = 0; i < splits; ++i) mm = fmaxf(mm, mine[i].x);
-    for (int i = 0; i < splits; ++i) {
-      mine[i].x = ex2(mine[i].x - mm);  // shares without keys hold -inf: 0
-      sum = fmaf(mine[i].x, mine[i].y, sum);
-    }
-    for (int i = 0; i < splits; ++i) mine[i].x /= sum;
-  }
-  __syncthreads();
-  const int cols = a.DV / 4, per = (cols + splits - 1) / splits, c0 = split * per, width = min(per, cols - c0);
-  for (int i = threadIdx.x; i < n_rows * width; i += kLatThreads) {
-    const int r = i / width, c = c0 + (i - r * width);
-    const uint32_t addr = ob_a + static_cast<uint32_t>(r * a.o_ld + 4 * c) * 4;
-    float4 v[8];
-#pragma unroll
-    for (int sh = 0; sh < 8; ++sh)
-      if (sh < splits) v[sh] = splits > 1 ? ld_cluster4(addr, sh) : *reinterpret_cast<const float4*>(gen + (addr - base));
+  if (clustered) cluster_wait();
+  const int c0 = split * per, quads = min(per, cols - c0) / 4;
+  const float* sums = reinterpret_cast<const float*>(gen + lay.swap);
+  for (int i = threadIdx.x; i < n_rows * quads; i += kLatThreads) {
+    const int r = i / quads, c = 4 * (i - r * quads);
     float4 o = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll
-    for (int sh = 0; sh < 8; ++sh)
-      if (sh < splits) {
-        const float w = share[r * 8 + sh].x;
-        o.x = fmaf(w, v[sh].x, o.x);
-        o.y = fmaf(w, v[sh].y, o.y);
-        o.z = fmaf(w, v[sh].z, o.z);
-        o.w = fmaf(w, v[sh].w, o.w);
-      }
+    for (int k = 0; k < splits; ++k) {
+      const float4 v = *reinterpret_cast<const float4*>(sums + (k * N + r) * per + c);
+      o.x += v.x;
+      o.y += v.y;
+      o.z += v.z;
+      o.w += v.w;
+    }
     const int rr = row0 + r, tok = rr / a.H, h = rr - tok * a.H;
-    bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV;
-    *reinterpret_cast<uint2*>(orow + 4 * c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + col0 + c0;
+    *reinterpret_cast<uint2*>(orow + c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
   }
-  if (splits > 1) cluster_sync();  // no CTA leaves while others read its shared memory
 }
 
 constexpr int kLatSmemLimit = 232448;
@@ -847,34 +923,34 @@ int for_rows(int n, F&& f) {
 
 // Ring sizes for row tiles of n; false if the sizes do not fit.
 bool plan_tc(int n, int d, int dv, LatTcArgs& a, int& smem) {
-  a.pairs = (dv + 127) / 128;
-  a.rests = d > 128 * a.pairs ? (d - 128 * a.pairs + 63) / 64 : 0;
+  a.blocks = (dv + 127) / 128;
+  a.halves = a.blocks > 1 ? 2 : 1;
+  a.pairs = (a.blocks + a.halves - 1) / a.halves;
+  a.rests = d > 128 * a.blocks ? (d - 128 * a.blocks + 63) / 64 : 0;
+  a.rest_slots = a.rests;
   uint32_t cols = 32;
   while (static_cast<int>(cols) < (a.pairs + 2) * n) cols *= 2;
   a.tmem_cols = cols;
-  a.o_ld = 128 * a.pairs + 4;
-  if (cols > 512) return false;
-  for (int tiles = 2; tiles >= 1; --tiles) {  // two whole tiles in flight, or one and what else fits
-    a.rest_slots = tiles * a.rests;
-    a.slots = (kLatSmemLimit - lat_smem(n, a.pairs, a.rests, 0, a.rest_slots).total) / kLatPair;
-    if (a.slots > kLatMaxSlots) a.slots = kLatMaxSlots;
-    if (a.slots > 3 * a.pairs) a.slots = 3 * a.pairs;
-    a.ahead = tiles == 2;
-    if (a.slots >= tiles * a.pairs && a.rest_slots <= kLatMaxSlots && a.slots * kLatPair >= n * a.o_ld * 4) {
-      smem = lat_smem(n, a.pairs, a.rests, a.slots, a.rest_slots).total;
-      return true;
-    }
-  }
-  return false;
+  if (cols > 512 || a.rests > kLatMaxSlots) return false;
+  const int left = kLatSmemLimit - lat_smem(n, a.halves, a.pairs, a.rests, 0, a.rest_slots).total;
+  if (left < 0) return false;
+  a.slots = left / kLatPair;
+  if (a.slots > kLatMaxSlots) a.slots = kLatMaxSlots;
+  if (a.slots > 3 * a.pairs) a.slots = 3 * a.pairs;
+  a.ahead = a.slots >= 2 * a.pairs;
+  if (a.slots < a.pairs || (n > 32 && !a.ahead)) return false;
+  if (a.ahead && a.slots >= a.pairs * 2 && a.rests && left - a.slots * kLatPair >= a.rests * kLatBox && 2 * a.rests <= kLatMaxSlots) a.rest_slots *= 2;
+  smem = lat_smem(n, a.halves, a.pairs, a.rests, a.slots, a.rest_slots).total;
+  return true;
 }
 
 // Clusters of `size` CTAs that can be resident at once (per device, worked out once).
 template <int N>
 int max_clusters(int size, int smem) {
-  static std::atomic<int> known[9][64];  // [size][shared memory in 4 KB steps]
+  static std::atomic<int> known[17][64];  // [size][shared memory in 4 KB steps]; -1: none
   std::atomic<int>& k = known[size][(smem >> 12) & 63];
   int v = k.load(std::memory_order_relaxed);
-  if (v > 0) return v;
+  if (v != 0) return v;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(size, 1, 1);
   cfg.blockDim = dim3(kLatThreads);
@@ -887,7 +963,7 @@ int max_clusters(int size, int smem) {
   cfg.numAttrs = 1;
   if (cudaOccupancyMaxActiveClusters(&v, latent_attention_kernel<N>, &cfg) != cudaSuccess || v < 1) {
     cudaGetLastError();
-    v = 1;
+    v = -1;
   }
   k.store(v, std::memory_order_relaxed);
   return v;
@@ -946,6 +1022,8 @@ int latent_attention_prepare() {
     for_rows(n, [&](auto nn) {
       if (e == cudaSuccess)
         e = cudaFuncSetAttribute(latent_attention_kernel<decltype(nn)::value>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLatSmemLimit);
+      if (e == cudaSuccess)
+        e = cudaFuncSetAttribute(latent_attention_kernel<decltype(nn)::value>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
       return 0;
     });
   if (e != cudaSuccess) return static_cast<int>(e);
@@ -993,18 +1071,20 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
         // shares of the keys per row tile: fewest rounds of tiles over all waves of clusters
         const long long work = static_cast<long long>(tiles) * n_seqs;
         const int key_tiles = (a.max_len + kLatTile - 1) / kLatTile;
-        int splits = 1;
+        int splits = 0;
         long long best = -1;
-        for (int c = 1; c <= 8 && c <= key_tiles; ++c) {
-          const long long waves = (work + max_clusters<N>(c, smem) - 1) / max_clusters<N>(c, smem);
-          const long long cost = waves * ((key_tiles + c - 1) / c);
+        for (int c = 1; c <= 8 && (c == 1 || c <= key_tiles); ++c) {
+          const int fit = max_clusters<N>(c * t.halves, smem);
+          if (fit < 1) continue;
+          const long long cost = ((work + fit - 1) / fit) * ((key_tiles + c - 1) / c);
           if (best < 0 || cost < best) {
             best = cost;
             splits = c;
           }
         }
-        launch_kernel(latent_attention_kernel<N>, dim3(splits, tiles, n_seqs), dim3(kLatThreads), smem, st, static_cast<unsigned>(splits), mc, mq, t,
-                      seqs);
+        if (splits == 0) return static_cast<int>(TEENY_ERR_BAD_ARG);
+        launch_kernel(latent_attention_kernel<N>, dim3(splits * t.halves, tiles, n_seqs), dim3(kLatThreads), smem, st,
+                      static_cast<unsigned>(splits * t.halves), mc, mq, t, seqs);
         return static_cast<int>(cudaGetLastError());
       });
     }
