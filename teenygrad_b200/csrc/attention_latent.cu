@@ -346,27 +346,28 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
   }
 }
 
-// Absorbed attention on the tensor cores (tcgen05).  A row tile is N consecutive (token, head) rows of one entry; a cluster shares
-// it: each CTA takes a share of the keys and, where there are 256 or more value dimensions, one of two halves of the dimensions,
-// so that two 128-key tiles fit into its shared memory.  The rows are the N side of both products (a few query heads waste
-// nothing), and the cache rows, loaded once per tile, are the A operand of both:
-//   S^T [128 keys, N]   = C [128 keys, D] Q^T          C K-major, Q in shared memory for the whole walk
-//   O^T [DV, N]        += C^T [DV, 128 keys] P^T       the same shared memory read MN-major; one M = 128 product per 128 values
-// Tensor memory: O^T in blocks of N columns per 128 values, two S^T buffers of N columns.
-//   warp 4   TMA producer: ring of 32 KB slots, each 128 keys x 128 value dimensions (two [128 keys][64 d] boxes); the dimensions
-//            behind the values (the rotated part) travel in a ring of single boxes.  A slot is free again when its product with P
-//            has completed, so the next tile's loads follow the current one's products block by block.  Starts before the
-//            dependency wait: only the queries come from the kernel in front of this one.
+// Absorbed attention on the tensor cores (tcgen05).  CTA = N consecutive (token, head) rows of one entry x one share of its keys;
+// the CTAs of a cluster hold the shares of one row tile.  The rows are the N side of both products (a few query heads waste
+// nothing), and the cache rows, loaded once per 64-key tile, are the A operand of both.  M = 128 holds 64 keys twice: a slot of
+// shared memory is 128 dimensions of the tile as two boxes [64 keys][64 d], one behind the other, which the two products read as
+//   S^T [2 x 64 keys, 2 N] += [boxes] [Q of the first box's dimensions; Q of the second's]^T     (K-major)
+//            the upper half of the lanes means something in the first N columns, the lower half in the others: their sum is S^T
+//   O^T [128 values, N]    += [boxes]^T P^T                                                    (the same memory MN-major)
+// so that two tiles are in shared memory at a time and no product is idle in half of its rows.
+// Tensor memory: O^T in blocks of N columns per 128 values, two S^T buffers of 2 N columns.
+//   warp 4   TMA producer: ring of 16 KB slots.  A slot is free again when its last product has completed (with P; for dimensions
+//            behind the values with Q), so the loads follow the products slot by slot.  Starts before the dependency wait: only
+//            the queries come from the kernel in front of this one.
 //   warp 5   allocates tensor memory, loads the queries, issues the MMAs (one thread); S of tile t + 1 goes ahead of P V of tile t
 //            where the ring holds two tiles.
-//   warps 0-3  thread = key in a tile: its N scores out of tensor memory -- with halved dimensions plus the partial scores of the
-//            other half's CTA, exchanged through distributed shared memory, after which both do the same --, mask, weights
-//            against the rows' running maxima (shared memory), sums in registers, weights as bf16 into shared memory ([row][key],
-//            the B operand).  The maxima only move when some score exceeds its row's by more than 2^8 (one vote per tile); then
-//            the tile's maxima are reduced across the lanes and O^T is rescaled.
-// At the end the shares tell one another their maxima and sums (while the last product runs), every CTA scales its O^T by its
-// weights and stores each column into the shared memory of the CTA that sums this column over the shares.
-constexpr int kLatTile = 128, kLatPair = 32768, kLatBox = 16384, kLatMaxSlots = 12, kLatThreads = 192;
+//   warps 0-3  thread = tensor-memory lane: its lane's N partial scores, half of which it trades with the thread of the same key in
+//            the other half (shared memory), so that each ends with N / 2 scores of its key; mask, weights against the rows'
+//            running maxima (shared memory), sums in registers, weights as bf16 into shared memory ([row][key], the B operand).
+//            The maxima only move when some score exceeds its row's by more than 2^8 (one vote per tile); then the tile's maxima
+//            are reduced across the lanes and O^T is rescaled.
+// At the end the shares tell one another their maxima and sums, every CTA scales its O^T by its weights and stores each column
+// into the shared memory of the CTA that sums this column over the shares.
+constexpr int kLatTile = 64, kLatSlot = 16384, kLatBox = 8192, kLatMaxSlots = 24, kLatThreads = 192;
 constexpr float kLatGrow = 8.0f;  // log2 units
 
 struct LatTcArgs {
@@ -374,28 +375,25 @@ struct LatTcArgs {
   long long ldo;
   int row_base;        // step row that row 0 of q and out stands for
   int H, D, DV;
-  int halves;          // CTAs that share the dimensions: 1 or 2
-  int blocks;          // 128-dimension blocks that hold values
-  int pairs, rests;    // of a tile: slots with values of one CTA (at most); single boxes behind the values (the last half's)
-  int slots, rest_slots, ahead;
+  int blocks;          // 128-dimension slots of a tile that hold values
+  int tile_slots;      // slots of a tile
+  int slots, ahead;    // of the ring; whether it holds two tiles
+  int sums_at;         // byte offset over the slots of what a CTA sums in the end
   uint32_t tmem_cols;
   float scale_log2;
   int* err;
 };
 
 struct LatSmem {  // byte offsets
-  int rest, q, p, swap, bars, stats, total;
+  int q, p, swap, bars, stats, total;
 };
-__host__ __device__ inline LatSmem lat_smem(int n, int halves, int pairs, int rests, int slots, int rest_slots) {
+__host__ __device__ inline LatSmem lat_smem(int n, int tile_slots, int slots) {
   LatSmem s;
-  s.rest = slots * kLatPair;
-  s.q = s.rest + rest_slots * kLatBox;
-  s.p = s.q + (2 * pairs + rests) * n * 128;
-  // partial scores from the other half, two tiles of [n / 4][128 keys] float4; in the end the columns to be summed here
-  s.swap = s.p + 2 * n * 128;
-  const int scores = halves > 1 ? 2 * n * 128 * 4 : 0, sums = n * (128 * pairs + 32) * 4;
-  s.bars = s.swap + (scores > sums ? scores : sums);
-  s.stats = s.bars + 8 * (4 * kLatMaxSlots + 8);
+  s.q = slots * kLatSlot;               // [boxes][n rows][64 d]
+  s.p = s.q + 2 * tile_slots * n * 128; // [n rows][64 keys]
+  s.swap = s.p + n * 128;               // partial scores between the lane halves: [n / 4][64 keys] float4
+  s.bars = s.swap + n * 64 * 4;
+  s.stats = s.bars + 8 * (2 * kLatMaxSlots + 8);
   s.total = s.stats + 4 * (8 + 16) * n + 1024;
   return s;
 }
@@ -407,17 +405,16 @@ __device__ __forceinline__ uint32_t map_rank(uint32_t local_addr, uint32_t rank)
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(local_addr), "r"(rank));
   return r;
 }
-__device__ __forceinline__ void st_cluster(uint32_t addr, float v) { asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
 __device__ __forceinline__ void st_cluster2(uint32_t addr, float x, float y) {
   asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(x), "f"(y) : "memory");
 }
-__device__ __forceinline__ void st_cluster4(uint32_t addr, float x, float y, float z, float w) {
-  asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(x), "f"(y), "f"(z), "f"(w) : "memory");
+// This CTA's shared memory -> another's (or its own), completion bytes on a barrier there.
+__device__ __forceinline__ void bulk_copy_cluster(uint32_t dst, uint32_t src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.shared::cta.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "r"(src), "r"(bytes), "r"(bar)
+               : "memory");
 }
-// This thread's stores to the other CTA's shared memory, then its arrival on a barrier there; mbar_wait_cluster sees them.
-__device__ __forceinline__ void mbar_arrive_remote(uint32_t addr) {
-  asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(addr) : "memory");
-}
+// mbar_wait for data that came from another CTA
 __device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity, int* err, int code) {
   uint64_t t0 = 0;
 #pragma unroll 1
@@ -485,15 +482,16 @@ __device__ __forceinline__ void tmem_st_cols(uint32_t addr, const float (&v)[N])
     }
   }
 }
-// Reduction of W columns over the warp's lanes, halving the columns a lane holds at every step; lane i ends with column i % W.
+// Reduction of W columns (8, 16 or 32) over the warp's lanes, halving the columns a lane holds at every step; lane i ends with
+// column i % W.
 template <int W, bool MAX>
 __device__ __forceinline__ float reduce_columns(float (&v)[W]) {
   const int lane = threadIdx.x & 31;
   auto op = [](float a, float b) { return MAX ? fmaxf(a, b) : a + b; };
-  if (W == 16) {
 #pragma unroll
-    for (int i = 0; i < 16; ++i) v[i] = op(v[i], __shfl_xor_sync(0xffffffffu, v[i], 16));
-  }
+  for (int w = 16; w >= W; w >>= 1)
+#pragma unroll
+    for (int i = 0; i < W; ++i) v[i] = op(v[i], __shfl_xor_sync(0xffffffffu, v[i], w));
 #pragma unroll
   for (int w = W / 2; w > 0; w >>= 1)
 #pragma unroll
@@ -504,49 +502,57 @@ __device__ __forceinline__ float reduce_columns(float (&v)[W]) {
     }
   return v[0];
 }
-// ... of all N columns, into dst[N] of this warp
-template <int N, bool MAX>
-__device__ __forceinline__ void reduce_to(const float (&v)[N], float* dst) {
-  constexpr int W = N < 32 ? N : 32;
-  const int lane = threadIdx.x & 31;
+// ... into dst[W] of this warp
+template <int W, bool MAX>
+__device__ __forceinline__ void reduce_to(const float (&v)[W], float* dst) {
+  float t[W];
 #pragma unroll
-  for (int i = 0; i < N / W; ++i) {
-    float t[W];
-#pragma unroll
-    for (int e = 0; e < W; ++e) t[e] = v[W * i + e];
-    const float r = reduce_columns<W, MAX>(t);
-    if (lane < W) dst[W * i + lane] = r;
-  }
+  for (int e = 0; e < W; ++e) t[e] = v[e];
+  const float r = reduce_columns<W, MAX>(t);
+  if ((threadIdx.x & 31) < W) dst[threadIdx.x & 31] = r;
 }
 
-// Straight-line runs of products: a lone thread with address arithmetic in between issues a product only every ~100 cycles.
-// Four K-steps over one K-major box of each operand (32 bytes along the rows per step).
-__device__ __forceinline__ void umma_box(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate_first) {
+// Whether the barrier's phase of this parity is complete, for the whole warp; does not wait.
+__device__ __forceinline__ bool mbar_test_wait(uint32_t bar, uint32_t parity) {
+  uint32_t done;
   asm volatile(
-      "{\n\t.reg .pred p, t;\n\t.reg .b64 x, y;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t setp.eq.b32 t, %3, %3;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
-      "add.u64 x, %1, 2;\n\t add.u64 y, %2, 2;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 4;\n\t add.u64 y, %2, 4;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 6;\n\t add.u64 y, %2, 6;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t}"
-      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate_first)
+      "{\n\t.reg .pred p;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(done) : "r"(bar), "r"(parity) : "memory");
+  return __all_sync(0xffffffffu, done != 0);
+}
+// Four K-steps of a product as straight-line code, the operands' addresses A_STEP and B_STEP (16-byte units) further at each.  The
+// whole warp comes here and the one lane with `lead` issues: in uniform control flow descriptors and counters stay in uniform
+// registers (a lone lane in a divergent branch issues a product only every ~100 cycles).
+template <int A_STEP, int B_STEP>
+__device__ __forceinline__ void umma_x4(uint32_t lead, uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate_first) {
+  asm volatile(
+      "{\n\t.reg .pred e, p, t;\n\t.reg .b64 x, y;\n\t"
+      "setp.ne.b32 e, %5, 0;\n\t setp.ne.b32 p, %4, 0;\n\t setp.eq.b32 t, %3, %3;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
+      "add.u64 x, %1, %6;\n\t add.u64 y, %2, %9;\n\t @e tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, %7;\n\t add.u64 y, %2, %10;\n\t @e tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
+      "add.u64 x, %1, %8;\n\t add.u64 y, %2, %11;\n\t @e tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate_first), "r"(lead), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP), "n"(B_STEP),
+        "n"(2 * B_STEP), "n"(3 * B_STEP)
       : "memory");
 }
-// The eight K-steps of 128 keys: A MN-major (2 KB per 16 keys), B K-major in two boxes BOX 16-byte units apart.
-template <int BOX>
-__device__ __forceinline__ void umma_keys(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate_first) {
+// 128 dimensions of a tile into a slot: two boxes [64 keys][64 d].
+__device__ __forceinline__ void load_slot(uint32_t lead, uint32_t dst, const CUtensorMap* m, uint32_t bar, int d, int key, int seq) {
   asm volatile(
-      "{\n\t.reg .pred p, t;\n\t.reg .b64 x, y;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t setp.eq.b32 t, %3, %3;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
-      "add.u64 x, %1, 128;\n\t add.u64 y, %2, 2;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 256;\n\t add.u64 y, %2, 4;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 384;\n\t add.u64 y, %2, 6;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 512;\n\t add.u64 y, %2, %5;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 640;\n\t add.u64 y, %2, %6;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 768;\n\t add.u64 y, %2, %7;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t"
-      "add.u64 x, %1, 896;\n\t add.u64 y, %2, %8;\n\t tcgen05.mma.cta_group::1.kind::f16 [%0], x, y, %3, t;\n\t}"
-      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate_first), "n"(BOX), "n"(BOX + 2), "n"(BOX + 4), "n"(BOX + 6)
+      "{\n\t.reg .pred e;\n\t.reg .b32 x, y;\n\t setp.ne.b32 e, %6, 0;\n\t add.u32 x, %0, %8;\n\t add.u32 y, %3, 64;\n\t"
+      "@e mbarrier.arrive.expect_tx.shared::cta.b64 _, [%2], %7;\n\t"
+      "@e cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n\t"
+      "@e cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [x], [%1, {y, %4, %5}], [%2];\n\t}"
+      ::"r"(dst), "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(d), "r"(key), "r"(seq), "r"(lead), "n"(kLatSlot), "n"(kLatBox)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_lead(uint32_t lead, uint32_t bar) {
+  asm volatile(
+      "{\n\t.reg .pred e;\n\t setp.ne.b32 e, %1, 0;\n\t"
+      "@e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+      ::"r"(bar), "r"(lead)
       : "memory");
 }
 
@@ -554,6 +560,7 @@ template <int N>
 __global__ void __launch_bounds__(kLatThreads, 1)
 latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid_constant__ CUtensorMap tmap_q, const LatTcArgs a,
                         const SeqDesc* __restrict__ seqs) {
+  constexpr int HN = N / 2;  // rows whose weights a thread works out
   extern __shared__ uint8_t lat_raw[];
   const SeqDesc seq = seqs[blockIdx.z];  // written well before the kernel in front of this one
   const int row0 = blockIdx.y * N, n_rows = min(N, seq.len * a.H - row0);
@@ -563,27 +570,22 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   }
   const uint32_t base = (smem_u32(lat_raw) + 1023u) & ~1023u;
   uint8_t* gen = lat_raw + (base - smem_u32(lat_raw));
-  const LatSmem lay = lat_smem(N, a.halves, a.pairs, a.rests, a.slots, a.rest_slots);
+  const LatSmem lay = lat_smem(N, a.tile_slots, a.slots);
   const uint32_t bar0 = base + lay.bars;
   auto full = [&](int i) { return bar0 + 8u * i; };
   auto empty = [&](int i) { return bar0 + 8u * (kLatMaxSlots + i); };
-  auto rfull = [&](int i) { return bar0 + 8u * (2 * kLatMaxSlots + i); };
-  auto rempty = [&](int i) { return bar0 + 8u * (3 * kLatMaxSlots + i); };
-  const uint32_t misc = bar0 + 8u * 4 * kLatMaxSlots;
-  const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40, x_full = misc + 48;  // two s_full, two x_full
+  const uint32_t misc = bar0 + 8u * 2 * kLatMaxSlots;
+  const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40;  // two s_full
   float* m_sh = reinterpret_cast<float*>(gen + lay.stats);  // [N] running maxima, log2 domain
   float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally this share's weights
   float* up_sh = alpha_sh + N;                              // [N] by how much the maxima just rose
-  float* red = up_sh + N;                                   // [4][N]
+  float* red = up_sh + N;                                   // [4][HN] of each warp
   int* lim = reinterpret_cast<int*>(red + 4 * N);           // [N] last key each row sees
   float2* share = reinterpret_cast<float2*>(lim + N);       // [N][8] maximum and sum of every share
 
-  const int rank = blockIdx.x, half = rank % a.halves, split = rank / a.halves, splits = gridDim.x / a.halves;
-  const bool clustered = gridDim.x > 1;
-  const int block0 = half * a.pairs;                                     // this CTA's blocks of 128 values ...
-  const int pairs = min(a.pairs, a.blocks - block0);
-  const int rests = half == a.halves - 1 ? a.rests : 0;                  // ... and single boxes behind the values
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int split = blockIdx.x, splits = gridDim.x;
+  const bool clustered = splits > 1;
+  const int warp = threadIdx.x >> 5;
   const int L = seq.pos + (row0 + n_rows - 1) / a.H + 1;  // keys the tile's last row sees
   const int span = ((L + splits - 1) / splits + kLatTile - 1) / kLatTile * kLatTile;
   const int key0 = split * span, key_end = min(L, key0 + span);
@@ -596,17 +598,12 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       mbar_init(full(i), 1);
       mbar_init(empty(i), 1);
     }
-    for (int i = 0; i < a.rest_slots; ++i) {
-      mbar_init(rfull(i), 1);
-      mbar_init(rempty(i), 1);
-    }
     mbar_init(q_full, 1);
     mbar_init(s_full, 1);
     mbar_init(s_full + 8, 1);
     mbar_init(p_ready, 128);
     mbar_init(pv_done, 1);
-    mbar_init(x_full, 128);
-    mbar_init(x_full + 8, 128);
+    mbar_init(misc + 48, 1);
     mbar_fence_init();
   }
   if (warp == 5) {
@@ -620,159 +617,158 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  if (clustered) cluster_arrive();  // [0] this CTA's barriers exist
-  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(gen + lay.bars + 8 * 4 * kLatMaxSlots + 40);
-  const uint32_t t_s = tmem + a.pairs * N;
+  if (clustered) cluster_arrive();  // [0] this CTA is there
+  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(gen + lay.bars + 8 * 2 * kLatMaxSlots + 40);
+  const uint32_t t_s = tmem + a.blocks * N;
   bool ok = true;
 
   if (warp == 4) {
     // ---------------- producer ----------------
-    if (lane == 0) {
-      bool waited = false;
-      for (int t = 0, g = 0, r = 0; ok && t < n_tiles; ++t) {
-        const int key = key0 + t * kLatTile;
-        for (int p = 0; p < pairs + rests; ++p) {
-          const bool pair = p < pairs;
-          const int idx = pair ? g++ : r++, n = pair ? a.slots : a.rest_slots, slot = idx % n;
-          if (idx >= n && !waited) {  // the rings are full: the queries' kernel has to be done by now anyway
+    const uint32_t lead = elect_one() ? 1u : 0u;
+    bool waited = false;
+    int slot = 0, key = key0;
+    uint32_t round = 0;
+    for (int t = 0; ok && t < n_tiles; ++t, key += kLatTile)
+      for (int p = 0; ok && p < a.tile_slots; ++p) {
+        if (round > 0) {
+          if (!waited) {  // the ring is full: the queries' kernel has to be done by now anyway
             pdl_wait();
             waited = true;
           }
-          if (!mbar_wait(pair ? empty(slot) : rempty(slot), ((idx / n) & 1) ^ 1, a.err, DEVERR_ATTN_PRODUCER)) { ok = false; break; }
-          if (pair) {
-            mbar_expect_tx(full(slot), kLatPair);
-            tma_load_3d(base + slot * kLatPair, &tmap_c, full(slot), 128 * (block0 + p), key, seq.slot);
-            tma_load_3d(base + slot * kLatPair + kLatBox, &tmap_c, full(slot), 128 * (block0 + p) + 64, key, seq.slot);
-          } else {
-            mbar_expect_tx(rfull(slot), kLatBox);
-            tma_load_3d(base + lay.rest + slot * kLatBox, &tmap_c, rfull(slot), 128 * a.blocks + 64 * (p - pairs), key, seq.slot);
-          }
+          ok = mbar_wait(empty(slot), (round & 1) ^ 1, a.err, DEVERR_ATTN_PRODUCER);
+          __syncwarp();
+        }
+        if (ok) load_slot(lead, base + slot * kLatSlot, &tmap_c, full(slot), 128 * p, key, seq.slot);
+        if (++slot == a.slots) {
+          slot = 0;
+          ++round;
         }
       }
-      if (!waited) pdl_wait();
-    } else {
-      pdl_wait();
-    }
+    if (!waited) pdl_wait();
     __syncwarp();
   } else if (warp == 5) {
     // ---------------- MMA issuer ----------------
     pdl_wait();
-    if (lane == 0 && n_tiles > 0) {
-      mbar_expect_tx(q_full, (2 * pairs + rests) * N * 128);
-      const int q_row = (seq.row0 - a.row_base) * a.H + row0;
-      for (int b = 0; b < 2 * pairs + rests; ++b)
-        tma_load_2d(base + lay.q + b * N * 128, &tmap_q, q_full, b < 2 * pairs ? 128 * block0 + 64 * b : 128 * a.blocks + 64 * (b - 2 * pairs), q_row);
-      constexpr uint32_t idesc_s = make_idesc_bf16(128, N, false, false), idesc_pv = make_idesc_bf16(128, N, true, false);
+    if (n_tiles > 0) {
+      const uint32_t lead = elect_one() ? 1u : 0u;
+      if (lead) {
+        mbar_expect_tx(q_full, 2 * a.tile_slots * N * 128);
+        for (int b = 0; b < 2 * a.tile_slots; ++b)
+          tma_load_2d(base + lay.q + b * N * 128, &tmap_q, q_full, 64 * b, (seq.row0 - a.row_base) * a.H + row0);
+      }
+      __syncwarp();
+      constexpr uint32_t idesc_s = make_idesc_bf16(128, 2 * N, false, false), idesc_pv = make_idesc_bf16(128, N, true, false);
       const uint64_t q_desc = make_smem_desc_sw128(base + lay.q, 16, 1024), p_desc = make_smem_desc_sw128(base + lay.p, 16, 1024);
       // cache rows: K-major for the scores; MN-major (64 values contiguous per key, 8 keys 1 KB apart, the next 64 values a box on) for O
-      const uint64_t c_desc0 = make_smem_desc_sw128(base, 16, 1024), v_desc0 = make_smem_desc_sw128(base, kLatBox, 1024);
+      const uint64_t c_desc = make_smem_desc_sw128(base, 16, 1024), v_desc = make_smem_desc_sw128(base, kLatBox, 1024);
       ok = mbar_wait(q_full, 0, a.err, DEVERR_ATTN_MMA);
-      // one 64-dimension box of cache rows times the queries' box (dimensions beyond D are zero in both)
-      auto box_products = [&](int offset, int box, uint32_t d, bool first) {
-        umma_box(d, c_desc0 + (offset >> 4), q_desc + static_cast<uint64_t>(box * N * 8), idesc_s, first ? 0u : 1u);
-      };
-      auto scores = [&](int t) {
-        const uint32_t d = t_s + (t & 1) * N;
-        for (int p = 0; ok && p < pairs; ++p) {
-          const int g = t * pairs + p, slot = g % a.slots;
-          ok = mbar_wait(full(slot), (g / a.slots) & 1, a.err, DEVERR_ATTN_MMA);
+      // Whichever product can go next: a slot of S as soon as it is loaded (S of a tile at most one ahead of P V, whose weights
+      // show that its buffer has been read; not ahead at all in a ring of less than two tiles), else P V as soon as its weights are
+      // there.
+      int s_tile = 0, s_part = 0, s_slot = 0, v_tile = 0, v_slot = 0;
+      uint32_t s_round = 0, spins = 0;
+      uint64_t t0 = 0;
+      while (ok && v_tile < n_tiles) {
+        if (s_tile < n_tiles && s_tile <= v_tile + (a.ahead ? 1 : 0) && mbar_test_wait(full(s_slot), s_round & 1)) {
           tc_fence_after();
-          box_products(slot * kLatPair, 2 * p, d, p == 0);
-          if (128 * (block0 + p) + 64 < a.D) box_products(slot * kLatPair + kLatBox, 2 * p + 1, d, false);
-        }
-        for (int r = 0; ok && r < rests; ++r) {
-          const int g = t * rests + r, slot = g % a.rest_slots;
-          ok = mbar_wait(rfull(slot), (g / a.rest_slots) & 1, a.err, DEVERR_ATTN_MMA);
+          // (32 bytes along the rows per step; dimensions beyond D are zero on both sides)
+          umma_x4<2, 2>(lead, t_s + (s_tile & 1) * 2 * N, c_desc + static_cast<uint64_t>(s_slot * (kLatSlot >> 4)),
+                        q_desc + static_cast<uint64_t>(s_part * 2 * N * 8), idesc_s, s_part > 0 ? 1u : 0u);
+          if (s_part >= a.blocks) umma_commit_lead(lead, empty(s_slot));
+          if (++s_part == a.tile_slots) {
+            umma_commit_lead(lead, s_full + 8 * (s_tile & 1));
+            s_part = 0;
+            ++s_tile;
+          }
+          if (++s_slot == a.slots) {
+            s_slot = 0;
+            ++s_round;
+          }
+          spins = 0;
+        } else if (mbar_test_wait(p_ready, v_tile & 1)) {
           tc_fence_after();
-          box_products(lay.rest + slot * kLatBox, 2 * pairs + r, d, false);
-          umma_commit(rempty(slot));
+          for (int i = 0; i < a.tile_slots; ++i) {
+            if (i < a.blocks) {  // 16 keys = 2 KB per step
+              umma_x4<128, 2>(lead, tmem + i * N, v_desc + static_cast<uint64_t>(v_slot * (kLatSlot >> 4)), p_desc, idesc_pv, v_tile > 0 ? 1u : 0u);
+              umma_commit_lead(lead, empty(v_slot));
+            }
+            if (++v_slot == a.slots) v_slot = 0;
+          }
+          umma_commit_lead(lead, pv_done);
+          ++v_tile;
+          spins = 0;
+        } else if ((++spins & 0xff) == 0) {  // (the limits of mbar_wait)
+          const uint64_t now = global_timer_ns();
+          if (spins == 0x100) t0 = now;
+          else if (*reinterpret_cast<volatile int*>(a.err) != 0) ok = false;
+          else if (now - t0 > kWaitLimitNs) {
+            atomicCAS(a.err, 0, static_cast<int>(DEVERR_ATTN_MMA));
+            ok = false;
+          }
         }
-        umma_commit(s_full + 8 * (t & 1));
-      };
-      auto values = [&](int t) {
-        if (ok) ok = mbar_wait(p_ready, t & 1, a.err, DEVERR_ATTN_MMA);
-        tc_fence_after();
-        for (int i = 0; ok && i < pairs; ++i) {
-          const int slot = (t * pairs + i) % a.slots;
-          umma_keys<N * 8>(tmem + i * N, v_desc0 + static_cast<uint64_t>(slot * (kLatPair >> 4)), p_desc, idesc_pv, t > 0 ? 1u : 0u);
-          umma_commit(empty(slot));
-        }
-        umma_commit(pv_done);
-      };
-      if (ok) scores(0);
-      for (int t = 0; ok && t < n_tiles; ++t) {
-        if (a.ahead && t + 1 < n_tiles) scores(t + 1);
-        values(t);
-        if (!a.ahead && ok && t + 1 < n_tiles) scores(t + 1);
+        ok = __all_sync(0xffffffffu, ok);
       }
     }
     __syncwarp();
-  }
-  if (warp >= 4) {
-    if (clustered) {
-      cluster_wait();    // [0]
-      cluster_arrive();  // [1]
-      cluster_wait();
-    }
   } else {
-    // ---------------- softmax: thread = key of the tile (tensor-memory lane) ----------------
+    // ---------------- softmax: thread = tensor-memory lane = (half, key of the tile) ----------------
     pdl_wait();
-    if (clustered) cluster_wait();  // [0]
-    const int r = threadIdx.x;
+    const int r = threadIdx.x, key = r & 63, half = r >> 6;
+    const int n0 = half * HN;  // first of the rows whose weights this thread works out
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    const uint32_t swap_peer = a.halves > 1 ? map_rank(base + lay.swap, rank ^ 1) : 0u, x_peer = a.halves > 1 ? map_rank(x_full, rank ^ 1) : 0u;
-    const float4* swap = reinterpret_cast<const float4*>(gen + lay.swap);
+    float4* swap = reinterpret_cast<float4*>(gen + lay.swap);
     const int min_lim = lim[0];  // rows are in token order
-    float l[N];
+    float l[HN];
 #pragma unroll
-    for (int n = 0; n < N; ++n) l[n] = 0.0f;
-    uint8_t* pw = gen + lay.p + (r >> 6) * (N * 128) + (r & 7) * 2;  // this key's column of the weights
-    const int pc = (r & 63) >> 3;
+    for (int n = 0; n < HN; ++n) l[n] = 0.0f;
+    uint8_t* pw = gen + lay.p + (key & 7) * 2 + n0 * 128;  // this key's column of the weights
+    const int pc = key >> 3;
     for (int t = 0; t < n_tiles; ++t) {
-      const int k0 = key0 + t * kLatTile, j = k0 + r;
+      const int k0 = key0 + t * kLatTile, j = k0 + key;
       if (ok) ok = mbar_wait(s_full + 8 * (t & 1), (t >> 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
       __syncwarp();
       tc_fence_after();
-      float s[N];
-      tmem_ld_cols<N>(t_s + lane_addr + (t & 1) * N, s);
-      tc_fence_before();
-      if (a.halves > 1) {
-        // A buffer is written again two tiles on, after this thread has seen the peer's arrivals of the tile in between, which
-        // follow the peer's reads.
-        const uint32_t buf = (t & 1) * (N * 512);
+      float s[HN];
+      {
+        float x[N];
+        tmem_ld_cols<N>(t_s + lane_addr + (t & 1) * 2 * N + half * N, x);
+        tc_fence_before();
+        // the other half's rows to the thread of the same key there; mine from it (everyone's reads are behind the vote below)
 #pragma unroll
-        for (int n = 0; n < N; n += 4) st_cluster4(swap_peer + buf + (n / 4 * 128 + r) * 16, s[n], s[n + 1], s[n + 2], s[n + 3]);
-        mbar_arrive_remote(x_peer + 8 * (t & 1));
-        if (ok) ok = mbar_wait_cluster(x_full + 8 * (t & 1), (t >> 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
-#pragma unroll
-        for (int n = 0; n < N; n += 4) {
-          const float4 o = swap[(buf >> 4) + n / 4 * 128 + r];
-          s[n] += o.x;
-          s[n + 1] += o.y;
-          s[n + 2] += o.z;
-          s[n + 3] += o.w;
+        for (int n = 0; n < HN; n += 4) {
+          const int give = half ? n : HN + n;
+          swap[give / 4 * 64 + key] = half ? make_float4(x[n], x[n + 1], x[n + 2], x[n + 3])
+                                           : make_float4(x[HN + n], x[HN + n + 1], x[HN + n + 2], x[HN + n + 3]);
         }
+#pragma unroll
+        for (int n = 0; n < HN; ++n) s[n] = half ? x[HN + n] : x[n];
+      }
+      named_barrier_sync(1, 128);
+#pragma unroll
+      for (int n = 0; n < HN; n += 4) {
+        const float4 o = swap[(n0 + n) / 4 * 64 + key];
+        s[n] += o.x;
+        s[n + 1] += o.y;
+        s[n + 2] += o.z;
+        s[n + 3] += o.w;
       }
       if (k0 + kLatTile > key_end || k0 + kLatTile - 1 > min_lim) {
         const bool live = j < key_end;
 #pragma unroll
-        for (int n = 0; n < N; ++n) s[n] = live && j <= lim[n] ? s[n] : -INFINITY;
+        for (int n = 0; n < HN; ++n) s[n] = live && j <= lim[n0 + n] ? s[n] : -INFINITY;
         if (k0 + kLatTile > key_end && !live)
           // rows past the live length hold whatever the cache had; their weights are zero, but 0 * NaN is NaN inside the product
-          for (int i = 0; i < pairs; ++i) {
-            uint8_t* row = gen + ((t * pairs + i) % a.slots) * kLatPair + r * 128;
+          for (int i = 0; i < a.blocks; ++i) {  // (in the last tile only)
+            uint8_t* row = gen + ((t * a.tile_slots + i) % a.slots) * kLatSlot + half * kLatBox + key * 128;
 #pragma unroll
-            for (int c = 0; c < 8; ++c) {
-              *reinterpret_cast<uint4*>(row + ((c ^ (r & 7)) << 4)) = make_uint4(0, 0, 0, 0);
-              *reinterpret_cast<uint4*>(row + kLatBox + ((c ^ (r & 7)) << 4)) = make_uint4(0, 0, 0, 0);
-            }
+            for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(row + ((c ^ (key & 7)) << 4)) = make_uint4(0, 0, 0, 0);
           }
       }
       // scores relative to the running maxima (first tile: to zero)
       bool grow = t == 0;
 #pragma unroll
-      for (int n = 0; n < N; n += 4) {
-        const float4 m4 = *reinterpret_cast<const float4*>(m_sh + n);
+      for (int n = 0; n < HN; n += 4) {
+        const float4 m4 = *reinterpret_cast<const float4*>(m_sh + n0 + n);
         s[n] = fmaf(s[n], a.scale_log2, -m4.x);
         s[n + 1] = fmaf(s[n + 1], a.scale_log2, -m4.y);
         s[n + 2] = fmaf(s[n + 2], a.scale_log2, -m4.z);
@@ -780,10 +776,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
         grow = grow || fmaxf(fmaxf(s[n], s[n + 1]), fmaxf(s[n + 2], s[n + 3])) > kLatGrow;
       }
       if (any128(grow)) {
-        reduce_to<N, true>(s, red + warp * N);
+        reduce_to<HN, true>(s, red + warp * HN);
         named_barrier_sync(1, 128);
         if (r < N) {
-          float up = fmaxf(fmaxf(red[r], red[N + r]), fmaxf(red[2 * N + r], red[3 * N + r]));
+          const float* mine = red + (r / HN) * 2 * HN + r % HN;
+          float up = fmaxf(mine[0], mine[HN]);
           up = t == 0 ? fmaxf(up, -1e30f) : fmaxf(up, 0.0f);  // finite also for rows that see none of this share's keys
           m_sh[r] += up;
           up_sh[r] = up;
@@ -794,7 +791,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
           if (ok) ok = mbar_wait(pv_done, (t - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);  // O^T is final for the tiles before
           __syncwarp();
           tc_fence_after();
-          for (int i = 0; i < pairs; ++i) {
+          for (int i = 0; i < a.blocks; ++i) {
             float o[N];
             tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
 #pragma unroll
@@ -805,14 +802,14 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
           tc_fence_before();
         }
 #pragma unroll
-        for (int n = 0; n < N; ++n) {
-          l[n] *= alpha_sh[n];
-          s[n] -= up_sh[n];
+        for (int n = 0; n < HN; ++n) {
+          l[n] *= alpha_sh[n0 + n];
+          s[n] -= up_sh[n0 + n];
         }
       }
-      uint32_t pk[N / 2];
+      uint32_t pk[HN / 2];
 #pragma unroll
-      for (int n = 0; n < N; n += 2) {
+      for (int n = 0; n < HN; n += 2) {
         const float p0 = ex2(s[n]), p1 = ex2(s[n + 1]);
         l[n] += p0;
         l[n + 1] += p1;
@@ -822,31 +819,42 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
         if (ok) ok = mbar_wait(pv_done, (t - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);  // the weights of the tile before have been read
       }
 #pragma unroll
-      for (int n = 0; n < N; ++n)
+      for (int n = 0; n < HN; ++n)  // (n0 is a multiple of 8: row n0 + n has n's swizzle)
         *reinterpret_cast<uint16_t*>(pw + n * 128 + ((pc ^ (n & 7)) << 4)) = static_cast<uint16_t>(n & 1 ? pk[n / 2] >> 16 : pk[n / 2] & 0xffffu);
       fence_proxy_async_smem();
       tc_fence_before();
       mbar_arrive(p_ready);
     }
-    // ---- maxima and sums of all shares, while the last product runs ----
-    reduce_to<N, false>(l, red + warp * N);
+    // ---- maxima and sums of all shares ----
+    reduce_to<HN, false>(l, red + warp * HN);
     named_barrier_sync(1, 128);
+    if (clustered) cluster_wait();  // [0]
     if (r < N) {
-      const float mine = n_tiles > 0 ? m_sh[r] : -INFINITY, sum = (red[r] + red[N + r]) + (red[2 * N + r] + red[3 * N + r]);
+      const float* part = red + (r / HN) * 2 * HN + r % HN;
+      const float mine = n_tiles > 0 ? m_sh[r] : -INFINITY, sum = part[0] + part[HN];
       if (clustered) {
         const uint32_t at = smem_u32(share + r * 8 + split);
-        for (int i = 0; i < splits; ++i) st_cluster2(map_rank(at, i * a.halves + half), mine, sum);
+        for (int i = 0; i < splits; ++i) st_cluster2(map_rank(at, i), mine, sum);
       } else {
         share[r * 8] = make_float2(mine, sum);
       }
     }
-    __syncwarp();
-    if (clustered) cluster_arrive();  // [1] maxima and sums are out; the partial scores here have been read
     if (n_tiles > 0 && ok) ok = mbar_wait(pv_done, (n_tiles - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
     __syncwarp();
     tc_fence_after();
-    if (clustered) cluster_wait();
+  }
+  if (clustered) {  // [1] maxima and sums are there; nobody's slots are in use any more
+    if (warp >= 4) cluster_wait();  // [0]
+    cluster_arrive();
+    cluster_wait();
+  }
+  // ---- columns: every CTA's scaled O^T as [column][row] over its slots (rows padded: no bank conflicts), `per` columns at a time
+  // copied to the CTA that sums them, which takes them as [share][column][row] behind its own ----
+  const int per = ((a.DV + splits - 1) / splits + 7) & ~7;
+  constexpr int RL = N + 4;
+  if (warp < 4) {
     named_barrier_sync(1, 128);
+    const int r = threadIdx.x;
     if (r < N) {
       float mm = -INFINITY, sum = 0.0f;
       for (int i = 0; i < splits; ++i) mm = fmaxf(mm, share[r * 8 + i].x);
@@ -854,12 +862,14 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       alpha_sh[r] = ex2(share[r * 8 + split].x - mm) / sum;
     }
     named_barrier_sync(1, 128);
-  }
-  // ---- columns: this half's values, `per` of them summed by each of its CTAs, from [share][row][column] ----
-  const int col0 = 128 * block0, cols = min(a.DV, col0 + 128 * pairs) - col0, per = ((cols + splits - 1) / splits + 3) & ~3;
-  if (warp < 4) {
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    for (int i = 0; i < pairs; ++i) {
+    float w[N];
+#pragma unroll
+    for (int n = 0; n < N; n += 4) {
+      const float4 w4 = *reinterpret_cast<const float4*>(alpha_sh + n);
+      w[n] = w4.x; w[n + 1] = w4.y; w[n + 2] = w4.z; w[n + 3] = w4.w;
+    }
+    for (int i = 0; i < a.blocks; ++i) {
       float o[N];
       if (n_tiles > 0) {
         tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
@@ -867,49 +877,55 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
 #pragma unroll
         for (int n = 0; n < N; ++n) o[n] = 0.0f;
       }
-      const int c = i * 128 + static_cast<int>(threadIdx.x), to = c / per;
-      if (c < cols) {
-        const uint32_t local = base + lay.swap + (static_cast<uint32_t>(split * N) * per + (c - to * per)) * 4;
-        if (clustered) {
-          const uint32_t at = map_rank(local, to * a.halves + half);
+      if (i * 128 + r < a.DV) {
+        float4* dst = reinterpret_cast<float4*>(gen + (i * 128 + r) * RL * 4);
 #pragma unroll
-          for (int n = 0; n < N; ++n) st_cluster(at + n * per * 4, o[n] * alpha_sh[n]);
-        } else {
-#pragma unroll
-          for (int n = 0; n < N; ++n) *reinterpret_cast<float*>(gen + (local - base) + n * per * 4) = o[n] * alpha_sh[n];
-        }
+        for (int n = 0; n < N; n += 4) dst[n / 4] = make_float4(o[n] * w[n], o[n + 1] * w[n + 1], o[n + 2] * w[n + 2], o[n + 3] * w[n + 3]);
       }
     }
     tc_fence_before();
+    if (clustered) fence_proxy_async_smem();
+  }
+  const uint32_t sums_full = misc + 48;
+  const int c0 = split * per, mine = max(0, min(per, a.DV - c0));  // columns summed here
+  if (clustered && threadIdx.x == 128 && mine > 0) mbar_expect_tx(sums_full, splits * mine * RL * 4);
+  __syncthreads();
+  const uint32_t taken = a.sums_at;  // where a CTA takes the shares
+  if (clustered && threadIdx.x < splits) {
+    const int to = threadIdx.x, n_cols = max(0, min(per, a.DV - to * per));
+    if (n_cols > 0)
+      bulk_copy_cluster(map_rank(base + taken + static_cast<uint32_t>(split * n_cols * RL) * 4, to), base + static_cast<uint32_t>(to * per * RL) * 4,
+                        n_cols * RL * 4, map_rank(sums_full, to));
   }
   pdl_trigger();
-  __syncthreads();
-  if (clustered) cluster_arrive();  // [2]
+  if (clustered && mine > 0) ok = mbar_wait_cluster(sums_full, 0, a.err, DEVERR_ATTN_SOFTMAX) && ok;
+  __syncwarp();
+  if (clustered) cluster_arrive();  // [2] the copies to this CTA have left their sources
   if (warp == 5) {
     if (*reinterpret_cast<volatile int*>(a.err) != 0) {  // a wait was given up: let copies and products in flight finish
       const uint64_t t0 = global_timer_ns();
       while (global_timer_ns() - t0 < 2000000ull) __nanosleep(1000);
     }
+    __syncwarp();
     tc_fence_after();
     tmem_dealloc(tmem, a.tmem_cols);
   }
-  if (clustered) cluster_wait();
-  const int c0 = split * per, quads = min(per, cols - c0) / 4;
-  const float* sums = reinterpret_cast<const float*>(gen + lay.swap);
-  for (int i = threadIdx.x; i < n_rows * quads; i += kLatThreads) {
-    const int r = i / quads, c = 4 * (i - r * quads);
-    float4 o = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  // thread = (row, eight columns); rows side by side in a warp
+  const float* sums = reinterpret_cast<const float*>(gen + (clustered ? taken : 0));
+  for (int i = threadIdx.x; i < mine / 8 * N; i += kLatThreads) {
+    const int r = i % N, c = i / N * 8;
+    if (r >= n_rows) continue;
+    float o[8] = {};
     for (int k = 0; k < splits; ++k) {
-      const float4 v = *reinterpret_cast<const float4*>(sums + (k * N + r) * per + c);
-      o.x += v.x;
-      o.y += v.y;
-      o.z += v.z;
-      o.w += v.w;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] += sums[(k * mine + c + e) * RL + r];
     }
     const int rr = row0 + r, tok = rr / a.H, h = rr - tok * a.H;
-    bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + col0 + c0;
-    *reinterpret_cast<uint2*>(orow + c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + c0;
+    st8(orow + c, o);
   }
+  __syncwarp();
+  if (clustered) cluster_wait();
 }
 
 constexpr int kLatSmemLimit = 232448;
@@ -921,33 +937,32 @@ int for_rows(int n, F&& f) {
   return f(std::integral_constant<int, 64>());
 }
 
-// Ring sizes for row tiles of n; false if the sizes do not fit.
+// Ring size for row tiles of n; false if the sizes do not fit.
 bool plan_tc(int n, int d, int dv, LatTcArgs& a, int& smem) {
   a.blocks = (dv + 127) / 128;
-  a.halves = a.blocks > 1 ? 2 : 1;
-  a.pairs = (a.blocks + a.halves - 1) / a.halves;
-  a.rests = d > 128 * a.blocks ? (d - 128 * a.blocks + 63) / 64 : 0;
-  a.rest_slots = a.rests;
+  a.tile_slots = (d + 127) / 128;
   uint32_t cols = 32;
-  while (static_cast<int>(cols) < (a.pairs + 2) * n) cols *= 2;
+  while (static_cast<int>(cols) < (a.blocks + 4) * n) cols *= 2;
   a.tmem_cols = cols;
-  if (cols > 512 || a.rests > kLatMaxSlots) return false;
-  const int left = kLatSmemLimit - lat_smem(n, a.halves, a.pairs, a.rests, 0, a.rest_slots).total;
-  if (left < 0) return false;
-  a.slots = left / kLatPair;
+  if (cols > 512) return false;
+  const int left = kLatSmemLimit - lat_smem(n, a.tile_slots, 0).total;
+  a.slots = left > 0 ? left / kLatSlot : 0;
   if (a.slots > kLatMaxSlots) a.slots = kLatMaxSlots;
-  if (a.slots > 3 * a.pairs) a.slots = 3 * a.pairs;
-  a.ahead = a.slots >= 2 * a.pairs;
-  if (a.slots < a.pairs || (n > 32 && !a.ahead)) return false;
-  if (a.ahead && a.slots >= a.pairs * 2 && a.rests && left - a.slots * kLatPair >= a.rests * kLatBox && 2 * a.rests <= kLatMaxSlots) a.rest_slots *= 2;
-  smem = lat_smem(n, a.halves, a.pairs, a.rests, a.slots, a.rest_slots).total;
-  return true;
+  if (a.slots > 3 * a.tile_slots) a.slots = 3 * a.tile_slots;
+  // in the end over the slots: O^T [values][n + 4] and the shares' columns (no more than values + 8 per share)
+  a.sums_at = (n + 4) * dv * 4;
+  const int bytes = a.sums_at + (n + 4) * (dv + 64) * 4;
+  if (a.slots * kLatSlot < bytes) a.slots = (bytes + kLatSlot - 1) / kLatSlot;
+  a.ahead = a.slots >= 2 * a.tile_slots;
+  if (a.slots < a.tile_slots || a.slots > kLatMaxSlots || (n > 32 && !a.ahead)) return false;
+  smem = lat_smem(n, a.tile_slots, a.slots).total;
+  return smem <= kLatSmemLimit;
 }
 
 // Clusters of `size` CTAs that can be resident at once (per device, worked out once).
 template <int N>
 int max_clusters(int size, int smem) {
-  static std::atomic<int> known[17][64];  // [size][shared memory in 4 KB steps]; -1: none
+  static std::atomic<int> known[9][64];  // [size][shared memory in 4 KB steps]; -1: none
   std::atomic<int>& k = known[size][(smem >> 12) & 63];
   int v = k.load(std::memory_order_relaxed);
   if (v != 0) return v;
@@ -1022,8 +1037,6 @@ int latent_attention_prepare() {
     for_rows(n, [&](auto nn) {
       if (e == cudaSuccess)
         e = cudaFuncSetAttribute(latent_attention_kernel<decltype(nn)::value>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLatSmemLimit);
-      if (e == cudaSuccess)
-        e = cudaFuncSetAttribute(latent_attention_kernel<decltype(nn)::value>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
       return 0;
     });
   if (e != cudaSuccess) return static_cast<int>(e);
@@ -1041,7 +1054,7 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
   }
   const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache);
   const int rows = longest * a.H;
-  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (a.ldo & 3) == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 7) == 0 &&
+  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (a.ldo & 7) == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 15) == 0 &&
       a.ldq == static_cast<long long>(a.H) * a.D) {
     LatTcArgs t{};
     int smem = 0, n = rows <= 16 ? 16 : (rows <= 32 ? 32 : 64);
@@ -1074,7 +1087,7 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
         int splits = 0;
         long long best = -1;
         for (int c = 1; c <= 8 && (c == 1 || c <= key_tiles); ++c) {
-          const int fit = max_clusters<N>(c * t.halves, smem);
+          const int fit = max_clusters<N>(c, smem);
           if (fit < 1) continue;
           const long long cost = ((work + fit - 1) / fit) * ((key_tiles + c - 1) / c);
           if (best < 0 || cost < best) {
@@ -1083,8 +1096,8 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
           }
         }
         if (splits == 0) return static_cast<int>(TEENY_ERR_BAD_ARG);
-        launch_kernel(latent_attention_kernel<N>, dim3(splits * t.halves, tiles, n_seqs), dim3(kLatThreads), smem, st,
-                      static_cast<unsigned>(splits * t.halves), mc, mq, t, seqs);
+        launch_kernel(latent_attention_kernel<N>, dim3(splits, tiles, n_seqs), dim3(kLatThreads), smem, st, static_cast<unsigned>(splits), mc, mq, t,
+                      seqs);
         return static_cast<int>(cudaGetLastError());
       });
     }
