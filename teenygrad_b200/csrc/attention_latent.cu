@@ -159,15 +159,10 @@ __device__ __forceinline__ void rotate_tail(const HeadLinear& a, int h, int r0, 
   const int base = a.seqs[0].row0;  // of row 0 of x and y
   for (int idx = threadIdx.x; idx < n * half; idx += blockDim.x) {
     const int r = r0 + idx / half, d = idx % half;
-    int pos = 0;
-    for (int s = 0; s < a.n_seqs; ++s) {
-      const SeqDesc q = a.seqs[s];
-      const int i = r + base - q.row0;
-      if (i >= 0 && i < q.len) {
-        pos = q.pos + i;
-        break;
-      }
-    }
+    int e = min(r, a.n_seqs - 1);  // entries lie in row order, each with at least one row
+    SeqDesc q = a.seqs[e];
+    while (q.row0 - base > r) q = a.seqs[--e];
+    const int pos = q.pos + r + base - q.row0;
     float sn, cs;
     sincosf(static_cast<float>(pos) * a.inv_freq[d], &sn, &cs);
     sn *= a.rot_scale;
@@ -365,8 +360,8 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
 //            running maxima (shared memory), sums in registers, weights as bf16 into shared memory ([row][key], the B operand).
 //            The maxima only move when some score exceeds its row's by more than 2^8 (one vote per tile); then the tile's maxima
 //            are reduced across the lanes and O^T is rescaled.
-// At the end the shares tell one another their maxima and sums, every CTA scales its O^T by its weights and stores each column
-// into the shared memory of the CTA that sums this column over the shares.
+// At the end the shares tell one another their maxima and sums, every CTA scales its O^T by its weights, rounds it to bf16 (the
+// exchange is what the end takes longest for) and copies the columns to the CTAs that sum them over the shares.
 constexpr int kLatTile = 64, kLatSlot = 16384, kLatBox = 8192, kLatMaxSlots = 24, kLatThreads = 192;
 constexpr float kLatGrow = 8.0f;  // log2 units
 
@@ -611,7 +606,6 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tmem_relinquish();
   }
   if (threadIdx.x < N) {
-    m_sh[threadIdx.x] = 0.0f;
     lim[threadIdx.x] = seq.pos + min(row0 + static_cast<int>(threadIdx.x), row0 + n_rows - 1) / a.H;
   }
   tc_fence_before();
@@ -764,8 +758,16 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
             for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(row + ((c ^ (key & 7)) << 4)) = make_uint4(0, 0, 0, 0);
           }
       }
-      // scores relative to the running maxima (first tile: to zero)
-      bool grow = t == 0;
+      if (t == 0) {
+        // a first maximum: the score of the share's first key (a row that does not see it sees none); finite
+        if (key == 0) {
+#pragma unroll
+          for (int n = 0; n < HN; ++n) m_sh[n0 + n] = fmaxf(s[n] * a.scale_log2, -1e30f);
+        }
+        named_barrier_sync(1, 128);
+      }
+      // scores relative to the running maxima
+      bool grow = false;
 #pragma unroll
       for (int n = 0; n < HN; n += 4) {
         const float4 m4 = *reinterpret_cast<const float4*>(m_sh + n0 + n);
@@ -780,11 +782,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
         named_barrier_sync(1, 128);
         if (r < N) {
           const float* mine = red + (r / HN) * 2 * HN + r % HN;
-          float up = fmaxf(mine[0], mine[HN]);
-          up = t == 0 ? fmaxf(up, -1e30f) : fmaxf(up, 0.0f);  // finite also for rows that see none of this share's keys
+          const float up = fmaxf(fmaxf(mine[0], mine[HN]), 0.0f);
           m_sh[r] += up;
           up_sh[r] = up;
-          alpha_sh[r] = t == 0 ? 0.0f : ex2(-up);
+          alpha_sh[r] = ex2(-up);
         }
         named_barrier_sync(1, 128);
         if (t > 0) {
@@ -851,7 +852,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   // ---- columns: every CTA's scaled O^T as [column][row] over its slots (rows padded: no bank conflicts), `per` columns at a time
   // copied to the CTA that sums them, which takes them as [share][column][row] behind its own ----
   const int per = ((a.DV + splits - 1) / splits + 7) & ~7;
-  constexpr int RL = N + 4;
+  constexpr int RL = N + 8;  // in bf16 elements
   if (warp < 4) {
     named_barrier_sync(1, 128);
     const int r = threadIdx.x;
@@ -878,9 +879,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
         for (int n = 0; n < N; ++n) o[n] = 0.0f;
       }
       if (i * 128 + r < a.DV) {
-        float4* dst = reinterpret_cast<float4*>(gen + (i * 128 + r) * RL * 4);
+        uint4* dst = reinterpret_cast<uint4*>(gen + (i * 128 + r) * RL * 2);
 #pragma unroll
-        for (int n = 0; n < N; n += 4) dst[n / 4] = make_float4(o[n] * w[n], o[n + 1] * w[n + 1], o[n + 2] * w[n + 2], o[n + 3] * w[n + 3]);
+        for (int n = 0; n < N; n += 8)
+          dst[n / 8] = make_uint4(pack_bf16x2(o[n] * w[n], o[n + 1] * w[n + 1]), pack_bf16x2(o[n + 2] * w[n + 2], o[n + 3] * w[n + 3]),
+                                  pack_bf16x2(o[n + 4] * w[n + 4], o[n + 5] * w[n + 5]), pack_bf16x2(o[n + 6] * w[n + 6], o[n + 7] * w[n + 7]));
       }
     }
     tc_fence_before();
@@ -888,14 +891,14 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   }
   const uint32_t sums_full = misc + 48;
   const int c0 = split * per, mine = max(0, min(per, a.DV - c0));  // columns summed here
-  if (clustered && threadIdx.x == 128 && mine > 0) mbar_expect_tx(sums_full, splits * mine * RL * 4);
+  if (clustered && threadIdx.x == 128 && mine > 0) mbar_expect_tx(sums_full, splits * mine * RL * 2);
   __syncthreads();
   const uint32_t taken = a.sums_at;  // where a CTA takes the shares
   if (clustered && threadIdx.x < splits) {
     const int to = threadIdx.x, n_cols = max(0, min(per, a.DV - to * per));
     if (n_cols > 0)
-      bulk_copy_cluster(map_rank(base + taken + static_cast<uint32_t>(split * n_cols * RL) * 4, to), base + static_cast<uint32_t>(to * per * RL) * 4,
-                        n_cols * RL * 4, map_rank(sums_full, to));
+      bulk_copy_cluster(map_rank(base + taken + static_cast<uint32_t>(split * n_cols * RL) * 2, to), base + static_cast<uint32_t>(to * per * RL) * 2,
+                        n_cols * RL * 2, map_rank(sums_full, to));
   }
   pdl_trigger();
   if (clustered && mine > 0) ok = mbar_wait_cluster(sums_full, 0, a.err, DEVERR_ATTN_SOFTMAX) && ok;
@@ -910,19 +913,25 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tc_fence_after();
     tmem_dealloc(tmem, a.tmem_cols);
   }
-  // thread = (row, eight columns); rows side by side in a warp
-  const float* sums = reinterpret_cast<const float*>(gen + (clustered ? taken : 0));
-  for (int i = threadIdx.x; i < mine / 8 * N; i += kLatThreads) {
-    const int r = i % N, c = i / N * 8;
+  // thread = (two rows, eight columns); rows side by side in a warp
+  const uint32_t* sums = reinterpret_cast<const uint32_t*>(gen + (clustered ? taken : 0));
+  for (int i = threadIdx.x; i < mine / 8 * (N / 2); i += kLatThreads) {
+    const int r = i % (N / 2) * 2, c = i / (N / 2) * 8;
     if (r >= n_rows) continue;
-    float o[8] = {};
+    float o[2][8] = {};
     for (int k = 0; k < splits; ++k) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] += sums[(k * mine + c + e) * RL + r];
+      for (int e = 0; e < 8; ++e) {
+        const uint32_t v = sums[((k * mine + c + e) * RL + r) >> 1];
+        o[0][e] += bf16_lo(v);
+        o[1][e] += bf16_hi(v);
+      }
     }
-    const int rr = row0 + r, tok = rr / a.H, h = rr - tok * a.H;
-    bf16* orow = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + c0;
-    st8(orow + c, o);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int rr = row0 + r + e, tok = rr / a.H, h = rr - tok * a.H;
+      if (r + e < n_rows) st8(a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + c0 + c, o[e]);
+    }
   }
   __syncwarp();
   if (clustered) cluster_wait();
@@ -949,9 +958,9 @@ bool plan_tc(int n, int d, int dv, LatTcArgs& a, int& smem) {
   a.slots = left > 0 ? left / kLatSlot : 0;
   if (a.slots > kLatMaxSlots) a.slots = kLatMaxSlots;
   if (a.slots > 3 * a.tile_slots) a.slots = 3 * a.tile_slots;
-  // in the end over the slots: O^T [values][n + 4] and the shares' columns (no more than values + 8 per share)
-  a.sums_at = (n + 4) * dv * 4;
-  const int bytes = a.sums_at + (n + 4) * (dv + 64) * 4;
+  // in the end over the slots: O^T [values][n + 8] and the shares' columns (no more than values + 8 per share)
+  a.sums_at = (n + 8) * dv * 2;
+  const int bytes = a.sums_at + (n + 8) * (dv + 64) * 2;
   if (a.slots * kLatSlot < bytes) a.slots = (bytes + kLatSlot - 1) / kLatSlot;
   a.ahead = a.slots >= 2 * a.tile_slots;
   if (a.slots < a.tile_slots || a.slots > kLatMaxSlots || (n > 32 && !a.ahead)) return false;
