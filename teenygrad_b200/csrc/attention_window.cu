@@ -141,21 +141,22 @@ __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormR
     }
   }
   const int partner = (lane - sub) + (sub < step ? sub + step : (sub < 2 * step ? sub - step : sub));
-  const bool in_head = d0 < a.D;
+  // heads of q that are not normed change in place in their rotated dimensions only
+  const bool in_k = d0 < a.D, in_q = a.q_w ? in_k : d0 < a.rot_dims;
   for (int base = 0; base < heads; base += per * kRopeTasks) {
     uint4 raw[kRopeTasks];
 #pragma unroll
     for (int t = 0; t < kRopeTasks; ++t) {
       const int u = base + t * per + h0;
       raw[t] = make_uint4(0u, 0u, 0u, 0u);
-      if (u < heads && in_head) raw[t] = *reinterpret_cast<const uint4*>((u < a.Hq ? qr + u * a.D : kr + (u - a.Hq) * a.D) + d0);
+      if (u < heads && (u < a.Hq ? in_q : in_k)) raw[t] = *reinterpret_cast<const uint4*>((u < a.Hq ? qr + u * a.D : kr + (u - a.Hq) * a.D) + d0);
     }
     if (base == 0) __syncthreads();  // the angles
 #pragma unroll
     for (int t = 0; t < kRopeTasks; ++t) {
       const int u = base + t * per + h0;
       if (base + t * per >= heads) break;  // uniform over the CTA
-      const bool is_q = u < a.Hq;
+      const bool is_q = u < a.Hq, in_head = is_q ? in_q : in_k;
       const uint32_t rw[4] = {raw[t].x, raw[t].y, raw[t].z, raw[t].w};
       float x[8], sq = 0.0f;
 #pragma unroll
@@ -506,7 +507,7 @@ int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, 
                           reinterpret_cast<uintptr_t>(a.k_w) | reinterpret_cast<uintptr_t>(a.v) | reinterpret_cast<uintptr_t>(a.v_first);
   if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && a.rot_dims % 16 == 0 && ((a.ldq | a.ldkr | a.ldk | a.ldv | a.ldvf) & 7) == 0 && (bases & 15) == 0) {
     int lph = 1;
-    while (lph * 8 < a.D) lph *= 2;
+    while (lph * 8 < (a.Hkv == 0 && !a.q_w ? a.rot_dims : a.D)) lph *= 2;
     launch_kernel(head_norm_rope_vec_kernel, grid, block, 0, st, 1, a, seqs, lph);
     return static_cast<int>(cudaGetLastError());
   }
