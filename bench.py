@@ -913,11 +913,13 @@ def molitar_kernels(size, peaks, timed, graph_timed):
         q1, k, v, D ** -0.5, one, softcap=30.0, sink=sink, gate=g1, out=o1, scratch=scratch)) for k, v in kvs]), "hbm", 2.0 * n * G * S * D * 2,
         "attention, decode")
     del kvs
-    caches = [bf(n, S, R + RD) for _ in range(copies + 2)]
     ql, ol = bf(n, H, R + RD), bf(n, H, R)
-    row("latent attention, absorbed, decode", graph_timed([(lambda c=c: ops.latent_attention(ql, c, R, KD ** -0.5, one[0], 1, out=ol)) for c in caches]),
-        "hbm", 2.0 * n * S * (R + RD), "attention, decode")
-    del caches
+    for length, name in ((S, ""), (4 * S, f", context {4 * S}")):
+        at = ops.seq_table([(b, length - 1, b, 1) for b in range(n)])
+        caches = [bf(n, length, R + RD) for _ in range(copies + 2 if length == S else 3)]
+        row("latent attention, absorbed, decode" + name, graph_timed([(lambda c=c, at=at: ops.latent_attention(ql, c, R, KD ** -0.5, at, 1, out=ol))
+                                                                       for c in caches]), "hbm", 2.0 * n * length * (R + RD), "attention, decode" + name)
+        del caches
     qh, vo = bf(n, H, KD), bf(n, H, V)
     many = max(8, (300 << 20) // (2 * H * R * lat["dim"]))
     ws = [bf(H, R, lat["dim"]) for _ in range(many)]
@@ -932,11 +934,14 @@ def molitar_kernels(size, peaks, timed, graph_timed):
     del ws
     qwen3_kernels(z, B, S, row, timed)
     from teenygrad_b200.ops import flash_attn_decode
-    kvs = [(bf(n, G, S, D), bf(n, G, S, D)) for _ in range(copies)]
     qd = bf(n, H, 1, D)
     od = torch.empty_like(qd)
-    row("attention, decode", graph_timed([(lambda k=k, v=v: flash_attn_decode(qd, k, v, S, D ** -0.5, out=od, scratch=scratch[0])) for k, v in kvs]),
-        "hbm", 2.0 * n * G * S * D * 2)
+    for length, name in ((S, ""), (4 * S, f", context {4 * S}")):
+        kvs = [(bf(n, G, length, D), bf(n, G, length, D)) for _ in range(copies if length == S else 2)]
+        sc = torch.empty(lib.teeny_attn_decode_scratch_bytes(n, H, D, length), dtype=torch.uint8, device="cuda")
+        row("attention, decode" + name, graph_timed([(lambda k=k, v=v, length=length: flash_attn_decode(qd, k, v, length, D ** -0.5, out=od, scratch=sc))
+                                                     for k, v in kvs]), "hbm", 2.0 * n * G * length * D * 2)
+        del kvs
     return rows
 
 

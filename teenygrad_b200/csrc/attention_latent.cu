@@ -460,6 +460,24 @@ __device__ __forceinline__ void tmem_ld_cols(uint32_t addr, float (&v)[N]) {
       for (int e = 0; e < 32; ++e) v[32 * i + e] = __uint_as_float(t[i][e]);
   }
 }
+// Two such blocks, side by side.
+template <int N>
+__device__ __forceinline__ void tmem_ld_cols2(uint32_t addr, float (&v)[2][N]) {
+  if constexpr (N == 32) {
+    uint32_t t[2][32];
+    tmem_ld_32x32(addr, t[0]);
+    tmem_ld_32x32(addr + 32, t[1]);
+    tmem_wait_ld();
+#pragma unroll
+    for (int e = 0; e < 32; ++e) {
+      v[0][e] = __uint_as_float(t[0][e]);
+      v[1][e] = __uint_as_float(t[1][e]);
+    }
+  } else {
+    tmem_ld_cols<N>(addr, v[0]);
+    tmem_ld_cols<N>(addr + N, v[1]);
+  }
+}
 template <int N>
 __device__ __forceinline__ void tmem_st_cols(uint32_t addr, const float (&v)[N]) {
   if constexpr (N == 16) {
@@ -541,6 +559,13 @@ __device__ __forceinline__ void load_slot(uint32_t lead, uint32_t dst, const CUt
       "@e cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n\t"
       "@e cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [x], [%1, {y, %4, %5}], [%2];\n\t}"
       ::"r"(dst), "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(d), "r"(key), "r"(seq), "r"(lead), "n"(kLatSlot), "n"(kLatBox)
+      : "memory");
+}
+__device__ __forceinline__ void load_queries(uint32_t lead, uint32_t dst, const CUtensorMap* m, uint32_t bar, int d, int row) {
+  asm volatile(
+      "{\n\t.reg .pred e;\n\t setp.ne.b32 e, %5, 0;\n\t"
+      "@e cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n\t}"
+      ::"r"(dst), "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(d), "r"(row), "r"(lead)
       : "memory");
 }
 __device__ __forceinline__ void umma_commit_lead(uint32_t lead, uint32_t bar) {
@@ -645,12 +670,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     pdl_wait();
     if (n_tiles > 0) {
       const uint32_t lead = elect_one() ? 1u : 0u;
-      if (lead) {
-        mbar_expect_tx(q_full, 2 * a.tile_slots * N * 128);
-        for (int b = 0; b < 2 * a.tile_slots; ++b)
-          tma_load_2d(base + lay.q + b * N * 128, &tmap_q, q_full, 64 * b, (seq.row0 - a.row_base) * a.H + row0);
-      }
+      if (lead) mbar_expect_tx(q_full, 2 * a.tile_slots * N * 128);
       __syncwarp();
+      const int q_row = (seq.row0 - a.row_base) * a.H + row0;
+      for (int b = 0; b < 2 * a.tile_slots; ++b) load_queries(lead, base + lay.q + b * N * 128, &tmap_q, q_full, 64 * b, q_row);
       constexpr uint32_t idesc_s = make_idesc_bf16(128, 2 * N, false, false), idesc_pv = make_idesc_bf16(128, N, true, false);
       const uint64_t q_desc = make_smem_desc_sw128(base + lay.q, 16, 1024), p_desc = make_smem_desc_sw128(base + lay.p, 16, 1024);
       // cache rows: K-major for the scores; MN-major (64 values contiguous per key, 8 keys 1 KB apart, the next 64 values a box on) for O
@@ -870,20 +893,32 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       const float4 w4 = *reinterpret_cast<const float4*>(alpha_sh + n);
       w[n] = w4.x; w[n + 1] = w4.y; w[n + 2] = w4.z; w[n + 3] = w4.w;
     }
-    for (int i = 0; i < a.blocks; ++i) {
-      float o[N];
-      if (n_tiles > 0) {
-        tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
-      } else {
-#pragma unroll
-        for (int n = 0; n < N; ++n) o[n] = 0.0f;
-      }
+    auto stage = [&](int i, const float (&o)[N]) {
       if (i * 128 + r < a.DV) {
         uint4* dst = reinterpret_cast<uint4*>(gen + (i * 128 + r) * RL * 2);
 #pragma unroll
         for (int n = 0; n < N; n += 8)
           dst[n / 8] = make_uint4(pack_bf16x2(o[n] * w[n], o[n + 1] * w[n + 1]), pack_bf16x2(o[n + 2] * w[n + 2], o[n + 3] * w[n + 3]),
                                   pack_bf16x2(o[n + 4] * w[n + 4], o[n + 5] * w[n + 5]), pack_bf16x2(o[n + 6] * w[n + 6], o[n + 7] * w[n + 7]));
+      }
+    };
+    float zero[N];
+#pragma unroll
+    for (int n = 0; n < N; ++n) zero[n] = 0.0f;
+    int i = 0;
+    for (; n_tiles > 0 && i + 2 <= a.blocks; i += 2) {  // two loads in flight
+      float o[2][N];
+      tmem_ld_cols2<N>(tmem + lane_addr + i * N, o);
+      stage(i, o[0]);
+      stage(i + 1, o[1]);
+    }
+    for (; i < a.blocks; ++i) {
+      if (n_tiles > 0) {
+        float o[N];
+        tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
+        stage(i, o);
+      } else {
+        stage(i, zero);
       }
     }
     tc_fence_before();
@@ -913,24 +948,30 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tc_fence_after();
     tmem_dealloc(tmem, a.tmem_cols);
   }
-  // thread = (two rows, eight columns); rows side by side in a warp
+  // thread = two rows, eight columns at a time; rows side by side in a warp
+  static_assert(kLatThreads % (N / 2) == 0, "a thread keeps its rows");
   const uint32_t* sums = reinterpret_cast<const uint32_t*>(gen + (clustered ? taken : 0));
-  for (int i = threadIdx.x; i < mine / 8 * (N / 2); i += kLatThreads) {
-    const int r = i % (N / 2) * 2, c = i / (N / 2) * 8;
-    if (r >= n_rows) continue;
-    float o[2][8] = {};
-    for (int k = 0; k < splits; ++k) {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        const uint32_t v = sums[((k * mine + c + e) * RL + r) >> 1];
-        o[0][e] += bf16_lo(v);
-        o[1][e] += bf16_hi(v);
-      }
-    }
+  const int r = threadIdx.x % (N / 2) * 2;
+  if (r < n_rows) {
+    bf16* orow[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int rr = row0 + r + e, tok = rr / a.H, h = rr - tok * a.H;
-      if (r + e < n_rows) st8(a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + c0 + c, o[e]);
+      orow[e] = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + c0;
+    }
+    for (int c = static_cast<int>(threadIdx.x) / (N / 2) * 8; c < mine; c += kLatThreads / (N / 2) * 8) {
+      float o[2][8] = {};
+      const uint32_t* at = sums + ((c * RL + r) >> 1);
+      for (int k = 0; k < splits; ++k, at += mine * RL / 2) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const uint32_t v = at[e * RL / 2];
+          o[0][e] += bf16_lo(v);
+          o[1][e] += bf16_hi(v);
+        }
+      }
+      st8(orow[0] + c, o[0]);
+      if (r + 1 < n_rows) st8(orow[1] + c, o[1]);
     }
   }
   __syncwarp();
