@@ -914,10 +914,11 @@ def molitar_kernels(size, peaks, timed, graph_timed):
         "attention, decode")
     del kvs
     ql, ol = bf(n, H, R + RD), bf(n, H, R)
+    part = torch.empty(lib.teeny_latent_attention_scratch_bytes(R), dtype=torch.uint8, device="cuda")
     for length, name in ((S, ""), (4 * S, f", context {4 * S}")):
         at = ops.seq_table([(b, length - 1, b, 1) for b in range(n)])
         caches = [bf(n, length, R + RD) for _ in range(copies + 2 if length == S else 3)]
-        row("latent attention, absorbed, decode" + name, graph_timed([(lambda c=c, at=at: ops.latent_attention(ql, c, R, KD ** -0.5, at, 1, out=ol))
+        row("latent attention, absorbed, decode" + name, graph_timed([(lambda c=c, at=at: ops.latent_attention(ql, c, R, KD ** -0.5, at, 1, out=ol, scratch=part))
                                                                        for c in caches]), "hbm", 2.0 * n * length * (R + RD), "attention, decode" + name)
         del caches
     qh, vo = bf(n, H, KD), bf(n, H, V)

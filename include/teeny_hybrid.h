@@ -198,10 +198,12 @@ int teeny_head_linear(int f32, const void* x, long long ldx, long long x_head, c
                       int heads, int n, int k, int rows, int rot_dims, int rot_off, const float* inv_freq, float rot_scale, const int* seqs,
                       int n_seqs, teeny_stream_t stream);
 /* Causal attention of `heads` query heads over one cached row per token (its first vdim elements are the value): q [rows, ldq]
- * with heads dim apart, cache [slots, max_cached, dim], out with heads vdim apart. */
+ * with heads dim apart, cache [slots, max_cached, dim], out with heads vdim apart.  scratch: teeny_latent_attention_scratch_bytes
+ * (or null: a long cache is then not shared between CTAs). */
+size_t teeny_latent_attention_scratch_bytes(int vdim);
 int teeny_latent_attention(int f32, const void* q, long long ldq, int rows, const void* cache, int slots, int max_cached, void* out,
-                           long long ldo, int heads, int dim, int vdim, float score_scale, const int* seqs, int n_seqs, int max_len,
-                           teeny_stream_t stream);
+                           long long ldo, int heads, int dim, int vdim, float score_scale, void* scratch, size_t scratch_bytes,
+                           const int* seqs, int n_seqs, int max_len, teeny_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -288,7 +288,8 @@ extern "C" {
     pub fn teeny_cached_attention(f32: c_int, q: *const c_void, ldq: c_longlong, k_cache: *mut c_void, v_cache: *mut c_void, slots: c_int, max_cached: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, kv_heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, softcap: f32, sink: *const f32, gate: *const c_void, ldg: c_longlong, scratch: *mut c_void, scratch_bytes: usize, counters: *mut c_uint, seqs: *const c_int, host_seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
     pub fn teeny_latent_prepare(f32: c_int, proj: *const c_void, ld: c_longlong, off_q: c_int, off_c: c_int, off_r: c_int, q_rank: c_int, rank: c_int, rot_dims: c_int, q_weight: *const f32, c_weight: *const f32, inv_freq: *const f32, eps: f32, rot_scale: f32, cq: *mut c_void, ldcq: c_longlong, latents: *mut c_void, cache: *mut c_void, max_cached: c_int, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
     pub fn teeny_head_linear(f32: c_int, x: *const c_void, ldx: c_longlong, x_head: c_longlong, w: *const c_void, y: *mut c_void, ldy: c_longlong, y_head: c_longlong, heads: c_int, n: c_int, k: c_int, rows: c_int, rot_dims: c_int, rot_off: c_int, inv_freq: *const f32, rot_scale: f32, seqs: *const c_int, n_seqs: c_int, stream: CUstream) -> c_int;
-    pub fn teeny_latent_attention(f32: c_int, q: *const c_void, ldq: c_longlong, rows: c_int, cache: *const c_void, slots: c_int, max_cached: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
+    pub fn teeny_latent_attention_scratch_bytes(vdim: c_int) -> usize;
+    pub fn teeny_latent_attention(f32: c_int, q: *const c_void, ldq: c_longlong, rows: c_int, cache: *const c_void, slots: c_int, max_cached: c_int, out: *mut c_void, ldo: c_longlong, heads: c_int, dim: c_int, vdim: c_int, score_scale: f32, scratch: *mut c_void, scratch_bytes: usize, seqs: *const c_int, n_seqs: c_int, max_len: c_int, stream: CUstream) -> c_int;
 }
 // ---- generated from include/*.h: end ----
 

@@ -80,7 +80,8 @@ SIGNATURES = {
                                      i32, i32, vp]),
     "teeny_latent_prepare": (i32, [i32, vp, i64] + [i32] * 6 + [vp, vp, vp, f32, f32, vp, i64, vp, vp, i32, vp, i32, i32, vp]),
     "teeny_head_linear": (i32, [i32, vp, i64, i64, vp, vp, i64, i64] + [i32] * 6 + [vp, f32, vp, i32, vp]),
-    "teeny_latent_attention": (i32, [i32, vp, i64, i32, vp, i32, i32, vp, i64, i32, i32, i32, f32, vp, i32, i32, vp]),
+    "teeny_latent_attention_scratch_bytes": (sz, [i32]),
+    "teeny_latent_attention": (i32, [i32, vp, i64, i32, vp, i32, i32, vp, i64, i32, i32, i32, f32, vp, sz, vp, i32, i32, vp]),
     "teeny_sample_merge": (i32, [vp, i32, sz, i32, f32, i32, f32, vp, vp, vp, vp]),
 }
 

@@ -9,8 +9,8 @@
 //   latent_prepare_kernel<T>          norms of the query latent and the latent, rotation of the shared key part, cache append
 //   head_linear_mma_kernel<MT>        the small per-head products, bf16 (mma.sync; weights fetched ahead of the dependency wait)
 //   head_linear_rows_kernel<T>        the same, anything
-//   latent_attention_kernel<N>        absorbed attention, bf16 (tcgen05; the key range is split over a cluster whose CTAs merge
-//                                     through distributed shared memory)
+//   latent_attention_kernel<N>        absorbed attention, bf16 (tcgen05; the key range is split over CTAs), and
+//   latent_merge_kernel               the sum over the shares of a split key range
 //   latent_attention_rows_kernel<T>   the same, anything: eight warps per (token, head)
 #include <atomic>
 #include <type_traits>
@@ -341,8 +341,8 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
   }
 }
 
-// Absorbed attention on the tensor cores (tcgen05).  CTA = N consecutive (token, head) rows of one entry x one share of its keys;
-// the CTAs of a cluster hold the shares of one row tile.  The rows are the N side of both products (a few query heads waste
+// Absorbed attention on the tensor cores (tcgen05).  CTA = N consecutive (token, head) rows of one entry x one share of its keys.
+// The rows are the N side of both products (a few query heads waste
 // nothing), and the cache rows, loaded once per 64-key tile, are the A operand of both.  M = 128 holds 64 keys twice: a slot of
 // shared memory is 128 dimensions of the tile as two boxes [64 keys][64 d], one behind the other, which the two products read as
 //   S^T [2 x 64 keys, 2 N] += [boxes] [Q of the first box's dimensions; Q of the second's]^T     (K-major)
@@ -360,20 +360,22 @@ __global__ void __launch_bounds__(256) latent_attention_rows_kernel(const Latent
 //            running maxima (shared memory), sums in registers, weights as bf16 into shared memory ([row][key], the B operand).
 //            The maxima only move when some score exceeds its row's by more than 2^8 (one vote per tile); then the tile's maxima
 //            are reduced across the lanes and O^T is rescaled.
-// At the end the shares tell one another their maxima and sums, every CTA scales its O^T by its weights, rounds it to bf16 (the
-// exchange is what the end takes longest for) and copies the columns to the CTAs that sum them over the shares.
+// At the end O^T over its row sums goes out as bf16 rows, one bulk store of N whole rows: to the output, or where the keys are
+// split to a partial result beside its maxima and sums, which latent_merge_kernel weighs and adds.  (Shares of a cluster meeting in
+// distributed shared memory were slower: the exchange of 64 KB per CTA took 5000 cycles, half as bf16, and clusters leave a
+// third of the SMs idle.)
 constexpr int kLatTile = 64, kLatSlot = 16384, kLatBox = 8192, kLatMaxSlots = 24, kLatThreads = 192;
 constexpr float kLatGrow = 8.0f;  // log2 units
 
 struct LatTcArgs {
-  bf16* out;
-  long long ldo;
+  bf16* out;           // [rows, DV]
+  bf16* part_o;        // split keys: [CTA][N][DV] and ...
+  float2* part_ml;     // ... [CTA][N] maximum (log2 domain) and sum
   int row_base;        // step row that row 0 of q and out stands for
   int H, D, DV;
   int blocks;          // 128-dimension slots of a tile that hold values
   int tile_slots;      // slots of a tile
   int slots, ahead;    // of the ring; whether it holds two tiles
-  int sums_at;         // byte offset over the slots of what a CTA sums in the end
   uint32_t tmem_cols;
   float scale_log2;
   int* err;
@@ -389,49 +391,14 @@ __host__ __device__ inline LatSmem lat_smem(int n, int tile_slots, int slots) {
   s.swap = s.p + n * 128;               // partial scores between the lane halves: [n / 4][64 keys] float4
   s.bars = s.swap + n * 64 * 4;
   s.stats = s.bars + 8 * (2 * kLatMaxSlots + 8);
-  s.total = s.stats + 4 * (8 + 16) * n + 1024;
+  s.total = s.stats + 4 * 8 * n + 1024;
   return s;
 }
 
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-__device__ __forceinline__ uint32_t map_rank(uint32_t local_addr, uint32_t rank) {
-  uint32_t r;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(local_addr), "r"(rank));
-  return r;
-}
-__device__ __forceinline__ void st_cluster2(uint32_t addr, float x, float y) {
-  asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(x), "f"(y) : "memory");
-}
-// This CTA's shared memory -> another's (or its own), completion bytes on a barrier there.
-__device__ __forceinline__ void bulk_copy_cluster(uint32_t dst, uint32_t src, uint32_t bytes, uint32_t bar) {
-  asm volatile("cp.async.bulk.shared::cluster.shared::cta.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-               ::"r"(dst), "r"(src), "r"(bytes), "r"(bar)
-               : "memory");
-}
-// mbar_wait for data that came from another CTA
-__device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity, int* err, int code) {
-  uint64_t t0 = 0;
-#pragma unroll 1
-  for (uint32_t it = 0;; ++it) {
-    uint32_t done;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(done) : "r"(bar), "r"(parity) : "memory");
-    if (done) return true;
-    if ((it & 0xff) == 0xff) {
-      if (*reinterpret_cast<volatile int*>(err) != 0) return false;
-      const uint64_t now = global_timer_ns();
-      if (t0 == 0) {
-        t0 = now;
-      } else if (now - t0 > kWaitLimitNs) {
-        atomicCAS(err, 0, code);
-        return false;
-      }
-    }
-  }
+// `bytes` of this CTA's shared memory to global memory, by one thread, which then waits until they have been read.
+__device__ __forceinline__ void bulk_store(void* dst, uint32_t src, uint32_t bytes) {
+  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst), "r"(src), "r"(bytes) : "memory");
+  asm volatile("cp.async.bulk.commit_group;\n\tcp.async.bulk.wait_group.read 0;" ::: "memory");
 }
 // whether `v` holds in any of the 128 softmax threads (barrier 1)
 __device__ __forceinline__ bool any128(bool v) {
@@ -584,7 +551,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   extern __shared__ uint8_t lat_raw[];
   const SeqDesc seq = seqs[blockIdx.z];  // written well before the kernel in front of this one
   const int row0 = blockIdx.y * N, n_rows = min(N, seq.len * a.H - row0);
-  if (n_rows <= 0) {  // the whole cluster
+  if (n_rows <= 0) {
     pdl_wait();
     return;
   }
@@ -597,14 +564,12 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   const uint32_t misc = bar0 + 8u * 2 * kLatMaxSlots;
   const uint32_t q_full = misc, s_full = misc + 8, p_ready = misc + 24, pv_done = misc + 32, tmem_slot = misc + 40;  // two s_full
   float* m_sh = reinterpret_cast<float*>(gen + lay.stats);  // [N] running maxima, log2 domain
-  float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally this share's weights
+  float* alpha_sh = m_sh + N;                               // [N] factor of the last rescale; finally 1 / the row sums
   float* up_sh = alpha_sh + N;                              // [N] by how much the maxima just rose
   float* red = up_sh + N;                                   // [4][HN] of each warp
   int* lim = reinterpret_cast<int*>(red + 4 * N);           // [N] last key each row sees
-  float2* share = reinterpret_cast<float2*>(lim + N);       // [N][8] maximum and sum of every share
 
   const int split = blockIdx.x, splits = gridDim.x;
-  const bool clustered = splits > 1;
   const int warp = threadIdx.x >> 5;
   const int L = seq.pos + (row0 + n_rows - 1) / a.H + 1;  // keys the tile's last row sees
   const int span = ((L + splits - 1) / splits + kLatTile - 1) / kLatTile * kLatTile;
@@ -623,7 +588,6 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     mbar_init(s_full + 8, 1);
     mbar_init(p_ready, 128);
     mbar_init(pv_done, 1);
-    mbar_init(misc + 48, 1);
     mbar_fence_init();
   }
   if (warp == 5) {
@@ -636,7 +600,6 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  if (clustered) cluster_arrive();  // [0] this CTA is there
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(gen + lay.bars + 8 * 2 * kLatMaxSlots + 40);
   const uint32_t t_s = tmem + a.blocks * N;
   bool ok = true;
@@ -849,96 +812,59 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
       tc_fence_before();
       mbar_arrive(p_ready);
     }
-    // ---- maxima and sums of all shares ----
+    // ---- row sums, then O^T as rows over the slots ----
     reduce_to<HN, false>(l, red + warp * HN);
     named_barrier_sync(1, 128);
-    if (clustered) cluster_wait();  // [0]
     if (r < N) {
       const float* part = red + (r / HN) * 2 * HN + r % HN;
-      const float mine = n_tiles > 0 ? m_sh[r] : -INFINITY, sum = part[0] + part[HN];
-      if (clustered) {
-        const uint32_t at = smem_u32(share + r * 8 + split);
-        for (int i = 0; i < splits; ++i) st_cluster2(map_rank(at, i), mine, sum);
-      } else {
-        share[r * 8] = make_float2(mine, sum);
+      const float sum = part[0] + part[HN];
+      alpha_sh[r] = sum > 0.0f ? 1.0f / sum : 0.0f;  // (no key of this share is visible to the row)
+      if (splits > 1) {
+        const size_t cta = (static_cast<size_t>(blockIdx.z) * gridDim.y + blockIdx.y) * splits + split;
+        a.part_ml[cta * N + r] = make_float2(sum > 0.0f ? m_sh[r] : -INFINITY, sum);
       }
     }
     if (n_tiles > 0 && ok) ok = mbar_wait(pv_done, (n_tiles - 1) & 1, a.err, DEVERR_ATTN_SOFTMAX);
     __syncwarp();
     tc_fence_after();
-  }
-  if (clustered) {  // [1] maxima and sums are there; nobody's slots are in use any more
-    if (warp >= 4) cluster_wait();  // [0]
-    cluster_arrive();
-    cluster_wait();
-  }
-  // ---- columns: every CTA's scaled O^T as [column][row] over its slots (rows padded: no bank conflicts), `per` columns at a time
-  // copied to the CTA that sums them, which takes them as [share][column][row] behind its own ----
-  const int per = ((a.DV + splits - 1) / splits + 7) & ~7;
-  constexpr int RL = N + 8;  // in bf16 elements
-  if (warp < 4) {
     named_barrier_sync(1, 128);
-    const int r = threadIdx.x;
-    if (r < N) {
-      float mm = -INFINITY, sum = 0.0f;
-      for (int i = 0; i < splits; ++i) mm = fmaxf(mm, share[r * 8 + i].x);
-      for (int i = 0; i < splits; ++i) sum = fmaf(ex2(share[r * 8 + i].x - mm), share[r * 8 + i].y, sum);  // shares without keys hold -inf: 0
-      alpha_sh[r] = ex2(share[r * 8 + split].x - mm) / sum;
-    }
-    named_barrier_sync(1, 128);
-    const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    float w[N];
+    if (n_tiles > 0) {
+      float w[N];
 #pragma unroll
-    for (int n = 0; n < N; n += 4) {
-      const float4 w4 = *reinterpret_cast<const float4*>(alpha_sh + n);
-      w[n] = w4.x; w[n + 1] = w4.y; w[n + 2] = w4.z; w[n + 3] = w4.w;
-    }
-    auto stage = [&](int i, const float (&o)[N]) {
-      if (i * 128 + r < a.DV) {
-        uint4* dst = reinterpret_cast<uint4*>(gen + (i * 128 + r) * RL * 2);
-#pragma unroll
-        for (int n = 0; n < N; n += 8)
-          dst[n / 8] = make_uint4(pack_bf16x2(o[n] * w[n], o[n + 1] * w[n + 1]), pack_bf16x2(o[n + 2] * w[n + 2], o[n + 3] * w[n + 3]),
-                                  pack_bf16x2(o[n + 4] * w[n + 4], o[n + 5] * w[n + 5]), pack_bf16x2(o[n + 6] * w[n + 6], o[n + 7] * w[n + 7]));
+      for (int n = 0; n < N; n += 4) {
+        const float4 w4 = *reinterpret_cast<const float4*>(alpha_sh + n);
+        w[n] = w4.x; w[n + 1] = w4.y; w[n + 2] = w4.z; w[n + 3] = w4.w;
       }
-    };
-    float zero[N];
+      auto stage = [&](int i, const float (&o)[N]) {
+        if (i * 128 + r < a.DV) {
+          bf16* dst = reinterpret_cast<bf16*>(gen) + i * 128 + r;
 #pragma unroll
-    for (int n = 0; n < N; ++n) zero[n] = 0.0f;
-    int i = 0;
-    for (; n_tiles > 0 && i + 2 <= a.blocks; i += 2) {  // two loads in flight
-      float o[2][N];
-      tmem_ld_cols2<N>(tmem + lane_addr + i * N, o);
-      stage(i, o[0]);
-      stage(i + 1, o[1]);
-    }
-    for (; i < a.blocks; ++i) {
-      if (n_tiles > 0) {
+          for (int n = 0; n < N; ++n) dst[n * a.DV] = __float2bfloat16_rn(o[n] * w[n]);
+        }
+      };
+      int i = 0;
+      for (; i + 2 <= a.blocks; i += 2) {  // two loads in flight
+        float o[2][N];
+        tmem_ld_cols2<N>(tmem + lane_addr + i * N, o);
+        stage(i, o[0]);
+        stage(i + 1, o[1]);
+      }
+      if (i < a.blocks) {
         float o[N];
         tmem_ld_cols<N>(tmem + lane_addr + i * N, o);
         stage(i, o);
-      } else {
-        stage(i, zero);
       }
+      fence_proxy_async_smem();
     }
     tc_fence_before();
-    if (clustered) fence_proxy_async_smem();
-  }
-  const uint32_t sums_full = misc + 48;
-  const int c0 = split * per, mine = max(0, min(per, a.DV - c0));  // columns summed here
-  if (clustered && threadIdx.x == 128 && mine > 0) mbar_expect_tx(sums_full, splits * mine * RL * 2);
-  __syncthreads();
-  const uint32_t taken = a.sums_at;  // where a CTA takes the shares
-  if (clustered && threadIdx.x < splits) {
-    const int to = threadIdx.x, n_cols = max(0, min(per, a.DV - to * per));
-    if (n_cols > 0)
-      bulk_copy_cluster(map_rank(base + taken + static_cast<uint32_t>(split * n_cols * RL) * 2, to), base + static_cast<uint32_t>(to * per * RL) * 2,
-                        n_cols * RL * 2, map_rank(sums_full, to));
   }
   pdl_trigger();
-  if (clustered && mine > 0) ok = mbar_wait_cluster(sums_full, 0, a.err, DEVERR_ATTN_SOFTMAX) && ok;
-  __syncwarp();
-  if (clustered) cluster_arrive();  // [2] the copies to this CTA have left their sources
+  __syncthreads();
+  if (threadIdx.x == 0 && n_tiles > 0) {  // (a share without keys has weight zero: its rows are never read)
+    bf16* dst = splits > 1 ? a.part_o + ((static_cast<size_t>(blockIdx.z) * gridDim.y + blockIdx.y) * splits + split) * N * a.DV
+                           : a.out + ((static_cast<long long>(seq.row0) - a.row_base) * a.H + row0) * a.DV;
+    bulk_store(dst, base, n_rows * a.DV * 2);
+  }
   if (warp == 5) {
     if (*reinterpret_cast<volatile int*>(a.err) != 0) {  // a wait was given up: let copies and products in flight finish
       const uint64_t t0 = global_timer_ns();
@@ -948,34 +874,52 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid
     tc_fence_after();
     tmem_dealloc(tmem, a.tmem_cols);
   }
-  // thread = two rows, eight columns at a time; rows side by side in a warp
-  static_assert(kLatThreads % (N / 2) == 0, "a thread keeps its rows");
-  const uint32_t* sums = reinterpret_cast<const uint32_t*>(gen + (clustered ? taken : 0));
-  const int r = threadIdx.x % (N / 2) * 2;
-  if (r < n_rows) {
-    bf16* orow[2];
+}
+
+// CTA = one row: thread = (eight columns, every `groups`-th share), so that a thread's few loads are all in flight together.
+constexpr int kLatMaxSplits = 32;
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatTcArgs a, const SeqDesc* __restrict__ seqs, int N, int tiles, int splits) {
+  __shared__ float weight[kLatMaxSplits];
+  __shared__ float sum[128][9];
+  const SeqDesc seq = seqs[blockIdx.y];
+  const int row = blockIdx.x;
+  pdl_wait();
+  pdl_trigger();
+  if (row >= seq.len * a.H) return;
+  const int tile = row / N, r = row - tile * N;
+  const size_t cta = (static_cast<size_t>(blockIdx.y) * tiles + tile) * splits;
+  const int chunks = a.DV / 8, groups = 128 / chunks, chunk = threadIdx.x % chunks, group = threadIdx.x / chunks;  // (DV <= 1024)
+  if (threadIdx.x < 32) {
+    const int s = threadIdx.x;
+    const float2 ml = s < splits ? a.part_ml[(cta + s) * N + r] : make_float2(-INFINITY, 0.0f);
+    const float w = ml.y * ex2(ml.x - warp_max(ml.x));  // shares without a visible key: 0
+    weight[s] = w / warp_sum(w);
+  }
+  __syncthreads();
+  float o[8] = {};
+  if (group < groups) {
+    const bf16* src = a.part_o + (cta * N + r) * a.DV + 8 * chunk;
+#pragma unroll 4
+    for (int s = group; s < splits; s += groups) {
+      const float w = weight[s];
+      if (w > 0.0f) {  // (the rows of a share without keys are not even written)
+        float v[8];
+        ld8(src + static_cast<size_t>(s) * N * a.DV, v);
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int rr = row0 + r + e, tok = rr / a.H, h = rr - tok * a.H;
-      orow[e] = a.out + (static_cast<long long>(seq.row0) - a.row_base + tok) * a.ldo + h * a.DV + c0;
-    }
-    for (int c = static_cast<int>(threadIdx.x) / (N / 2) * 8; c < mine; c += kLatThreads / (N / 2) * 8) {
-      float o[2][8] = {};
-      const uint32_t* at = sums + ((c * RL + r) >> 1);
-      for (int k = 0; k < splits; ++k, at += mine * RL / 2) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const uint32_t v = at[e * RL / 2];
-          o[0][e] += bf16_lo(v);
-          o[1][e] += bf16_hi(v);
-        }
+        for (int e = 0; e < 8; ++e) o[e] = fmaf(w, v[e], o[e]);
       }
-      st8(orow[0] + c, o[0]);
-      if (r + 1 < n_rows) st8(orow[1] + c, o[1]);
     }
   }
-  __syncwarp();
-  if (clustered) cluster_wait();
+  if (groups > 1) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum[threadIdx.x][e] = o[e];
+    __syncthreads();
+    if (group == 0)
+      for (int g = 1; g < groups; ++g)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] += sum[g * chunks + chunk][e];
+  }
+  if (group == 0) st8(a.out + ((static_cast<long long>(seq.row0) - a.row_base) * a.H + row) * a.DV + 8 * chunk, o);
 }
 
 constexpr int kLatSmemLimit = 232448;
@@ -999,39 +943,12 @@ bool plan_tc(int n, int d, int dv, LatTcArgs& a, int& smem) {
   a.slots = left > 0 ? left / kLatSlot : 0;
   if (a.slots > kLatMaxSlots) a.slots = kLatMaxSlots;
   if (a.slots > 3 * a.tile_slots) a.slots = 3 * a.tile_slots;
-  // in the end over the slots: O^T [values][n + 8] and the shares' columns (no more than values + 8 per share)
-  a.sums_at = (n + 8) * dv * 2;
-  const int bytes = a.sums_at + (n + 8) * (dv + 64) * 2;
-  if (a.slots * kLatSlot < bytes) a.slots = (bytes + kLatSlot - 1) / kLatSlot;
+  const int rows = n * dv * 2;  // in the end over the slots
+  if (a.slots * kLatSlot < rows) a.slots = (rows + kLatSlot - 1) / kLatSlot;
   a.ahead = a.slots >= 2 * a.tile_slots;
   if (a.slots < a.tile_slots || a.slots > kLatMaxSlots || (n > 32 && !a.ahead)) return false;
   smem = lat_smem(n, a.tile_slots, a.slots).total;
   return smem <= kLatSmemLimit;
-}
-
-// Clusters of `size` CTAs that can be resident at once (per device, worked out once).
-template <int N>
-int max_clusters(int size, int smem) {
-  static std::atomic<int> known[9][64];  // [size][shared memory in 4 KB steps]; -1: none
-  std::atomic<int>& k = known[size][(smem >> 12) & 63];
-  int v = k.load(std::memory_order_relaxed);
-  if (v != 0) return v;
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(size, 1, 1);
-  cfg.blockDim = dim3(kLatThreads);
-  cfg.dynamicSmemBytes = smem;
-  cudaLaunchAttribute attr;
-  attr.id = cudaLaunchAttributeClusterDimension;
-  attr.val.clusterDim.x = size;
-  attr.val.clusterDim.y = attr.val.clusterDim.z = 1;
-  cfg.attrs = &attr;
-  cfg.numAttrs = 1;
-  if (cudaOccupancyMaxActiveClusters(&v, latent_attention_kernel<N>, &cfg) != cudaSuccess || v < 1) {
-    cudaGetLastError();
-    v = -1;
-  }
-  k.store(v, std::memory_order_relaxed);
-  return v;
 }
 
 }  // namespace
@@ -1094,6 +1011,11 @@ int latent_attention_prepare() {
   return 0;
 }
 
+size_t latent_attention_scratch_bytes(int dv) {
+  // as many partial results as rows of CTAs that a launch with a split key range has: at most two rounds of 64-row tiles
+  return static_cast<size_t>(2 * sm_count()) * 64 * (static_cast<size_t>(dv) * 2 + 8) + 16;
+}
+
 int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int longest, cudaStream_t st) {
   if (!a.q || !a.cache || !a.out || !seqs || n_seqs <= 0 || n_seqs > 65535 || longest <= 0 || a.H <= 0 || a.D <= 0 || a.D > kLatMax ||
       a.DV <= 0 || a.DV > a.D || a.max_len <= 0 || static_cast<long long>(longest) * a.H > 0x7fffffffLL)
@@ -1104,15 +1026,14 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
   }
   const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache);
   const int rows = longest * a.H;
-  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (a.ldo & 7) == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 15) == 0 &&
-      a.ldq == static_cast<long long>(a.H) * a.D) {
+  if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 15) == 0 &&
+      a.ldq == static_cast<long long>(a.H) * a.D && a.ldo == static_cast<long long>(a.H) * a.DV) {
     LatTcArgs t{};
     int smem = 0, n = rows <= 16 ? 16 : (rows <= 32 ? 32 : 64);
     while (n >= 16 && !plan_tc(n, a.D, a.DV, t, smem)) n /= 2;
     const int tiles = n >= 16 ? (rows + n - 1) / n : 0;
     if (n >= 16 && tiles <= 65535) {
       t.out = static_cast<bf16*>(a.out);
-      t.ldo = a.ldo;
       t.row_base = a.row_base;
       t.H = a.H; t.D = a.D; t.DV = a.DV;
       t.scale_log2 = a.scale * 1.4426950408889634f;
@@ -1129,27 +1050,30 @@ int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int l
       const uint32_t qb[2] = {64, static_cast<uint32_t>(n)};
       rc = encode_tensor_map_bf16(&mq, a.q, 2, qd, qs, qb);
       if (rc) return rc;
-      return for_rows(n, [&](auto nn) {
-        constexpr int N = decltype(nn)::value;
-        // shares of the keys per row tile: fewest rounds of tiles over all waves of clusters
-        const long long work = static_cast<long long>(tiles) * n_seqs;
-        const int key_tiles = (a.max_len + kLatTile - 1) / kLatTile;
-        int splits = 0;
-        long long best = -1;
-        for (int c = 1; c <= 8 && (c == 1 || c <= key_tiles); ++c) {
-          const int fit = max_clusters<N>(c, smem);
-          if (fit < 1) continue;
-          const long long cost = ((work + fit - 1) / fit) * ((key_tiles + c - 1) / c);
-          if (best < 0 || cost < best) {
-            best = cost;
-            splits = c;
-          }
+      // shares of the keys per row tile: fewest rounds of tiles, each CTA's start and end counted as four; as far as there is
+      // scratch for the partial results
+      const long long work = static_cast<long long>(tiles) * n_seqs;
+      const int key_tiles = (a.max_len + kLatTile - 1) / kLatTile;
+      int splits = 1;
+      long long best = -1;
+      for (int c = 1; c <= kLatMaxSplits && (c == 1 || (c <= key_tiles && a.scratch && work * c * n * (a.DV * 2 + 8) + 16 <= static_cast<long long>(a.scratch_bytes)));
+           ++c) {
+        const long long cost = ((work * c + sm_count() - 1) / sm_count()) * ((key_tiles + c - 1) / c + 4) + (c > 1 ? 3 : 0);
+        if (best < 0 || cost < best) {
+          best = cost;
+          splits = c;
         }
-        if (splits == 0) return static_cast<int>(TEENY_ERR_BAD_ARG);
-        launch_kernel(latent_attention_kernel<N>, dim3(splits, tiles, n_seqs), dim3(kLatThreads), smem, st, static_cast<unsigned>(splits), mc, mq, t,
-                      seqs);
+      }
+      t.part_ml = static_cast<float2*>(a.scratch);
+      t.part_o = reinterpret_cast<bf16*>(static_cast<uint8_t*>(a.scratch) + (work * splits * n * 8 + 15) / 16 * 16);
+      rc = for_rows(n, [&](auto nn) {
+        constexpr int N = decltype(nn)::value;
+        launch_kernel(latent_attention_kernel<N>, dim3(splits, tiles, n_seqs), dim3(kLatThreads), smem, st, 1, mc, mq, t, seqs);
         return static_cast<int>(cudaGetLastError());
       });
+      if (rc || splits == 1) return rc;
+      launch_kernel(latent_merge_kernel, dim3(rows, n_seqs), dim3(128), 0, st, 1, t, seqs, n, tiles, splits);
+      return static_cast<int>(cudaGetLastError());
     }
   }
   const dim3 grid(static_cast<unsigned>(rows), n_seqs);

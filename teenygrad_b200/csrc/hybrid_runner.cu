@@ -63,7 +63,7 @@ struct Plan {
   std::vector<Layer> layers;
   size_t x, y, proj, mix, delta, act, gu, o32, low, wz, kbuf, yrows, logits, logits16;
   size_t attn_scratch, attn_counters, attn_scratch_bytes;
-  size_t v_first, cq, lat_q, lat_rows, lat_kv, lat_qa, lat_oa;  // value mixing; latent attention
+  size_t v_first, cq, lat_q, lat_rows, lat_kv, lat_qa, lat_oa, lat_scratch, lat_scratch_bytes;  // value mixing; latent attention
   int v_first_ld, cq_ld, lat_q_ld, lat_row_ld, lat_kv_ld, lat_qa_ld, lat_oa_ld;
   int absorb_rows;  // most rows of one absorbed run
   size_t seqs, rows, sample_u, best_val, next_ids, cur_ids, history, state, total;
@@ -100,6 +100,7 @@ bool make_plan(const teeny_hybrid_config& c, const teeny_hybrid_layer* layers, c
   p.proj_ld = p.mix_ld = p.o_ld = p.low_ld = p.wz_ld = p.k_ld = 8;
   p.act_ld = 64;
   p.v_first_ld = p.cq_ld = p.lat_q_ld = p.lat_row_ld = p.lat_kv_ld = p.lat_qa_ld = p.lat_oa_ld = 0;
+  p.lat_scratch_bytes = 0;
   int mixed_values = 0;  // columns of the first branch that mixes values
   p.attn_scratch_bytes = 0;
   int kv_heads = 1;
@@ -158,6 +159,10 @@ bool make_plan(const teeny_hybrid_config& c, const teeny_hybrid_layer* layers, c
           up(p.lat_kv_ld, H * (b.head() + V));
           up(p.lat_qa_ld, H * b.row());
           up(p.lat_oa_ld, H * b.latent());
+          if (!c.f32) {
+            const size_t need = latent_attention_scratch_bytes(b.latent());
+            if (need > p.lat_scratch_bytes) p.lat_scratch_bytes = need;
+          }
           break;
         case TEENY_HYBRID_DELTA:
           for (; n < 5; ++n) sizes[n] = H * D;
@@ -215,6 +220,7 @@ bool make_plan(const teeny_hybrid_config& c, const teeny_hybrid_layer* layers, c
   p.absorb_rows = c.max_tokens < 2048 ? c.max_tokens : (c.max_batch > 2048 ? c.max_batch : 2048);
   p.lat_qa = take(static_cast<size_t>(p.absorb_rows) * p.lat_qa_ld * es);
   p.lat_oa = take(static_cast<size_t>(p.absorb_rows) * p.lat_oa_ld * es);
+  p.lat_scratch = take(p.lat_scratch_bytes);
   p.yrows = take(static_cast<size_t>(c.max_rows) * p.width_ld * es);
   p.logits = take(static_cast<size_t>(c.max_rows) * p.vocab_ld * es);
   p.logits16 = take(c.f32 ? Bm * p.vocab_ld * 2 : 0);
@@ -363,6 +369,8 @@ int run_latent_absorbed(teeny_hybrid* m, const Layer& L, const Branch& b, int e0
   a.out = m->at<void>(p.lat_oa); a.ldo = H * KR;
   a.H = H; a.D = DL; a.DV = KR;
   a.scale = c.score_scale;
+  a.scratch = m->at<void>(p.lat_scratch);
+  a.scratch_bytes = p.lat_scratch_bytes;
   TEENY_TRY(latent_attention(a, seqs, n, longest, st));
   HeadLinear out{};
   out.f32 = m->cfg.f32;
@@ -974,10 +982,12 @@ int teeny_head_linear(int f32, const void* x, long long ldx, long long x_head, c
   return head_linear(a, reinterpret_cast<cudaStream_t>(stream));
 }
 
+size_t teeny_latent_attention_scratch_bytes(int vdim) { return vdim > 0 ? latent_attention_scratch_bytes(vdim) : 0; }
+
 int teeny_latent_attention(int f32, const void* q, long long ldq, int rows, const void* cache, int slots, int max_cached, void* out,
-                           long long ldo, int heads, int dim, int vdim, float score_scale, const int* seqs, int n_seqs, int max_len,
-                           teeny_stream_t stream) {
-  const LatentAttn a{f32, q, ldq, rows, 0, cache, slots, max_cached, out, ldo, heads, dim, vdim, score_scale};
+                           long long ldo, int heads, int dim, int vdim, float score_scale, void* scratch, size_t scratch_bytes,
+                           const int* seqs, int n_seqs, int max_len, teeny_stream_t stream) {
+  const LatentAttn a{f32, q, ldq, rows, 0, cache, slots, max_cached, out, ldo, heads, dim, vdim, score_scale, scratch, scratch_bytes};
   return latent_attention(a, reinterpret_cast<const SeqDesc*>(seqs), n_seqs, max_len, reinterpret_cast<cudaStream_t>(stream));
 }
 

@@ -418,7 +418,10 @@ struct LatentAttn {
   long long ldo;
   int H, D, DV;
   float scale;
+  void* scratch;             // latent_attention_scratch_bytes(DV), or null (the keys are then not split over CTAs)
+  size_t scratch_bytes;
 };
+size_t latent_attention_scratch_bytes(int dv);
 int latent_attention_prepare();
 int latent_attention(const LatentAttn& a, const SeqDesc* seqs, int n_seqs, int longest, cudaStream_t st);
 

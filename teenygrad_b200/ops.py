@@ -503,11 +503,15 @@ def head_linear(x, w, rot_dims=0, rot_off=0, inv_freq=None, rot_scale=1.0, seqs=
     return out
 
 
-def latent_attention(q, cache, vdim, score_scale, seqs, max_len, out=None):
+def latent_attention(q, cache, vdim, score_scale, seqs, max_len, out=None, scratch=None):
     """q [rows, heads, dim] over ``cache`` [slots, max_len, dim], whose rows' first ``vdim`` elements are the values; causal, the
-    entries' own rows are in the cache already.  Returns [rows, heads, vdim]."""
+    entries' own rows are in the cache already.  ``scratch``: uint8, for a key range shared between CTAs (made here when missing).
+    Returns [rows, heads, vdim]."""
     _req(q, name="q"); _req(cache, q.dtype, "cache")
     out = torch.zeros(q.shape[0], q.shape[1], vdim, dtype=q.dtype, device=q.device) if out is None else out
+    if scratch is None and q.dtype == _BF16:
+        scratch = torch.empty(lib.teeny_latent_attention_scratch_bytes(vdim), dtype=torch.uint8, device=q.device)
     check(lib.teeny_latent_attention(_f32_flag(q), _ptr(q), q.stride(0), q.shape[0], _ptr(cache), cache.shape[0], cache.shape[1], _ptr(out),
-                                     out.stride(0), q.shape[1], q.shape[2], vdim, float(score_scale), _ptr(seqs), seqs.shape[0], max_len, _stream()), "latent_attention")
+                                     out.stride(0), q.shape[1], q.shape[2], vdim, float(score_scale), _ptr(scratch),
+                                     0 if scratch is None else scratch.numel(), _ptr(seqs), seqs.shape[0], max_len, _stream()), "latent_attention")
     return out
