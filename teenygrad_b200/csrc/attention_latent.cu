@@ -889,6 +889,13 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatTcArgs a, co
   const int tile = row / N, r = row - tile * N;
   const size_t cta = (static_cast<size_t>(blockIdx.y) * tiles + tile) * splits;
   const int chunks = a.DV / 8, groups = 128 / chunks, chunk = threadIdx.x % chunks, group = threadIdx.x / chunks;  // (DV <= 1024)
+  // the rows are on their way while the weights are worked out
+  constexpr int kAhead = 8;
+  const bf16* src = a.part_o + (cta * N + r) * a.DV + 8 * chunk;
+  uint4 v[kAhead];
+#pragma unroll
+  for (int i = 0; i < kAhead; ++i)
+    if (group < groups && group + i * groups < splits) v[i] = *reinterpret_cast<const uint4*>(src + static_cast<size_t>(group + i * groups) * N * a.DV);
   if (threadIdx.x < 32) {
     const int s = threadIdx.x;
     const float2 ml = s < splits ? a.part_ml[(cta + s) * N + r] : make_float2(-INFINITY, 0.0f);
@@ -897,18 +904,22 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatTcArgs a, co
   }
   __syncthreads();
   float o[8] = {};
-  if (group < groups) {
-    const bf16* src = a.part_o + (cta * N + r) * a.DV + 8 * chunk;
-#pragma unroll 4
-    for (int s = group; s < splits; s += groups) {
-      const float w = weight[s];
-      if (w > 0.0f) {  // (the rows of a share without keys are not even written)
-        float v[8];
-        ld8(src + static_cast<size_t>(s) * N * a.DV, v);
+  auto add = [&](int s, uint4 x) {
+    const float w = weight[s];
+    if (w > 0.0f) {  // (the rows of a share without keys are not even written)
+      const uint32_t u[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(w, v[e], o[e]);
+      for (int e = 0; e < 4; ++e) {
+        o[2 * e] = fmaf(w, bf16_lo(u[e]), o[2 * e]);
+        o[2 * e + 1] = fmaf(w, bf16_hi(u[e]), o[2 * e + 1]);
       }
     }
+  };
+  if (group < groups) {
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+      if (group + i * groups < splits) add(group + i * groups, v[i]);
+    for (int s = group + kAhead * groups; s < splits; s += groups) add(s, *reinterpret_cast<const uint4*>(src + static_cast<size_t>(s) * N * a.DV));
   }
   if (groups > 1) {
 #pragma unroll

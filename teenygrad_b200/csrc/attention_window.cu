@@ -105,6 +105,7 @@ __global__ void head_norm_rope_rows_kernel(const HeadNormRope a, const SeqDesc* 
 // The same for bf16 heads of whole 16-byte vectors: `lph` (a power of two) lanes hold a head, eight elements each; the
 // rotation partner of a lane is rot_dims / 16 lanes away.
 constexpr int kRopeTasks = 4;  // (head, lane) tasks per thread whose loads are in flight together
+template <bool PLAIN>  // normed heads and no values
 __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormRope a, const SeqDesc* __restrict__ seqs, int lph) {
   __shared__ __align__(16) float cs[kMaxHead / 2], sn[kMaxHead / 2];
   const SeqDesc seq = seqs[blockIdx.y];  // written well before the kernel in front of this one
@@ -123,7 +124,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormR
   const int per = 256 / lph, heads = a.Hq + a.Hkv, h0 = threadIdx.x / lph;
   const int step = half >> 3;
   const int at = a.ring ? (seq.pos + i) % a.ring : 0;
-  if (a.v) {
+  if (!PLAIN && a.v) {
     const float lam = a.v_mode == kMixWith ? *a.mix : 0.0f, keep = 1.0f - lam;
     for (int c = threadIdx.x * 8; c < a.Hkv * a.DV; c += 256 * 8) {
       uint4 v = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(a.v) + row * a.ldv + c);
@@ -142,7 +143,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_vec_kernel(const HeadNormR
   }
   const int partner = (lane - sub) + (sub < step ? sub + step : (sub < 2 * step ? sub - step : sub));
   // heads of q that are not normed change in place in their rotated dimensions only
-  const bool in_k = d0 < a.D, in_q = a.q_w ? in_k : d0 < a.rot_dims;
+  const bool in_k = d0 < a.D, in_q = PLAIN || a.q_w ? in_k : d0 < a.rot_dims;
   for (int base = 0; base < heads; base += per * kRopeTasks) {
     uint4 raw[kRopeTasks];
 #pragma unroll
@@ -508,7 +509,8 @@ int head_norm_rope_rows(const HeadNormRope& a, const SeqDesc* seqs, int n_seqs, 
   if (!a.f32 && a.D % 8 == 0 && a.DV % 8 == 0 && a.rot_dims % 16 == 0 && ((a.ldq | a.ldkr | a.ldk | a.ldv | a.ldvf) & 7) == 0 && (bases & 15) == 0) {
     int lph = 1;
     while (lph * 8 < (a.Hkv == 0 && !a.q_w ? a.rot_dims : a.D)) lph *= 2;
-    launch_kernel(head_norm_rope_vec_kernel, grid, block, 0, st, 1, a, seqs, lph);
+    if (a.q_w && !a.v) launch_kernel(head_norm_rope_vec_kernel<true>, grid, block, 0, st, 1, a, seqs, lph);
+    else launch_kernel(head_norm_rope_vec_kernel<false>, grid, block, 0, st, 1, a, seqs, lph);
     return static_cast<int>(cudaGetLastError());
   }
   if (a.f32) launch_kernel(head_norm_rope_rows_kernel<float>, grid, block, 0, st, 1, a, seqs);
