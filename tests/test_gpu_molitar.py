@@ -472,6 +472,21 @@ def test_first_tokens_of_a_sequence():
             close(o, want[n][1:3], dtype)
 
 
+@DTYPES
+@pytest.mark.parametrize("n", [1, 2, 9, 63, 65, 129])
+def test_capacity_of_exactly_the_sequence(dtype, n):
+    """A runner that holds no token more than the request, at once and token by token."""
+    cfg, w, toks, want = case("b")
+    r = build("b", dtype, max_batch=1, max_len=n, max_rows=n)
+    for sizes in ([n], [1] * n):
+        s, at, out = r.open(), 0, []
+        for c in sizes:
+            out += r.step([(s, toks[201][at:at + c], range(c))])
+            at += c
+        r.close(s)
+        close(torch.cat(out), want[201][:n], dtype)
+
+
 def test_command_line_and_trace_replay(tmp_path):
     from teenygrad_b200 import safetensors
     cfg, w, toks, want = case("a")
